@@ -272,6 +272,11 @@ int32_t runit_moe_router_f32(runit_ctx_t*, const void* router_w, const void* x, 
  * out_idx: int32 [T][k]; out_w: f32 [T][k].  E <= 256, k <= 32. */
 int32_t runit_moe_route_topk(runit_ctx_t*, const void* logits, int32_t logits_f16, uint32_t E, uint32_t k, int32_t renorm,
                              uint32_t T, void* out_idx, void* out_w);
+/* The same with the scoring function as a parameter: rows of ld logits (the first E are the experts'), softmax over the
+ * experts or the sigmoid of each logit.  f32 logits. */
+enum { RUNIT_SCORE_SOFTMAX = 0, RUNIT_SCORE_SIGMOID = 1 };
+int32_t runit_moe_route_scored(runit_ctx_t*, const void* logits, uint32_t ld, uint32_t E, uint32_t k, int32_t score, int32_t renorm,
+                               uint32_t T, void* out_idx, void* out_w);
 /* Scratch bytes runit_moe_layer_q4k needs for these shapes. */
 size_t runit_moe_scratch_bytes(uint32_t T, uint32_t h, uint32_t ff, uint32_t E, uint32_t k);
 /* One MoE block over T tokens, all on the device:

@@ -25,6 +25,7 @@
 #include <cuda_bf16.h>
 
 #include "gemv_common.cuh"
+#include "moe_internal.h"
 #include "runit_internal.h"
 #include "tcgen05.cuh"
 #include "tma.cuh"
@@ -408,90 +409,6 @@ grouped_gemm_pair_kernel(const __grid_constant__ CUtensorMap map_b, const __grid
 
 // ───────────────────────── token permutation ─────────────────────────
 
-// counts[e] = slots routed to expert e; slots with an id outside [0, E) get position -1.
-__global__ void __launch_bounds__(256) count_kernel(const int32_t* __restrict__ idx, uint32_t S, uint32_t E,
-                                                     int32_t* __restrict__ counts, int32_t* __restrict__ pos_of_slot) {
-    __shared__ int hist[256];
-    hist[threadIdx.x] = 0;
-    __syncthreads();
-    for (uint32_t s = blockIdx.x * 4096 + threadIdx.x, i = 0; i < 16 && s < S; i++, s += 256) {
-        const int32_t e = idx[s];
-        if (e >= 0 && (uint32_t)e < E) atomicAdd(&hist[e], 1);
-        else pos_of_slot[s] = -1;
-    }
-    __syncthreads();
-    if (threadIdx.x < E && hist[threadIdx.x]) atomicAdd(&counts[threadIdx.x], hist[threadIdx.x]);
-}
-
-// One CTA per expert: first row of the expert in the permuted order (experts in index order, each padded to a
-// multiple of 128 rows), the token-tile table (tiles of `tile_tok` slots, 128 or 256, never across experts), and the
-// position of each of its slots (slot order kept).
-__global__ void __launch_bounds__(1024) place_kernel(const int32_t* __restrict__ idx, uint32_t S, uint32_t E,
-                                                      const int32_t* __restrict__ counts, int tile_tok,
-                                                      int32_t* __restrict__ pos_of_slot, int32_t* __restrict__ tile_expert,
-                                                      int32_t* __restrict__ tile_nvalid, int32_t* __restrict__ tile_row0,
-                                                      int32_t* __restrict__ n_tok_tiles) {
-    __shared__ int s_cnt[256];
-    __shared__ int s_warp[32];
-    __shared__ int s_off, s_tile0, s_chunk;
-    const uint32_t e = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    if (tid < 256) s_cnt[tid] = tid < E ? counts[tid] : 0;
-    __syncthreads();
-    if (tid == 0) {
-        int off = 0, tiles = 0;
-        for (uint32_t i = 0; i < E; i++) {
-            if (i == e) { s_off = off; s_tile0 = tiles; }
-            off += ((s_cnt[i] + kTok - 1) / kTok) * kTok;
-            tiles += (s_cnt[i] + tile_tok - 1) / tile_tok;
-        }
-        if (e == 0) n_tok_tiles[0] = tiles;
-    }
-    __syncthreads();
-    const int cnt = s_cnt[e], off = s_off, tile0 = s_tile0;
-    for (int i = tid; i * tile_tok < cnt; i += 1024) {
-        tile_expert[tile0 + i] = (int32_t)e;
-        tile_nvalid[tile0 + i] = min(tile_tok, cnt - i * tile_tok);
-        tile_row0[tile0 + i] = off + i * tile_tok;
-    }
-    // every thread takes 4 consecutive slots per round, so a round covers 4096 slots in slot order
-    int running = 0;
-    for (uint32_t s0 = 0; s0 < S; s0 += 4096) {
-        const uint32_t s = s0 + 4 * tid;
-        bool hit[4];
-        int mine = 0;
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-            hit[i] = s + i < S && idx[s + i] == (int32_t)e;
-            mine += hit[i];
-        }
-        int incl = mine;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const int t = __shfl_up_sync(0xffffffffu, incl, o);
-            if ((int)lane >= o) incl += t;
-        }
-        if (lane == 31) s_warp[warp] = incl;
-        __syncthreads();
-        if (warp == 0) {
-            int v = s_warp[lane], wi = v;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const int t = __shfl_up_sync(0xffffffffu, wi, o);
-                if ((int)lane >= o) wi += t;
-            }
-            s_warp[lane] = wi - v;   // exclusive prefix over the warps
-            if (lane == 31) s_chunk = wi;
-        }
-        __syncthreads();
-        int p = off + running + s_warp[warp] + incl - mine;
-#pragma unroll
-        for (int i = 0; i < 4; i++)
-            if (hit[i]) pos_of_slot[s + i] = p++;
-        running += s_chunk;
-        __syncthreads();
-    }
-}
-
 // xperm[pos(s)][:] = bf16(x[s / k][:]); one warp per slot, 8 slots per CTA.
 __global__ void __launch_bounds__(256) gather_kernel(const float* __restrict__ x, const int32_t* __restrict__ pos_of_slot,
                                                       __nv_bfloat16* __restrict__ xperm, uint32_t S, uint32_t h, uint32_t k) {
@@ -510,18 +427,6 @@ __global__ void __launch_bounds__(256) gather_kernel(const float* __restrict__ x
     }
 }
 
-// The same permutation for rows that are bf16 already (slots received from other ranks): xperm[pos(s)][:] = x[s][:].
-__global__ void __launch_bounds__(256) gather_bf16_kernel(const __nv_bfloat16* __restrict__ x, const int32_t* __restrict__ pos_of_slot,
-                                                           __nv_bfloat16* __restrict__ xperm, uint32_t S, uint32_t h) {
-    const uint32_t s = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (s >= S) return;
-    const int32_t pos = pos_of_slot[s];
-    if (pos < 0) return;
-    const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)s * h);
-    uint4* dst = reinterpret_cast<uint4*>(xperm + (size_t)pos * h);
-    for (uint32_t c = lane; c < h / 8; c += 32) dst[c] = src[c];
-}
-
 // Destination of every permuted row of an expert-parallel block: receive row i (region r = i / cap_src of rank r, used
 // while i % cap_src < cnt[r]) came from slot meta[i].y of rank r and goes back to row meta[i].y of that rank's return buffer.
 struct ReturnPeers {
@@ -536,27 +441,6 @@ __global__ void __launch_bounds__(256) row_ptr_kernel(const int32_t* __restrict_
     if (j >= (uint32_t)cnt[r]) return;
     const int32_t pos = pos_of_slot[i];
     if (pos >= 0) table[pos] = ry.p[r] + (size_t)meta[i].y * h;
-}
-
-// out[t] = (residual ? residual[t] : 0) + sum_i w[t][i] * y[pos(t, i)]   (routing order; product and sum rounded
-// separately, like the reference's scale-accumulate followed by the residual add).
-__global__ void __launch_bounds__(256) combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pos_of_slot,
-                                                       const float* __restrict__ w, const float* __restrict__ residual,
-                                                       float* __restrict__ out, uint32_t h, uint32_t k) {
-    const uint32_t t = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
-    if (c >= h / 4) return;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (uint32_t i = 0; i < k; i++) {
-        const int32_t pos = pos_of_slot[t * k + i];
-        if (pos < 0) continue;
-        const float wi = w[t * k + i];
-        const float4 v = __ldg(reinterpret_cast<const float4*>(y + (size_t)pos * h) + c);
-        acc.x = __fadd_rn(acc.x, __fmul_rn(wi, v.x)); acc.y = __fadd_rn(acc.y, __fmul_rn(wi, v.y));
-        acc.z = __fadd_rn(acc.z, __fmul_rn(wi, v.z)); acc.w = __fadd_rn(acc.w, __fmul_rn(wi, v.w));
-    }
-    float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (residual) b = reinterpret_cast<const float4*>(residual + (size_t)t * h)[c];
-    reinterpret_cast<float4*>(out + (size_t)t * h)[c] = make_float4(b.x + acc.x, b.y + acc.y, b.z + acc.z, b.w + acc.w);
 }
 
 // ───────────────────────── host side ─────────────────────────
@@ -629,16 +513,13 @@ static int32_t experts_impl(runit_ctx* ctx, const Scratch& s, const void* gate, 
                             const int2* ret_meta = nullptr, const int32_t* ret_cnt = nullptr, const ReturnPeers* ret_peers = nullptr,
                             uint32_t cap_src = 0) {
     const uint32_t S = T * k;
-    RUNIT_CUDA_TRY(ctx, cudaMemsetAsync(s.counts, 0, 4 * 256, ctx->stream));
-    count_kernel<<<(S + 4095) / 4096, 256, 0, ctx->stream>>>(idx, S, E, s.counts, s.pos_of_slot);
-    int32_t st = runit_after_launch(ctx, "moe_grouped_count");
+    MoePermutation p{s.counts, s.n_tok_tiles, s.tile_expert, s.tile_nvalid, s.tile_row0, s.pos_of_slot};
+    int32_t st = moe_permute(ctx, idx, S, E, pair::kTokPair, p);
     if (st != RUNIT_OK) return st;
-    place_kernel<<<E, 1024, 0, ctx->stream>>>(idx, S, E, s.counts, pair::kTokPair, s.pos_of_slot, s.tile_expert,
-                                              s.tile_nvalid, s.tile_row0, s.n_tok_tiles);
-    if ((st = runit_after_launch(ctx, "moe_grouped_place")) != RUNIT_OK) return st;
-    if (x_bf16) gather_bf16_kernel<<<(S + 7) / 8, 256, 0, ctx->stream>>>((const __nv_bfloat16*)x_bf16, s.pos_of_slot, s.xperm, S, h);
-    else gather_kernel<<<(S + 7) / 8, 256, 0, ctx->stream>>>(x, s.pos_of_slot, s.xperm, S, h, k);
-    if ((st = runit_after_launch(ctx, "moe_grouped_gather")) != RUNIT_OK) return st;
+    if (x_bf16) {
+        if ((st = moe_gather_rows(ctx, x_bf16, s.pos_of_slot, s.xperm, S, (size_t)h * 2, 1)) != RUNIT_OK) return st;
+    } else gather_kernel<<<(S + 7) / 8, 256, 0, ctx->stream>>>(x, s.pos_of_slot, s.xperm, S, h, k);
+    if (!x_bf16 && (st = runit_after_launch(ctx, "moe_grouped_gather")) != RUNIT_OK) return st;
 
     const uint32_t rows = s.max_tiles * kTok + 256;
     Args a1{};
@@ -659,8 +540,7 @@ static int32_t experts_impl(runit_ctx* ctx, const Scratch& s, const void* gate, 
     if ((st = launch_pair<true>(ctx, "moe_grouped_gate_up", a1, s.xperm, rows, E, s.max_tiles * (ff / 128))) != RUNIT_OK) return st;
     if ((st = launch_pair<false>(ctx, "moe_grouped_down", a2, s.act, rows, E, s.max_tiles * (h / 256))) != RUNIT_OK) return st;
     if (!out) return RUNIT_OK;
-    combine_kernel<<<dim3((h / 4 + 255) / 256, T), 256, 0, ctx->stream>>>(s.y, s.pos_of_slot, w, residual, out, h, k);
-    return runit_after_launch(ctx, "moe_grouped_combine");
+    return moe_grouped_combine(ctx, s.y, s.pos_of_slot, w, residual, out, T, h, k);
 }
 
 static int32_t check_shapes(runit_ctx* ctx, const char* who, uint32_t T, uint32_t h, uint32_t ff, uint32_t E, uint32_t k) {
@@ -671,17 +551,7 @@ static int32_t check_shapes(runit_ctx* ctx, const char* who, uint32_t T, uint32_
     return RUNIT_OK;
 }
 
-// ── dense use of the same kernels: one "expert" that owns the whole matrix, tokens in their own order ──
-__global__ void dense_tiles_kernel(uint32_t T, int32_t* tile_expert, int32_t* tile_nvalid, int32_t* tile_row0, int32_t* n_tok_tiles) {
-    const uint32_t n = (T + pair::kTokPair - 1) / pair::kTokPair;
-    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
-        tile_expert[i] = 0;
-        tile_nvalid[i] = (int32_t)min((uint32_t)pair::kTokPair, T - i * pair::kTokPair);
-        tile_row0[i] = (int32_t)(i * pair::kTokPair);
-    }
-    if (threadIdx.x == 0) n_tok_tiles[0] = (int32_t)n;
-}
-
+// (dense use of the same kernels: one "expert" that owns the whole matrix, tokens in their own order)
 }  // namespace gg
 
 // Expert outputs of S slots whose rows are bf16 already (slot s: expert idx[s] of the E local ones, or an id outside
@@ -710,18 +580,10 @@ int32_t moe_grouped_slots_bf16(runit_ctx* ctx, const void* gate, const void* up,
     return gg::experts_impl(ctx, s, gate, up, down, nullptr, idx, nullptr, nullptr, nullptr, S, h, ff, E, 1, x_bf16);
 }
 
-// The weighted sum of the batched block by itself: out[t] = residual[t] + sum_i w[t][i] * y[pos_of_slot[t*k+i]].
-int32_t moe_grouped_combine(runit_ctx* ctx, const float* y, const int32_t* pos_of_slot, const float* w, const float* residual, float* out,
-                            uint32_t T, uint32_t h, uint32_t k) {
-    gg::combine_kernel<<<dim3((h / 4 + 255) / 256, T), 256, 0, ctx->stream>>>(y, pos_of_slot, w, residual, out, h, k);
-    return runit_after_launch(ctx, "moe_grouped_combine");
-}
-
 // Tile tables for dense_gemm_q4k_bf16 over T tokens: `tables` holds 3 * ceil(T / 256) + 4 int32.
 int32_t dense_tiles_prepare(runit_ctx* ctx, int32_t* tables, uint32_t T) {
     const uint32_t n = (T + gg::pair::kTokPair - 1) / gg::pair::kTokPair;
-    gg::dense_tiles_kernel<<<1, 256, 0, ctx->stream>>>(T, tables + 4, tables + 4 + n, tables + 4 + 2 * n, tables);
-    return runit_after_launch(ctx, "dense_tiles");
+    return moe_dense_tiles(ctx, T, gg::pair::kTokPair, tables + 4, tables + 4 + n, tables + 4 + 2 * n, tables);
 }
 
 // out[t][r] = sum_k bf16(W[r][k]) * x[t][k] (f32 out, w_up == nullptr), or out[t][r] = bf16(silu(W.x) * (W_up.x)) (bf16 out):
@@ -749,10 +611,6 @@ int32_t dense_gemm_q4k_bf16(runit_ctx* ctx, const char* name, const void* w, con
     if (w_up) return gg::launch_pair<true>(ctx, name, a, x_bf16, x_rows, 1, n * (rows / 128));
     return gg::launch_pair<false>(ctx, name, a, x_bf16, x_rows, 1, n * (rows / 256));
 }
-
-// moe.cu
-int32_t moe_router(runit_ctx* ctx, const float* router_w, const float* x, float* logits, uint32_t E, uint32_t h, uint32_t T);
-int32_t moe_topk(runit_ctx* ctx, const float* logits, uint32_t E, uint32_t k, int32_t renorm, uint32_t T, int32_t* idx, float* w);
 
 }  // namespace runit
 

@@ -21,6 +21,7 @@ OK = 0
 ERR_NO_DEVICE, ERR_BAD_ARG, ERR_BUFFER_SIZE, ERR_LAUNCH, ERR_NCCL, ERR_TIMEOUT, ERR_UNSUPPORTED, ERR_ALLOC = range(1, 9)
 FMT_Q8_0, FMT_Q4_0, FMT_Q4K, FMT_Q5_0, FMT_Q5K, FMT_Q6K = 0, 1, 2, 3, 4, 5
 BUF_DEVICE, BUF_HOST_VISIBLE = 0, 1
+SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
 
 BLOCK_ELEMS = {FMT_Q8_0: 32, FMT_Q4_0: 32, FMT_Q4K: 256, FMT_Q5_0: 32, FMT_Q5K: 256, FMT_Q6K: 256}     # dispatch.rs:735-747
 BLOCK_BYTES = {FMT_Q8_0: 34, FMT_Q4_0: 18, FMT_Q4K: 144, FMT_Q5_0: 22, FMT_Q5K: 176, FMT_Q6K: 210}
@@ -264,6 +265,7 @@ _TWINS = [
     ("argmax_f32", "no twin: f32 logits"),
     ("moe_router_f32", "no twin: (router_w, x, logits, E, h, T)"),
     ("moe_route_topk", "forward.rs:2420-2448 on the device: (logits, logits_f16, E, k, renorm, T, out_idx, out_w)"),
+    ("moe_route_scored", "no twin: (logits, ld, E, k, score, renorm, T, out_idx, out_w), score = SCORE_SOFTMAX / SCORE_SIGMOID"),
     ("moe_layer_q4k", "forward.rs:1644-1679 as one call: (router_w, gate, up, down, x, residual, out, idx_out, w_out, "
                       "scratch, scratch_bytes, T, h, ff, E, k, renorm)"),
     ("moe_experts_q4k", "no twin: (gate, up, down, x_slots, slot_expert, y_slots, act_scratch, n_slots, h, ff, n_experts)"),
