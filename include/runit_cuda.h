@@ -466,6 +466,61 @@ size_t  runit_ffn_q4k_bf16_scratch_bytes(uint32_t T, uint32_t h, uint32_t ff);
 int32_t runit_ffn_q4k_bf16(runit_ctx_t*, const void* w_gate, const void* w_up, const void* w_down, const void* x, const void* gamma,
                            float eps, const void* residual, void* out, void* scratch, size_t scratch_bytes, uint32_t T, uint32_t h,
                            uint32_t ff);
+/* A portion of a sequence through the batched pass: tokens at positions start_pos .. start_pos + n - 1 on top of the
+ * start_pos cached ones (one token runs as a recorded decode step).  want: places inside the portion whose logits are
+ * returned, logits: host, f32 [n_want][vocab] in the order of want.  Layered decoders only (RUNIT_ERR_UNSUPPORTED else);
+ * start_pos must not exceed what the cache holds, a smaller one drops what comes after it. */
+int32_t runit_model_forward(runit_model_t* model, const int32_t* tokens, uint32_t n, uint32_t start_pos, const uint32_t* want,
+                            uint32_t n_want, float* logits);
+
+/* ── decoders described layer by layer (no twin), weights in bf16 ──
+ * Every matrix is row-major [rows][pad8(columns)] bf16 with zero padding; norms and router are f32.  Linear maps W x.
+ * Residual stream, norms, scores, softmax, router and angles are f32.  Pre-norm layers:
+ *   x += mixer(norm1(x));  x += ff(norm2(x));  norm(x) = x / sqrt(mean(x^2) + eps) * gain, one gain for all coordinates.
+ * exact = 0: activations and cache bf16 with f32 accumulation (batched passes on the tensor cores); exact = 1: activations
+ * and cache f32 throughout.  The step, the generate and sampling loops, prefill and forward are those of any runit_model_t. */
+enum { RUNIT_FF_NONE = 0, RUNIT_FF_DENSE = 1, RUNIT_FF_MOE = 2 };
+enum { RUNIT_ACT_SILU_GLU = 0,    /* rows 2i and 2i+1 of the up matrix are gate and up of unit i: silu(g) * u */
+       RUNIT_ACT_RELU2 = 1 };     /* max(u, 0)^2 */
+typedef struct {
+    /* latent attention: q rows [heads][dim | rot_dim]; latent of kv_rank values and a rotated key part of rot_dim values per
+     * position, in the cache of this layer (kv_from < 0) or of the earlier layer kv_from.  Rotation: pairs (2i, 2i+1), angle
+     * position * rot_base^(-2i/rot_dim). */
+    int32_t heads, dim, rot_dim, vdim, kv_rank, kv_from;
+    float   scale, rot_base;
+    /* feed-forward: ff units (per expert for RUNIT_FF_MOE); routing weights are the scores of the top_k largest of n_experts,
+     * and multiply an expert's input; a shared block of shared_ff units (0 = none) runs for every token, its output times the
+     * sigmoid of its own gate row */
+    int32_t ff_kind, ff_act, ff, n_experts, top_k, score, renorm, shared_ff;
+    const void* norm1;        /* f32 [1] */
+    const void* norm2;        /* f32 [1]; NULL without feed-forward */
+    const void* w_q;          /* [heads*(dim+rot_dim) (+ kv_rank+rot_dim when the layer owns its latent)][width] */
+    const void* kv_norm;      /* f32 [kv_rank]; NULL when kv_from >= 0 */
+    const void* w_ukv;        /* [heads*dim + heads*vdim][kv_rank]: keys of all heads, then values */
+    const void* w_o;          /* [width][heads*vdim] */
+    const void* ff_up;        /* [ff (2 ff for a gated block)][width], experts stacked */
+    const void* ff_down;      /* [width][ff], experts stacked */
+    const void* router;       /* f32 [n_experts (+ 1 gate row of the shared block)][width], no padding */
+    const void* shared_up;    /* [shared_ff (2 shared_ff)][width] */
+    const void* shared_down;  /* [width][shared_ff] */
+} runit_layer_desc;
+typedef struct {
+    int32_t n_layers, width, vocab, max_seq, exact;
+    float   eps;
+} runit_layered_cfg;
+typedef struct {
+    const void* embed;        /* [vocab][width] */
+    const void* embed_norm;   /* f32 [1] */
+    const void* final_norm;   /* f32 [1] */
+    const void* head;         /* [vocab][width] */
+} runit_layered_weights;
+/* Device pointers; the model keeps them, the caller keeps the memory alive. */
+int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cfg, const runit_layer_desc* layers,
+                                   const runit_layered_weights* weights, runit_model_t** out);
+/* Device pointer, f32 [n][width]: the residual stream of the last portion's tokens after its last layer; and the number of
+ * layers a portion runs (tests bring a model up layer by layer): n_layers < 0 restores all of them. */
+void*   runit_model_residual(runit_model_t* model);
+int32_t runit_model_set_depth(runit_model_t* model, int32_t n_layers);
 void*   runit_model_logits(runit_model_t* model);           /* device pointer, f32 [vocab], of the last step */
 uint64_t runit_model_launches_per_token(runit_model_t* model);
 

@@ -22,6 +22,7 @@ _CTYPES = {
     "const int32_t*": C.POINTER(C.c_int32), "const uint64_t*": C.POINTER(C.c_uint64), "const uint32_t*": C.POINTER(C.c_uint32),
     "const runit_model_cfg*": C.c_void_p, "const runit_sampler_cfg*": C.c_void_p, "const runit_model_weights*": C.c_void_p, "runit_model_t*": C.c_void_p,
     "int32_t*": C.POINTER(C.c_int32),
+    "const runit_layered_cfg*": C.c_void_p, "const runit_layer_desc*": C.c_void_p, "const runit_layered_weights*": C.c_void_p,
     "runit_model_t**": C.POINTER(C.c_void_p), "const void* const*": C.POINTER(C.c_void_p),
     "void* const*": C.POINTER(C.c_void_p), "float*": C.POINTER(C.c_float),
     "uint64_t*": C.POINTER(C.c_uint64), "runit_graph_t*": C.c_void_p, "runit_graph_t**": C.POINTER(C.c_void_p),
@@ -72,16 +73,18 @@ def prototypes():
     return _protos
 
 
-def load():
-    """dlopen the library and type every exported function; raise if anything is missing."""
+def load(path: Path | None = None):
+    """dlopen the library and type every exported function; raise if anything is missing.  `path`: a part of the library
+    (build.PARTS), which may lack functions outside of it; only the first call in a process chooses."""
     global _lib
     if _lib is not None:
         return _lib
-    if not LIB_PATH.exists():
+    path = LIB_PATH if path is None else Path(path)
+    if not path.exists():
         raise ImportError(
             "%s is missing: build it with `python -m runit_mac_b200.build` (needs nvcc). "
-            "There is no CPU or PyTorch fallback for this library." % LIB_PATH)
-    lib = C.CDLL(str(LIB_PATH), mode=C.RTLD_GLOBAL)
+            "There is no CPU or PyTorch fallback for this library." % path)
+    lib = C.CDLL(str(path), mode=C.RTLD_GLOBAL)
     missing = []
     for name, (ret, args) in prototypes().items():
         try:
@@ -91,7 +94,7 @@ def load():
             continue
         fn.restype = _ctype(ret)
         fn.argtypes = [_ctype(a) for a in args]
-    if missing:
+    if missing and path == LIB_PATH:
         raise ImportError("librunit_cuda.so does not export: %s" % ", ".join(missing))
     _lib = lib
     return lib

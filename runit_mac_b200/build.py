@@ -6,6 +6,7 @@ cross-compiles without a GPU.  Objects are rebuilt only when a source or header 
 """
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -18,6 +19,14 @@ CSRC = PKG / "csrc"
 INCLUDE = PKG.parent / "include"
 OBJ = PKG / "build"
 LIB = PKG / "librunit_cuda.so"
+
+# Parts of the library that are useful alone: {name: (shared library, sources)}.  A part exports the subset of the C ABI its
+# sources define; it exists so that serving one kind of model does not compile the kernels of all others.
+PARTS = {
+    "layered": (PKG / "librunit_layered.so",
+                ("ctx", "gemv_stream", "model_core", "layered_model", "gemv_bf16", "gemm_bf16", "latent_attention", "moe_route",
+                 "moe_permute", "sampler")),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -38,11 +47,30 @@ def _newest_header() -> float:
     return max(h.stat().st_mtime for h in hs)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def _fresh(lib: Path, srcs) -> bool:
+    """The library exists and is newer than everything it is made from."""
+    return lib.exists() and lib.stat().st_mtime >= max([_newest_header()] + [s.stat().st_mtime for s in srcs])
+
+
+def ensure(part: str) -> Path:
+    """A library that holds `part`: the full one when it is built and current, else the part's own, compiled on demand."""
+    if _fresh(LIB, CSRC.glob("*.cu")):
+        return LIB
+    lib, names = PARTS[part]
+    if not _fresh(lib, [CSRC / (n + ".cu") for n in names]):
+        OBJ.mkdir(exist_ok=True)
+        with open(OBJ / ".lock", "w") as lock:      # one builder at a time
+            fcntl.flock(lock, fcntl.LOCK_EX)
+            build(part=part)
+    return lib
+
+
+def build(force: bool = False, verbose: bool = False, part: str | None = None) -> Path:
     nvcc = _nvcc()
     OBJ.mkdir(exist_ok=True)
     hdr = _newest_header()
-    srcs = sorted(CSRC.glob("*.cu"))
+    out, names = PARTS[part] if part else (LIB, None)
+    srcs = [CSRC / (n + ".cu") for n in names] if names else sorted(CSRC.glob("*.cu"))
     todo = []
     for s in srcs:
         o = OBJ / (s.stem + ".o")
@@ -62,12 +90,14 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     with ThreadPoolExecutor(max_workers=min(8, max(1, len(todo)))) as ex:
         list(ex.map(compile_one, todo))
     objs = [OBJ / (s.stem + ".o") for s in srcs]
-    if todo or not LIB.exists():
-        cmd = [nvcc, "-shared", "-o", str(LIB), *map(str, objs), "-lcudart"]
+    if todo or not out.exists() or out.stat().st_mtime < max(o.stat().st_mtime for o in objs):
+        tmp = out.with_name("%s.%d.tmp" % (out.name, os.getpid()))
+        cmd = [nvcc, "-shared", "-Xlinker", "-z,defs", "-o", str(tmp), *map(str, objs), "-lcudart"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError("link failed:\n%s\n%s" % (r.stdout, r.stderr))
-    return LIB
+        os.replace(tmp, out)
+    return out
 
 
 if __name__ == "__main__":

@@ -1,0 +1,394 @@
+// One-token operators of decoders with bf16 weights: GEMV with the norm in front and the activation behind fused in, and the
+// row operators of a pass (embedding, norms with one gain for all coordinates).
+//
+// A warp owns 1, 2 or 4 weight rows (rows 2i and 2i+1 together for a gated block) and keeps eight 16-byte loads per lane in
+// flight; the first group of them does not depend on the previous kernel of the chain and is requested before the dependency
+// wait.  The input vector is staged in shared memory as f32; the norm's factor multiplies the dot product (the gain is one
+// number), so the vector is read once.  Sums are f32.
+#include "bf16_ops.cuh"
+#include "model_core.h"
+#include "tma.cuh"
+
+namespace runit {
+namespace gv {
+
+constexpr int kWarps = 8;
+constexpr int kLoads = 8;      // 16-byte loads per lane and group
+
+__device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
+// eight products of one 16-byte piece of a row with x (xa: elements 0..3, xb: 4..7)
+__device__ __forceinline__ float dot8(const uint4& w, const float4& xa, const float4& xb, float acc) {
+    acc = fmaf(bf_lo(w.x), xa.x, acc); acc = fmaf(bf_hi(w.x), xa.y, acc);
+    acc = fmaf(bf_lo(w.y), xa.z, acc); acc = fmaf(bf_hi(w.y), xa.w, acc);
+    acc = fmaf(bf_lo(w.z), xb.x, acc); acc = fmaf(bf_hi(w.z), xb.y, acc);
+    acc = fmaf(bf_lo(w.w), xb.z, acc); acc = fmaf(bf_hi(w.w), xb.w, acc);
+    return acc;
+}
+__device__ __forceinline__ float warp_add(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float silu_mul(float g, float u) { return g / (1.0f + expf(-g)) * u; }
+__device__ __forceinline__ float relu2(float v) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+}
+
+// x (K values) into shared memory as two planes of 16-byte pieces (elements 0..3 and 4..7 of every chunk of eight), zero
+// padded; returns the sum of squares of this thread's elements.
+__device__ __forceinline__ float stage_x(const float* x, uint32_t K, uint32_t nch, float4* xa, float4* xb) {
+    float sq = 0.f;
+    const bool vec = (K & 3u) == 0 && (reinterpret_cast<uintptr_t>(x) & 15u) == 0;
+    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        const uint32_t e = 4 * i;
+        if (vec) {
+            if (e < K) v = *reinterpret_cast<const float4*>(x + e);
+        } else {
+            if (e < K) v.x = x[e];
+            if (e + 1 < K) v.y = x[e + 1];
+            if (e + 2 < K) v.z = x[e + 2];
+            if (e + 3 < K) v.w = x[e + 3];
+        }
+        sq = fmaf(v.x, v.x, sq); sq = fmaf(v.y, v.y, sq); sq = fmaf(v.z, v.z, sq); sq = fmaf(v.w, v.w, sq);
+        ((i & 1u) ? xb : xa)[i >> 1] = v;
+    }
+    return sq;
+}
+
+struct Args {
+    const uint8_t* w;
+    uint32_t rows, K, ldw;
+    const float* x;
+    const float* gain;
+    float eps;
+    float* out;
+    const float* res;
+    int32_t* argmax;
+    unsigned long long* argmax_ctl;
+    uint32_t n_routed, slot_stride;
+    const int32_t* slot_expert;
+    const float* pre;
+    const uint8_t* w_extra;
+    uint32_t rows_extra;
+    const float* post_extra;
+};
+
+template <int EPI, int RPU, bool SLOTS>
+__global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
+    constexpr int U = kLoads / RPU;
+    extern __shared__ __align__(16) float4 smem4[];
+    __shared__ float part[kWarps];
+    __shared__ unsigned long long best_s[kWarps];
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t nch = (a.K + 7) / 8;
+    float4 *xa = smem4, *xb = smem4 + nch;
+    const uint32_t slot = SLOTS ? blockIdx.y : 0;
+    const bool extra = SLOTS && slot == a.n_routed;
+    const uint32_t rows = extra ? a.rows_extra : a.rows;
+    const uint32_t units = (rows + RPU - 1) / RPU;
+    const uint8_t* w = extra ? a.w_extra : a.w;
+    const size_t row_bytes = (size_t)a.ldw * 2;
+    uint32_t unit = blockIdx.x * kWarps + warp;
+    uint4 v[RPU][U];
+    auto load = [&](uint32_t u, uint32_t c0) {
+#pragma unroll
+        for (int r = 0; r < RPU; r++) {
+            const uint8_t* row = w + (size_t)(u * RPU + r) * row_bytes;
+#pragma unroll
+            for (int i = 0; i < U; i++) {
+                const uint32_t c = c0 + 32 * i + lane;
+                v[r][i] = (c < nch && u * RPU + r < rows) ? __ldg(reinterpret_cast<const uint4*>(row) + c) : make_uint4(0, 0, 0, 0);
+            }
+        }
+    };
+    const bool early = !SLOTS || extra;
+    if (early && unit < units) load(unit, 0);
+    grid_dependency_wait();
+    grid_launch_dependents();
+    float pre = 1.f, post = 1.f;
+    if (SLOTS) {
+        if (extra) {
+            if (a.post_extra) post = *a.post_extra;
+        } else {
+            const int32_t e = a.slot_expert[slot];
+            if (e < 0) return;
+            w += (size_t)e * a.rows * row_bytes;
+            if (a.pre) pre = a.pre[slot];
+        }
+    }
+    if (!early && unit < units) load(unit, 0);
+    float scale = stage_x(a.x, a.K, nch, xa, xb);
+    if (a.gain) {
+        scale = warp_add(scale);
+        if (lane == 0) part[warp] = scale;
+    }
+    __syncthreads();
+    scale = 1.f;
+    if (a.gain) {
+        float tot = 0.f;
+#pragma unroll
+        for (int i = 0; i < kWarps; i++) tot += part[i];
+        scale = rsqrtf(tot / (float)a.K + a.eps) * *a.gain;
+    }
+    unsigned long long best = 0;
+    bool first = true;
+    for (; unit < units; unit += gridDim.x * kWarps) {
+        float acc[RPU];
+#pragma unroll
+        for (int r = 0; r < RPU; r++) acc[r] = 0.f;
+        for (uint32_t c0 = 0; c0 < nch; c0 += 32 * U) {
+            if (!first) load(unit, c0);
+            first = false;
+#pragma unroll
+            for (int i = 0; i < U; i++) {
+                const uint32_t c = c0 + 32 * i + lane;
+                if (c < nch) {
+                    const float4 p = xa[c], q = xb[c];
+#pragma unroll
+                    for (int r = 0; r < RPU; r++) acc[r] = dot8(v[r][i], p, q, acc[r]);
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < RPU; r++) acc[r] = warp_add(acc[r]) * scale;
+        if (lane == 0) {
+            float* out = a.out + (size_t)slot * a.slot_stride;
+            if (EPI == EPI_SILU_GLU) {
+#pragma unroll
+                for (int r = 0; r + 1 < RPU; r += 2)
+                    if (unit * RPU + r + 1 < rows) out[(unit * RPU + r) / 2] = silu_mul(acc[r] * pre, acc[r + 1] * pre) * post;
+            } else {
+#pragma unroll
+                for (int r = 0; r < RPU; r++) {
+                    const uint32_t row = unit * RPU + r;
+                    if (row >= rows) continue;
+                    float o;
+                    if (EPI == EPI_RELU2) o = relu2(acc[r] * pre) * post;
+                    else o = acc[r] + (a.res ? a.res[row] : 0.f);
+                    out[row] = o;
+                    if (EPI == EPI_F32 && a.argmax) {
+                        uint32_t b = __float_as_uint(o);
+                        b = (b & 0x80000000u) ? ~b : (b | 0x80000000u);
+                        const unsigned long long key = ((unsigned long long)b << 32) | (0xFFFFFFFFu - row);
+                        best = key > best ? key : best;
+                    }
+                }
+            }
+        }
+    }
+    if (EPI == EPI_F32 && a.argmax) {
+        if (lane == 0) best_s[warp] = best;
+        __syncthreads();
+        if (threadIdx.x == 0) {
+#pragma unroll
+            for (int i = 1; i < kWarps; i++) best = best_s[i] > best ? best_s[i] : best;
+            atomicMax(a.argmax_ctl, best);
+            __threadfence();
+            if (atomicAdd(a.argmax_ctl + 1, 1ull) == gridDim.x - 1) {
+                const unsigned long long k = atomicExch(a.argmax_ctl, 0ull);
+                a.argmax_ctl[1] = 0;
+                *a.argmax = (int32_t)(0xFFFFFFFFu - (uint32_t)k);
+            }
+        }
+    }
+}
+
+struct SumArgs {
+    const uint8_t* w;
+    uint32_t rows, K, ldw, n_routed, x_stride;
+    const int32_t* slot_expert;
+    const uint8_t* w_extra;
+    uint32_t K_extra, ldw_extra;
+    const float* x;
+    const float* res;
+    float* out;
+};
+
+// The inputs of all slots lie one after the other in shared memory, each padded to chunks of eight; a lane walks the chunks of
+// all slots as one list, so the loads of small blocks are in flight together.
+template <int RPU>
+__global__ void __launch_bounds__(kWarps * 32) gemv_bf16_sum_kernel(const SumArgs a) {
+    constexpr int U = kLoads / RPU;
+    extern __shared__ __align__(16) float4 smem4[];
+    __shared__ const uint8_t* base_s[33];
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t chs = (a.K + 7) / 8, routed = a.n_routed * chs, chx = a.w_extra ? (a.K_extra + 7) / 8 : 0, total = routed + chx;
+    float4 *xa = smem4, *xb = smem4 + total;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    if (threadIdx.x < a.n_routed) {
+        const int32_t e = a.slot_expert ? a.slot_expert[threadIdx.x] : 0;
+        base_s[threadIdx.x] = e < 0 ? nullptr : a.w + (size_t)e * a.rows * a.ldw * 2;
+    }
+    for (uint32_t s = 0; s < a.n_routed; s++) stage_x(a.x + (size_t)s * a.x_stride, a.K, chs, xa + s * chs, xb + s * chs);
+    if (chx) stage_x(a.x + (size_t)a.n_routed * a.x_stride, a.K_extra, chx, xa + routed, xb + routed);
+    __syncthreads();
+    const uint32_t units = (a.rows + RPU - 1) / RPU;
+    for (uint32_t unit = blockIdx.x * kWarps + warp; unit < units; unit += gridDim.x * kWarps) {
+        float acc[RPU];
+#pragma unroll
+        for (int r = 0; r < RPU; r++) acc[r] = 0.f;
+        for (uint32_t c0 = 0; c0 < total; c0 += 32 * U) {
+            uint4 v[RPU][U];
+#pragma unroll
+            for (int i = 0; i < U; i++) {
+                const uint32_t c = c0 + 32 * i + lane;
+                const uint8_t* p = nullptr;
+                size_t pitch = 0;
+                if (c < routed) {
+                    const uint32_t s = c / chs;
+                    pitch = (size_t)a.ldw * 2;
+                    if (base_s[s]) p = base_s[s] + (size_t)(c - s * chs) * 16;
+                } else if (c < total) {
+                    pitch = (size_t)a.ldw_extra * 2;
+                    p = a.w_extra + (size_t)(c - routed) * 16;
+                }
+#pragma unroll
+                for (int r = 0; r < RPU; r++) {
+                    const uint32_t row = unit * RPU + r;
+                    v[r][i] = (p && row < a.rows) ? __ldg(reinterpret_cast<const uint4*>(p + row * pitch)) : make_uint4(0, 0, 0, 0);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < U; i++) {
+                const uint32_t c = c0 + 32 * i + lane;
+                if (c < total) {
+                    const float4 p = xa[c], q = xb[c];
+#pragma unroll
+                    for (int r = 0; r < RPU; r++) acc[r] = dot8(v[r][i], p, q, acc[r]);
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < RPU; r++) {
+            acc[r] = warp_add(acc[r]);
+            const uint32_t row = unit * RPU + r;
+            if (lane == 0 && row < a.rows) a.out[row] = (a.res ? a.res[row] : 0.f) + acc[r];
+        }
+    }
+}
+
+// ── rows ──
+// sum over the CTA (256 threads)
+__device__ __forceinline__ float block_sum(float s) {
+    __shared__ float part[8];
+    s = warp_add(s);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = s;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) tot += part[i];
+    return tot;
+}
+
+__global__ void __launch_bounds__(256) embed_norm_kernel(const __nv_bfloat16* __restrict__ emb, uint32_t ld, const int32_t* __restrict__ tokens,
+                                                          const int32_t* state, const int32_t* __restrict__ forced, uint32_t n_forced,
+                                                          uint32_t vocab, const float* __restrict__ gain, float eps, float* __restrict__ x,
+                                                          uint32_t width) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const uint32_t t = blockIdx.x;
+    const int32_t tok = tokens ? tokens[t] : model_step_token(state, forced, n_forced, vocab);
+    const __nv_bfloat16* row = emb + (size_t)tok * ld;
+    float s = 0.f;
+    for (uint32_t i = threadIdx.x; i < width; i += 256) {
+        const float v = __bfloat162float(row[i]);
+        s = fmaf(v, v, s);
+    }
+    const float r = rsqrtf(block_sum(s) / (float)width + eps) * *gain;
+    for (uint32_t i = threadIdx.x; i < width; i += 256) x[(size_t)t * width + i] = __bfloat162float(row[i]) * r;
+}
+
+template <typename TY>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index,
+                                                         const float* __restrict__ gain, float eps, TY* __restrict__ y, uint32_t ldy,
+                                                         float* __restrict__ y2, uint32_t width) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const uint32_t t = blockIdx.x;
+    const float* row = x + (size_t)(row_index ? row_index[t] : (int32_t)t) * width;
+    float s = 0.f;
+    for (uint32_t i = threadIdx.x; i < width; i += 256) s = fmaf(row[i], row[i], s);
+    const float r = rsqrtf(block_sum(s) / (float)width + eps) * *gain;
+    for (uint32_t i = threadIdx.x; i < ldy; i += 256) {
+        const float v = i < width ? row[i] * r : 0.f;
+        if constexpr (sizeof(TY) == 2) y[(size_t)t * ldy + i] = __float2bfloat16_rn(v);
+        else y[(size_t)t * ldy + i] = v;
+        if (y2 && i < width) y2[(size_t)t * width + i] = v;
+    }
+}
+
+__global__ void sigmoid_column_kernel(const float* __restrict__ logits, uint32_t ld, uint32_t col, float* __restrict__ out, uint32_t T) {
+    const uint32_t t = blockIdx.x * blockDim.x + threadIdx.x;
+    if (t < T) out[t] = 1.0f / (1.0f + expf(-logits[(size_t)t * ld + col]));
+}
+
+template <int EPI, int RPU, bool SLOTS>
+static int32_t launch(runit_ctx* ctx, const char* name, const Args& a, uint32_t max_rows, uint32_t slots) {
+    const size_t smem = (size_t)((a.K + 7) / 8) * 32;
+    RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 1024, "%s: %u columns do not fit shared memory", name, a.K);
+    if (smem > 48 * 1024)
+        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, SLOTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * 8;
+    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, SLOTS>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
+    return runit_after_launch(ctx, name);
+}
+
+}  // namespace gv
+
+int32_t gemv_bf16(runit_ctx* ctx, const char* name, const GemvDesc& d) {
+    RUNIT_REQUIRE(ctx, d.w && d.x && d.out && d.rows > 0 && d.K > 0 && d.ldw % 8 == 0 && d.ldw >= d.K, "%s: bad argument", name);
+    gv::Args a{(const uint8_t*)d.w, d.rows, d.K, d.ldw, d.x, d.gain, d.eps, d.out, d.res, d.argmax, d.argmax_ctl, d.n_routed, d.slot_stride,
+               d.slot_expert, d.pre, (const uint8_t*)d.w_extra, d.rows_extra, d.post_extra};
+    const bool slots = d.slot_expert != nullptr;
+    const uint32_t n_slots = slots ? d.n_routed + (d.w_extra ? 1 : 0) : 1;
+    const uint32_t rows = slots && d.w_extra && d.rows_extra > d.rows ? d.rows_extra : d.rows;
+    const int rpu = d.K > 1024 ? 1 : (d.K > 512 ? 2 : 4);
+#define RUNIT_GV(E, R) (slots ? gv::launch<E, R, true>(ctx, name, a, rows, n_slots) : gv::launch<E, R, false>(ctx, name, a, rows, n_slots))
+    if (d.epi == EPI_SILU_GLU) return rpu == 4 ? RUNIT_GV(EPI_SILU_GLU, 4) : RUNIT_GV(EPI_SILU_GLU, 2);
+    if (d.epi == EPI_RELU2) return rpu == 4 ? RUNIT_GV(EPI_RELU2, 4) : (rpu == 2 ? RUNIT_GV(EPI_RELU2, 2) : RUNIT_GV(EPI_RELU2, 1));
+    return rpu == 4 ? RUNIT_GV(EPI_F32, 4) : (rpu == 2 ? RUNIT_GV(EPI_F32, 2) : RUNIT_GV(EPI_F32, 1));
+#undef RUNIT_GV
+}
+
+int32_t gemv_bf16_sum(runit_ctx* ctx, const char* name, const GemvSumDesc& d) {
+    RUNIT_REQUIRE(ctx, (d.w || d.n_routed == 0) && d.x && d.out && d.rows > 0 && d.n_routed <= 32 && (d.n_routed > 0 || d.w_extra),
+                  "%s: bad argument", name);
+    gv::SumArgs a{(const uint8_t*)d.w, d.rows, d.K, d.ldw, d.n_routed, d.x_stride, d.slot_expert, (const uint8_t*)d.w_extra, d.K_extra,
+                  d.ldw_extra, d.x, d.res, d.out};
+    const uint32_t total = d.n_routed * ((d.K + 7) / 8) + (d.w_extra ? (d.K_extra + 7) / 8 : 0);
+    const size_t smem = (size_t)total * 32;
+    RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 1024, "%s: the slots' inputs do not fit shared memory", name);
+    auto go = [&](auto kern, uint32_t rpu) -> int32_t {
+        if (smem > 48 * 1024) RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        const uint32_t units = (d.rows + rpu - 1) / rpu, want = (units + gv::kWarps - 1) / gv::kWarps, cap = (uint32_t)ctx->sm_count * 8;
+        runit_launch_chain_smem(ctx, kern, dim3(want < cap ? want : cap), dim3(gv::kWarps * 32), smem, a);
+        return runit_after_launch(ctx, name);
+    };
+    if (total > 128) return go(gv::gemv_bf16_sum_kernel<1>, 1);
+    return go(gv::gemv_bf16_sum_kernel<2>, 2);
+}
+
+int32_t embed_norm_rows(runit_ctx* ctx, const void* embed, uint32_t ld, const int32_t* tokens, const int32_t* state, const int32_t* forced,
+                        uint32_t n_forced, uint32_t vocab, const float* gain, float eps, float* x, uint32_t T, uint32_t width) {
+    runit_launch_chain(ctx, gv::embed_norm_kernel, dim3(T), dim3(256), (const __nv_bfloat16*)embed, ld, tokens, state, forced, n_forced, vocab,
+                       gain, eps, x, width);
+    return runit_after_launch(ctx, "embed_norm");
+}
+
+int32_t norm_rows(runit_ctx* ctx, const float* x, const int32_t* row_index, const float* gain, float eps, void* y, bool y_f32, uint32_t ldy,
+                  float* y2, uint32_t T, uint32_t width) {
+    if (y_f32) runit_launch_chain(ctx, gv::norm_rows_kernel<float>, dim3(T), dim3(256), x, row_index, gain, eps, (float*)y, ldy, y2, width);
+    else runit_launch_chain(ctx, gv::norm_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), x, row_index, gain, eps, (__nv_bfloat16*)y, ldy, y2, width);
+    return runit_after_launch(ctx, "norm_rows");
+}
+
+int32_t sigmoid_column(runit_ctx* ctx, const float* logits, uint32_t ld, uint32_t col, float* out, uint32_t T) {
+    gv::sigmoid_column_kernel<<<(T + 255) / 256, 256, 0, ctx->stream>>>(logits, ld, col, out, T);
+    return runit_after_launch(ctx, "sigmoid_column");
+}
+
+}  // namespace runit

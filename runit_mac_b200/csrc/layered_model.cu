@@ -1,0 +1,450 @@
+// Decoders described layer by layer (runit_layer_desc): latent attention with an optional latent borrowed from an earlier
+// layer, dense or mixture-of-experts feed-forward with a shared block, norms with one gain, bf16 weights.
+//
+// The step bookkeeping, command lists, generate loop and sampler are the shared core's (model_core.cu); routing and token
+// permutation are those of the other mixture-of-experts blocks (moe_route.cu, moe_permute.cu).  Here: how one decode step and
+// one batched portion are issued.
+//   Decode step, per layer: norm + q | latent projection; folded queries + rotation + cache row; split attention over the
+//   cached rows; merge + value projection; output projection + residual; then either norm + gate/up + activation and down +
+//   residual (dense), or norm + router + top-k, all selected blocks' up + activation, all their downs + residual.  Vectors are
+//   f32, weights bf16.
+//   Portion: the same with GEMMs; long portions in bf16 expand keys and values of the whole context per layer, the others use
+//   the folded arrangement.  A prompt is cut into portions of at most portion_cap tokens.
+#include <algorithm>
+#include <cmath>
+#include <new>
+#include <vector>
+
+#include "bf16_ops.cuh"
+#include "decode_ops.cuh"
+#include "model_core.h"
+#include "moe_internal.h"
+
+namespace runit {
+
+struct Layer {
+    runit_layer_desc d;
+    LatentDims lat;
+    uint32_t q_rows;           // rows of w_q
+    const float* freq;         // [rot_dim / 2]
+    void* cache;               // its own or the lending layer's
+    const void* w_uv;          // inside w_ukv
+    uint32_t gates;            // rows of the router past the experts
+};
+
+struct LayeredModel : runit_model {
+    runit_layered_cfg cfg;
+    runit_layered_weights w;
+    std::vector<Layer> layers;
+    bool exact = false;
+    uint32_t depth = 0;             // layers that run
+    uint32_t portion_cap = 0;       // tokens of one batched portion
+    uint32_t nsplit1 = 1;           // key splits of a decode step
+    unsigned long long* argmax_ctl = nullptr;
+    uint32_t* counter = nullptr;    // ticket word of the routing launch
+    // one token (f32)
+    float *x1 = nullptr, *xn1 = nullptr, *qkv1 = nullptr, *qeff1 = nullptr, *po1 = nullptr, *pml1 = nullptr, *ao1 = nullptr, *act1 = nullptr,
+          *rl1 = nullptr, *rw1 = nullptr, *gate1 = nullptr;
+    int32_t* idx1 = nullptr;
+    uint32_t act_stride = 0;
+    // portions (allocated on first use)
+    struct {
+        float *x = nullptr, *xf = nullptr, *qkv = nullptr, *qeff = nullptr, *po = nullptr, *pml = nullptr, *rl = nullptr, *rw = nullptr,
+              *gate = nullptr, *pre = nullptr, *y = nullptr, *logits = nullptr;
+        void *h = nullptr, *ao = nullptr, *act = nullptr, *kv = nullptr, *xperm = nullptr, *actp = nullptr;
+        int32_t *tokens = nullptr, *idx = nullptr, *want = nullptr;
+        MoePermutation perm{};
+        uint32_t rows_perm = 0, po_rows = 0;
+    } pf;
+    static constexpr uint32_t kWantRows = 64;       // rows of one head product
+
+    int32_t issue_step(bool with_logits, uint32_t n_forced, bool sampled) override;
+    int32_t prefill(const int32_t* tokens, uint32_t n, int32_t* next_token) override;
+    int32_t forward(const int32_t* tokens, uint32_t n, uint32_t start_pos, const uint32_t* want, uint32_t n_want, float* logits_host) override;
+    uint64_t launches_per_token() override;
+
+    int32_t alloc_portions();
+    int32_t portion(const int32_t* tokens, uint32_t T, uint32_t start);
+    int32_t attention_rows(const Layer& l, uint32_t T, uint32_t start);
+    int32_t ff_rows(const Layer& l, uint32_t T);
+    size_t es() const { return exact ? 4 : 2; }
+    uint32_t width() const { return (uint32_t)cfg.width; }
+    uint32_t ldw() const { return pad8(width()); }
+    // long portions in bf16 expand keys and values; in 32-bit and for short portions the folded form reads less
+    bool expands(const Layer& l, uint32_t T) const { return !exact && T >= 32 && latent_prefill_supported(l.lat); }
+};
+
+static uint32_t up_rows(const runit_layer_desc& d, uint32_t ff) { return d.ff_act == RUNIT_ACT_SILU_GLU ? 2 * ff : ff; }
+static int act_epi(const runit_layer_desc& d) { return d.ff_act == RUNIT_ACT_SILU_GLU ? EPI_SILU_GLU : EPI_RELU2; }
+
+int32_t LayeredModel::issue_step(bool with_logits, uint32_t n_forced, bool sampled) {
+    int32_t st;
+    const LatentPos pos{state + 1, 0};
+    const uint32_t wd = width();
+    if ((st = embed_norm_rows(ctx, w.embed, ldw(), nullptr, state, forced, n_forced, (uint32_t)vocab, (const float*)w.embed_norm, cfg.eps, x1, 1, wd)))
+        return st;
+    for (uint32_t i = 0; i < depth; i++) {
+        const Layer& l = layers[i];
+        const runit_layer_desc& d = l.d;
+        const uint32_t hv = l.lat.heads * l.lat.vdim, ldk = pad8(l.lat.kv_rank);
+        GemvDesc g;
+        g.w = d.w_q; g.rows = l.q_rows; g.K = wd; g.ldw = ldw(); g.x = x1; g.gain = (const float*)d.norm1; g.eps = cfg.eps; g.out = qkv1;
+        if ((st = gemv_bf16(ctx, "layer_qkv", g))) return st;
+        if ((st = latent_query(ctx, l.lat, exact, qkv1, 0, d.w_ukv, ldk, (const float*)d.kv_norm, l.freq, l.cache, qeff1, 1, pos))) return st;
+        if ((st = latent_attention(ctx, l.lat, exact, qeff1, l.cache, po1, pml1, nsplit1, 1, pos))) return st;
+        if ((st = latent_value(ctx, l.lat, po1, pml1, nsplit1, l.w_uv, ldk, ao1, true, 0, 1))) return st;
+        g = GemvDesc();
+        g.w = d.w_o; g.rows = wd; g.K = hv; g.ldw = pad8(hv); g.x = ao1; g.out = x1; g.res = x1;
+        if ((st = gemv_bf16(ctx, "layer_out", g))) return st;
+        if (d.ff_kind == RUNIT_FF_DENSE) {
+            g = GemvDesc();
+            g.w = d.ff_up; g.rows = up_rows(d, d.ff); g.K = wd; g.ldw = ldw(); g.x = x1; g.gain = (const float*)d.norm2; g.eps = cfg.eps;
+            g.out = act1; g.epi = act_epi(d);
+            if ((st = gemv_bf16(ctx, "layer_up", g))) return st;
+            g = GemvDesc();
+            g.w = d.ff_down; g.rows = wd; g.K = d.ff; g.ldw = pad8(d.ff); g.x = act1; g.out = x1; g.res = x1;
+            if ((st = gemv_bf16(ctx, "layer_down", g))) return st;
+        } else if (d.ff_kind == RUNIT_FF_MOE) {
+            const uint32_t E = d.n_experts, k = d.top_k;
+            if ((st = moe_route_gated(ctx, (const float*)d.router, x1, rl1, E + l.gates, E, wd, k, d.score, d.renorm, idx1, rw1, gate1, counter,
+                                      (const float*)d.norm2, cfg.eps, xn1)))
+                return st;
+            g = GemvDesc();
+            g.w = d.ff_up; g.rows = up_rows(d, d.ff); g.K = wd; g.ldw = ldw(); g.x = xn1; g.out = act1; g.epi = act_epi(d);
+            g.n_routed = k; g.slot_stride = act_stride; g.slot_expert = idx1; g.pre = rw1;
+            if (d.shared_ff) { g.w_extra = d.shared_up; g.rows_extra = up_rows(d, d.shared_ff); g.post_extra = gate1; }
+            if ((st = gemv_bf16(ctx, "layer_experts_up", g))) return st;
+            GemvSumDesc s;
+            s.w = d.ff_down; s.rows = wd; s.K = d.ff; s.ldw = pad8(d.ff); s.n_routed = k; s.x_stride = act_stride; s.slot_expert = idx1;
+            if (d.shared_ff) { s.w_extra = d.shared_down; s.K_extra = d.shared_ff; s.ldw_extra = pad8(d.shared_ff); }
+            s.x = act1; s.res = x1; s.out = x1;
+            if ((st = gemv_bf16_sum(ctx, "layer_experts_down", s))) return st;
+        }
+    }
+    if (with_logits) {
+        GemvDesc g;
+        g.w = w.head; g.rows = (uint32_t)vocab; g.K = wd; g.ldw = ldw(); g.x = x1; g.gain = (const float*)w.final_norm; g.eps = cfg.eps; g.out = logits;
+        if (!sampled) { g.argmax = state + 3; g.argmax_ctl = argmax_ctl; }
+        if ((st = gemv_bf16(ctx, "layer_head", g))) return st;
+        // the context of the draw: what has been generated so far, out_tokens[state[4] .. state[5])
+        if (sampled && (st = runit_sample_f32(ctx, logits, scores, (uint32_t)vocab, &sampler_cfg, out_tokens, state + 4, 0, 0, eos, sampler_n_eos, rng,
+                                              state + 3)))
+            return st;
+    }
+    model_issue_advance(this, with_logits);
+    return runit_after_launch(ctx, "advance");
+}
+
+int32_t LayeredModel::alloc_portions() {
+    if (pf.x) return RUNIT_OK;
+    int32_t st = RUNIT_OK;
+    auto A = [&](void** p, size_t b) {
+        if (st == RUNIT_OK && b) st = model_dev_alloc(this, p, b);
+        if (st == RUNIT_OK && b) cudaMemsetAsync(*p, 0, b, ctx->stream);       // padding stays finite
+    };
+    const uint32_t P = portion_cap, wd = width();
+    uint32_t q = 0, hv = 0, kvw = 0, ffd = 0, ffe = 0, k = 0, E = 0, R = 0, heads = 0, cp = 0, pitch = 0;
+    bool all_expand = true;
+    for (const Layer& l : layers) {
+        const runit_layer_desc& d = l.d;
+        q = std::max(q, l.q_rows);
+        hv = std::max(hv, pad8(l.lat.heads * l.lat.vdim));
+        kvw = std::max(kvw, pad8(l.lat.heads * (l.lat.dim + l.lat.vdim)));
+        heads = std::max(heads, l.lat.heads); cp = std::max(cp, l.lat.cp()); pitch = std::max(pitch, l.lat.pitch());
+        all_expand = all_expand && expands(l, 1u << 30);
+        if (d.ff_kind == RUNIT_FF_DENSE) ffd = std::max(ffd, pad8(d.ff));
+        if (d.ff_kind == RUNIT_FF_MOE) {
+            ffe = std::max(ffe, pad8(d.ff)); ffd = std::max(ffd, pad8(d.shared_ff));
+            k = std::max(k, (uint32_t)d.top_k); E = std::max(E, (uint32_t)d.n_experts); R = std::max(R, d.n_experts + l.gates);
+        }
+    }
+    q = (q + 1) & ~1u;
+    // rows of the folded arrangement: every portion in 32-bit or with sizes the expanded kernel does not take, else short ones
+    const uint32_t fold_T = all_expand ? std::min(P, 32u) : P;
+    pf.po_rows = fold_T * heads + 16 * (2 * ctx->sm_count + 64);
+    A((void**)&pf.tokens, (size_t)P * 4); A((void**)&pf.xf, (size_t)P * wd * 4); A((void**)&pf.qkv, (size_t)P * q * 4);
+    A((void**)&pf.qeff, (size_t)fold_T * heads * pitch * 4); A((void**)&pf.po, (size_t)pf.po_rows * cp * 4); A((void**)&pf.pml, (size_t)pf.po_rows * 8);
+    A(&pf.h, (size_t)P * ldw() * es()); A(&pf.ao, (size_t)P * hv * es()); A(&pf.act, (size_t)P * ffd * es());
+    if (!exact) A(&pf.kv, (size_t)max_seq * kvw * 2);
+    A((void**)&pf.logits, (size_t)kWantRows * vocab * 4); A((void**)&pf.want, (size_t)kWantRows * 4);
+    if (E) {
+        const size_t S = (size_t)P * k;
+        pf.rows_perm = ((uint32_t)((S + kMoeRowAlign - 1) / kMoeRowAlign) + E) * kMoeRowAlign;
+        const size_t tiles = S / 64 + E + 1;
+        A((void**)&pf.rl, (size_t)P * R * 4); A((void**)&pf.idx, S * 4); A((void**)&pf.rw, S * 4); A((void**)&pf.gate, (size_t)P * 4);
+        A((void**)&pf.pre, (size_t)pf.rows_perm * 4); A((void**)&pf.y, (size_t)pf.rows_perm * wd * 4);
+        A(&pf.xperm, (size_t)pf.rows_perm * ldw() * es()); A(&pf.actp, (size_t)pf.rows_perm * ffe * es());
+        A((void**)&pf.perm.counts, 1024); A((void**)&pf.perm.n_tok_tiles, 16); A((void**)&pf.perm.tile_expert, tiles * 4);
+        A((void**)&pf.perm.tile_nvalid, tiles * 4); A((void**)&pf.perm.tile_row0, tiles * 4); A((void**)&pf.perm.pos_of_slot, S * 4);
+    }
+    A((void**)&pf.x, (size_t)P * wd * 4);       // last: its pointer says that all of them are there
+    return st;
+}
+
+int32_t LayeredModel::attention_rows(const Layer& l, uint32_t T, uint32_t start) {
+    int32_t st;
+    const runit_layer_desc& d = l.d;
+    const uint32_t wd = width(), ldk = pad8(l.lat.kv_rank), hv = l.lat.heads * l.lat.vdim, ldh = pad8(hv), ldq = (l.q_rows + 1) & ~1u;
+    if ((st = norm_rows(ctx, pf.x, nullptr, (const float*)d.norm1, cfg.eps, pf.h, exact, ldw(), nullptr, T, wd))) return st;
+    GemmDesc g;
+    g.w = d.w_q; g.rows = l.q_rows; g.K = wd; g.ldw = ldw(); g.x = pf.h; g.ldx = ldw(); g.x_rows = portion_cap; g.T = T; g.out = pf.qkv; g.ldo = ldq;
+    if ((st = gemm_bf16(ctx, "rows_qkv", g, exact))) return st;
+    const LatentPos pos{nullptr, start};
+    if (expands(l, T)) {
+        if ((st = latent_rows(ctx, l.lat, false, pf.qkv, ldq, (const float*)d.kv_norm, l.freq, l.cache, T, pos))) return st;
+        const uint32_t kvw = l.lat.heads * (l.lat.dim + l.lat.vdim), S = start + T;
+        g = GemmDesc();
+        g.w = d.w_ukv; g.rows = kvw; g.K = l.lat.kv_rank; g.ldw = ldk; g.x = l.cache; g.ldx = l.lat.pitch(); g.x_rows = (uint32_t)max_seq; g.T = S;
+        g.out = pf.kv; g.ldo = pad8(kvw); g.epi = EPI_CAST;
+        if ((st = gemm_bf16(ctx, "rows_expand", g, false))) return st;
+        if ((st = latent_prefill(ctx, l.lat, pf.qkv, ldq, pf.kv, pad8(kvw), l.cache, pf.ao, ldh, T, start))) return st;
+    } else {
+        uint32_t ns = latent_splits(ctx, l.lat, exact, T);
+        while (ns > 1 && (uint64_t)ns * T * l.lat.heads > pf.po_rows) ns--;
+        if ((st = latent_query(ctx, l.lat, exact, pf.qkv, ldq, d.w_ukv, ldk, (const float*)d.kv_norm, l.freq, l.cache, pf.qeff, T, pos))) return st;
+        if ((st = latent_attention(ctx, l.lat, exact, pf.qeff, l.cache, pf.po, pf.pml, ns, T, pos))) return st;
+        if ((st = latent_value(ctx, l.lat, pf.po, pf.pml, ns, l.w_uv, ldk, pf.ao, exact, ldh, T))) return st;
+    }
+    g = GemmDesc();
+    g.w = d.w_o; g.rows = wd; g.K = hv; g.ldw = ldh; g.x = pf.ao; g.ldx = ldh; g.x_rows = portion_cap; g.T = T; g.out = pf.x; g.ldo = wd; g.epi = EPI_ADD;
+    return gemm_bf16(ctx, "rows_out", g, exact);
+}
+
+int32_t LayeredModel::ff_rows(const Layer& l, uint32_t T) {
+    const runit_layer_desc& d = l.d;
+    if (d.ff_kind == RUNIT_FF_NONE) return RUNIT_OK;
+    int32_t st;
+    const uint32_t wd = width();
+    const bool moe = d.ff_kind == RUNIT_FF_MOE;
+    if ((st = norm_rows(ctx, pf.x, nullptr, (const float*)d.norm2, cfg.eps, pf.h, exact, ldw(), moe ? pf.xf : nullptr, T, wd))) return st;
+    auto block = [&](const void* up, const void* down, uint32_t ff, const float* post) -> int32_t {
+        GemmDesc g;
+        g.w = up; g.rows = up_rows(d, ff); g.K = wd; g.ldw = ldw(); g.x = pf.h; g.ldx = ldw(); g.x_rows = portion_cap; g.T = T;
+        g.out = pf.act; g.ldo = pad8(ff); g.epi = act_epi(d); g.post = post;
+        if ((st = gemm_bf16(ctx, "rows_up", g, exact))) return st;
+        g = GemmDesc();
+        g.w = down; g.rows = wd; g.K = ff; g.ldw = pad8(ff); g.x = pf.act; g.ldx = pad8(ff); g.x_rows = portion_cap; g.T = T; g.out = pf.x; g.ldo = wd;
+        g.epi = EPI_ADD;
+        return gemm_bf16(ctx, "rows_down", g, exact);
+    };
+    if (!moe) return block(d.ff_up, d.ff_down, d.ff, nullptr);
+    const uint32_t E = d.n_experts, k = d.top_k, R = E + l.gates, S = T * k;
+    if ((st = moe_router(ctx, (const float*)d.router, pf.xf, pf.rl, R, wd, T))) return st;
+    if ((st = moe_topk_rows(ctx, pf.rl, 0, R, E, k, d.score, d.renorm, T, pf.idx, pf.rw))) return st;
+    if (d.shared_ff) {
+        if ((st = sigmoid_column(ctx, pf.rl, R, E, pf.gate, T))) return st;
+        if ((st = block(d.shared_up, d.shared_down, d.shared_ff, pf.gate))) return st;
+    }
+    const uint32_t tt = gemm_bf16_tile_tok(S / E, exact);
+    if ((st = moe_permute(ctx, pf.idx, S, E, tt, pf.perm))) return st;
+    if ((st = moe_gather_rows(ctx, pf.h, pf.perm.pos_of_slot, pf.xperm, S, (size_t)ldw() * es(), k))) return st;
+    if ((st = moe_gather_values(ctx, pf.rw, pf.perm.pos_of_slot, pf.pre, S))) return st;
+    GemmDesc g;
+    g.n_experts = E; g.T = S; g.x_rows = pf.rows_perm; g.tile_tok = tt; g.max_tiles = S / tt + E;
+    g.tile_expert = pf.perm.tile_expert; g.tile_nvalid = pf.perm.tile_nvalid; g.tile_row0 = pf.perm.tile_row0; g.n_tok_tiles = pf.perm.n_tok_tiles;
+    g.w = d.ff_up; g.rows = up_rows(d, d.ff); g.K = wd; g.ldw = ldw(); g.x = pf.xperm; g.ldx = ldw(); g.out = pf.actp; g.ldo = pad8(d.ff);
+    g.epi = act_epi(d); g.pre = pf.pre;
+    if ((st = gemm_bf16(ctx, "rows_experts_up", g, exact))) return st;
+    g.w = d.ff_down; g.rows = wd; g.K = d.ff; g.ldw = pad8(d.ff); g.x = pf.actp; g.ldx = pad8(d.ff); g.out = pf.y; g.ldo = wd; g.epi = EPI_F32; g.pre = nullptr;
+    if ((st = gemm_bf16(ctx, "rows_experts_down", g, exact))) return st;
+    return moe_grouped_combine(ctx, pf.y, pf.perm.pos_of_slot, nullptr, pf.x, pf.x, T, wd, k);
+}
+
+// One batched portion at positions start .. start + T - 1; the residual stream of its tokens is left in pf.x.
+int32_t LayeredModel::portion(const int32_t* tokens, uint32_t T, uint32_t start) {
+    int32_t st;
+    RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(pf.tokens, tokens, (size_t)T * 4, cudaMemcpyHostToDevice, ctx->stream));
+    if ((st = embed_norm_rows(ctx, w.embed, ldw(), pf.tokens, nullptr, nullptr, 0, (uint32_t)vocab, (const float*)w.embed_norm, cfg.eps, pf.x, T, width())))
+        return st;
+    for (uint32_t i = 0; i < depth; i++) {
+        if ((st = attention_rows(layers[i], T, start))) return st;
+        if ((st = ff_rows(layers[i], T))) return st;
+    }
+    cached = start + T;
+    return RUNIT_OK;
+}
+
+int32_t LayeredModel::prefill(const int32_t* tokens, uint32_t n, int32_t* next_token) {
+    int32_t st = alloc_portions();
+    if (st != RUNIT_OK) return st;
+    uint32_t last = 0;
+    for (uint32_t i = 0; i < n; i += portion_cap) {
+        last = std::min(portion_cap, n - i);
+        if ((st = portion(tokens + i, last, i))) return st;
+    }
+    // final norm + head on the last position only, through the decode path's launch
+    GemvDesc g;
+    g.w = w.head; g.rows = (uint32_t)vocab; g.K = width(); g.ldw = ldw(); g.x = pf.x + (size_t)(last - 1) * width(); g.gain = (const float*)w.final_norm;
+    g.eps = cfg.eps; g.out = logits; g.argmax = state + 3; g.argmax_ctl = argmax_ctl;
+    if ((st = gemv_bf16(ctx, "layer_head", g))) return st;
+    return model_finish_prefill(this, n, next_token);
+}
+
+int32_t LayeredModel::forward(const int32_t* tokens, uint32_t n, uint32_t start_pos, const uint32_t* want, uint32_t n_want, float* logits_host) {
+    int32_t st;
+    RUNIT_REQUIRE(ctx, start_pos <= cached, "model_forward: position %u, but the cache holds %u", start_pos, cached);
+    if (n == 1) {       // a decode step: the recorded command list
+        if ((st = runit_model_reset(this, tokens[0], (int32_t)start_pos))) return st;
+        RUNIT_CUDA_TRY(ctx, cudaMemsetAsync(forced, 0xFF, 4, ctx->stream));     // not forced by an earlier prompt
+        RUNIT_CUDA_TRY(ctx, cudaGraphLaunch(n_want ? graph_full : graph_prompt, ctx->stream));
+        for (uint32_t i = 0; i < n_want; i++)
+            RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(logits_host + (size_t)i * vocab, logits, (size_t)vocab * 4, cudaMemcpyDeviceToHost, ctx->stream));
+        cached = start_pos + 1;
+        return runit_flush(ctx);
+    }
+    if ((st = alloc_portions())) return st;
+    const uint32_t want_rows = portion_cap < kWantRows ? portion_cap : kWantRows;
+    for (uint32_t i = 0; i < n; i += portion_cap) {
+        const uint32_t T = std::min(portion_cap, n - i);
+        if ((st = portion(tokens + i, T, start_pos + i))) return st;
+        // the wanted places of this portion, a few rows at a time (their order in the output is the caller's)
+        std::vector<uint32_t> at;
+        for (uint32_t j = 0; j < n_want; j++)
+            if (want[j] >= i && want[j] < i + T) at.push_back(j);
+        for (size_t a = 0; a < at.size(); a += want_rows) {
+            const uint32_t m = (uint32_t)std::min<size_t>(want_rows, at.size() - a);
+            int32_t rows[kWantRows];
+            for (uint32_t j = 0; j < m; j++) rows[j] = (int32_t)(want[at[a + j]] - i);
+            RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(pf.want, rows, (size_t)m * 4, cudaMemcpyHostToDevice, ctx->stream));
+            if ((st = norm_rows(ctx, pf.x, pf.want, (const float*)w.final_norm, cfg.eps, pf.h, exact, ldw(), nullptr, m, width()))) return st;
+            GemmDesc g;
+            g.w = w.head; g.rows = (uint32_t)vocab; g.K = width(); g.ldw = ldw(); g.x = pf.h; g.ldx = ldw(); g.x_rows = portion_cap; g.T = m;
+            g.out = pf.logits; g.ldo = (uint32_t)vocab;
+            if ((st = gemm_bf16(ctx, "rows_head", g, exact))) return st;
+            for (uint32_t j = 0; j < m; j++)
+                RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(logits_host + (size_t)at[a + j] * vocab, pf.logits + (size_t)j * vocab, (size_t)vocab * 4,
+                                                    cudaMemcpyDeviceToHost, ctx->stream));
+            if ((st = runit_flush(ctx))) return st;
+        }
+    }
+    return runit_flush(ctx);
+}
+
+uint64_t LayeredModel::launches_per_token() {
+    uint64_t n = 1 + 2;      // embed + norm; head with its norm and the argmax, advance
+    for (uint32_t i = 0; i < depth; i++) n += 5 + (layers[i].d.ff_kind == RUNIT_FF_MOE ? 3 : (layers[i].d.ff_kind == RUNIT_FF_DENSE ? 2 : 0));
+    return n;
+}
+
+static int32_t check_layer(runit_ctx* ctx, const runit_layered_cfg& c, const runit_layer_desc* all, int32_t i) {
+    const runit_layer_desc& d = all[i];
+    RUNIT_REQUIRE(ctx, d.heads > 0 && d.dim > 0 && d.rot_dim > 0 && d.rot_dim % 2 == 0 && d.vdim > 0 && d.kv_rank > 0 && d.kv_rank <= 1024,
+                  "model_create_layered: layer %d: bad attention sizes (rot_dim even, kv_rank <= 1024)", i);
+    RUNIT_REQUIRE(ctx, d.rot_base > 0.f && d.norm1 && d.w_q && d.w_ukv && d.w_o, "model_create_layered: layer %d: null pointer", i);
+    if (d.kv_from >= 0) {
+        RUNIT_REQUIRE(ctx, d.kv_from < i && all[d.kv_from].kv_from < 0, "model_create_layered: layer %d borrows from layer %d, which has no latent of its own before it", i, d.kv_from);
+        const runit_layer_desc& s = all[d.kv_from];
+        RUNIT_REQUIRE(ctx, s.kv_rank == d.kv_rank && s.rot_dim == d.rot_dim && s.rot_base == d.rot_base,
+                      "model_create_layered: layer %d and the layer it borrows from differ in latent size or rotation", i);
+    } else {
+        RUNIT_REQUIRE(ctx, d.kv_norm, "model_create_layered: layer %d: null latent norm", i);
+    }
+    if (d.ff_kind == RUNIT_FF_NONE) return RUNIT_OK;
+    RUNIT_REQUIRE(ctx, d.ff_kind == RUNIT_FF_DENSE || d.ff_kind == RUNIT_FF_MOE, "model_create_layered: layer %d: unknown feed-forward kind %d", i, d.ff_kind);
+    RUNIT_REQUIRE(ctx, d.ff_act == RUNIT_ACT_SILU_GLU || d.ff_act == RUNIT_ACT_RELU2, "model_create_layered: layer %d: unknown activation %d", i, d.ff_act);
+    RUNIT_REQUIRE(ctx, d.ff > 0 && d.norm2 && d.ff_up && d.ff_down, "model_create_layered: layer %d: bad feed-forward", i);
+    if (d.ff_kind == RUNIT_FF_DENSE) return RUNIT_OK;
+    RUNIT_REQUIRE(ctx, d.n_experts > 0 && d.n_experts <= 256 && d.top_k > 0 && d.top_k <= d.n_experts && d.top_k <= 32 && d.router,
+                  "model_create_layered: layer %d: bad experts (at most 256, top_k at most 32)", i);
+    RUNIT_REQUIRE(ctx, d.score == RUNIT_SCORE_SOFTMAX || d.score == RUNIT_SCORE_SIGMOID, "model_create_layered: layer %d: unknown scoring function", i);
+    RUNIT_REQUIRE(ctx, d.shared_ff == 0 || (d.shared_ff > 0 && d.shared_up && d.shared_down), "model_create_layered: layer %d: bad shared block", i);
+    (void)c;
+    return RUNIT_OK;
+}
+
+}  // namespace runit
+
+using namespace runit;
+
+extern "C" {
+
+int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cfg, const runit_layer_desc* layers,
+                                   const runit_layered_weights* weights, runit_model_t** out) {
+    if (!ctx || !out) return RUNIT_ERR_BAD_ARG;
+    *out = nullptr;
+    RUNIT_REQUIRE(ctx, cfg && layers && weights && weights->embed && weights->embed_norm && weights->final_norm && weights->head,
+                  "model_create_layered: null configuration or weights");
+    const runit_layered_cfg& c = *cfg;
+    RUNIT_REQUIRE(ctx, c.n_layers > 0 && c.n_layers <= 1024 && c.width > 0 && c.width <= 12000 && c.vocab > 0 && c.max_seq > 0,
+                  "model_create_layered: bad width, depth, vocabulary or length");
+    int32_t st;
+    for (int32_t i = 0; i < c.n_layers; i++)
+        if ((st = check_layer(ctx, c, layers, i)) != RUNIT_OK) return st;
+    LayeredModel* m = new (std::nothrow) LayeredModel();
+    if (!m) return RUNIT_ERR_ALLOC;
+    m->ctx = ctx;
+    m->cfg = c;
+    m->w = *weights;
+    m->vocab = c.vocab;
+    m->max_seq = c.max_seq;
+    m->exact = c.exact != 0;
+    m->depth = (uint32_t)c.n_layers;
+    m->portion_cap = std::min<uint32_t>((uint32_t)c.max_seq, m->exact ? 256u : 2048u);
+    st = model_alloc_common(m);
+    auto A = [&](void** p, size_t b) {
+        if (st == RUNIT_OK) st = model_dev_alloc(m, p, b);
+        if (st == RUNIT_OK) cudaMemsetAsync(*p, 0, b, ctx->stream);
+    };
+    size_t q = 0, qe = 0, po = 0, hv = 0, rows = 0, act = 0, routers = 0;
+    uint32_t splits = 1;
+    for (int32_t i = 0; i < c.n_layers && st == RUNIT_OK; i++) {
+        Layer l{};
+        l.d = layers[i];
+        const runit_layer_desc& d = l.d;
+        l.lat = LatentDims{(uint32_t)d.heads, (uint32_t)d.dim, (uint32_t)d.rot_dim, (uint32_t)d.vdim, (uint32_t)d.kv_rank, d.scale, c.eps};
+        const bool own = d.kv_from < 0;
+        l.q_rows = l.lat.q_width() + (own ? d.kv_rank + d.rot_dim : 0);
+        l.gates = d.ff_kind == RUNIT_FF_MOE && d.shared_ff ? 1 : 0;
+        l.w_uv = (const uint8_t*)d.w_ukv + (size_t)d.heads * d.dim * pad8(d.kv_rank) * 2;
+        if (own) A(&l.cache, (size_t)c.max_seq * l.lat.pitch() * m->es());
+        else l.cache = m->layers[d.kv_from].cache;
+        std::vector<float> f(d.rot_dim / 2);
+        for (int32_t j = 0; j < d.rot_dim / 2; j++) f[j] = (float)std::pow((double)d.rot_base, -2.0 * j / d.rot_dim);
+        A((void**)&l.freq, f.size() * 4);
+        if (st == RUNIT_OK) {
+            cudaMemcpyAsync((void*)l.freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice, ctx->stream);
+            cudaStreamSynchronize(ctx->stream);      // f lives in this iteration
+        }
+        splits = std::max(splits, latent_splits(ctx, l.lat, m->exact, 1));
+        q = std::max<size_t>(q, l.q_rows);
+        qe = std::max<size_t>(qe, (size_t)d.heads * l.lat.pitch());
+        po = std::max<size_t>(po, (size_t)d.heads * l.lat.cp());
+        hv = std::max<size_t>(hv, (size_t)d.heads * d.vdim);
+        rows = std::max<size_t>(rows, d.heads);
+        if (d.ff_kind == RUNIT_FF_DENSE) act = std::max<size_t>(act, d.ff);
+        if (d.ff_kind == RUNIT_FF_MOE) {
+            const uint32_t stride = pad8((uint32_t)std::max(d.ff, d.shared_ff));
+            m->act_stride = std::max(m->act_stride, stride);
+            act = std::max<size_t>(act, (size_t)m->act_stride * 34);
+            routers = std::max<size_t>(routers, d.n_experts + l.gates);
+        }
+        m->layers.push_back(l);
+    }
+    m->nsplit1 = splits;
+    A((void**)&m->x1, (size_t)c.width * 4); A((void**)&m->xn1, (size_t)c.width * 4); A((void**)&m->qkv1, q * 4); A((void**)&m->qeff1, qe * 4);
+    A((void**)&m->po1, po * splits * 4); A((void**)&m->pml1, rows * splits * 8); A((void**)&m->ao1, hv * 4); A((void**)&m->act1, (act + 8) * 4);
+    A((void**)&m->rl1, (routers + 1) * 4); A((void**)&m->rw1, 128); A((void**)&m->gate1, 16); A((void**)&m->idx1, 128); A((void**)&m->counter, 16);
+    A((void**)&m->argmax_ctl, 16);
+    if (st == RUNIT_OK) st = model_record(m);
+    if (st != RUNIT_OK) {
+        runit_model_destroy(m);
+        return st;
+    }
+    *out = m;
+    return RUNIT_OK;
+}
+
+void* runit_model_residual(runit_model_t* model) {
+    LayeredModel* m = dynamic_cast<LayeredModel*>(model);
+    return m ? (void*)m->pf.x : nullptr;
+}
+
+int32_t runit_model_set_depth(runit_model_t* model, int32_t n_layers) {
+    if (!model) return RUNIT_ERR_BAD_ARG;
+    LayeredModel* m = dynamic_cast<LayeredModel*>(model);
+    RUNIT_REQUIRE(model->ctx, m && n_layers <= m->cfg.n_layers, "model_set_depth: not a layered decoder, or more layers than it has");
+    m->depth = n_layers < 0 ? (uint32_t)m->cfg.n_layers : (uint32_t)n_layers;
+    return RUNIT_OK;
+}
+
+}  // extern "C"

@@ -119,6 +119,7 @@ __global__ void prefill_finish_kernel(int32_t* state, int32_t n) {
 
 int32_t model_finish_prefill(runit_model* m, uint32_t n, int32_t* next_token) {
     runit_ctx* ctx = m->ctx;
+    m->cached = n;
     prefill_finish_kernel<<<1, 32, 0, ctx->stream>>>(m->state, (int32_t)n);
     int32_t st = runit_after_launch(ctx, "prefill_finish");
     if (st != RUNIT_OK) return st;
@@ -191,6 +192,7 @@ int32_t runit_model_forward_greedy(runit_model_t* m, int32_t token_id, int32_t p
     RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(&tok, m->state, 4, cudaMemcpyDeviceToHost, ctx->stream));
     st = runit_flush(ctx);
     if (st != RUNIT_OK) return st;
+    m->cached = (uint32_t)pos + 1;
     if (next_token) *next_token = tok;
     return RUNIT_OK;
 }
@@ -264,6 +266,7 @@ static int32_t generate_impl(runit_model_t* m, const int32_t* prompt, uint32_t n
         // the flush below reports it
         if (ctx->h_status && *reinterpret_cast<volatile int32_t*>(ctx->h_status) != 0) break;
     }
+    m->cached = (uint32_t)start_pos + n_steps;
     RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(out_tokens, m->out_tokens, (size_t)n_steps * 4, cudaMemcpyDeviceToHost, ctx->stream));
     return runit_flush(ctx);
 }

@@ -24,6 +24,7 @@ struct runit_model {
     float* scores = nullptr;                 // [vocab]
     int32_t* eos = nullptr;                  // [16]
     unsigned long long* rng = nullptr;
+    uint32_t cached = 0;                     // positions the cache holds
     std::vector<void*> owned;
 
     virtual ~runit_model() {}

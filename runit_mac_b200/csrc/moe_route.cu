@@ -500,6 +500,8 @@ int32_t moe_route_fused(runit_ctx* ctx, const float* w, const float* x, float* l
 int32_t moe_route_gated(runit_ctx* ctx, const float* w, const float* x, float* logits, uint32_t R, uint32_t E, uint32_t K, uint32_t k,
                         int32_t score, int32_t renorm, int32_t* idx, float* wts, float* gates, uint32_t* counter, const float* gain,
                         float eps, float* xn_out) {
+    if ((size_t)K * 4 > 40 * 1024)
+        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(route_gated_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(K * 4)));
     runit_launch_chain_smem(ctx, route_gated_kernel, dim3((R + 7) / 8), dim3(256), (size_t)K * 4, w, x, logits, R, E, K, k, (int)score,
                             (int)renorm, idx, wts, gates, counter, gain, eps, xn_out);
     return runit_after_launch(ctx, "moe_route_gated");

@@ -369,6 +369,26 @@ class Model:
         self.ctx._check(self.ctx.lib.runit_model_prefill(self.handle, tokens.ctypes.data_as(C.POINTER(C.c_int32)), len(tokens), C.byref(nxt)))
         return nxt.value
 
+    def generate(self, prompt, n: int) -> np.ndarray:
+        """n greedy tokens after the prompt: one batched pass over it, then recorded decode steps."""
+        if n <= 0:
+            return np.empty(0, np.int32)
+        first = self.prefill(prompt)
+        if n == 1:
+            return np.array([first], np.int32)
+        return np.concatenate([[first], self.generate_greedy([first], n - 2, len(prompt))]).astype(np.int32)
+
+    def forward(self, tokens, start_pos: int, want=()) -> np.ndarray:
+        """A portion of a sequence at positions start_pos ..; logits [len(want)][vocab] of the wanted places (layered
+        decoders only)."""
+        tokens = np.ascontiguousarray(tokens, np.int32)
+        want = np.ascontiguousarray(np.asarray(want, np.uint32))
+        out = np.empty((len(want), self.cfg.vocab), np.float32)
+        self.ctx._check(self.ctx.lib.runit_model_forward(
+            self.handle, tokens.ctypes.data_as(C.POINTER(C.c_int32)), len(tokens), start_pos, want.ctypes.data_as(C.POINTER(C.c_uint32)),
+            len(want), out.ctypes.data_as(C.POINTER(C.c_float))))
+        return out
+
     def logits(self) -> np.ndarray:
         out = np.empty(self.cfg.vocab, np.float32)
         p = self.ctx.lib.runit_model_logits(self.handle)
@@ -384,6 +404,54 @@ class Model:
         if self.handle:
             self.ctx.lib.runit_model_destroy(self.handle)
             self.handle = None
+
+
+FF_NONE, FF_DENSE, FF_MOE = 0, 1, 2
+ACT_SILU_GLU, ACT_RELU2 = 0, 1
+
+
+class LayerDesc(C.Structure):
+    """runit_layer_desc: mixer and feed-forward of one layer, sizes, constants and device pointers."""
+    _fields_ = ([(n, C.c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "kv_from")] +
+                [(n, C.c_float) for n in ("scale", "rot_base")] +
+                [(n, C.c_int32) for n in ("ff_kind", "ff_act", "ff", "n_experts", "top_k", "score", "renorm", "shared_ff")] +
+                [(n, C.c_void_p) for n in ("norm1", "norm2", "w_q", "kv_norm", "w_ukv", "w_o", "ff_up", "ff_down", "router", "shared_up",
+                                           "shared_down")])
+
+
+class LayeredCfg(C.Structure):
+    """runit_layered_cfg"""
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "width", "vocab", "max_seq", "exact")] + [("eps", C.c_float)]
+
+
+class LayeredWeights(C.Structure):
+    """runit_layered_weights"""
+    _fields_ = [(n, C.c_void_p) for n in ("embed", "embed_norm", "final_norm", "head")]
+
+
+class LayeredModel(Model):
+    """Decoder described layer by layer (bf16 weights).  The step, prefill, generation and sampling are those of Model."""
+
+    def __init__(self, ctx: Context, cfg: LayeredCfg, layers, weights: dict, keep=()):
+        """layers: LayerDesc list; weights: embed, embed_norm, final_norm, head; keep: owners of the memory behind the
+        pointers."""
+        self.ctx, self.cfg, self._keep = ctx, cfg, (layers, weights, keep)
+        arr = (LayerDesc * len(layers))(*layers)
+        w = LayeredWeights(**{k: _ptr(v) for k, v in weights.items()})
+        h = C.c_void_p()
+        ctx._check(ctx.lib.runit_model_create_layered(ctx.handle, C.byref(cfg), arr, C.byref(w), C.byref(h)))
+        self.handle = h
+
+    def set_depth(self, n_layers: int):
+        """Portions run the first n_layers layers only (-1: all); for bringing a model up layer by layer."""
+        self.ctx._check(self.ctx.lib.runit_model_set_depth(self.handle, n_layers))
+
+    def residual(self, n: int) -> np.ndarray:
+        """Residual stream [n][width] of the last portion's tokens."""
+        out = np.empty((n, self.cfg.width), np.float32)
+        self.ctx._check(self.ctx.lib.runit_memcpy_d2h(self.ctx.handle, out.ctypes.data, self.ctx.lib.runit_model_residual(self.handle), out.nbytes))
+        self.ctx.flush()
+        return out
 
 
 def moe_scratch_bytes(ctx: Context, T: int, h: int, ff: int, E: int, k: int) -> int:
@@ -434,5 +502,6 @@ def moe_layer_q4k_host(ctx: Context, router, gate, up, down, x, *, h, ff, E, top
             w.download(np.float32, T * top_k).reshape(T, top_k))
 
 
-__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
+__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc",
+           "FF_NONE", "FF_DENSE", "FF_MOE", "ACT_SILU_GLU", "ACT_RELU2", "SCORE_SOFTMAX", "SCORE_SIGMOID", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
            "FMT_Q8_0", "FMT_Q4_0", "FMT_Q4K", "FMT_Q5_0", "FMT_Q5K", "FMT_Q6K"] + [n for n, _ in _TWINS]
