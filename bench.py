@@ -606,6 +606,213 @@ def run_extras(R, ctx, torch, dist, stream, rank, world, args, decode_only=False
     return out
 
 
+# ───────────────────────── layered decoders (bf16 weights, latent attention) ─────────────────────────
+# (width, layers, heads, kv_rank, experts, top, expert ff, dense ff, vocab); heads of 128 + 64 rotated, values of 128
+LAYERED_SIZES = {"1024": (1024, 12, 8, 256, 32, 4, 512, 2048, 50304), "2048": (2048, 16, 16, 512, 64, 8, 1024, 8192, 50304),
+                 "4096": (4096, 4, 32, 512, 64, 8, 1024, 16384, 50304)}
+
+
+def build_layered(R, ctx, torch, size, max_seq):
+    """A Nuvilorn decoder with random weights: one dense layer, then mixture-of-experts layers with a shared block; every third
+    layer lends its latent to the two after it."""
+    W, L, H, rank, E, top, ff, dff, V = size
+    keep = []
+
+    def mat(rows, cols, s=1.0):
+        t = torch.empty(rows, cols, dtype=torch.bfloat16, device="cuda").normal_(0, s / cols ** 0.5)
+        keep.append(t)
+        return t.data_ptr()
+
+    def f32(t):
+        keep.append(t)
+        return t.data_ptr()
+    one = f32(torch.ones(1, device="cuda"))
+    layers = []
+    for i in range(L):
+        d = R.LayerDesc(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=rank, kv_from=-1 if i % 3 == 0 else i - i % 3, scale=192 ** -0.5,
+                        rot_base=10000.0, norm1=one, norm2=one)
+        q = H * 192 + (rank + 64 if i % 3 == 0 else 0)
+        d.w_q, d.w_ukv, d.w_o = mat(q, W), mat(H * 256, rank), mat(W, H * 128)
+        if i % 3 == 0:
+            d.kv_norm = f32(torch.ones(rank, device="cuda"))
+        if i == 0:
+            d.ff_kind, d.ff_act, d.ff, d.ff_up, d.ff_down = R.FF_DENSE, R.ACT_SILU_GLU, dff, mat(2 * dff, W), mat(W, dff)
+        else:
+            d.ff_kind, d.ff_act, d.ff, d.n_experts, d.top_k, d.score, d.shared_ff = R.FF_MOE, R.ACT_RELU2, ff, E, top, R.SCORE_SIGMOID, ff
+            d.ff_up, d.ff_down = mat(E * ff, W), mat(E * W, ff)
+            d.router = f32(torch.randn(E + 1, W, device="cuda") / W ** 0.5)
+            d.shared_up, d.shared_down = mat(ff, W), mat(W, ff)
+        layers.append(d)
+    w = {"embed": mat(V, W), "embed_norm": one, "final_norm": one, "head": mat(V, W)}
+    cfg = R.LayeredCfg(n_layers=L, width=W, vocab=V, max_seq=max_seq, exact=0, eps=1e-6)
+    torch.cuda.synchronize()
+    return R.LayeredModel(ctx, cfg, layers, w, keep=keep)
+
+
+def build_olmoe(R, ctx, size, max_seq):
+    """The Q4_K decoder at the same width, depth, heads, experts and vocabulary."""
+    W, L, H, _rank, E, top, ff, _dff, V = size
+    rbq = lambda kk: kk // 256 * 144
+    shapes = {"wq": (L * H * 128, W), "wk": (L * H * 128, W), "wv": (L * H * 128, W), "wo": (L * W, H * 128), "gate": (L * E * ff, W),
+              "up": (L * E * ff, W), "down": (L * E * W, ff), "lm_head": (V, W)}
+    dev = {}
+    for i, (name, (rows, kk)) in enumerate(shapes.items()):
+        dev[name] = ctx.new_buffer(rows * rbq(kk))
+        R.fill_weights_q4k_zero_mean(ctx, dev[name], rows * (kk // 256), 31 + i, 6e-5)
+    for name, n, sig in (("tok_emb", V * W, 1.0), ("router", L * E * W, 0.02)):
+        dev[name] = ctx.new_buffer(n * 4)
+        R.fill_normal_f32(ctx, dev[name], n, 7, sig)
+    for name, n in (("attn_norm", L * W), ("ffn_norm", L * W), ("out_norm", W)):
+        dev[name] = ctx.buffer_from(np.ones(n, np.float32))
+    cfg = R.ModelCfg(n_layers=L, hidden=W, n_heads=H, n_kv_heads=H, head_dim=128, vocab=V, n_experts=E, top_k=top, ff=ff, max_seq=max_seq,
+                     renorm=0, eps=1e-5, theta=10000.0)
+    return R.Model(ctx, cfg, dev)
+
+
+def time_model(model, vocab, contexts=(128, 2048), steps=64):
+    """Prompt and decode throughput of a decoder (wall clock around calls that synchronise once)."""
+    out = {"launches_per_token": int(model.launches_per_token), "prefill": {}, "decode": {}}
+    for T in (128, 512, 2048):
+        pr = np.random.default_rng(T).integers(0, vocab, T).astype(np.int32)
+        for _ in range(3):
+            model.prefill(pr)
+        t0 = time.perf_counter()
+        for _ in range(5):
+            model.prefill(pr)
+        dt = (time.perf_counter() - t0) / 5
+        out["prefill"]["T%d" % T] = {"ms": dt * 1e3, "tokens_per_s": T / dt}
+    for n in contexts:
+        pr = np.random.default_rng(n).integers(0, vocab, n).astype(np.int32)
+        nxt = np.array([model.prefill(pr)], np.int32)
+        model.generate_greedy(nxt, 3, start_pos=n)
+        t0 = time.perf_counter()
+        model.generate_greedy(nxt, steps - 1, start_pos=n)
+        dt = (time.perf_counter() - t0) / steps
+        out["decode"]["context%d" % n] = {"us_per_token": dt * 1e6, "tokens_per_s": 1 / dt}
+    return out
+
+
+def time_layered_kernels(R, ctx, torch, stream, size, reps=20):
+    """The kernels of a layer by themselves beside the like kernels of the Q4_K decoder: fraction of measured HBM bandwidth
+    (one token) or of the measured tensor peak (2048 tokens).  Inputs rotate over sets larger than L2."""
+    import ctypes as C
+    W, _L, H, rank, E, top, ff, dff, V = size
+    hbm = measured_peak()[0]
+    tc, _ = measured_tensor_peak()
+    rows = []
+
+    def timed(fns):
+        for f in fns[:3]:
+            f()
+        ctx.flush()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        n = max(reps, len(fns))
+        a.record(stream)
+        for i in range(n):
+            fns[i % len(fns)]()
+        b.record(stream)
+        torch.cuda.synchronize()
+        return a.elapsed_time(b) / n * 1e3
+
+    def add(name, us, us_like, nbytes=0, flops=0, nbytes_like=0, flops_like=0):
+        f = lambda t, by, fl: by / (t * 1e-6) / 1e9 / hbm if by else fl / (t * 1e-6) / 1e12 / tc
+        rows.append({"kernel": name, "us": us, "frac_of_roofline": f(us, nbytes, flops), "like_us": us_like,
+                     "like_frac_of_roofline": f(us_like, nbytes_like, flops_like)})
+    rbq = lambda kk: kk // 256 * 144
+    bf = lambda *s: torch.empty(*s, dtype=torch.bfloat16, device="cuda").normal_(0, 0.05)
+    one = torch.ones(1, device="cuda")
+    ones = torch.ones(65536, device="cuda")
+    # one token: projections
+    for name, m, k in (("q|latent projection, 1 token", H * 192 + rank + 64, W), ("output projection, 1 token", W, H * 128), ("head, 1 token", V, W)):
+        sets = max(2, min(64, int(300e6 // (m * k * 2)) + 1))
+        ws, x, y = [bf(m, k) for _ in range(sets)], torch.randn(k, device="cuda"), torch.empty(m, device="cuda")
+        us = timed([(lambda w=w: R.gemv_bf16_f32(ctx, w, x, one, 1e-6, y, None, m, k)) for w in ws])
+        m4 = m // 32 * 32
+        qs = max(2, min(128, int(300e6 // (m4 * rbq(k))) + 1))
+        wq = [ctx.new_buffer(m4 * rbq(k)) for _ in range(qs)]
+        for i, b in enumerate(wq):
+            R.fill_weights(ctx, R.FMT_Q4K, b, m4 * (k // 256), 3 + i, 0.01)
+        us4 = timed([(lambda w=w: R.rms_norm_gemv_f32(ctx, R.FMT_Q4K, w, x, ones, 1e-6, y, None, m4, k)) for w in wq])
+        add(name, us, us4, nbytes=m * k * 2, nbytes_like=m4 * rbq(k))
+        for b in wq:
+            b.free()
+        del ws
+    # one token: attention over 4096 positions (bytes: cache rows; folded queries and value projection apart)
+    S, pitch = 4096, rank + 64
+    lc = R.LatentCfg(H, 128, 64, 128, rank, 192 ** -0.5, 1e-6)
+    caches = [bf(S, pitch) for _ in range(64)]
+    ns = max(1, min(64, 296 // ((H + 15) // 16)))
+    qe, po, ml = torch.randn(H * pitch, device="cuda"), torch.empty(H * ns * rank, device="cuda"), torch.empty(H * ns * 2, device="cuda")
+    us = timed([(lambda c=c: R.latent_attention(ctx, C.byref(lc), 0, qe, c, po, ml, ns, 1, S - 1)) for c in caches])
+    kc = [torch.randn(2, H, S, 128, device="cuda").half() for _ in range(8)]
+    q1, o1 = torch.randn(H * 128, device="cuda"), torch.empty(H * 128, device="cuda")
+    us4 = timed([(lambda c=c: R.decode_attention_f32q_f16kv(ctx, q1, c[0], c[1], o1, 1, S, H, H, 128, S)) for c in kc])
+    add("attention over 4096 positions, 1 token", us, us4, nbytes=S * pitch * 2, nbytes_like=2 * H * S * 128 * 2)
+    ukv = [bf(H * 256, rank) for _ in range(64)]
+    qkv, freq = torch.randn(H * 192 + rank + 64, device="cuda"), torch.rand(32, device="cuda")
+    kvn, ao = torch.ones(rank, device="cuda"), torch.empty(H * 128, device="cuda")
+    us = timed([(lambda w=w: R.latent_query(ctx, C.byref(lc), 0, qkv, H * 192 + rank + 64, w, kvn, freq, caches[0], qe, 1, 7)) for w in ukv])
+    wq = [ctx.new_buffer(H * 128 * rbq(rank)) for _ in range(128)]
+    for i, b in enumerate(wq):
+        R.fill_weights(ctx, R.FMT_Q4K, b, H * 128 * (rank // 256), 3 + i, 0.01)
+    xr, yr = torch.randn(rank, device="cuda"), torch.empty(H * 128, device="cuda")
+    us4 = timed([(lambda w=w: R.gemv_q4k_f32in_f32out(ctx, w, xr, yr, H * 128, rank)) for w in wq])
+    add("folded queries + cache row, 1 token (like: Q4_K GEMV of the same shape)", us, us4, nbytes=H * 128 * rank * 2, nbytes_like=H * 128 * rbq(rank))
+    us = timed([(lambda w=w: R.latent_value(ctx, C.byref(lc), po, ml, ns, w[H * 128:], ao, 1)) for w in ukv])
+    add("merge + value projection, 1 token (like: the same)", us, us4, nbytes=H * 128 * rank * 2 + H * ns * rank * 4, nbytes_like=H * 128 * rbq(rank))
+    del caches, kc, ukv
+    # 2048 tokens: dense products
+    T = 2048
+    for name, m, k, epi in (("q|latent projection, 2048 tokens", H * 192 + rank + 64, W, R.EPI_F32), ("output projection + residual, 2048 tokens", W, H * 128, R.EPI_ADD),
+                            ("gate/up + silu, 2048 tokens", 2 * dff, W, R.EPI_SILU_GLU), ("down + residual, 2048 tokens", W, dff, R.EPI_ADD)):
+        ws, x = [bf(m, k) for _ in range(4)], bf(T, k)
+        n_out = m // 2 if epi == R.EPI_SILU_GLU else m
+        y = torch.empty(T, n_out, device="cuda")
+        us = timed([(lambda w=w: R.gemm_bf16_rows(ctx, w, x, y, n_out, T, m, k, 0, epi, None, None)) for w in ws])
+        rows.append({"kernel": name, "us": us, "frac_of_roofline": 2.0 * T * m * k / (us * 1e-6) / 1e12 / tc})
+        del ws
+    f4 = [ctx.new_buffer(r * rbq(kk)) for r, kk in ((dff, W), (dff, W), (W, dff))]
+    for i, (b, (r, kk)) in enumerate(zip(f4, ((dff, W), (dff, W), (W, dff)))):
+        R.fill_weights(ctx, R.FMT_Q4K, b, r * (kk // 256), 611 + i, 0.01)
+    xd, od = torch.randn(T, W, device="cuda"), torch.empty(T, W, device="cuda")
+    nbd = ctx.lib.runit_ffn_q4k_bf16_scratch_bytes(T, W, dff)
+    sd = ctx.new_buffer(nbd)
+    us4 = timed([lambda: R.ffn_q4k_bf16(ctx, f4[0], f4[1], f4[2], xd, None, 0.0, xd, od, sd, nbd, T, W, dff)])
+    rows.append({"kernel": "like: dense feed-forward block of the Q4_K decoder, 2048 tokens", "us": us4,
+                 "frac_of_roofline": 2.0 * 3 * T * W * dff / (us4 * 1e-6) / 1e12 / tc})
+    for b in f4 + [sd]:
+        b.free()
+    # 2048 tokens: causal attention (half of the pairs)
+    kv, cache = bf(T, H * 256), bf(T, pitch)
+    q, out = torch.randn(T, H * 192, device="cuda"), torch.empty(T, H * 128, dtype=torch.bfloat16, device="cuda")
+    us = timed([lambda: R.latent_prefill_attention(ctx, C.byref(lc), q, H * 192, kv, H * 256, cache, out, H * 128, T, 0)])
+    kc, q4 = torch.randn(2, H, T, 128, device="cuda").half(), torch.randn(T, H * 128, device="cuda")
+    us4 = timed([lambda: R.prefill_attention_f16kv(ctx, q4, kc[0], kc[1], out, T, H, H, 128, T, 0)])
+    add("causal attention, 2048 tokens", us, us4, flops=T * T * H * (192 + 128), flops_like=T * T * H * 256)
+    return rows
+
+
+def run_layered(R, ctx, torch, stream, sizes):
+    out = {"note": "random weights; the closest model is the Q4_K OLMoE-shaped decoder at equal width, depth, heads, experts and vocabulary"}
+    for name in sizes:
+        size = LAYERED_SIZES[name]
+        res = {"size": dict(zip(("width", "layers", "heads", "kv_rank", "experts", "top", "expert_ff", "dense_ff", "vocab"), size))}
+        m = build_layered(R, ctx, torch, size, 2304)
+        res["nuvilorn_bf16"] = time_model(m, size[-1])
+        m.close()
+        del m
+        torch.cuda.empty_cache()
+        m = build_olmoe(R, ctx, size, 2304)
+        res["olmoe_q4k"] = time_model(m, size[-1])
+        m.close()
+        del m
+        if name == "2048":
+            res["kernels"] = time_layered_kernels(R, ctx, torch, stream, size)
+        out[name] = res
+        torch.cuda.empty_cache()
+    return out
+
+
 # ───────────────────────── sharded paths (N > 1) ─────────────────────────
 
 def _time_steps(torch, dist, stream, ctx, fn, steps, world):
@@ -936,6 +1143,8 @@ def main():
     ap.add_argument("--ffn", default="", help="T: the dense feed-forward block (Qwen2.5-7B shape) on T tokens, three times, then exit "
                                               "(the small case for ncu captures of the dense tcgen05 GEMM)")
     ap.add_argument("--shapes", action="store_true", help="per-shape GEMV table (one JSON line per shape) instead of the headline run")
+    ap.add_argument("--layered", nargs="?", const="1024,2048,4096", default="",
+                    help="prefill and decode throughput of the layered (latent attention) decoder at these widths beside the Q4_K decoder, then exit")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -981,6 +1190,9 @@ def main():
                 getattr(R, "gemv_%s_f32in_f32out" % f)(ctx, w, x, y, m, k)
         ctx.flush()
         print(json.dumps({"one": args.one, "launches": ctx.launches}))
+        return
+    if args.layered:
+        print(json.dumps(run_layered(R, ctx, torch, stream, args.layered.split(","))))
         return
     if args.ffn:
         T = int(args.ffn)

@@ -473,6 +473,47 @@ int32_t runit_ffn_q4k_bf16(runit_ctx_t*, const void* w_gate, const void* w_up, c
 int32_t runit_model_forward(runit_model_t* model, const int32_t* tokens, uint32_t n, uint32_t start_pos, const uint32_t* want,
                             uint32_t n_want, float* logits);
 
+/* ── operators over bf16 weight matrices (no twin): rows of pad8(k) elements, zero padding ── */
+/* y[m] = W . x (+ residual, may be y); gain f32 [1] not NULL: x is first divided by its root mean square and multiplied by it */
+int32_t runit_gemv_bf16_f32(runit_ctx_t*, const void* weight, const void* x, const void* gain, float eps, void* y, const void* residual,
+                            uint32_t m, uint32_t k);
+/* What becomes of a product: stored as f32; added to the f32 output; stored in the activation type; pairs of rows (2i, 2i+1)
+ * as silu(g) * u, or max(v, 0)^2, in the activation type.  pre / post (f32 per token, may be NULL) multiply the product / the
+ * activated value of the last two. */
+enum { RUNIT_EPI_F32 = 0, RUNIT_EPI_ADD = 1, RUNIT_EPI_CAST = 2, RUNIT_EPI_SILU_GLU = 3, RUNIT_EPI_RELU2 = 4 };
+/* y[T][outputs] = epilogue(W[m][k] . x[t]); x rows of pad8(k) elements: bf16 on the tensor cores (exact = 0; the activation
+ * type is bf16), or f32 with f32 multiply-adds (exact = 1; f32).  y rows of ldy elements. */
+int32_t runit_gemm_bf16_rows(runit_ctx_t*, const void* weight, const void* x, void* y, uint32_t ldy, uint32_t T, uint32_t m, uint32_t k,
+                             int32_t exact, int32_t epi, const void* pre, const void* post);
+/* y[t] = x[t] / sqrt(mean(x[t]^2) + eps) * gain[0], x f32 [T][width], y f32 or bf16 rows of pad8(width) */
+int32_t runit_norm_gain_rows(runit_ctx_t*, const void* x, const void* gain, float eps, void* y, int32_t y_f32, uint32_t T, uint32_t width);
+/* Latent attention.  One cache row per position: the normed latent (kv_rank values padded to a multiple of 16), then the
+ * rotated shared key part (rot_dim padded likewise), bf16 or f32 (cache_f32).  qkv: f32 rows of ldq values, the queries of all
+ * heads [dim | rot_dim] and then, when kv_norm is not NULL, the raw latent and key part of the token, which become the cache
+ * row of its position.  freq f32 [rot_dim / 2]: angle = position * freq[i] for the pair (2i, 2i+1). */
+typedef struct {
+    uint32_t heads, dim, rot_dim, vdim, kv_rank;
+    float    scale, eps;
+} runit_latent_cfg;
+/* folded queries q_eff f32 [T * heads][row] (row = elements of a cache row): [W_uk^T q_un | rotated q_rot]; w_uk [heads*dim][pad8(kv_rank)] */
+int32_t runit_latent_query(runit_ctx_t*, const runit_latent_cfg* cfg, int32_t cache_f32, const void* qkv, uint32_t ldq, const void* w_uk,
+                           const void* kv_norm, const void* freq, void* cache, void* q_eff, uint32_t T, uint32_t start);
+/* softmax over positions 0 .. start+t per (token, head), keys split nsplit ways: part_o f32 [T*heads][nsplit][pad16(kv_rank)]
+ * (weighted latent sums), part_ml f32 [T*heads][nsplit][2] (maximum, sum of weights) */
+int32_t runit_latent_attention(runit_ctx_t*, const runit_latent_cfg* cfg, int32_t cache_f32, const void* q_eff, const void* cache,
+                               void* part_o, void* part_ml, uint32_t nsplit, uint32_t T, uint32_t start);
+/* merges the splits and applies W_uv [heads*vdim][pad8(kv_rank)]: out f32 [T][heads*vdim] */
+int32_t runit_latent_value(runit_ctx_t*, const runit_latent_cfg* cfg, const void* part_o, const void* part_ml, uint32_t nsplit,
+                           const void* w_uv, void* out, uint32_t T);
+/* cache rows (bf16 or f32) of T tokens, and the rotated parts of their queries in place */
+int32_t runit_latent_rows(runit_ctx_t*, const runit_latent_cfg* cfg, int32_t cache_f32, void* qkv, uint32_t ldq, const void* kv_norm,
+                          const void* freq, void* cache, uint32_t T, uint32_t start);
+/* the same attention over expanded keys and values, kv bf16 [start + T][ldkv] = [keys of all heads (dim each) | values (vdim)];
+ * q f32 with rotated parts; bf16 cache (for the shared key part); out bf16 [T][ldo].  dim, rot_dim, vdim multiples of 8,
+ * dim + rot_dim <= 192, vdim <= 128, ldq even, ldkv a multiple of 8, ldo even. */
+int32_t runit_latent_prefill_attention(runit_ctx_t*, const runit_latent_cfg* cfg, const void* q, uint32_t ldq, const void* kv, uint32_t ldkv,
+                                       const void* cache, void* out, uint32_t ldo, uint32_t T, uint32_t start);
+
 /* ── decoders described layer by layer (no twin), weights in bf16 ──
  * Every matrix is row-major [rows][pad8(columns)] bf16 with zero padding; norms and router are f32.  Linear maps W x.
  * Residual stream, norms, scores, softmax, router and angles are f32.  Pre-norm layers:

@@ -18,6 +18,10 @@
 namespace runit {
 namespace gm {
 
+static_assert(EPI_F32 == RUNIT_EPI_F32 && EPI_ADD == RUNIT_EPI_ADD && EPI_CAST == RUNIT_EPI_CAST && EPI_SILU_GLU == RUNIT_EPI_SILU_GLU &&
+                  EPI_RELU2 == RUNIT_EPI_RELU2,
+              "the epilogues of the C interface");
+
 struct Args {
     const __nv_bfloat16* w;
     const float* x32;
@@ -357,3 +361,19 @@ int32_t gemm_bf16(runit_ctx* ctx, const char* name, const GemmDesc& d, bool exac
 }
 
 }  // namespace runit
+
+using namespace runit;
+
+extern "C" {
+
+int32_t runit_gemm_bf16_rows(runit_ctx_t* ctx, const void* weight, const void* x, void* y, uint32_t ldy, uint32_t T, uint32_t m, uint32_t k,
+                             int32_t exact, int32_t epi, const void* pre, const void* post) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, weight && x && y && T > 0 && m > 0 && k > 0 && epi >= RUNIT_EPI_F32 && epi <= RUNIT_EPI_RELU2, "gemm_bf16_rows: bad argument");
+    GemmDesc d;
+    d.w = weight; d.rows = m; d.K = k; d.ldw = pad8(k); d.x = x; d.ldx = pad8(k); d.x_rows = T; d.T = T; d.epi = epi; d.out = y; d.ldo = ldy;
+    d.pre = (const float*)pre; d.post = (const float*)post;
+    return gemm_bf16(ctx, "gemm_bf16_rows", d, exact != 0);
+}
+
+}  // extern "C"

@@ -392,3 +392,25 @@ int32_t sigmoid_column(runit_ctx* ctx, const float* logits, uint32_t ld, uint32_
 }
 
 }  // namespace runit
+
+using namespace runit;
+
+extern "C" {
+
+int32_t runit_gemv_bf16_f32(runit_ctx_t* ctx, const void* weight, const void* x, const void* gain, float eps, void* y, const void* residual,
+                            uint32_t m, uint32_t k) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, weight && x && y && m > 0 && k > 0 && runit_aligned(weight, 16), "gemv_bf16_f32: bad argument");
+    GemvDesc d;
+    d.w = weight; d.rows = m; d.K = k; d.ldw = pad8(k); d.x = (const float*)x; d.gain = (const float*)gain; d.eps = eps; d.out = (float*)y;
+    d.res = (const float*)residual;
+    return gemv_bf16(ctx, "gemv_bf16_f32", d);
+}
+
+int32_t runit_norm_gain_rows(runit_ctx_t* ctx, const void* x, const void* gain, float eps, void* y, int32_t y_f32, uint32_t T, uint32_t width) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, x && gain && y && T > 0 && width > 0, "norm_gain_rows: bad argument");
+    return norm_rows(ctx, (const float*)x, nullptr, (const float*)gain, eps, y, y_f32 != 0, pad8(width), nullptr, T, width);
+}
+
+}  // extern "C"

@@ -705,3 +705,68 @@ int32_t latent_prefill(runit_ctx* ctx, const LatentDims& d, const float* q, uint
 }
 
 }  // namespace runit
+
+using namespace runit;
+
+static int32_t latent_check(runit_ctx* ctx, const char* who, const runit_latent_cfg* c, LatentDims* d, uint32_t T) {
+    RUNIT_REQUIRE(ctx, c && T > 0 && T <= 65535 && c->heads > 0 && c->dim > 0 && c->rot_dim > 0 && c->rot_dim % 2 == 0 && c->vdim > 0 && c->kv_rank > 0 &&
+                           c->kv_rank <= 1024, "%s: bad sizes", who);
+    *d = LatentDims{c->heads, c->dim, c->rot_dim, c->vdim, c->kv_rank, c->scale, c->eps};
+    return RUNIT_OK;
+}
+
+extern "C" {
+
+int32_t runit_latent_query(runit_ctx_t* ctx, const runit_latent_cfg* cfg, int32_t cache_f32, const void* qkv, uint32_t ldq, const void* w_uk,
+                           const void* kv_norm, const void* freq, void* cache, void* q_eff, uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    LatentDims d;
+    int32_t st = latent_check(ctx, "latent_query", cfg, &d, T);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, qkv && w_uk && freq && cache && q_eff && ldq >= d.q_width() + (kv_norm ? d.kv_rank + d.rot_dim : 0), "latent_query: bad argument");
+    return latent_query(ctx, d, cache_f32 != 0, (const float*)qkv, ldq, w_uk, pad8(d.kv_rank), (const float*)kv_norm, (const float*)freq, cache,
+                        (float*)q_eff, T, LatentPos{nullptr, start});
+}
+
+int32_t runit_latent_attention(runit_ctx_t* ctx, const runit_latent_cfg* cfg, int32_t cache_f32, const void* q_eff, const void* cache,
+                               void* part_o, void* part_ml, uint32_t nsplit, uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    LatentDims d;
+    int32_t st = latent_check(ctx, "latent_attention", cfg, &d, T);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, q_eff && cache && part_o && part_ml && nsplit > 0 && nsplit <= 1024, "latent_attention: bad argument");
+    return latent_attention(ctx, d, cache_f32 != 0, (const float*)q_eff, cache, (float*)part_o, (float*)part_ml, nsplit, T, LatentPos{nullptr, start});
+}
+
+int32_t runit_latent_value(runit_ctx_t* ctx, const runit_latent_cfg* cfg, const void* part_o, const void* part_ml, uint32_t nsplit,
+                           const void* w_uv, void* out, uint32_t T) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    LatentDims d;
+    int32_t st = latent_check(ctx, "latent_value", cfg, &d, T);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, part_o && part_ml && w_uv && out && nsplit > 0 && nsplit <= 1024, "latent_value: bad argument");
+    return latent_value(ctx, d, (const float*)part_o, (const float*)part_ml, nsplit, w_uv, pad8(d.kv_rank), out, true, d.heads * d.vdim, T);
+}
+
+int32_t runit_latent_rows(runit_ctx_t* ctx, const runit_latent_cfg* cfg, int32_t cache_f32, void* qkv, uint32_t ldq, const void* kv_norm,
+                          const void* freq, void* cache, uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    LatentDims d;
+    int32_t st = latent_check(ctx, "latent_rows", cfg, &d, T);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, qkv && freq && cache && ldq >= d.q_width() + (kv_norm ? d.kv_rank + d.rot_dim : 0), "latent_rows: bad argument");
+    return latent_rows(ctx, d, cache_f32 != 0, (float*)qkv, ldq, (const float*)kv_norm, (const float*)freq, cache, T, LatentPos{nullptr, start});
+}
+
+int32_t runit_latent_prefill_attention(runit_ctx_t* ctx, const runit_latent_cfg* cfg, const void* q, uint32_t ldq, const void* kv, uint32_t ldkv,
+                                       const void* cache, void* out, uint32_t ldo, uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    LatentDims d;
+    int32_t st = latent_check(ctx, "latent_prefill_attention", cfg, &d, T);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, q && kv && cache && out && ldq >= d.q_width() && ldkv >= d.heads * (d.dim + d.vdim) && ldo >= d.heads * d.vdim,
+                  "latent_prefill_attention: bad argument");
+    return latent_prefill(ctx, d, (const float*)q, ldq, kv, ldkv, cache, out, ldo, T, start);
+}
+
+}  // extern "C"

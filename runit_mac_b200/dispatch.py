@@ -277,6 +277,14 @@ _TWINS = [
     ("peer_barrier", "no twin: (signal_pads[world] pointer table, world, rank, epoch)"),
     ("moe_layer_q4k_ep", "no twin: expert-parallel decode block with replicated tokens, combine fused over peer memory"),
     ("moe_layer_q4k_bf16_ep", "no twin: expert-parallel batched block, token rows exchanged by peer stores"),
+    ("gemv_bf16_f32", "no twin: (weight_bf16, x, gain or None, eps, y, residual or None, m, k)"),
+    ("gemm_bf16_rows", "no twin: (weight_bf16, x, y, ldy, T, m, k, exact, epi, pre or None, post or None)"),
+    ("norm_gain_rows", "no twin: (x, gain, eps, y, y_f32, T, width)"),
+    ("latent_query", "no twin: (LatentCfg ref, cache_f32, qkv, ldq, w_uk, kv_norm or None, freq, cache, q_eff, T, start)"),
+    ("latent_attention", "no twin: (LatentCfg ref, cache_f32, q_eff, cache, part_o, part_ml, nsplit, T, start)"),
+    ("latent_value", "no twin: (LatentCfg ref, part_o, part_ml, nsplit, w_uv, out, T)"),
+    ("latent_rows", "no twin: (LatentCfg ref, cache_f32, qkv, ldq, kv_norm or None, freq, cache, T, start)"),
+    ("latent_prefill_attention", "no twin: (LatentCfg ref, q, ldq, kv, ldkv, cache, out, ldo, T, start)"),
     ("fill_weights", "no twin: (fmt, dst, n_blocks, seed, sigma)"),
     ("fill_weights_q4k_zero_mean", "no twin: (dst, n_blocks, seed, sigma), Q4_K blocks with zero-mean weights"),
     ("fill_normal_f32", "no twin: (dst, n, seed, sigma)"),
@@ -410,6 +418,14 @@ FF_NONE, FF_DENSE, FF_MOE = 0, 1, 2
 ACT_SILU_GLU, ACT_RELU2 = 0, 1
 
 
+EPI_F32, EPI_ADD, EPI_CAST, EPI_SILU_GLU, EPI_RELU2 = 0, 1, 2, 3, 4
+
+
+class LatentCfg(C.Structure):
+    """runit_latent_cfg; pass ``ctypes.byref(cfg)`` to the latent_* operators."""
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank")] + [("scale", C.c_float), ("eps", C.c_float)]
+
+
 class LayerDesc(C.Structure):
     """runit_layer_desc: mixer and feed-forward of one layer, sizes, constants and device pointers."""
     _fields_ = ([(n, C.c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "kv_from")] +
@@ -502,6 +518,6 @@ def moe_layer_q4k_host(ctx: Context, router, gate, up, down, x, *, h, ff, E, top
             w.download(np.float32, T * top_k).reshape(T, top_k))
 
 
-__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc",
+__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc", "LatentCfg", "EPI_F32", "EPI_ADD", "EPI_CAST", "EPI_SILU_GLU", "EPI_RELU2",
            "FF_NONE", "FF_DENSE", "FF_MOE", "ACT_SILU_GLU", "ACT_RELU2", "SCORE_SOFTMAX", "SCORE_SIGMOID", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
            "FMT_Q8_0", "FMT_Q4_0", "FMT_Q4K", "FMT_Q5_0", "FMT_Q5K", "FMT_Q6K"] + [n for n, _ in _TWINS]
