@@ -495,7 +495,8 @@ typedef struct {
     uint32_t heads, dim, rot_dim, vdim, kv_rank;
     float    scale, eps;
 } runit_latent_cfg;
-/* folded queries q_eff f32 [T * heads][row] (row = elements of a cache row): [W_uk^T q_un | rotated q_rot]; w_uk [heads*dim][pad8(kv_rank)] */
+/* folded queries q_eff [T * heads][row] (row = elements of a cache row): [W_uk^T q_un | rotated q_rot], f32 with an f32 cache,
+ * else the high bf16 parts of a row followed by its low parts; w_uk [heads*dim][pad8(kv_rank)] */
 int32_t runit_latent_query(runit_ctx_t*, const runit_latent_cfg* cfg, int32_t cache_f32, const void* qkv, uint32_t ldq, const void* w_uk,
                            const void* kv_norm, const void* freq, void* cache, void* q_eff, uint32_t T, uint32_t start);
 /* softmax over positions 0 .. start+t per (token, head), keys split nsplit ways: part_o f32 [T*heads][nsplit][pad16(kv_rank)]

@@ -101,16 +101,17 @@ struct LatentPos {
     const int32_t* pos_ptr;
     uint32_t start;
 };
-// Query side folded with W_uk: q_eff[t*heads+h] = [W_uk,h^T q_un | rotated q_rot], f32 rows of pitch().  One more CTA per token
+// Query side folded with W_uk: q_eff[t*heads+h] = [W_uk,h^T q_un | rotated q_rot], rows of pitch() values: f32, or with a bf16
+// cache the high bf16 parts of all and then their low parts (4 bytes a value either way).  One more CTA per token
 // writes the cache row of its position from qkv[t][q_width() ..] when kv_norm is not null (the layer owns its latent).
 int32_t latent_query(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const float* qkv, uint32_t ldq, const void* w_uk, uint32_t ldk,
-                     const float* kv_norm, const float* freq, void* cache, float* q_eff, uint32_t T, LatentPos pos);
+                     const float* kv_norm, const float* freq, void* cache, void* q_eff, uint32_t T, LatentPos pos);
 // The same without W_uk: cache rows, and the rotated parts of q in place (f32).
 int32_t latent_rows(runit_ctx* ctx, const LatentDims& d, bool cache_f32, float* qkv, uint32_t ldq, const float* kv_norm, const float* freq,
                     void* cache, uint32_t T, LatentPos pos);
 // Attention over cached rows: query row r = t*heads+h sees positions 0 .. pos(t); keys split nsplit ways.  part_o f32
 // [row][nsplit][cp()], part_ml f32 [row][nsplit][2] (maximum, sum).
-int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const float* q_eff, const void* cache, float* part_o,
+int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const void* q_eff, const void* cache, float* part_o,
                          float* part_ml, uint32_t nsplit, uint32_t T, LatentPos pos);
 uint32_t latent_splits(const runit_ctx* ctx, const LatentDims& d, bool cache_f32, uint32_t T);
 // out[t][h*vdim + j] = W_uv,h (merged latent output), f32 or bf16 rows of ldo

@@ -191,6 +191,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                             out[(size_t)(tok0 + jj) * a.ldo + (r >> 1)] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u * post);
                         }
                     }
+                } else if constexpr (EPI == EPI_ADD) {
+                    // all loads of the group before its first store (the compiler may not reorder them across one)
+                    float* out = reinterpret_cast<float*>(a.out) + (size_t)tok0 * a.ldo + r;
+                    float old[32];
+#pragma unroll
+                    for (int j = 0; j < 32; j++) old[j] = (live && (uint32_t)j < cnt) ? out[(size_t)j * a.ldo] : 0.f;
+#pragma unroll
+                    for (int j = 0; j < 32; j++)
+                        if (live && (uint32_t)j < cnt) out[(size_t)j * a.ldo] = old[j] + __uint_as_float(v[j]);
                 } else {
 #pragma unroll
                     for (int j = 0; j < 32; j++) {
@@ -198,7 +207,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         const float f = __uint_as_float(v[j]);
                         const size_t o = (size_t)(tok0 + j) * a.ldo + r;
                         if constexpr (EPI == EPI_F32) reinterpret_cast<float*>(a.out)[o] = f;
-                        else if constexpr (EPI == EPI_ADD) reinterpret_cast<float*>(a.out)[o] += f;
                         else if constexpr (EPI == EPI_CAST) reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16_rn(f);
                         else {
                             const float pre = a.pre ? a.pre[tok0 + j] : 1.f, post = a.post ? a.post[tok0 + j] : 1.f;

@@ -217,41 +217,51 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_sum_kernel(const SumArg
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t chs = (a.K + 7) / 8, routed = a.n_routed * chs, chx = a.w_extra ? (a.K_extra + 7) / 8 : 0, total = routed + chx;
     float4 *xa = smem4, *xb = smem4 + total;
-    grid_dependency_wait();
-    grid_launch_dependents();
+    // The expert ids come from the launch before the one this depends on: that launch has waited for it, so they are final
+    // and the first weights can be requested before the wait.
     if (threadIdx.x < a.n_routed) {
         const int32_t e = a.slot_expert ? a.slot_expert[threadIdx.x] : 0;
         base_s[threadIdx.x] = e < 0 ? nullptr : a.w + (size_t)e * a.rows * a.ldw * 2;
     }
+    __syncthreads();
+    const uint32_t units = (a.rows + RPU - 1) / RPU;
+    uint32_t unit = blockIdx.x * kWarps + warp;
+    uint4 v[RPU][U];
+    auto load = [&](uint32_t u, uint32_t c0) {
+#pragma unroll
+        for (int i = 0; i < U; i++) {
+            const uint32_t c = c0 + 32 * i + lane;
+            const uint8_t* p = nullptr;
+            size_t pitch = 0;
+            if (c < routed) {
+                const uint32_t s = c / chs;
+                pitch = (size_t)a.ldw * 2;
+                if (base_s[s]) p = base_s[s] + (size_t)(c - s * chs) * 16;
+            } else if (c < total) {
+                pitch = (size_t)a.ldw_extra * 2;
+                p = a.w_extra + (size_t)(c - routed) * 16;
+            }
+#pragma unroll
+            for (int r = 0; r < RPU; r++) {
+                const uint32_t row = u * RPU + r;
+                v[r][i] = (p && row < a.rows) ? __ldg(reinterpret_cast<const uint4*>(p + row * pitch)) : make_uint4(0, 0, 0, 0);
+            }
+        }
+    };
+    if (unit < units) load(unit, 0);
+    grid_dependency_wait();
+    grid_launch_dependents();
     for (uint32_t s = 0; s < a.n_routed; s++) stage_x(a.x + (size_t)s * a.x_stride, a.K, chs, xa + s * chs, xb + s * chs);
     if (chx) stage_x(a.x + (size_t)a.n_routed * a.x_stride, a.K_extra, chx, xa + routed, xb + routed);
     __syncthreads();
-    const uint32_t units = (a.rows + RPU - 1) / RPU;
-    for (uint32_t unit = blockIdx.x * kWarps + warp; unit < units; unit += gridDim.x * kWarps) {
+    bool first = true;
+    for (; unit < units; unit += gridDim.x * kWarps) {
         float acc[RPU];
 #pragma unroll
         for (int r = 0; r < RPU; r++) acc[r] = 0.f;
         for (uint32_t c0 = 0; c0 < total; c0 += 32 * U) {
-            uint4 v[RPU][U];
-#pragma unroll
-            for (int i = 0; i < U; i++) {
-                const uint32_t c = c0 + 32 * i + lane;
-                const uint8_t* p = nullptr;
-                size_t pitch = 0;
-                if (c < routed) {
-                    const uint32_t s = c / chs;
-                    pitch = (size_t)a.ldw * 2;
-                    if (base_s[s]) p = base_s[s] + (size_t)(c - s * chs) * 16;
-                } else if (c < total) {
-                    pitch = (size_t)a.ldw_extra * 2;
-                    p = a.w_extra + (size_t)(c - routed) * 16;
-                }
-#pragma unroll
-                for (int r = 0; r < RPU; r++) {
-                    const uint32_t row = unit * RPU + r;
-                    v[r][i] = (p && row < a.rows) ? __ldg(reinterpret_cast<const uint4*>(p + row * pitch)) : make_uint4(0, 0, 0, 0);
-                }
-            }
+            if (!first) load(unit, c0);
+            first = false;
 #pragma unroll
             for (int i = 0; i < U; i++) {
                 const uint32_t c = c0 + 32 * i + lane;

@@ -73,7 +73,7 @@ template <typename TC>
 __global__ void __launch_bounds__(256) latent_query_kernel(const Dims d, const float* __restrict__ qkv, uint32_t ldq,
                                                             const __nv_bfloat16* __restrict__ w_uk, uint32_t ldk, uint32_t nchunk,
                                                             const float* __restrict__ kv_norm, const float* __restrict__ freq,
-                                                            TC* __restrict__ cache, float* __restrict__ q_eff, const LatentPos lp) {
+                                                            TC* __restrict__ cache, void* __restrict__ q_eff, const LatentPos lp) {
     __shared__ float red[32][65];
     const uint32_t t = blockIdx.y;
     const float* q = qkv + (size_t)t * ldq;
@@ -112,13 +112,24 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const Dims d, const f
 #pragma unroll
     for (int i = 0; i < 8; i++) red[g][cg * 8 + i] = acc[i];
     __syncthreads();
-    float* out = q_eff + ((size_t)t * d.heads + h) * d.pitch;
+    // a row of the folded query: f32, or the high and the low bf16 half of every value (same bytes)
+    float* out = reinterpret_cast<float*>(q_eff) + ((size_t)t * d.heads + h) * d.pitch;
+    auto put_q = [&](uint32_t col, float v) {
+        if constexpr (sizeof(TC) == 4) {
+            out[col] = v;
+        } else {
+            __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(out);
+            const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+            o[col] = hi;
+            o[d.pitch + col] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        }
+    };
     if (threadIdx.x < 64) {
         const uint32_t col = ch * 64 + threadIdx.x;
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < 32; i++) s += red[i][threadIdx.x];
-        if (col < d.cp) out[col] = s;          // columns past kv_rank are zero: so is the padding of W_uk
+        if (col < d.cp) put_q(col, s);          // columns past kv_rank are zero: so is the padding of W_uk
     } else if (ch == 0) {
         const uint32_t pos = (lp.pos_ptr ? (uint32_t)*lp.pos_ptr : lp.start) + t;
         for (uint32_t i = threadIdx.x - 64; i < (d.pitch - d.cp) / 2; i += 192) {
@@ -128,8 +139,8 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const Dims d, const f
                 v = qh[d.dim + 2 * i + 1];
                 rotate_pair(u, v, pos, freq[i]);
             }
-            out[d.cp + 2 * i] = u;
-            out[d.cp + 2 * i + 1] = v;
+            put_q(d.cp + 2 * i, u);
+            put_q(d.cp + 2 * i + 1, v);
         }
     }
 }
@@ -154,7 +165,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const Dims d, float* _
 // ── folded attention ──
 // The keys of a tile whose last row sees `len` of them, cut for split `split` of `nsplit`.
 __device__ __forceinline__ void split_range(uint32_t len, uint32_t split, uint32_t nsplit, uint32_t& beg, uint32_t& end) {
-    const uint32_t chunk = max(64u, ((len + nsplit - 1) / nsplit + 31) / 32 * 32);
+    const uint32_t chunk = max(64u, ((len + nsplit - 1) / nsplit + 63) / 64 * 64);
     beg = min(len, split * chunk);
     end = min(len, beg + chunk);
 }
@@ -176,21 +187,22 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
                  : "r"(addr));
 }
 
-// Tensor cores, bf16 cache.  grid (ceil(rows / 16), nsplit), 4 warps; blocks of 32 keys, two stages (cp.async).  Scores: warp w
-// takes keys 8w .. 8w+7 over the whole row; values: warp w takes the 16-column groups w, w+4, ... of the latent for all 32 keys.
+// Tensor cores, bf16 cache.  grid (ceil(rows / 16), nsplit), 8 warps; blocks of KB keys, two stages (cp.async).  Scores: warp w
+// takes keys 8w .. 8w+7 over the whole row; values: warp w takes the 16-column groups w, w+8, ... of the latent for all keys.
 // The query is carried as the sum of two bf16 numbers, so that its rounding does not add to the cache's.
-constexpr int kKB = 32;
-template <int NG>      // 16-column groups of the latent per warp
-__global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const float* __restrict__ q_eff, const __nv_bfloat16* __restrict__ cache,
+// KB = 64, or 32 for rows that would not fit shared memory otherwise.
+template <int NG, int KB>      // 16-column groups of the latent per warp, keys per block
+__global__ void __launch_bounds__(256) latent_attn_kernel(const Dims d, const __nv_bfloat16* __restrict__ q_eff, const __nv_bfloat16* __restrict__ cache,
                                                            float* __restrict__ part_o, float* __restrict__ part_ml, uint32_t rows,
                                                            const LatentPos lp) {
     extern __shared__ __align__(16) uint8_t smem[];
-    __shared__ float wmax[4][16], wl[4][16];
+    constexpr int LP = KB + 8;
+    __shared__ float wmax[8][16], wl[8][16];
     const uint32_t ld = d.pitch + 8;                                   // row pitch in shared memory (elements)
     __nv_bfloat16* qh = reinterpret_cast<__nv_bfloat16*>(smem);        // [16][ld] high part
     __nv_bfloat16* ql = qh + 16 * ld;                                  // [16][ld] low part
-    __nv_bfloat16* kv = ql + 16 * ld;                                  // [2][32][ld]
-    __nv_bfloat16* ps = kv + 2 * kKB * ld;                             // [16][40]
+    __nv_bfloat16* kv = ql + 16 * ld;                                  // [2][KB][ld]
+    __nv_bfloat16* ps = kv + 2 * KB * ld;                             // [16][LP]
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const uint32_t r0 = blockIdx.x * 16, split = blockIdx.y, nsplit = gridDim.y;
     grid_dependency_wait();
@@ -199,24 +211,24 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
     const uint32_t last = min(rows, r0 + 16) - 1, len = start + last / d.heads + 1;
     uint32_t beg, end;
     split_range(len, split, nsplit, beg, end);
-    const uint32_t cpr = d.pitch / 8, nblk = (end - beg + kKB - 1) / kKB;
+    const uint32_t cpr = d.pitch / 8, nblk = (end - beg + KB - 1) / KB;
     auto stage = [&](uint32_t b) {
-        __nv_bfloat16* dst = kv + (b & 1) * kKB * ld;
-        for (uint32_t i = tid; i < kKB * cpr; i += 128) {
-            const uint32_t r = i / cpr, c = i - r * cpr, key = beg + b * kKB + r;
+        __nv_bfloat16* dst = kv + (b & 1) * KB * ld;
+        for (uint32_t i = tid; i < KB * cpr; i += 256) {
+            const uint32_t r = i / cpr, c = i - r * cpr, key = beg + b * KB + r;
             if (key < end) cp_async16(smem_u32(dst + r * ld + c * 8), cache + (size_t)key * d.pitch + c * 8);
             else *reinterpret_cast<uint4*>(dst + r * ld + c * 8) = make_uint4(0, 0, 0, 0);
         }
         cp_async_commit();
     };
-    if (nblk) stage(0);
-    for (uint32_t i = tid; i < 16 * (d.pitch / 2); i += 128) {
-        const uint32_t r = i / (d.pitch / 2), c = 2 * (i % (d.pitch / 2));
-        float2 v = make_float2(0.f, 0.f);
-        if (r0 + r < rows) v = *reinterpret_cast<const float2*>(q_eff + (size_t)(r0 + r) * d.pitch + c);
-        const __nv_bfloat162 hi = __floats2bfloat162_rn(v.x, v.y);
-        *reinterpret_cast<__nv_bfloat162*>(qh + r * ld + c) = hi;
-        *reinterpret_cast<__nv_bfloat162*>(ql + r * ld + c) = __floats2bfloat162_rn(v.x - __low2float(hi), v.y - __high2float(hi));
+    if (nblk) {
+        for (uint32_t i = tid; i < 32 * cpr; i += 256) {               // the tile's queries: 16 high rows, 16 low rows
+            const uint32_t r = i / cpr, c = i - r * cpr, row = r0 + (r & 15);
+            __nv_bfloat16* dst = qh + r * ld + c * 8;
+            if (row < rows) cp_async16(smem_u32(dst), q_eff + ((size_t)row * 2 + (r >> 4)) * d.pitch + c * 8);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        }
+        stage(0);                                                      // one group with the queries
     }
     const uint32_t ra = r0 + g, rb = ra + 8;                           // this thread's two query rows
     const uint32_t lim_a = ra < rows ? start + ra / d.heads : 0, lim_b = rb < rows ? start + rb / d.heads : 0;   // last visible position
@@ -237,10 +249,12 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
             cp_async_wait<0>();
         }
         __syncthreads();
-        const __nv_bfloat16* kb = kv + (b & 1) * kKB * ld;
+        const __nv_bfloat16* kb = kv + (b & 1) * KB * ld;
         float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+        const bool scores = warp * 8 < KB;
         const uint32_t qh_u = smem_u32(qh + a_off), ql_u = smem_u32(ql + a_off);
         const uint32_t k_u = smem_u32(kb + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
+        if (scores)
 #pragma unroll 4
         for (uint32_t ks = 0; ks < d.pitch / 16; ks++) {
             uint32_t ah[4], al[4], b0, b1;
@@ -250,11 +264,11 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
             mma_bf16(s, ah, b0, b1);
             mma_bf16(s2, al, b0, b1);
         }
-        const uint32_t key0 = beg + b * kKB + warp * 8 + 2 * tq;
+        const uint32_t key0 = beg + b * KB + warp * 8 + 2 * tq;
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const uint32_t key = key0 + (j & 1);
-            const bool vis = key < end && key <= (j < 2 ? lim_a : lim_b);
+            const bool vis = scores && key < end && key <= (j < 2 ? lim_a : lim_b);
             s[j] = vis ? (s[j] + s2[j]) * d.scale : -INFINITY;
         }
         float xa = fmaxf(s[0], s[1]), xb = fmaxf(s[2], s[3]);
@@ -262,8 +276,12 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
         xb = fmaxf(xb, __shfl_xor_sync(0xffffffffu, xb, 1)); xb = fmaxf(xb, __shfl_xor_sync(0xffffffffu, xb, 2));
         if (tq == 0) { wmax[warp][g] = xa; wmax[warp][g + 8] = xb; }
         __syncthreads();
-        const float n_a = fmaxf(m_a, fmaxf(fmaxf(wmax[0][g], wmax[1][g]), fmaxf(wmax[2][g], wmax[3][g])));
-        const float n_b = fmaxf(m_b, fmaxf(fmaxf(wmax[0][g + 8], wmax[1][g + 8]), fmaxf(wmax[2][g + 8], wmax[3][g + 8])));
+        float n_a = m_a, n_b = m_b;
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            n_a = fmaxf(n_a, wmax[i][g]);
+            n_b = fmaxf(n_b, wmax[i][g + 8]);
+        }
         // a row may see none of the block's keys (and none so far): its maximum stays -inf and its weights are 0
         const float base_a = n_a == -INFINITY ? 0.f : n_a, base_b = n_b == -INFINITY ? 0.f : n_b;
         const float f_a = expf(m_a - base_a), f_b = expf(m_b - base_b);
@@ -272,20 +290,22 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
         m_b = n_b;
         l_a = l_a * f_a + p0 + p1;
         l_b = l_b * f_b + p2 + p3;
-        *reinterpret_cast<uint32_t*>(ps + g * 40 + warp * 8 + 2 * tq) = pack_bf2(p0, p1);
-        *reinterpret_cast<uint32_t*>(ps + (g + 8) * 40 + warp * 8 + 2 * tq) = pack_bf2(p2, p3);
+        if (scores) {
+            *reinterpret_cast<uint32_t*>(ps + g * LP + warp * 8 + 2 * tq) = pack_bf2(p0, p1);
+            *reinterpret_cast<uint32_t*>(ps + (g + 8) * LP + warp * 8 + 2 * tq) = pack_bf2(p2, p3);
+        }
         __syncthreads();
-        uint32_t pa[2][4];
+        uint32_t pa[KB / 16][4];
 #pragma unroll
-        for (int kk = 0; kk < 2; kk++) ldsm_x4(pa[kk], smem_u32(ps + (lane & 15) * 40 + (lane >> 4) * 8 + kk * 16));
+        for (int kk = 0; kk < KB / 16; kk++) ldsm_x4(pa[kk], smem_u32(ps + (lane & 15) * LP + (lane >> 4) * 8 + kk * 16));
 #pragma unroll
         for (int i = 0; i < NG; i++) {
-            const uint32_t grp = warp + 4 * i;
+            const uint32_t grp = warp + 8 * i;
             if (grp >= ngroups) break;
             o[i][0] *= f_a; o[i][1] *= f_a; o[i][2] *= f_b; o[i][3] *= f_b;
             o[i][4] *= f_a; o[i][5] *= f_a; o[i][6] *= f_b; o[i][7] *= f_b;
 #pragma unroll
-            for (int kk = 0; kk < 2; kk++) {
+            for (int kk = 0; kk < KB / 16; kk++) {
                 // 16 keys x 16 columns: transposed tiles (keys 0-7 | 8-15) x (columns 0-7 | 8-15)
                 uint32_t v[4];
                 ldsm_x4_trans(v, smem_u32(kb + (kk * 16 + (lane & 15)) * ld + grp * 16 + (lane >> 4) * 8));
@@ -301,22 +321,28 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const Dims d, const fl
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
     if (tq == 0) { wl[warp][g] = l_a; wl[warp][g + 8] = l_b; }
     __syncthreads();
+    auto sum_l = [&](uint32_t r) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; i++) s += wl[i][r];
+        return s;
+    };
     if (warp == 0 && tq == 0) {
         if (ra < rows) {
             float* p = part_ml + ((size_t)ra * nsplit + split) * 2;
             p[0] = m_a;
-            p[1] = wl[0][g] + wl[1][g] + wl[2][g] + wl[3][g];
+            p[1] = sum_l(g);
         }
         if (rb < rows) {
             float* p = part_ml + ((size_t)rb * nsplit + split) * 2;
             p[0] = m_b;
-            p[1] = wl[0][g + 8] + wl[1][g + 8] + wl[2][g + 8] + wl[3][g + 8];
+            p[1] = sum_l(g + 8);
         }
     }
     if (!nblk) return;         // an empty split: its maximum is -inf and its sums are not read
 #pragma unroll
     for (int i = 0; i < NG; i++) {
-        const uint32_t grp = warp + 4 * i;
+        const uint32_t grp = warp + 8 * i;
         if (grp >= ngroups) break;
         const uint32_t col = grp * 16 + 2 * tq;
         if (ra < rows) {
@@ -398,8 +424,9 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const Dims d, const f
                                                             uint32_t nsplit, const __nv_bfloat16* __restrict__ w_uv, uint32_t ldk,
                                                             TO* __restrict__ out, uint32_t ldo) {
     extern __shared__ __align__(16) uint8_t smem[];
-    float* c = reinterpret_cast<float*>(smem);             // [cp]
-    float* wt = c + d.cp;                                  // [nsplit]
+    float* c = reinterpret_cast<float*>(smem);             // [max(1024, cp)]: shares of the merged latent
+    float* wt = c + (d.cp < 1024 ? 1024 : d.cp);           // [nsplit]
+    __shared__ uint32_t live_s;
     const uint32_t h = blockIdx.x, t = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t j0 = blockIdx.y * 32 + warp * 4, nch = (d.rank + 7) / 8;
     const uint4* w = reinterpret_cast<const uint4*>(w_uv + (size_t)(h * d.vdim + j0) * ldk);
@@ -415,27 +442,59 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const Dims d, const f
     const size_t row = (size_t)t * d.heads + h;
     if (warp == 0) {
         float M = -INFINITY, L = 0.f;
-        for (uint32_t s = lane; s < nsplit; s += 32) M = fmaxf(M, part_ml[(row * nsplit + s) * 2]);
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+        uint32_t live = 0;
         for (uint32_t s = lane; s < nsplit; s += 32) {
-            const float m = part_ml[(row * nsplit + s) * 2], f = m == -INFINITY ? 0.f : expf(m - M);
+            const float m = part_ml[(row * nsplit + s) * 2];
+            M = fmaxf(M, m);
+            if (m != -INFINITY) live = s + 1;         // the splits in which the row sees keys are the first ones
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+            live = max(live, __shfl_xor_sync(0xffffffffu, live, o));
+        }
+        for (uint32_t s = lane; s < live; s += 32) {
+            const float2 ml = *reinterpret_cast<const float2*>(part_ml + (row * nsplit + s) * 2);
+            const float f = expf(ml.x - M);
             wt[s] = f;
-            L = fmaf(f, part_ml[(row * nsplit + s) * 2 + 1], L);
+            L = fmaf(f, ml.y, L);
         }
         L = wsum(L);
-        for (uint32_t s = lane; s < nsplit; s += 32) wt[s] /= L;
+        for (uint32_t s = lane; s < live; s += 32) wt[s] /= L;
+        if (lane == 0) live_s = live;
     }
     __syncthreads();
-    for (uint32_t i = threadIdx.x; i < d.cp; i += 256) {
-        float v = 0.f;
-        for (uint32_t s = 0; s < nsplit; s++) {
-            const float f = wt[s];
-            if (f != 0.f) v = fmaf(f, part_o[(row * nsplit + s) * d.cp + i], v);
+    // weighted sum of the splits' rows: thread = 4 columns x every G-th split, eight loads in flight; shares added in order
+    const uint32_t c4 = d.cp / 4, G = c4 < 256 ? 256 / c4 : 1, live = live_s;
+    for (uint32_t i = threadIdx.x; i < G * c4; i += 256) {
+        const uint32_t grp = i / c4, col = i - grp * c4;
+        const float4* p = reinterpret_cast<const float4*>(part_o + row * nsplit * d.cp) + col;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (uint32_t s0 = grp; s0 < live; s0 += 8 * G) {
+            float4 x[8];
+#pragma unroll
+            for (int k = 0; k < 8; k++) {
+                const uint32_t s = s0 + k * G;
+                x[k] = s < live ? p[(size_t)s * c4] : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int k = 0; k < 8; k++) {
+                const uint32_t s = s0 + k * G;
+                const float f = s < live ? wt[s] : 0.f;
+                v.x = fmaf(f, x[k].x, v.x); v.y = fmaf(f, x[k].y, v.y); v.z = fmaf(f, x[k].z, v.z); v.w = fmaf(f, x[k].w, v.w);
+            }
         }
-        c[i] = v;
+        reinterpret_cast<float4*>(c)[grp * c4 + col] = v;
     }
     __syncthreads();
+    if (G > 1) {
+        for (uint32_t i = threadIdx.x; i < d.cp; i += 256) {
+            float v = c[i];
+            for (uint32_t k = 1; k < G; k++) v += c[k * d.cp + i];
+            c[i] = v;
+        }
+        __syncthreads();
+    }
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     auto step = [&](const uint4& v, uint32_t ch, float a) {
         const float4 x0 = *reinterpret_cast<const float4*>(c + ch * 8), x1 = *reinterpret_cast<const float4*>(c + ch * 8 + 4);
@@ -611,7 +670,7 @@ static int32_t allow_smem(runit_ctx* ctx, const char* name, K kern, size_t smem)
 using namespace la;
 
 int32_t latent_query(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const float* qkv, uint32_t ldq, const void* w_uk, uint32_t ldk,
-                     const float* kv_norm, const float* freq, void* cache, float* q_eff, uint32_t T, LatentPos pos) {
+                     const float* kv_norm, const float* freq, void* cache, void* q_eff, uint32_t T, LatentPos pos) {
     const uint32_t nchunk = (d.cp() + 63) / 64;
     const dim3 grid(d.heads * nchunk + (kv_norm ? 1 : 0), T);
     if (cache_f32)
@@ -637,7 +696,7 @@ uint32_t latent_splits(const runit_ctx* ctx, const LatentDims& d, bool cache_f32
     return n < 1 ? 1u : (n > 64 ? 64u : (uint32_t)n);
 }
 
-int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const float* q_eff, const void* cache, float* part_o,
+int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, const void* q_eff, const void* cache, float* part_o,
                          float* part_ml, uint32_t nsplit, uint32_t T, LatentPos pos) {
     const uint32_t rows = T * d.heads;
     int32_t st;
@@ -645,7 +704,7 @@ int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, co
         const size_t smem = (size_t)(d.pitch() + 4 * d.cp()) * 4;
         auto go = [&](auto kern) -> int32_t {
             if ((st = allow_smem(ctx, "latent_attention", kern, smem)) != RUNIT_OK) return st;
-            runit_launch_chain_smem(ctx, kern, dim3(rows, nsplit), dim3(128), smem, dims_of(d), q_eff, (const float*)cache, part_o, part_ml, pos);
+            runit_launch_chain_smem(ctx, kern, dim3(rows, nsplit), dim3(128), smem, dims_of(d), (const float*)q_eff, (const float*)cache, part_o, part_ml, pos);
             return runit_after_launch(ctx, "latent_attention_f32");
         };
         if (d.cp() <= 128) return go(latent_attn_f32_kernel<4>);
@@ -653,23 +712,27 @@ int32_t latent_attention(runit_ctx* ctx, const LatentDims& d, bool cache_f32, co
         RUNIT_REQUIRE(ctx, d.cp() <= 1024, "latent_attention: a latent of more than 1024 values");
         return go(latent_attn_f32_kernel<32>);
     }
-    const size_t ld = d.pitch() + 8, smem = (32 * ld + 2 * kKB * ld + 16 * 40) * 2;
-    auto go = [&](auto kern) -> int32_t {
+    const size_t ld = d.pitch() + 8;
+    auto go = [&](auto kern, size_t kb) -> int32_t {
+        const size_t smem = (32 * ld + 2 * kb * ld + 16 * (kb + 8)) * 2;
         if ((st = allow_smem(ctx, "latent_attention", kern, smem)) != RUNIT_OK) return st;
-        runit_launch_chain_smem(ctx, kern, dim3((rows + 15) / 16, nsplit), dim3(128), smem, dims_of(d), q_eff, (const __nv_bfloat16*)cache, part_o,
-                                part_ml, rows, pos);
+        runit_launch_chain_smem(ctx, kern, dim3((rows + 15) / 16, nsplit), dim3(256), smem, dims_of(d), (const __nv_bfloat16*)q_eff,
+                                (const __nv_bfloat16*)cache, (float*)part_o, (float*)part_ml, rows, pos);
         return runit_after_launch(ctx, "latent_attention");
     };
-    if (d.cp() <= 128) return go(latent_attn_kernel<2>);
-    if (d.cp() <= 512) return go(latent_attn_kernel<8>);
     RUNIT_REQUIRE(ctx, d.cp() <= 1024, "latent_attention: a latent of more than 1024 values");
-    return go(latent_attn_kernel<16>);
+    if (d.pitch() <= 672) {
+        if (d.cp() <= 128) return go(latent_attn_kernel<1, 64>, 64);
+        if (d.cp() <= 512) return go(latent_attn_kernel<4, 64>, 64);
+        return go(latent_attn_kernel<8, 64>, 64);
+    }
+    return go(latent_attn_kernel<8, 32>, 32);
 }
 
 int32_t latent_value(runit_ctx* ctx, const LatentDims& d, const float* part_o, const float* part_ml, uint32_t nsplit, const void* w_uv,
                      uint32_t ldk, void* out, bool out_f32, uint32_t ldo, uint32_t T) {
     const dim3 grid(d.heads, (d.vdim + 31) / 32, T);
-    const size_t smem = (size_t)(d.cp() + nsplit) * 4;
+    const size_t smem = (size_t)((d.cp() < 1024 ? 1024 : d.cp()) + nsplit) * 4;
     if (out_f32)
         runit_launch_chain_smem(ctx, latent_value_kernel<float>, grid, dim3(256), smem, dims_of(d), part_o, part_ml, nsplit,
                                 (const __nv_bfloat16*)w_uv, ldk, (float*)out, ldo);
@@ -725,7 +788,7 @@ int32_t runit_latent_query(runit_ctx_t* ctx, const runit_latent_cfg* cfg, int32_
     if (st != RUNIT_OK) return st;
     RUNIT_REQUIRE(ctx, qkv && w_uk && freq && cache && q_eff && ldq >= d.q_width() + (kv_norm ? d.kv_rank + d.rot_dim : 0), "latent_query: bad argument");
     return latent_query(ctx, d, cache_f32 != 0, (const float*)qkv, ldq, w_uk, pad8(d.kv_rank), (const float*)kv_norm, (const float*)freq, cache,
-                        (float*)q_eff, T, LatentPos{nullptr, start});
+                        q_eff, T, LatentPos{nullptr, start});
 }
 
 int32_t runit_latent_attention(runit_ctx_t* ctx, const runit_latent_cfg* cfg, int32_t cache_f32, const void* q_eff, const void* cache,
@@ -735,7 +798,7 @@ int32_t runit_latent_attention(runit_ctx_t* ctx, const runit_latent_cfg* cfg, in
     int32_t st = latent_check(ctx, "latent_attention", cfg, &d, T);
     if (st != RUNIT_OK) return st;
     RUNIT_REQUIRE(ctx, q_eff && cache && part_o && part_ml && nsplit > 0 && nsplit <= 1024, "latent_attention: bad argument");
-    return latent_attention(ctx, d, cache_f32 != 0, (const float*)q_eff, cache, (float*)part_o, (float*)part_ml, nsplit, T, LatentPos{nullptr, start});
+    return latent_attention(ctx, d, cache_f32 != 0, q_eff, cache, (float*)part_o, (float*)part_ml, nsplit, T, LatentPos{nullptr, start});
 }
 
 int32_t runit_latent_value(runit_ctx_t* ctx, const runit_latent_cfg* cfg, const void* part_o, const void* part_ml, uint32_t nsplit,

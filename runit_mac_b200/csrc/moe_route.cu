@@ -394,10 +394,16 @@ __global__ void __launch_bounds__(256) route_gated_kernel(const float* __restric
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r = blockIdx.x * 8 + warp;
     const float g = *gain;
     const float* wrow = w + (size_t)r * K;
+    const bool vec = (K & 3u) == 0;
+    const float4* w4 = reinterpret_cast<const float4*>(wrow);
     // the first part of the row does not depend on the previous kernel of the chain: requested before the wait
-    float wv[16];
+    constexpr int P = 16;
+    float4 wv[P];
 #pragma unroll
-    for (int i = 0; i < 16; i++) wv[i] = (r < R && lane + 32 * i < K) ? wrow[lane + 32 * i] : 0.f;
+    for (int i = 0; i < P; i++) {
+        const uint32_t c = lane + 32 * i;
+        wv[i] = (vec && r < R && c < K / 4) ? __ldg(w4 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     grid_dependency_wait();
     grid_launch_dependents();
     float sq = 0.f;
@@ -418,10 +424,19 @@ __global__ void __launch_bounds__(256) route_gated_kernel(const float* __restric
         for (uint32_t i = threadIdx.x; i < K; i += 256) xn_out[i] = xs[i] * sc;
     if (r < R) {
         float acc = 0.f;
+        if (vec) {
+            const float4* x4 = reinterpret_cast<const float4*>(xs);
+            auto step = [&](const float4& a, const float4& v) {
+                acc = fmaf(a.x, v.x, acc); acc = fmaf(a.y, v.y, acc); acc = fmaf(a.z, v.z, acc); acc = fmaf(a.w, v.w, acc);
+            };
 #pragma unroll
-        for (int i = 0; i < 16; i++)
-            if (lane + 32 * i < K) acc = fmaf(wv[i], xs[lane + 32 * i], acc);
-        for (uint32_t c = lane + 512; c < K; c += 32) acc = fmaf(wrow[c], xs[c], acc);
+            for (int i = 0; i < P; i++)
+                if (lane + 32 * i < K / 4) step(wv[i], x4[lane + 32 * i]);
+#pragma unroll 8
+            for (uint32_t c = lane + 32 * P; c < K / 4; c += 32) step(__ldg(w4 + c), x4[c]);
+        } else {
+            for (uint32_t c = lane; c < K; c += 32) acc = fmaf(wrow[c], xs[c], acc);
+        }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
         if (lane == 0) {

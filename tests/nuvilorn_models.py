@@ -112,3 +112,21 @@ def row_errors(got, ref):
     d = np.asarray(got, np.float64) - ref
     d -= d.mean(-1, keepdims=True)
     return np.sqrt((d * d).mean(-1)) / np.std(ref)
+
+
+def routing_margins(cfg, w, toks):
+    """Per token the smallest distance, over the layers, between the logits of the last chosen and the first left-out expert."""
+    out = np.full(len(toks), np.inf)
+    real = N.route_sigmoid
+
+    def watch(h, w_router, top):
+        z = -np.sort(-(h @ w_router.T), axis=-1)
+        if top < z.shape[1]:
+            out[:] = np.minimum(out, z[:, top - 1] - z[:, top])
+        return real(h, w_router, top)
+    N.route_sigmoid = watch
+    try:
+        N.forward(cfg, w, toks)
+    finally:
+        N.route_sigmoid = real
+    return out

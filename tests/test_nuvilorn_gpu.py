@@ -21,9 +21,10 @@ def bf16_rows(a):
 
 
 def close(got, ref, tol):
+    """Within tol of the larger of the value itself and the root mean square."""
     got, ref = np.asarray(got, np.float64), np.asarray(ref, np.float64)
     assert np.isfinite(got).all()
-    err = np.abs(got - ref).max() / max(np.sqrt((ref ** 2).mean()), 1e-30)
+    err = (np.abs(got - ref) / np.maximum(np.abs(ref), max(np.sqrt((ref ** 2).mean()), 1e-30))).max()
     assert err <= tol, err
 
 
@@ -90,7 +91,7 @@ def test_gemm(ctx, T, m, k):
             ctx.flush()
             f32 = exact or epi in (R.EPI_F32, R.EPI_ADD)
             got = y.download(np.float32, T * n) if f32 else N.from_bf16(y.download(np.uint16, T * n))
-            close(got.reshape(T, n), ref, 3e-5 if f32 else 4e-2)
+            close(got.reshape(T, n), ref, 3e-5 if f32 else 1e-2)
 
 
 def test_gemm_repeats_bit_for_bit(ctx):
@@ -133,7 +134,7 @@ def _latent_case(mix, T, start, seed, f32, spike=None):
     raw = g.normal(size=(n, rank + r)).astype(np.float32)
     q = g.normal(size=(n, H * (d + r))).astype(np.float32)
     if spike is not None:                             # a query whose scores stand out
-        q[spike] *= 6.0
+        q[spike] *= 3.0
     kvn = g.uniform(0.5, 1.5, rank).astype(np.float32)
     uk_u, uk = bf16_rows(g.normal(size=(H * d, rank)) / np.sqrt(rank))
     uv_u, uv = bf16_rows(g.normal(size=(H * dv, rank)) / np.sqrt(rank))
@@ -187,7 +188,7 @@ def test_expanded_attention(ctx, H, d, r, dv, rank, T, start):
     import runit_mac_b200 as R
     mix = M.mixer(H, d, r, dv, rank, scale=0.5)
     # the last query points sharply at its keys: a key that is dropped or let in shows
-    raw, q, kvn, uk, uv, ref, p = _latent_case(mix, T, start, T, 0, spike=start + T - 1)
+    raw, q, kvn, uk, uv, _, _ = _latent_case(mix, T, start, T, 0, spike=start + T - 1)
     n, cp = start + T, (rank + 15) // 16 * 16
     pitch, ldq = cp + (r + 15) // 16 * 16, H * (d + r) + rank + r
     cfg = R.LatentCfg(H, d, r, dv, rank, 0.5, 1e-5)
@@ -199,11 +200,17 @@ def test_expanded_attention(ctx, H, d, r, dv, rank, T, start):
     lat = N.from_bf16(cache.download(np.uint16, n * pitch)).reshape(n, pitch)[:, :rank].astype(np.float64)
     ukv = np.concatenate([uk, uv]).astype(np.uint16)
     w = N.from_bf16(ukv)[:, :rank].astype(np.float64)
-    kv, _ = bf16_rows(lat @ w.T)
+    kv, kvv = bf16_rows(lat @ w.T)
     ldo = (H * dv + 7) // 8 * 8
     out = ctx.new_buffer(T * ldo * 2)
     R.latent_prefill_attention(ctx, C.byref(cfg), qkv.ptr + start * ldq * 4, ldq, ctx.buffer_from(kv), kv.shape[1], cache, out, ldo, T, start)
     ctx.flush()
+    # the plain result from the same expanded keys and values
+    rows = N.from_bf16(cache.download(np.uint16, n * pitch)).reshape(n, pitch).astype(np.float64)
+    qq = q.reshape(n, H, d + r).astype(np.float64)
+    q_rot = N.rotate_interleaved(qq[..., d:], np.arange(n), r, mix["rot"]["base"])
+    s = np.einsum("ihd,jhd->hij", qq[..., :d], kvv[:, :H * d].reshape(n, H, d)) + np.einsum("ihd,jd->hij", q_rot, rows[:, cp:cp + r])
+    ref = np.einsum("hij,jhd->ihd", N.causal_softmax(s * 0.5), kvv[:, H * d:].reshape(n, H, dv)).reshape(n, H * dv)[start:]
     close(N.from_bf16(out.download(np.uint16, T * ldo)).reshape(T, ldo)[:, :H * dv], ref, 6e-2)
 
 
@@ -231,13 +238,15 @@ def dtype(request):
     return request.param
 
 
-def check_rows(got, ref, dtype):
+def check_rows(got, ref, dtype, margins=None):
+    """margins (bf16): tokens whose routing is a close call may go to another expert than in the plain implementation."""
     e = M.row_errors(got, ref)
     if dtype == "float32":
         assert e.max() <= EXACT, e.max()
-    else:      # a close call of a router may send a token elsewhere: few rows may be off
-        assert np.median(e) <= 0.02 and (e > 0.08).mean() <= 0.08, (np.median(e), np.sort(e)[-5:])
-    return e
+        return
+    clear = e if margins is None else e[margins[:len(e)] > 0.2]
+    if len(clear):
+        assert np.median(clear) <= 0.02 and (clear > 0.08).mean() <= 0.02, (np.median(clear), np.sort(clear)[-5:])
 
 
 @pytest.mark.parametrize("name", sorted(M.CONFIGS))
@@ -245,17 +254,17 @@ def check_rows(got, ref, dtype):
 def test_prompt(ctx, tmp_path, dtype, name, n):
     s = Served(ctx, tmp_path, M.CONFIGS[name], dtype)
     t = M.tokens(s.cfg, n)
-    check_rows(s.run(t, [n]), N.forward(s.cfg, s.w, t), dtype)
+    check_rows(s.run(t, [n]), N.forward(s.cfg, s.w, t), dtype, M.routing_margins(s.cfg, s.w, t))
 
 
 @pytest.mark.parametrize("name", sorted(M.CONFIGS))
 def test_prefill_against_token_by_token_and_portions(ctx, tmp_path, dtype, name):
     s = Served(ctx, tmp_path, M.CONFIGS[name], dtype, gain=2.0)
     t = M.tokens(s.cfg, 100)
-    ref = N.forward(s.cfg, s.w, t)
+    ref, mg = N.forward(s.cfg, s.w, t), M.routing_margins(s.cfg, s.w, t)
     whole = s.run(t, [100])
     for cuts in ([1], [2], [3, 2], [31, 1, 33], [64, 36], [99, 1], [7, 50, 2]):
-        check_rows(s.run(t, cuts), ref, dtype)
+        check_rows(s.run(t, cuts), ref, dtype, mg)
     if dtype == "float32":
         assert M.row_errors(s.run(t, [1]), whole).max() <= EXACT
 
@@ -293,9 +302,9 @@ def test_mechanism_alone(ctx, tmp_path, dtype, name):
             w["l0.mix.o"][:] = 0
     s = Served(ctx, tmp_path, cfg, dtype, edit=edit)
     t = M.tokens(cfg, 60)
-    ref = N.forward(cfg, s.w, t)
-    check_rows(s.run(t, [60]), ref, dtype)
-    check_rows(s.run(t, [1]), ref, dtype)
+    ref, mg = N.forward(cfg, s.w, t), M.routing_margins(cfg, s.w, t)
+    check_rows(s.run(t, [60]), ref, dtype, mg)
+    check_rows(s.run(t, [1]), ref, dtype, mg)
 
 
 def _only(monkeypatch, name, fault):
@@ -399,15 +408,15 @@ def test_cache_is_reused_and_cut_back(ctx, tmp_path, dtype):
     """Another sequence after the first, a shorter one after a longer one, and a sequence taken up again from the middle."""
     s = Served(ctx, tmp_path, M.CONFIGS["mixed"], dtype)
     a, b = M.tokens(s.cfg, 120, 5), M.tokens(s.cfg, 50, 6)
-    ra = N.forward(s.cfg, s.w, a)
-    check_rows(s.run(a, [120]), ra, dtype)
-    check_rows(s.run(b, [20, 1, 29]), N.forward(s.cfg, s.w, b), dtype)
-    first = s.run(a, [60, 1])
-    check_rows(first, ra, dtype)
+    ra, mg = N.forward(s.cfg, s.w, a), lambda t: M.routing_margins(s.cfg, s.w, t)
+    ma = mg(a)
+    check_rows(s.run(a, [120]), ra, dtype, ma)
+    check_rows(s.run(b, [20, 1, 29]), N.forward(s.cfg, s.w, b), dtype, mg(b))
+    check_rows(s.run(a, [60, 1]), ra, dtype, ma)
     mixed = a[:40] + b[:30]
     got = s.m.forward(mixed[40:], 40, range(30))          # positions 40.. are overwritten
-    check_rows(got, N.forward(s.cfg, s.w, mixed)[40:], dtype)
-    check_rows(s.run(a, [17]), ra, dtype)
+    check_rows(got, N.forward(s.cfg, s.w, mixed)[40:], dtype, mg(mixed)[40:])
+    check_rows(s.run(a, [17]), ra, dtype, ma)
 
 
 def test_long_prompt_is_cut_inside(ctx, tmp_path, dtype):
@@ -450,7 +459,7 @@ def test_greedy_generation(ctx, tmp_path):
         seq.append(got[-1])
     assert got == ref[:5]
     # portions continue from where generation left the cache
-    lg = s.m.forward(ref[5:8], len(p) + 5, [2])
+    lg = s.m.forward(ref[4:8], len(p) + 4, [3])
     assert int(np.argmax(lg[0])) == ref[8]
 
 
