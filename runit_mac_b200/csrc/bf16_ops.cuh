@@ -80,10 +80,10 @@ uint32_t gemm_bf16_tile_tok(uint32_t tokens_per_expert, bool exact);
 // x[t] = RMSNorm(embed[token[t]]) * gain; tokens == nullptr: one row, the step's token (state, forced; see model_core.h)
 int32_t embed_norm_rows(runit_ctx* ctx, const void* embed, uint32_t ld, const int32_t* tokens, const int32_t* state, const int32_t* forced,
                         uint32_t n_forced, uint32_t vocab, const float* gain, float eps, float* x, uint32_t T, uint32_t width);
-// y = RMSNorm(x[rows]) * gain as bf16 or f32 rows of ldy elements (padding zero), and f32 rows of `width` in y2 when it is not null
+// y = RMSNorm(x[rows]) * gain as bf16 or f32 rows of ldy elements (padding zero), and f32 rows of `width` in y2 when it is not
+// null; gate_row not null: gate_out[t] = sigmoid(gate_row . y[t])
 int32_t norm_rows(runit_ctx* ctx, const float* x, const int32_t* row_index, const float* gain, float eps, void* y, bool y_f32, uint32_t ldy,
-                  float* y2, uint32_t T, uint32_t width);
-int32_t sigmoid_column(runit_ctx* ctx, const float* logits, uint32_t ld, uint32_t col, float* out, uint32_t T);
+                  float* y2, uint32_t T, uint32_t width, const float* gate_row = nullptr, float* gate_out = nullptr);
 
 // ── latent attention ──
 // Keys and values of all heads come from one cached row per position: the normed latent c (kv_rank values, padded to a

@@ -69,6 +69,31 @@ __device__ __forceinline__ float relu2(float v) {
     return v * v;
 }
 
+// Lane l of a quad holds v[0..3] = its row's values of tokens 0..3; afterwards y[0..3] = the quad's four rows of token l & 3.
+__device__ __forceinline__ void quad_transpose(const uint32_t* v, float (&y)[4], bool odd, bool high) {
+    const uint32_t a = __shfl_xor_sync(0xffffffffu, odd ? v[0] : v[1], 1), b = __shfl_xor_sync(0xffffffffu, odd ? v[2] : v[3], 1);
+    // even lanes: rows (0, 1) of tokens 0 and 2; odd lanes: of tokens 1 and 3
+    const uint32_t p0 = odd ? a : v[0], p1 = odd ? v[1] : a, q0 = odd ? b : v[2], q1 = odd ? v[3] : b;
+    const uint32_t c = __shfl_xor_sync(0xffffffffu, high ? p0 : q0, 2), d = __shfl_xor_sync(0xffffffffu, high ? p1 : q1, 2);
+    y[0] = __uint_as_float(high ? c : p0);
+    y[1] = __uint_as_float(high ? d : p1);
+    y[2] = __uint_as_float(high ? q0 : c);
+    y[3] = __uint_as_float(high ? q1 : d);
+}
+// N neighbouring outputs of one token, `left` of them inside the matrix
+template <int N>
+__device__ __forceinline__ void store_rows(__nv_bfloat16* o, const float (&y)[4], uint32_t left, uint32_t ldo) {
+    if (left >= N && ldo % N == 0) {
+        __nv_bfloat162 p[N / 2];
+#pragma unroll
+        for (int i = 0; i < N / 2; i++) p[i] = __floats2bfloat162_rn(y[2 * i], y[2 * i + 1]);
+        if constexpr (N == 4) *reinterpret_cast<uint2*>(o) = *reinterpret_cast<const uint2*>(p);
+        else *reinterpret_cast<uint32_t*>(o) = *reinterpret_cast<const uint32_t*>(p);
+    } else {
+        for (uint32_t i = 0; i < N && i < left; i++) o[i] = __float2bfloat16_rn(y[i]);
+    }
+}
+
 constexpr int kThreads = 192, kRowsTile = 128, kABytes = kRowsTile * 128;
 template <int NT>
 struct Cfg {
@@ -176,19 +201,36 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 tmem_ld32(taddr + cg * 32, v);
                 tmem_ld_wait();
                 const uint32_t tok0 = t.row0 + cg * 32, cnt = min(32u, t.nvalid - cg * 32);
-                if constexpr (EPI == EPI_SILU_GLU) {
-                    // lanes 2i, 2i+1 hold gate and up of output i: the even lane finishes token j, the odd one token j + 1
+                if constexpr (EPI == EPI_SILU_GLU || EPI == EPI_RELU2 || EPI == EPI_CAST) {
+                    // Four lanes exchange their values of four tokens, so that each holds four neighbouring rows of one token: one
+                    // wide store and one pair of factors instead of four.
                     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out);
-                    const bool odd = lane & 1;
+                    const bool odd = lane & 1, high = lane & 2;
+                    const uint32_t r4 = r & ~3u;
 #pragma unroll
-                    for (int j = 0; j < 32; j += 2) {
-                        const float v0 = __uint_as_float(v[j]), v1 = __uint_as_float(v[j + 1]);
-                        const float got = __shfl_xor_sync(0xffffffffu, odd ? v0 : v1, 1);
-                        const uint32_t jj = j + (odd ? 1 : 0);
-                        if (live && jj < cnt) {
-                            const float pre = a.pre ? a.pre[tok0 + jj] : 1.f, post = a.post ? a.post[tok0 + jj] : 1.f;
-                            const float g = (odd ? got : v0) * pre, u = (odd ? v1 : got) * pre;
-                            out[(size_t)(tok0 + jj) * a.ldo + (r >> 1)] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u * post);
+                    for (int j = 0; j < 32; j += 4) {
+                        float y[4];
+                        quad_transpose(v + j, y, odd, high);
+                        const uint32_t jj = j + (lane & 3);
+                        if (jj >= cnt || r4 >= a.rows) continue;
+                        const uint32_t tok = tok0 + jj;
+                        __nv_bfloat16* o = out + (size_t)tok * a.ldo;
+                        if constexpr (EPI == EPI_CAST) {
+                            store_rows<4>(o + r4, y, a.rows - r4, a.ldo);
+                        } else {
+                            const float pre = a.pre ? a.pre[tok] : 1.f, post = a.post ? a.post[tok] : 1.f;
+                            if constexpr (EPI == EPI_SILU_GLU) {      // rows 2i, 2i+1: gate and up of output i
+#pragma unroll
+                                for (int i = 0; i < 2; i++) {
+                                    const float g = y[2 * i] * pre, u = y[2 * i + 1] * pre;
+                                    y[i] = __fdividef(g, 1.0f + __expf(-g)) * u * post;
+                                }
+                                store_rows<2>(o + r4 / 2, y, (a.rows - r4) / 2, a.ldo);
+                            } else {
+#pragma unroll
+                                for (int i = 0; i < 4; i++) y[i] = relu2(y[i] * pre) * post;
+                                store_rows<4>(o + r4, y, a.rows - r4, a.ldo);
+                            }
                         }
                     }
                 } else if constexpr (EPI == EPI_ADD) {
@@ -206,12 +248,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         if (!live || (uint32_t)j >= cnt) continue;
                         const float f = __uint_as_float(v[j]);
                         const size_t o = (size_t)(tok0 + j) * a.ldo + r;
-                        if constexpr (EPI == EPI_F32) reinterpret_cast<float*>(a.out)[o] = f;
-                        else if constexpr (EPI == EPI_CAST) reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16_rn(f);
-                        else {
-                            const float pre = a.pre ? a.pre[tok0 + j] : 1.f, post = a.post ? a.post[tok0 + j] : 1.f;
-                            reinterpret_cast<__nv_bfloat16*>(a.out)[o] = __float2bfloat16_rn(relu2(f * pre) * post);
-                        }
+                        reinterpret_cast<float*>(a.out)[o] = f;
                     }
                 }
             }

@@ -1,8 +1,8 @@
 // One-token operators of decoders with bf16 weights: GEMV with the norm in front and the activation behind fused in, and the
 // row operators of a pass (embedding, norms with one gain for all coordinates).
 //
-// A warp owns 1, 2 or 4 weight rows (rows 2i and 2i+1 together for a gated block) and keeps eight 16-byte loads per lane in
-// flight; the first group of them does not depend on the previous kernel of the chain and is requested before the dependency
+// A warp owns 1, 2 or 4 weight rows (rows 2i and 2i+1 together for a gated block) and keeps eight to sixteen 16-byte loads per
+// lane in flight; the first group of them does not depend on the previous kernel of the chain and is requested before the dependency
 // wait.  The input vector is staged in shared memory as f32; the norm's factor multiplies the dot product (the gain is one
 // number), so the vector is read once.  Sums are f32.
 #include "bf16_ops.cuh"
@@ -13,7 +13,6 @@ namespace runit {
 namespace gv {
 
 constexpr int kWarps = 8;
-constexpr int kLoads = 8;      // 16-byte loads per lane and group
 
 __device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
 __device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
@@ -76,9 +75,9 @@ struct Args {
     const float* post_extra;
 };
 
-template <int EPI, int RPU, bool SLOTS>
+// RPU: rows of a warp's unit; U: 16-byte loads per lane, row and group
+template <int EPI, int RPU, int U, bool SLOTS>
 __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
-    constexpr int U = kLoads / RPU;
     extern __shared__ __align__(16) float4 smem4[];
     __shared__ float part[kWarps];
     __shared__ unsigned long long best_s[kWarps];
@@ -207,11 +206,10 @@ struct SumArgs {
     float* out;
 };
 
-// The inputs of all slots lie one after the other in shared memory, each padded to chunks of eight; a lane walks the chunks of
-// all slots as one list, so the loads of small blocks are in flight together.
-template <int RPU>
+// The inputs of all slots lie one after the other in shared memory, each padded to chunks of eight.  A warp walks steps of 32
+// chunks of one slot after the other, U steps in flight, so the loads of small blocks overlap across slots.
+template <int RPU, int U>
 __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_sum_kernel(const SumArgs a) {
-    constexpr int U = kLoads / RPU;
     extern __shared__ __align__(16) float4 smem4[];
     __shared__ const uint8_t* base_s[33];
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -223,53 +221,82 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_sum_kernel(const SumArg
         const int32_t e = a.slot_expert ? a.slot_expert[threadIdx.x] : 0;
         base_s[threadIdx.x] = e < 0 ? nullptr : a.w + (size_t)e * a.rows * a.ldw * 2;
     }
+    if (threadIdx.x == a.n_routed) base_s[threadIdx.x] = a.w_extra;
     __syncthreads();
     const uint32_t units = (a.rows + RPU - 1) / RPU;
+    const uint32_t steps_s = (chs + 31) / 32, steps = a.n_routed * steps_s + (chx + 31) / 32;
     uint32_t unit = blockIdx.x * kWarps + warp;
     uint4 v[RPU][U];
-    auto load = [&](uint32_t u, uint32_t c0) {
+    uint32_t slot = 0, k = 0;                     // position of the next step to load
+    uint32_t fslot = 0, fk = 0;                   // and of the next step to multiply
+    auto advance = [&](uint32_t& s, uint32_t& kk) {
+        if (++kk == steps_s && s < a.n_routed) { kk = 0; s++; }
+    };
+    auto load = [&](uint32_t u, uint32_t s0) {
 #pragma unroll
         for (int i = 0; i < U; i++) {
-            const uint32_t c = c0 + 32 * i + lane;
-            const uint8_t* p = nullptr;
-            size_t pitch = 0;
-            if (c < routed) {
-                const uint32_t s = c / chs;
-                pitch = (size_t)a.ldw * 2;
-                if (base_s[s]) p = base_s[s] + (size_t)(c - s * chs) * 16;
-            } else if (c < total) {
-                pitch = (size_t)a.ldw_extra * 2;
-                p = a.w_extra + (size_t)(c - routed) * 16;
-            }
+            const bool extra = slot == a.n_routed;
+            const uint32_t c = k * 32 + lane, n = extra ? chx : chs, pitch = (extra ? a.ldw_extra : a.ldw) * 2;
+            const uint8_t* p = (s0 + i < steps && c < n) ? base_s[slot] : nullptr;
 #pragma unroll
             for (int r = 0; r < RPU; r++) {
                 const uint32_t row = u * RPU + r;
-                v[r][i] = (p && row < a.rows) ? __ldg(reinterpret_cast<const uint4*>(p + row * pitch)) : make_uint4(0, 0, 0, 0);
+                v[r][i] = (p && row < a.rows) ? __ldg(reinterpret_cast<const uint4*>(p + (size_t)row * pitch) + c) : make_uint4(0, 0, 0, 0);
             }
+            advance(slot, k);
         }
     };
     if (unit < units) load(unit, 0);
     grid_dependency_wait();
     grid_launch_dependents();
-    for (uint32_t s = 0; s < a.n_routed; s++) stage_x(a.x + (size_t)s * a.x_stride, a.K, chs, xa + s * chs, xb + s * chs);
-    if (chx) stage_x(a.x + (size_t)a.n_routed * a.x_stride, a.K_extra, chx, xa + routed, xb + routed);
+    // inputs: four 16-byte pieces per thread in flight
+    {
+        const bool vec = (a.K & 3u) == 0 && (a.K_extra & 3u) == 0 && (a.x_stride & 3u) == 0 && (reinterpret_cast<uintptr_t>(a.x) & 15u) == 0;
+        for (uint32_t i0 = threadIdx.x; i0 < 2 * total; i0 += 4 * kWarps * 32) {
+            float4 t[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const uint32_t i = i0 + j * kWarps * 32;
+                t[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (i >= 2 * total) continue;
+                const uint32_t s = i < 2 * routed ? i / (2 * chs) : a.n_routed, e = 4 * (i - s * 2 * chs), n = s == a.n_routed ? a.K_extra : a.K;
+                const float* x = a.x + (size_t)s * a.x_stride + e;
+                if (vec) {
+                    if (e < n) t[j] = *reinterpret_cast<const float4*>(x);
+                } else {
+                    if (e < n) t[j].x = x[0];
+                    if (e + 1 < n) t[j].y = x[1];
+                    if (e + 2 < n) t[j].z = x[2];
+                    if (e + 3 < n) t[j].w = x[3];
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const uint32_t i = i0 + j * kWarps * 32;
+                if (i < 2 * total) ((i & 1u) ? xb : xa)[i >> 1] = t[j];
+            }
+        }
+    }
     __syncthreads();
     bool first = true;
     for (; unit < units; unit += gridDim.x * kWarps) {
         float acc[RPU];
 #pragma unroll
         for (int r = 0; r < RPU; r++) acc[r] = 0.f;
-        for (uint32_t c0 = 0; c0 < total; c0 += 32 * U) {
-            if (!first) load(unit, c0);
+        if (!first) slot = k = 0;
+        fslot = fk = 0;
+        for (uint32_t s0 = 0; s0 < steps; s0 += U) {
+            if (!first) load(unit, s0);
             first = false;
 #pragma unroll
             for (int i = 0; i < U; i++) {
-                const uint32_t c = c0 + 32 * i + lane;
-                if (c < total) {
-                    const float4 p = xa[c], q = xb[c];
+                const uint32_t c = fk * 32 + lane, n = fslot == a.n_routed ? chx : chs;
+                if (s0 + i < steps && c < n) {
+                    const float4 p = xa[fslot * chs + c], q = xb[fslot * chs + c];
 #pragma unroll
                     for (int r = 0; r < RPU; r++) acc[r] = dot8(v[r][i], p, q, acc[r]);
                 }
+                advance(fslot, fk);
             }
         }
 #pragma unroll
@@ -315,7 +342,8 @@ __global__ void __launch_bounds__(256) embed_norm_kernel(const __nv_bfloat16* __
 template <typename TY>
 __global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index,
                                                          const float* __restrict__ gain, float eps, TY* __restrict__ y, uint32_t ldy,
-                                                         float* __restrict__ y2, uint32_t width) {
+                                                         float* __restrict__ y2, uint32_t width, const float* __restrict__ gate_row,
+                                                         float* __restrict__ gate_out) {
     grid_dependency_wait();
     grid_launch_dependents();
     const uint32_t t = blockIdx.x;
@@ -329,21 +357,23 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict_
         else y[(size_t)t * ldy + i] = v;
         if (y2 && i < width) y2[(size_t)t * width + i] = v;
     }
+    if (gate_row) {          // sigmoid of one product of the normed row (the gate of a block that runs for every token)
+        float z = 0.f;
+        for (uint32_t i = threadIdx.x; i < width; i += 256) z = fmaf(row[i] * r, gate_row[i], z);
+        __syncthreads();     // block_sum's partial sums are rewritten
+        z = block_sum(z);
+        if (threadIdx.x == 0) gate_out[t] = 1.0f / (1.0f + expf(-z));
+    }
 }
 
-__global__ void sigmoid_column_kernel(const float* __restrict__ logits, uint32_t ld, uint32_t col, float* __restrict__ out, uint32_t T) {
-    const uint32_t t = blockIdx.x * blockDim.x + threadIdx.x;
-    if (t < T) out[t] = 1.0f / (1.0f + expf(-logits[(size_t)t * ld + col]));
-}
-
-template <int EPI, int RPU, bool SLOTS>
+template <int EPI, int RPU, int U, bool SLOTS>
 static int32_t launch(runit_ctx* ctx, const char* name, const Args& a, uint32_t max_rows, uint32_t slots) {
     const size_t smem = (size_t)((a.K + 7) / 8) * 32;
     RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 1024, "%s: %u columns do not fit shared memory", name, a.K);
     if (smem > 48 * 1024)
-        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, SLOTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, U, SLOTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * 8;
-    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, SLOTS>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
+    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, U, SLOTS>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
     return runit_after_launch(ctx, name);
 }
 
@@ -356,11 +386,15 @@ int32_t gemv_bf16(runit_ctx* ctx, const char* name, const GemvDesc& d) {
     const bool slots = d.slot_expert != nullptr;
     const uint32_t n_slots = slots ? d.n_routed + (d.w_extra ? 1 : 0) : 1;
     const uint32_t rows = slots && d.w_extra && d.rows_extra > d.rows ? d.rows_extra : d.rows;
-    const int rpu = d.K > 1024 ? 1 : (d.K > 512 ? 2 : 4);
-#define RUNIT_GV(E, R) (slots ? gv::launch<E, R, true>(ctx, name, a, rows, n_slots) : gv::launch<E, R, false>(ctx, name, a, rows, n_slots))
-    if (d.epi == EPI_SILU_GLU) return rpu == 4 ? RUNIT_GV(EPI_SILU_GLU, 4) : RUNIT_GV(EPI_SILU_GLU, 2);
-    if (d.epi == EPI_RELU2) return rpu == 4 ? RUNIT_GV(EPI_RELU2, 4) : (rpu == 2 ? RUNIT_GV(EPI_RELU2, 2) : RUNIT_GV(EPI_RELU2, 1));
-    return rpu == 4 ? RUNIT_GV(EPI_F32, 4) : (rpu == 2 ? RUNIT_GV(EPI_F32, 2) : RUNIT_GV(EPI_F32, 1));
+    // small rows: several per warp, so that as many loads are in flight; several blocks: fewer, larger CTAs
+#define RUNIT_GV(E, R, U) (slots ? gv::launch<E, R, U, true>(ctx, name, a, rows, n_slots) : gv::launch<E, R, U, false>(ctx, name, a, rows, n_slots))
+    const bool mid = d.K > 512 && !(slots && d.K > 1024);
+    if (d.epi == EPI_SILU_GLU) return d.K <= 512 ? RUNIT_GV(EPI_SILU_GLU, 4, 2) : (mid ? RUNIT_GV(EPI_SILU_GLU, 2, 4) : RUNIT_GV(EPI_SILU_GLU, 2, 8));
+    if (d.epi == EPI_RELU2)
+        return d.K <= 512 ? RUNIT_GV(EPI_RELU2, 4, 2) : (mid && d.K <= 1024 ? RUNIT_GV(EPI_RELU2, 2, 4) : (slots ? RUNIT_GV(EPI_RELU2, 2, 8) : RUNIT_GV(EPI_RELU2, 1, 8)));
+    if (d.K <= 512) return RUNIT_GV(EPI_F32, 4, 2);
+    if (d.K <= 1024) return RUNIT_GV(EPI_F32, 2, 4);
+    return d.K <= 4096 ? RUNIT_GV(EPI_F32, 1, 8) : RUNIT_GV(EPI_F32, 1, 16);
 #undef RUNIT_GV
 }
 
@@ -378,8 +412,8 @@ int32_t gemv_bf16_sum(runit_ctx* ctx, const char* name, const GemvSumDesc& d) {
         runit_launch_chain_smem(ctx, kern, dim3(want < cap ? want : cap), dim3(gv::kWarps * 32), smem, a);
         return runit_after_launch(ctx, name);
     };
-    if (total > 128) return go(gv::gemv_bf16_sum_kernel<1>, 1);
-    return go(gv::gemv_bf16_sum_kernel<2>, 2);
+    if (total > 128) return go(gv::gemv_bf16_sum_kernel<1, 12>, 1);
+    return go(gv::gemv_bf16_sum_kernel<2, 4>, 2);
 }
 
 int32_t embed_norm_rows(runit_ctx* ctx, const void* embed, uint32_t ld, const int32_t* tokens, const int32_t* state, const int32_t* forced,
@@ -390,15 +424,11 @@ int32_t embed_norm_rows(runit_ctx* ctx, const void* embed, uint32_t ld, const in
 }
 
 int32_t norm_rows(runit_ctx* ctx, const float* x, const int32_t* row_index, const float* gain, float eps, void* y, bool y_f32, uint32_t ldy,
-                  float* y2, uint32_t T, uint32_t width) {
-    if (y_f32) runit_launch_chain(ctx, gv::norm_rows_kernel<float>, dim3(T), dim3(256), x, row_index, gain, eps, (float*)y, ldy, y2, width);
-    else runit_launch_chain(ctx, gv::norm_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), x, row_index, gain, eps, (__nv_bfloat16*)y, ldy, y2, width);
+                  float* y2, uint32_t T, uint32_t width, const float* gate_row, float* gate_out) {
+    if (y_f32) runit_launch_chain(ctx, gv::norm_rows_kernel<float>, dim3(T), dim3(256), x, row_index, gain, eps, (float*)y, ldy, y2, width, gate_row, gate_out);
+    else runit_launch_chain(ctx, gv::norm_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), x, row_index, gain, eps, (__nv_bfloat16*)y, ldy, y2, width,
+                            gate_row, gate_out);
     return runit_after_launch(ctx, "norm_rows");
-}
-
-int32_t sigmoid_column(runit_ctx* ctx, const float* logits, uint32_t ld, uint32_t col, float* out, uint32_t T) {
-    gv::sigmoid_column_kernel<<<(T + 255) / 256, 256, 0, ctx->stream>>>(logits, ld, col, out, T);
-    return runit_after_launch(ctx, "sigmoid_column");
 }
 
 }  // namespace runit

@@ -143,7 +143,7 @@ int32_t LayeredModel::alloc_portions() {
         if (st == RUNIT_OK && b) cudaMemsetAsync(*p, 0, b, ctx->stream);       // padding stays finite
     };
     const uint32_t P = portion_cap, wd = width();
-    uint32_t q = 0, hv = 0, kvw = 0, ffd = 0, ffe = 0, k = 0, E = 0, R = 0, heads = 0, cp = 0, pitch = 0;
+    uint32_t q = 0, hv = 0, kvw = 0, ffd = 0, ffe = 0, k = 0, E = 0, heads = 0, cp = 0, pitch = 0;
     bool all_expand = true;
     for (const Layer& l : layers) {
         const runit_layer_desc& d = l.d;
@@ -155,7 +155,7 @@ int32_t LayeredModel::alloc_portions() {
         if (d.ff_kind == RUNIT_FF_DENSE) ffd = std::max(ffd, pad8(d.ff));
         if (d.ff_kind == RUNIT_FF_MOE) {
             ffe = std::max(ffe, pad8(d.ff)); ffd = std::max(ffd, pad8(d.shared_ff));
-            k = std::max(k, (uint32_t)d.top_k); E = std::max(E, (uint32_t)d.n_experts); R = std::max(R, d.n_experts + l.gates);
+            k = std::max(k, (uint32_t)d.top_k); E = std::max(E, (uint32_t)d.n_experts);
         }
     }
     q = (q + 1) & ~1u;
@@ -171,7 +171,7 @@ int32_t LayeredModel::alloc_portions() {
         const size_t S = (size_t)P * k;
         pf.rows_perm = ((uint32_t)((S + kMoeRowAlign - 1) / kMoeRowAlign) + E) * kMoeRowAlign;
         const size_t tiles = S / 64 + E + 1;
-        A((void**)&pf.rl, (size_t)P * R * 4); A((void**)&pf.idx, S * 4); A((void**)&pf.rw, S * 4); A((void**)&pf.gate, (size_t)P * 4);
+        A((void**)&pf.rl, (size_t)P * E * 4); A((void**)&pf.idx, S * 4); A((void**)&pf.rw, S * 4); A((void**)&pf.gate, (size_t)P * 4);
         A((void**)&pf.pre, (size_t)pf.rows_perm * 4); A((void**)&pf.y, (size_t)pf.rows_perm * wd * 4);
         A(&pf.xperm, (size_t)pf.rows_perm * ldw() * es()); A(&pf.actp, (size_t)pf.rows_perm * ffe * es());
         A((void**)&pf.perm.counts, 1024); A((void**)&pf.perm.n_tok_tiles, 16); A((void**)&pf.perm.tile_expert, tiles * 4);
@@ -216,7 +216,8 @@ int32_t LayeredModel::ff_rows(const Layer& l, uint32_t T) {
     int32_t st;
     const uint32_t wd = width();
     const bool moe = d.ff_kind == RUNIT_FF_MOE;
-    if ((st = norm_rows(ctx, pf.x, nullptr, (const float*)d.norm2, cfg.eps, pf.h, exact, ldw(), moe ? pf.xf : nullptr, T, wd))) return st;
+    const float* gate_row = moe && d.shared_ff ? (const float*)d.router + (size_t)d.n_experts * wd : nullptr;
+    if ((st = norm_rows(ctx, pf.x, nullptr, (const float*)d.norm2, cfg.eps, pf.h, exact, ldw(), moe ? pf.xf : nullptr, T, wd, gate_row, pf.gate))) return st;
     auto block = [&](const void* up, const void* down, uint32_t ff, const float* post) -> int32_t {
         GemmDesc g;
         g.w = up; g.rows = up_rows(d, ff); g.K = wd; g.ldw = ldw(); g.x = pf.h; g.ldx = ldw(); g.x_rows = portion_cap; g.T = T;
@@ -228,13 +229,10 @@ int32_t LayeredModel::ff_rows(const Layer& l, uint32_t T) {
         return gemm_bf16(ctx, "rows_down", g, exact);
     };
     if (!moe) return block(d.ff_up, d.ff_down, d.ff, nullptr);
-    const uint32_t E = d.n_experts, k = d.top_k, R = E + l.gates, S = T * k;
-    if ((st = moe_router(ctx, (const float*)d.router, pf.xf, pf.rl, R, wd, T))) return st;
-    if ((st = moe_topk_rows(ctx, pf.rl, 0, R, E, k, d.score, d.renorm, T, pf.idx, pf.rw))) return st;
-    if (d.shared_ff) {
-        if ((st = sigmoid_column(ctx, pf.rl, R, E, pf.gate, T))) return st;
-        if ((st = block(d.shared_up, d.shared_down, d.shared_ff, pf.gate))) return st;
-    }
+    const uint32_t E = d.n_experts, k = d.top_k, S = T * k;
+    if ((st = moe_router(ctx, (const float*)d.router, pf.xf, pf.rl, E, wd, T))) return st;
+    if ((st = moe_topk_rows(ctx, pf.rl, 0, E, E, k, d.score, d.renorm, T, pf.idx, pf.rw))) return st;
+    if (d.shared_ff && (st = block(d.shared_up, d.shared_down, d.shared_ff, pf.gate))) return st;
     const uint32_t tt = gemm_bf16_tile_tok(S / E, exact);
     if ((st = moe_permute(ctx, pf.idx, S, E, tt, pf.perm))) return st;
     if ((st = moe_gather_rows(ctx, pf.h, pf.perm.pos_of_slot, pf.xperm, S, (size_t)ldw() * es(), k))) return st;
