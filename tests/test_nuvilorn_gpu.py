@@ -182,7 +182,7 @@ def test_folded_attention(ctx, case, f32, nsplit):
     close(out.download(np.float32, T * H * dv).reshape(T, H * dv), ref, 2e-5 if f32 else 2e-2)
 
 
-@pytest.mark.parametrize("H,d,r,dv,rank,T,start", [(2, 24, 8, 40, 48, 70, 0), (3, 64, 32, 64, 64, 129, 50), (2, 96, 32, 64, 40, 65, 64),
+@pytest.mark.parametrize("H,d,r,dv,rank,T,start", [(2, 24, 8, 40, 48, 70, 0), (3, 64, 32, 56, 72, 129, 50), (2, 96, 32, 64, 40, 65, 64),
                                                    (2, 64, 64, 128, 80, 200, 1), (2, 128, 64, 128, 512, 150, 37), (1, 8, 8, 8, 16, 64, 63)])
 def test_expanded_attention(ctx, H, d, r, dv, rank, T, start):
     import runit_mac_b200 as R
