@@ -66,6 +66,7 @@ void*   runit_ctx_stream(runit_ctx_t* ctx);
 int32_t runit_flush(runit_ctx_t* ctx);
 const char* runit_last_error_string(runit_ctx_t* ctx);
 const char* runit_status_string(int32_t status);
+/* Device buffers are 1024-byte aligned. */
 int32_t runit_buf_alloc(runit_ctx_t* ctx, size_t bytes, int32_t flags, void** dptr);
 int32_t runit_buf_free(runit_ctx_t* ctx, void* dptr);
 int32_t runit_memcpy_h2d(runit_ctx_t* ctx, void* dst_dev, const void* src_host, size_t bytes);

@@ -8,7 +8,15 @@
 
 #include <cstdarg>
 #include <cstdlib>
+#include <mutex>
 #include <new>
+#include <unordered_map>
+
+// Device buffers start at a multiple of this (what the batched blocks ask of their scratch); the ones whose start had to be
+// moved for it, with the address to free.
+static constexpr size_t kBufAlign = 1024;
+static std::unordered_map<void*, void*> g_shifted;
+static std::mutex g_shifted_mutex;
 
 const char* runit_status_name(int32_t st) {
     switch (st) {
@@ -317,8 +325,21 @@ int32_t runit_buf_alloc(runit_ctx_t* ctx, size_t bytes, int32_t flags, void** dp
         e = cudaHostAlloc(dptr, bytes, cudaHostAllocMapped | cudaHostAllocPortable);
     } else {
         e = cudaMalloc(dptr, bytes);
+        if (e == cudaSuccess && !runit_aligned(*dptr, kBufAlign)) {      // small allocations come 256- or 512-byte aligned
+            cudaFree(*dptr);
+            void* raw = nullptr;
+            e = cudaMalloc(&raw, bytes + kBufAlign);
+            if (e == cudaSuccess) {
+                *dptr = reinterpret_cast<void*>((reinterpret_cast<uintptr_t>(raw) + kBufAlign - 1) & ~(uintptr_t)(kBufAlign - 1));
+                if (*dptr != raw) {
+                    std::lock_guard<std::mutex> lock(g_shifted_mutex);
+                    g_shifted[*dptr] = raw;
+                }
+            }
+        }
     }
     if (e != cudaSuccess) {
+        *dptr = nullptr;
         cudaGetLastError();
         return runit_fail(ctx, RUNIT_ERR_ALLOC, "allocation of %zu bytes failed: %s", bytes, cudaGetErrorString(e));
     }
@@ -336,7 +357,17 @@ int32_t runit_buf_free(runit_ctx_t* ctx, void* dptr) {
     }
     cudaStreamSynchronize(ctx->stream);
     if (a.type == cudaMemoryTypeHost) RUNIT_CUDA_TRY(ctx, cudaFreeHost(dptr));
-    else RUNIT_CUDA_TRY(ctx, cudaFree(dptr));
+    else {
+        {
+            std::lock_guard<std::mutex> lock(g_shifted_mutex);
+            auto it = g_shifted.find(dptr);
+            if (it != g_shifted.end()) {
+                dptr = it->second;
+                g_shifted.erase(it);
+            }
+        }
+        RUNIT_CUDA_TRY(ctx, cudaFree(dptr));
+    }
     return RUNIT_OK;
 }
 

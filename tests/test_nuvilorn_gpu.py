@@ -531,3 +531,14 @@ def test_bad_calls_are_refused(ctx, tmp_path):
         with pytest.raises(R.KernelError):
             call()
     assert ctx.launches == before
+
+
+def test_buffers_are_aligned_whatever_was_allocated_before(ctx):
+    """Odd small buffers first: the scratch of the batched blocks must still start at a multiple of 1024 bytes."""
+    keep = [ctx.new_buffer(n) for n in (16, 700, 513, 1 << 12, 300, 90000, 256, 1100)]
+    assert all(b.ptr % 1024 == 0 for b in keep)
+    for b in keep[::2]:
+        b.free()
+    again = [ctx.new_buffer(n) for n in (512, 40, 5000)]
+    a = np.arange(10, dtype=np.int32)
+    assert all(b.ptr % 1024 == 0 for b in again) and (again[0].upload(a).download(np.int32, 10) == a).all()
