@@ -324,7 +324,7 @@ uint64_t LayeredModel::launches_per_token() {
     return n;
 }
 
-static int32_t check_layer(runit_ctx* ctx, const runit_layered_cfg& c, const runit_layer_desc* all, int32_t i) {
+static int32_t check_layer(runit_ctx* ctx, const runit_layer_desc* all, int32_t i) {
     const runit_layer_desc& d = all[i];
     RUNIT_REQUIRE(ctx, d.heads > 0 && d.dim > 0 && d.rot_dim > 0 && d.rot_dim % 2 == 0 && d.vdim > 0 && d.kv_rank > 0 && d.kv_rank <= 1024,
                   "model_create_layered: layer %d: bad attention sizes (rot_dim even, kv_rank <= 1024)", i);
@@ -346,7 +346,6 @@ static int32_t check_layer(runit_ctx* ctx, const runit_layered_cfg& c, const run
                   "model_create_layered: layer %d: bad experts (at most 256, top_k at most 32)", i);
     RUNIT_REQUIRE(ctx, d.score == RUNIT_SCORE_SOFTMAX || d.score == RUNIT_SCORE_SIGMOID, "model_create_layered: layer %d: unknown scoring function", i);
     RUNIT_REQUIRE(ctx, d.shared_ff == 0 || (d.shared_ff > 0 && d.shared_up && d.shared_down), "model_create_layered: layer %d: bad shared block", i);
-    (void)c;
     return RUNIT_OK;
 }
 
@@ -367,7 +366,7 @@ int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cf
                   "model_create_layered: bad width, depth, vocabulary or length");
     int32_t st;
     for (int32_t i = 0; i < c.n_layers; i++)
-        if ((st = check_layer(ctx, c, layers, i)) != RUNIT_OK) return st;
+        if ((st = check_layer(ctx, layers, i)) != RUNIT_OK) return st;
     LayeredModel* m = new (std::nothrow) LayeredModel();
     if (!m) return RUNIT_ERR_ALLOC;
     m->ctx = ctx;
