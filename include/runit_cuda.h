@@ -518,11 +518,17 @@ int32_t runit_latent_prefill_attention(runit_ctx_t*, const runit_latent_cfg* cfg
 
 /* ── decoders described layer by layer (no twin), weights in bf16 ──
  * Every matrix is row-major [rows][pad8(columns)] bf16 with zero padding; norms and router are f32.  Linear maps W x.
- * Residual stream, norms, scores, softmax, router and angles are f32.  Pre-norm layers:
- *   x += mixer(norm1(x));  x += ff(norm2(x));  norm(x) = x / sqrt(mean(x^2) + eps) * gain, one gain for all coordinates.
+ * Residual stream, norms, scores, softmax, router, angles and recurrent state are f32.  norm(x) = x / sqrt(mean(x^2) + eps) * gain.
+ *   post_norm = 0: x += mixer(norm1(x));  x += ff(norm2(x));  one gain for all coordinates.
+ *   post_norm = 1: x += norm1(mixer(x));  x += norm2(ff(x));  a gain per coordinate (dense feed-forward only).
+ * A decoder with retention or state-space layers carries state from token to token: a pass starts at position 0 (from a zero
+ * state) or where the last one ended.
  * exact = 0: activations and cache bf16 with f32 accumulation (batched passes on the tensor cores); exact = 1: activations
  * and cache f32 throughout.  The step, the generate and sampling loops, prefill and forward are those of any runit_model_t. */
 enum { RUNIT_FF_NONE = 0, RUNIT_FF_DENSE = 1, RUNIT_FF_MOE = 2 };
+enum { RUNIT_MIX_LATENT = 0,      /* latent attention */
+       RUNIT_MIX_HEADS = 1,       /* attention over keys and values per head and / or retention, side by side */
+       RUNIT_MIX_SSM = 2 };       /* state-space layer with a scalar decay per head and token */
 enum { RUNIT_ACT_SILU_GLU = 0,    /* rows 2i and 2i+1 of the up matrix are gate and up of unit i: silu(g) * u */
        RUNIT_ACT_RELU2 = 1 };     /* max(u, 0)^2 */
 typedef struct {
@@ -535,26 +541,51 @@ typedef struct {
      * and multiply an expert's input; a shared block of shared_ff units (0 = none) runs for every token, its output times the
      * sigmoid of its own gate row */
     int32_t ff_kind, ff_act, ff, n_experts, top_k, score, renorm, shared_ff;
-    const void* norm1;        /* f32 [1] */
-    const void* norm2;        /* f32 [1]; NULL without feed-forward */
-    const void* w_q;          /* [heads*(dim+rot_dim) (+ kv_rank+rot_dim when the layer owns its latent)][width] */
+    const void* norm1;        /* f32 [1] ([width] with post_norm) */
+    const void* norm2;        /* the same; NULL without feed-forward */
+    /* projections of the mixer's input, one under the other.  Latent attention: [heads*(dim+rot_dim) (+ kv_rank+rot_dim when the
+     * layer owns its latent)][width]; RUNIT_MIX_HEADS: q, k, v of the attention, then q, k, v, gate of the retention;
+     * RUNIT_MIX_SSM: gate, x, B, C, step sizes */
+    const void* w_q;
     const void* kv_norm;      /* f32 [kv_rank]; NULL when kv_from >= 0 */
     const void* w_ukv;        /* [heads*dim + heads*vdim][kv_rank]: keys of all heads, then values */
-    const void* w_o;          /* [width][heads*vdim] */
+    const void* w_o;          /* [width][outputs of the mixer]; RUNIT_MIX_HEADS: attention heads, then retention heads */
     const void* ff_up;        /* [ff (2 ff for a gated block)][width], experts stacked */
     const void* ff_down;      /* [width][ff], experts stacked */
     const void* router;       /* f32 [n_experts (+ 1 gate row of the shared block)][width], no padding */
     const void* shared_up;    /* [shared_ff (2 shared_ff)][width] */
     const void* shared_down;  /* [width][shared_ff] */
+    int32_t mixer;
+    /* RUNIT_MIX_HEADS, attention (at_heads = 0: none): query head h uses key / value head h / (at_heads / at_kv_heads); score
+     * (q . k) * at_scale - at_slopes[h] * (i - j); position i sees the at_window positions up to its own (0: all of them);
+     * at_unit_qk: q and k are divided by their root mean square per head; the output is multiplied by at_out_scale */
+    int32_t at_heads, at_kv_heads, at_dim, at_vdim, at_window, at_unit_qk;
+    /* retention (rt_heads = 0: none): S <- decay_h S + k v^T, o = S^T q; the first rt_rot_dims coordinates of q and k are rotated
+     * (pairs (i, i + rt_rot_dims / 2), angle position * rt_rot_base^(-2i / rt_rot_dims)), k is multiplied by rt_dim^(-1/2); o is
+     * divided by its root mean square per head and multiplied by silu(gate) and rt_out_scale */
+    int32_t rt_heads, rt_dim, rt_vdim, rt_rot_dims;
+    /* RUNIT_MIX_SSM: x, B, C pass a causal convolution over ss_taps tokens and silu; dt = softplus(. + ss_dt_bias);
+     * S <- exp(ss_a dt) S + dt B x^T, y = (S^T C + ss_skip x) * silu(gate), normed in ss_norm_groups parts */
+    int32_t ss_heads, ss_vdim, ss_state, ss_groups, ss_taps, ss_norm_groups;
+    float   at_scale, at_out_scale, rt_rot_base, rt_out_scale;
+    const void* at_slopes;    /* f32 [at_heads]; NULL: no bias */
+    const void* rt_decay;     /* f32 [2][rt_heads]: the decays, then their logarithms */
+    const void* ss_conv;      /* f32 [channels][ss_taps], last column: the current token; channels = ss_heads*ss_vdim + 2*ss_groups*ss_state */
+    const void* ss_conv_b;    /* f32 [channels] */
+    const void* ss_dt_bias;   /* f32 [ss_heads] */
+    const void* ss_a;         /* f32 [ss_heads], negative: logarithm of the decay per unit of dt */
+    const void* ss_skip;      /* f32 [ss_heads] */
+    const void* ss_norm;      /* f32 [ss_heads*ss_vdim] */
 } runit_layer_desc;
 typedef struct {
-    int32_t n_layers, width, vocab, max_seq, exact;
-    float   eps;
+    int32_t n_layers, width, vocab, max_seq, exact, post_norm;
+    float   eps, embed_scale;   /* embed_scale: factor of the embedding when embed_norm is NULL */
+    float   logit_cap;          /* 0: none; else logits = cap * tanh(logits / cap) */
 } runit_layered_cfg;
 typedef struct {
     const void* embed;        /* [vocab][width] */
-    const void* embed_norm;   /* f32 [1] */
-    const void* final_norm;   /* f32 [1] */
+    const void* embed_norm;   /* f32 [1]; NULL: no norm */
+    const void* final_norm;   /* f32 [1] ([width] with post_norm) */
     const void* head;         /* [vocab][width] */
 } runit_layered_weights;
 /* Device pointers; the model keeps them, the caller keeps the memory alive. */

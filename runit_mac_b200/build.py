@@ -24,7 +24,7 @@ LIB = PKG / "librunit_cuda.so"
 # sources define; it exists so that serving one kind of model does not compile the kernels of all others.
 PARTS = {
     "layered": (PKG / "librunit_layered.so",
-                ("ctx", "gemv_stream", "model_core", "layered_model", "gemv_bf16", "gemm_bf16", "latent_attention", "moe_route",
+                ("ctx", "gemv_stream", "model_core", "layered_model", "gemv_bf16", "gemm_bf16", "latent_attention", "head_attention", "linear_state", "moe_route",
                  "moe_permute", "sampler")),
 }
 

@@ -30,6 +30,9 @@ struct Args {
     void* out;
     uint32_t ldo;
     const float *pre, *post;
+    float* tail;
+    uint32_t tail_from, ldt;
+    float cap;
     int32_t* status;
 };
 
@@ -216,7 +219,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         const uint32_t tok = tok0 + jj;
                         __nv_bfloat16* o = out + (size_t)tok * a.ldo;
                         if constexpr (EPI == EPI_CAST) {
-                            store_rows<4>(o + r4, y, a.rows - r4, a.ldo);
+                            if (r4 + 4 <= a.tail_from) {
+                                store_rows<4>(o + r4, y, a.rows - r4, a.ldo);
+                            } else {
+                                for (uint32_t i = 0; i < 4 && r4 + i < a.rows; i++) {
+                                    if (r4 + i < a.tail_from) o[r4 + i] = __float2bfloat16_rn(y[i]);
+                                    else a.tail[(size_t)tok * a.ldt + r4 + i - a.tail_from] = y[i];
+                                }
+                            }
                         } else {
                             const float pre = a.pre ? a.pre[tok] : 1.f, post = a.post ? a.post[tok] : 1.f;
                             if constexpr (EPI == EPI_SILU_GLU) {      // rows 2i, 2i+1: gate and up of output i
@@ -246,7 +256,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                     for (int j = 0; j < 32; j++) {
                         if (!live || (uint32_t)j >= cnt) continue;
-                        const float f = __uint_as_float(v[j]);
+                        float f = __uint_as_float(v[j]);
+                        if (a.cap != 0.f) f = a.cap * tanhf(f / a.cap);
                         const size_t o = (size_t)(tok0 + j) * a.ldo + r;
                         reinterpret_cast<float*>(a.out)[o] = f;
                     }
@@ -319,7 +330,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const Args a) {
                     o[r >> 1] = g / (1.0f + expf(-g)) * u * post;
                 } else if constexpr (EPI == EPI_RELU2) o[r] = relu2(acc[i][j] * pre) * post;
                 else if constexpr (EPI == EPI_ADD) o[r] += acc[i][j];
-                else o[r] = acc[i][j];
+                else if (r >= a.tail_from) a.tail[(size_t)(t.row0 + tok) * a.ldt + r - a.tail_from] = acc[i][j];
+                else o[r] = a.cap != 0.f ? a.cap * tanhf(acc[i][j] / a.cap) : acc[i][j];
             }
         }
     }
@@ -380,7 +392,8 @@ int32_t gemm_bf16(runit_ctx* ctx, const char* name, const GemmDesc& d, bool exac
     RUNIT_REQUIRE(ctx, d.epi != EPI_SILU_GLU || d.rows % 2 == 0, "%s: a gated product needs pairs of rows", name);
     const bool grouped = d.tile_expert != nullptr;
     gm::Args a{(const __nv_bfloat16*)d.w, (const float*)d.x, d.rows, d.K, d.ldw, d.ldx, 0, d.T, 0, d.tile_expert, d.tile_nvalid, d.tile_row0,
-               d.n_tok_tiles, d.out, d.ldo, d.pre, d.post, ctx->d_status};
+               d.n_tok_tiles, d.out, d.ldo, d.pre, d.post, d.tail, d.tail ? d.tail_from : 0xFFFFFFFFu, d.ldt, d.cap, ctx->d_status};
+    RUNIT_REQUIRE(ctx, (!d.tail || d.epi == EPI_CAST) && (d.cap == 0.f || d.epi == EPI_F32), "%s: f32 columns go with EPI_CAST, a cap with EPI_F32", name);
     if (exact) {
         a.nb = (d.rows + 63) / 64;
         a.tile_tok = 64;

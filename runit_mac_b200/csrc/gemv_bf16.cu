@@ -1,5 +1,5 @@
 // One-token operators of decoders with bf16 weights: GEMV with the norm in front and the activation behind fused in, and the
-// row operators of a pass (embedding, norms with one gain for all coordinates).
+// row operators of a pass (embedding; norms with one gain for all coordinates, or with one per coordinate on a sublayer's output).
 //
 // A warp owns 1, 2 or 4 weight rows (rows 2i and 2i+1 together for a gated block) and keeps eight to sixteen 16-byte loads per
 // lane in flight; the first group of them does not depend on the previous kernel of the chain and is requested before the dependency
@@ -57,6 +57,129 @@ __device__ __forceinline__ float stage_x(const float* x, uint32_t K, uint32_t nc
     return sq;
 }
 
+// sum over the CTA of up to two values at a time (kWarps warps); every thread gets it
+__device__ __forceinline__ float cta_sum(float s, float* part) {
+    s = warp_add(s);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = s;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int i = 0; i < kWarps; i++) tot += part[i];
+    return tot;
+}
+__device__ __forceinline__ float4 load4(const float* p, uint32_t e, uint32_t n, bool vec) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vec) {
+        if (e < n) v = *reinterpret_cast<const float4*>(p + e);
+    } else {
+        if (e < n) v.x = p[e];
+        if (e + 1 < n) v.y = p[e + 1];
+        if (e + 2 < n) v.z = p[e + 2];
+        if (e + 3 < n) v.w = p[e + 3];
+    }
+    return v;
+}
+__device__ __forceinline__ bool aligned4(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
+
+// GEMV_PRO_RESIDUAL: returns the factor of the products (that of the second norm).  A thread handles the same pieces in every
+// pass; ya / yb are two more planes like xa / xb.
+__device__ __forceinline__ float stage_residual(const float* x, const GemvPrologue& p, float eps, uint32_t K, uint32_t nch, float4* xa, float4* xb,
+                                                 float4* ya, float4* yb, float* part) {
+    const bool vec = (K & 3u) == 0 && aligned4(x) && aligned4(p.y) && aligned4(p.y_gain) && aligned4(p.gain) && aligned4(p.x_out);
+    float r = 0.f;
+    if (p.y) {
+        float sq = 0.f;
+        for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+            const float4 xv = load4(x, 4 * i, K, vec), g = load4(p.y_gain, 4 * i, K, vec);
+            float4 y = load4(p.y, 4 * i, K, vec);
+            sq = fmaf(y.x, y.x, sq); sq = fmaf(y.y, y.y, sq); sq = fmaf(y.z, y.z, sq); sq = fmaf(y.w, y.w, sq);
+            y.x *= g.x; y.y *= g.y; y.z *= g.z; y.w *= g.w;
+            ((i & 1u) ? xb : xa)[i >> 1] = xv;
+            ((i & 1u) ? yb : ya)[i >> 1] = y;
+        }
+        r = rsqrtf(cta_sum(sq, part) / (float)K + eps);
+    }
+    float sq = 0.f;
+    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+        float4& s = ((i & 1u) ? xb : xa)[i >> 1];
+        float4 v;
+        if (p.y) {
+            const float4 y = ((i & 1u) ? yb : ya)[i >> 1];
+            v = s;
+            v.x = fmaf(y.x, r, v.x); v.y = fmaf(y.y, r, v.y); v.z = fmaf(y.z, r, v.z); v.w = fmaf(y.w, r, v.w);
+            if (p.x_out && blockIdx.x == 0) {
+                const uint32_t e = 4 * i;
+                if (vec) {
+                    if (e < K) *reinterpret_cast<float4*>(p.x_out + e) = v;
+                } else {
+                    if (e < K) p.x_out[e] = v.x;
+                    if (e + 1 < K) p.x_out[e + 1] = v.y;
+                    if (e + 2 < K) p.x_out[e + 2] = v.z;
+                    if (e + 3 < K) p.x_out[e + 3] = v.w;
+                }
+            }
+        } else {
+            v = load4(x, 4 * i, K, vec);
+        }
+        if (p.gain) {
+            sq = fmaf(v.x, v.x, sq); sq = fmaf(v.y, v.y, sq); sq = fmaf(v.z, v.z, sq); sq = fmaf(v.w, v.w, sq);
+            const float4 g = load4(p.gain, 4 * i, K, vec);
+            v.x *= g.x; v.y *= g.y; v.z *= g.z; v.w *= g.w;
+        }
+        s = v;
+    }
+    if (!p.gain) return 1.f;
+    __syncthreads();           // part is rewritten
+    return rsqrtf(cta_sum(sq, part) / (float)K + eps);
+}
+
+// GEMV_PRO_GROUPS: the values and their factors go to shared memory first, then the groups are summed there.  fac: one word per
+// group and warp of it.
+__device__ __forceinline__ void stage_groups(const float* x, const GemvPrologue& p, float eps, uint32_t K, uint32_t nch, float4* xa, float4* xb,
+                                             float4* ya, float4* yb, float* fac) {
+    const bool vec = (K & 3u) == 0 && (p.plain & 3u) == 0 && aligned4(x) && aligned4(p.factor);
+    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+        const uint32_t e = 4 * i;
+        ((i & 1u) ? xb : xa)[i >> 1] = load4(x, e, K, vec);
+        float4 f;
+        if (vec) {
+            f = e >= p.plain ? load4(p.factor, e - p.plain, K - p.plain, true) : make_float4(1.f, 1.f, 1.f, 1.f);
+        } else {
+            auto one = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? p.factor[j - p.plain] : 0.f); };
+            f = make_float4(one(e), one(e + 1), one(e + 2), one(e + 3));
+        }
+        ((i & 1u) ? yb : ya)[i >> 1] = f;
+    }
+    __syncthreads();
+    const uint32_t groups = (K - p.plain) / p.group, wpg = groups >= 8 ? 1u : (groups >= 3 ? 2u : (groups == 2 ? 4u : 8u));
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = warp % wpg;
+    auto at = [&](uint32_t e) -> float { return reinterpret_cast<const float*>(((e >> 2) & 1u) ? xb : xa)[(e >> 3) * 4 + (e & 3u)]; };
+    for (uint32_t g = warp / wpg; g < groups; g += kWarps / wpg) {
+        const uint32_t lo = p.plain + g * p.group;
+        float sq = 0.f;
+        for (uint32_t i = sub * 32 + lane; i < p.group; i += 32 * wpg) {
+            const float v = at(lo + i);
+            sq = fmaf(v, v, sq);
+        }
+        sq = warp_add(sq);
+        if (lane == 0) fac[g * wpg + sub] = sq;
+    }
+    __syncthreads();
+    for (uint32_t g = threadIdx.x; g < groups; g += kWarps * 32) {
+        float sq = 0.f;
+        for (uint32_t i = 0; i < wpg; i++) sq += fac[g * wpg + i];
+        fac[g * wpg] = rsqrtf(sq / (float)p.group + eps);
+    }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+        const uint32_t e = 4 * i;
+        float4& v = ((i & 1u) ? xb : xa)[i >> 1];
+        const float4 f = ((i & 1u) ? yb : ya)[i >> 1];
+        auto r = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? fac[(j - p.plain) / p.group * wpg] : 0.f); };
+        v.x *= f.x * r(e); v.y *= f.y * r(e + 1); v.z *= f.z * r(e + 2); v.w *= f.w * r(e + 3);
+    }
+}
+
 struct Args {
     const uint8_t* w;
     uint32_t rows, K, ldw;
@@ -73,10 +196,12 @@ struct Args {
     const uint8_t* w_extra;
     uint32_t rows_extra;
     const float* post_extra;
+    GemvPrologue pro;
+    float cap;
 };
 
 // RPU: rows of a warp's unit; U: 16-byte loads per lane, row and group
-template <int EPI, int RPU, int U, bool SLOTS>
+template <int EPI, int RPU, int U, bool SLOTS, bool PRO = false>
 __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
     extern __shared__ __align__(16) float4 smem4[];
     __shared__ float part[kWarps];
@@ -119,18 +244,26 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
         }
     }
     if (!early && unit < units) load(unit, 0);
-    float scale = stage_x(a.x, a.K, nch, xa, xb);
-    if (a.gain) {
-        scale = warp_add(scale);
-        if (lane == 0) part[warp] = scale;
-    }
-    __syncthreads();
-    scale = 1.f;
-    if (a.gain) {
-        float tot = 0.f;
+    float scale = 1.f;
+    if constexpr (PRO) {
+        float4 *ya = xb + nch, *yb = ya + nch;
+        if (a.pro.kind == GEMV_PRO_RESIDUAL) scale = stage_residual(a.x, a.pro, a.eps, a.K, nch, xa, xb, ya, yb, part);
+        else stage_groups(a.x, a.pro, a.eps, a.K, nch, xa, xb, ya, yb, reinterpret_cast<float*>(yb + nch));
+        __syncthreads();
+    } else {
+        scale = stage_x(a.x, a.K, nch, xa, xb);
+        if (a.gain) {
+            scale = warp_add(scale);
+            if (lane == 0) part[warp] = scale;
+        }
+        __syncthreads();
+        scale = 1.f;
+        if (a.gain) {
+            float tot = 0.f;
 #pragma unroll
-        for (int i = 0; i < kWarps; i++) tot += part[i];
-        scale = rsqrtf(tot / (float)a.K + a.eps) * *a.gain;
+            for (int i = 0; i < kWarps; i++) tot += part[i];
+            scale = rsqrtf(tot / (float)a.K + a.eps) * *a.gain;
+        }
     }
     unsigned long long best = 0;
     bool first = true;
@@ -167,6 +300,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
                     float o;
                     if (EPI == EPI_RELU2) o = relu2(acc[r] * pre) * post;
                     else o = acc[r] + (a.res ? a.res[row] : 0.f);
+                    if (EPI == EPI_F32 && a.cap != 0.f) o = a.cap * tanhf(o / a.cap);
                     out[row] = o;
                     if (EPI == EPI_F32 && a.argmax) {
                         uint32_t b = __float_as_uint(o);
@@ -324,18 +458,21 @@ __device__ __forceinline__ float block_sum(float s) {
 __global__ void __launch_bounds__(256) embed_norm_kernel(const __nv_bfloat16* __restrict__ emb, uint32_t ld, const int32_t* __restrict__ tokens,
                                                           const int32_t* state, const int32_t* __restrict__ forced, uint32_t n_forced,
                                                           uint32_t vocab, const float* __restrict__ gain, float eps, float* __restrict__ x,
-                                                          uint32_t width) {
+                                                          uint32_t width, float scale) {
     grid_dependency_wait();
     grid_launch_dependents();
     const uint32_t t = blockIdx.x;
     const int32_t tok = tokens ? tokens[t] : model_step_token(state, forced, n_forced, vocab);
     const __nv_bfloat16* row = emb + (size_t)tok * ld;
-    float s = 0.f;
-    for (uint32_t i = threadIdx.x; i < width; i += 256) {
-        const float v = __bfloat162float(row[i]);
-        s = fmaf(v, v, s);
+    float r = scale;
+    if (gain) {
+        float s = 0.f;
+        for (uint32_t i = threadIdx.x; i < width; i += 256) {
+            const float v = __bfloat162float(row[i]);
+            s = fmaf(v, v, s);
+        }
+        r = rsqrtf(block_sum(s) / (float)width + eps) * *gain;
     }
-    const float r = rsqrtf(block_sum(s) / (float)width + eps) * *gain;
     for (uint32_t i = threadIdx.x; i < width; i += 256) x[(size_t)t * width + i] = __bfloat162float(row[i]) * r;
 }
 
@@ -366,14 +503,48 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const float* __restrict_
     }
 }
 
-template <int EPI, int RPU, int U, bool SLOTS>
+// x += y / rms(y) * gain (y null: x as it is), and y_out = x in the operand type; T rows.  With out_gain the stored row is x
+// divided by its own root mean square and multiplied by out_gain (a final norm), and x stays as it is.
+template <typename TY>
+__global__ void __launch_bounds__(256) add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ gain, float eps,
+                                                        const int32_t* __restrict__ row_index, const float* __restrict__ out_gain,
+                                                        TY* __restrict__ out, uint32_t ldo, uint32_t width) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const uint32_t t = blockIdx.x;
+    float* xr = x + (size_t)(row_index ? row_index[t] : (int32_t)t) * width;
+    float r = 0.f, q = 1.f;
+    if (y) {
+        const float* yr = y + (size_t)t * width;
+        float s = 0.f;
+        for (uint32_t i = threadIdx.x; i < width; i += 256) s = fmaf(yr[i], yr[i], s);
+        r = rsqrtf(block_sum(s) / (float)width + eps);
+        for (uint32_t i = threadIdx.x; i < width; i += 256) xr[i] = fmaf(yr[i] * gain[i], r, xr[i]);
+    }
+    if (out_gain) {
+        float s = 0.f;
+        for (uint32_t i = threadIdx.x; i < width; i += 256) s = fmaf(xr[i], xr[i], s);      // this thread's own elements
+        __syncthreads();
+        q = rsqrtf(block_sum(s) / (float)width + eps);
+    }
+    if (!out) return;
+    for (uint32_t i = threadIdx.x; i < ldo; i += 256) {
+        const float v = i < width ? (out_gain ? xr[i] * q * out_gain[i] : xr[i]) : 0.f;
+        if constexpr (sizeof(TY) == 2) out[(size_t)t * ldo + i] = __float2bfloat16_rn(v);
+        else out[(size_t)t * ldo + i] = v;
+    }
+}
+
+template <int EPI, int RPU, int U, bool SLOTS, bool PRO = false>
 static int32_t launch(runit_ctx* ctx, const char* name, const Args& a, uint32_t max_rows, uint32_t slots) {
-    const size_t smem = (size_t)((a.K + 7) / 8) * 32;
+    size_t smem = (size_t)((a.K + 7) / 8) * 32 * (PRO ? 2 : 1);
+    if (PRO && a.pro.kind == GEMV_PRO_GROUPS) smem += ((size_t)(a.K - a.pro.plain) / a.pro.group + 8) * 4;
     RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 1024, "%s: %u columns do not fit shared memory", name, a.K);
     if (smem > 48 * 1024)
-        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, U, SLOTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * 8;
-    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, U, SLOTS>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
+        RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, U, SLOTS, PRO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    // every CTA forms the whole vector: with a prologue that reads several vectors, fewer and longer-lived ones
+    const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * (PRO ? 3 : 8);
+    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, U, SLOTS, PRO>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
     return runit_after_launch(ctx, name);
 }
 
@@ -382,7 +553,19 @@ static int32_t launch(runit_ctx* ctx, const char* name, const Args& a, uint32_t 
 int32_t gemv_bf16(runit_ctx* ctx, const char* name, const GemvDesc& d) {
     RUNIT_REQUIRE(ctx, d.w && d.x && d.out && d.rows > 0 && d.K > 0 && d.ldw % 8 == 0 && d.ldw >= d.K, "%s: bad argument", name);
     gv::Args a{(const uint8_t*)d.w, d.rows, d.K, d.ldw, d.x, d.gain, d.eps, d.out, d.res, d.argmax, d.argmax_ctl, d.n_routed, d.slot_stride,
-               d.slot_expert, d.pre, (const uint8_t*)d.w_extra, d.rows_extra, d.post_extra};
+               d.slot_expert, d.pre, (const uint8_t*)d.w_extra, d.rows_extra, d.post_extra, d.pro, d.cap};
+    if (d.pro.kind != GEMV_PRO_NONE) {
+        RUNIT_REQUIRE(ctx, !d.slot_expert && !d.gain && (d.epi == EPI_F32 || d.epi == EPI_RELU2 || d.epi == EPI_SILU_GLU),
+                      "%s: a prologue goes with a plain product", name);
+        RUNIT_REQUIRE(ctx, d.pro.kind != GEMV_PRO_GROUPS || (d.pro.group > 0 && d.pro.plain < d.K && (d.K - d.pro.plain) % d.pro.group == 0 && d.pro.factor),
+                      "%s: bad groups", name);
+        RUNIT_REQUIRE(ctx, d.pro.kind != GEMV_PRO_RESIDUAL || !d.pro.y || d.pro.y_gain, "%s: bad residual", name);
+#define RUNIT_GVP(E, R, U) gv::launch<E, R, U, false, true>(ctx, name, a, d.rows, 1)
+        if (d.epi == EPI_SILU_GLU) return d.K <= 512 ? RUNIT_GVP(EPI_SILU_GLU, 4, 2) : RUNIT_GVP(EPI_SILU_GLU, 2, 8);
+        if (d.epi == EPI_RELU2) return d.K <= 512 ? RUNIT_GVP(EPI_RELU2, 4, 2) : (d.K <= 1024 ? RUNIT_GVP(EPI_RELU2, 2, 4) : RUNIT_GVP(EPI_RELU2, 1, 8));
+        return d.K <= 512 ? RUNIT_GVP(EPI_F32, 4, 2) : (d.K <= 1024 ? RUNIT_GVP(EPI_F32, 2, 4) : RUNIT_GVP(EPI_F32, 1, 8));
+#undef RUNIT_GVP
+    }
     const bool slots = d.slot_expert != nullptr;
     const uint32_t n_slots = slots ? d.n_routed + (d.w_extra ? 1 : 0) : 1;
     const uint32_t rows = slots && d.w_extra && d.rows_extra > d.rows ? d.rows_extra : d.rows;
@@ -417,9 +600,9 @@ int32_t gemv_bf16_sum(runit_ctx* ctx, const char* name, const GemvSumDesc& d) {
 }
 
 int32_t embed_norm_rows(runit_ctx* ctx, const void* embed, uint32_t ld, const int32_t* tokens, const int32_t* state, const int32_t* forced,
-                        uint32_t n_forced, uint32_t vocab, const float* gain, float eps, float* x, uint32_t T, uint32_t width) {
+                        uint32_t n_forced, uint32_t vocab, const float* gain, float eps, float* x, uint32_t T, uint32_t width, float scale) {
     runit_launch_chain(ctx, gv::embed_norm_kernel, dim3(T), dim3(256), (const __nv_bfloat16*)embed, ld, tokens, state, forced, n_forced, vocab,
-                       gain, eps, x, width);
+                       gain, eps, x, width, scale);
     return runit_after_launch(ctx, "embed_norm");
 }
 
@@ -429,6 +612,14 @@ int32_t norm_rows(runit_ctx* ctx, const float* x, const int32_t* row_index, cons
     else runit_launch_chain(ctx, gv::norm_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), x, row_index, gain, eps, (__nv_bfloat16*)y, ldy, y2, width,
                             gate_row, gate_out);
     return runit_after_launch(ctx, "norm_rows");
+}
+
+int32_t add_norm_rows(runit_ctx* ctx, float* x, const float* y, const float* gain, float eps, const int32_t* row_index, const float* out_gain,
+                      void* out, bool out_f32, uint32_t ldo, uint32_t T, uint32_t width) {
+    if (out_f32) runit_launch_chain(ctx, gv::add_norm_kernel<float>, dim3(T), dim3(256), x, y, gain, eps, row_index, out_gain, (float*)out, ldo, width);
+    else runit_launch_chain(ctx, gv::add_norm_kernel<__nv_bfloat16>, dim3(T), dim3(256), x, y, gain, eps, row_index, out_gain, (__nv_bfloat16*)out, ldo,
+                            width);
+    return runit_after_launch(ctx, "add_norm_rows");
 }
 
 }  // namespace runit

@@ -1,0 +1,579 @@
+// Layers with a decaying linear state per head, S <- decay S + k v^T, o = S^T q: retention (decay fixed per head) and the
+// state-space layer (decay and step size per token).  S is f32 and so is everything that enters the recurrence besides the
+// projections and the short convolution.  A sequence that starts at position 0 starts from a zero state: the kernels look at
+// the position, nothing has to be cleared.
+//   * ssm_step_kernel: one token, convolution to gate (the retention's step is in head_attention.cu, beside the attention).
+//   * ssm_conv_kernel: convolution, silu and softplus of a portion.
+//   * linear_scan_kernel: the recurrence token by token, state in registers.  32-bit runs, short portions, odd sizes.
+//   * chunk_state_kernel + chunk_out_kernel: long portions in bf16, in chunks of 64 tokens on tensor cores.  The first walks the
+//     chunks of one head and 32 value columns with the state in accumulators and leaves the state at the start of every chunk
+//     (as the sum of two bf16 numbers); the second forms all chunks at once: what the starting state contributes, and the masked
+//     products within the chunk, weighted by decays in f32.
+//   * gated_norm_kernel: gate and norm of groups of the result.
+#include "bf16_ops.cuh"
+#include "gemv_common.cuh"
+#include "linear_state.cuh"
+#include "tma.cuh"
+
+namespace runit {
+namespace ls {
+
+__device__ __forceinline__ float wsum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+// ── one token ──
+// Convolved and activated value of channel c at position pos; raw: its projection at pos.
+__device__ __forceinline__ float conv_step(const Ssm& m, uint32_t c, float raw, uint32_t pos) {
+    const uint32_t ch = m.channels();
+    float s = m.conv_b[c];
+    for (uint32_t j = 0; j + 1 < m.taps; j++) {
+        const uint32_t back = m.taps - 1 - j;
+        if (pos >= back) s = fmaf(m.conv_w[(size_t)c * m.taps + j], m.ring[(size_t)((pos - back) % m.taps) * ch + c], s);
+    }
+    return silu(fmaf(m.conv_w[(size_t)c * m.taps + m.taps - 1], raw, s));
+}
+
+// grid (heads, ceil(vdim / 32)).  The ring row of this position is not read by anyone in this launch.
+__global__ void __launch_bounds__(256) ssm_step_kernel(const Ssm m, const float* proj, float* y, const int32_t* pos_ptr) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[8][33];
+    float *qs = sm, *ks = sm + m.state;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, h = blockIdx.x, j = blockIdx.y * 32 + lane, inner = m.inner(), ch = m.channels();
+    const uint32_t rep = m.heads / m.groups, g = h / rep;
+    float* S = m.s + (size_t)h * m.state * m.vdim;
+    StateRows st;
+    load_rows(st, S, m.state, m.vdim, j, 0);         // the state is that of the last step: final long before this launch
+    const float a = m.a[h], bias = m.dt_bias[h], skip = m.skip[h];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const uint32_t pos = (uint32_t)*pos_ptr;
+    float* slot = m.ring + (size_t)(pos % m.taps) * ch;
+    const float dt = softplus(proj[2 * inner + 2 * m.groups * m.state + h] + bias);
+    const float* xbc = proj + inner;
+    const bool writes = blockIdx.y == 0 && h % rep == 0;
+    for (uint32_t i = tid; i < 2 * m.state; i += 256) {
+        const bool is_c = i >= m.state;
+        const uint32_t n = is_c ? i - m.state : i, c = inner + (is_c ? m.groups * m.state : 0) + g * m.state + n;
+        const float raw = xbc[c], v = conv_step(m, c, raw, pos);
+        if (is_c) qs[n] = v;
+        else ks[n] = v * dt;
+        if (writes) slot[c] = raw;
+    }
+    float v = 0.f, z = 0.f;
+    if (j < m.vdim) {
+        const uint32_t c = h * m.vdim + j;
+        const float raw = xbc[c];
+        v = conv_step(m, c, raw, pos);
+        z = proj[c];
+        if (tid < 32) slot[c] = raw;
+    }
+    __syncthreads();
+    const float o = state_step(st, S, m.state, m.vdim, j, qs, ks, v, expf(a * dt), pos == 0, red);
+    if (tid < 32 && j < m.vdim) y[h * m.vdim + j] = fmaf(skip, v, o) * silu(z);
+}
+
+// ── many tokens: convolution ──
+// grid (channel blocks + 1, token blocks of kConvTok), a thread walks one channel; the last column of blocks does the step
+// sizes.  Only the first token block reads the ring, and each of its threads rewrites it for its channel afterwards.
+constexpr uint32_t kConvTok = 32;
+template <typename TA, int TAPS>
+__global__ void __launch_bounds__(256) ssm_conv_kernel(const Ssm m, const TA* __restrict__ proj, uint32_t ld, TA* __restrict__ out, uint32_t ld_out,
+                                                        float* __restrict__ dt, uint32_t T, uint32_t start) {
+    const uint32_t t0 = blockIdx.y * kConvTok, t1 = min(T, t0 + kConvTok);
+    if (blockIdx.x == gridDim.x - 1) {
+        for (uint32_t i = t0 * m.heads + threadIdx.x; i < t1 * m.heads; i += 256) dt[i] = softplus(dt[i] + m.dt_bias[i % m.heads]);
+        return;
+    }
+    const uint32_t c = blockIdx.x * 256 + threadIdx.x, ch = m.channels(), taps = TAPS ? TAPS : m.taps;
+    if (c >= ch) return;
+    const TA* x = proj + m.inner() + c;
+    const float* w = m.conv_w + (size_t)c * taps;
+    const float b = m.conv_b[c];
+    auto input = [&](int32_t t) -> float {           // t relative to the portion
+        if (t >= 0) return to_f32(x[(size_t)t * ld]);
+        return (int32_t)start + t >= 0 ? m.ring[(size_t)((start + t) % taps) * ch + c] : 0.f;
+    };
+    if constexpr (TAPS > 0) {
+        float win[TAPS], wr[TAPS];
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) wr[j] = w[j];
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; j++) win[j + 1] = input((int32_t)t0 - (TAPS - 1 - j));
+#pragma unroll 4
+        for (uint32_t t = t0; t < t1; t++) {
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; j++) win[j] = win[j + 1];
+            win[TAPS - 1] = to_f32(x[(size_t)t * ld]);
+            float s = b;
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) s = fmaf(wr[j], win[j], s);
+            put(out + (size_t)t * ld_out + c, silu(s));
+        }
+    } else {
+        for (uint32_t t = t0; t < t1; t++) {
+            float s = b;
+            for (uint32_t j = 0; j < taps; j++) s = fmaf(w[j], input((int32_t)t - (int32_t)(taps - 1 - j)), s);
+            put(out + (size_t)t * ld_out + c, silu(s));
+        }
+    }
+    if (blockIdx.y == 0)
+        for (uint32_t t = T > taps ? T - taps : 0; t < T; t++) m.ring[(size_t)((start + t) % taps) * ch + c] = to_f32(x[(size_t)t * ld]);
+}
+
+// ── many tokens: the recurrence token by token ──
+// grid (heads, ceil(dv / 32)), 256 threads: lane = column, warp w keeps rows w, w + 8, ... of the state in registers.
+template <typename TA, int NR>
+__global__ void __launch_bounds__(256) linear_scan_kernel(const LinearRows d, uint32_t T, uint32_t fresh) {
+    __shared__ float qs[2][NR * 8], ks[2][NR * 8], red[2][8][33];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, j = blockIdx.y * 32 + lane, g = h / (d.heads / d.groups);
+    const bool live = j < d.dv;
+    const TA *q = (const TA*)d.q + g * d.dk, *k = (const TA*)d.k + g * d.dk, *v = (const TA*)d.v + h * d.dv + j;
+    float* S = d.state + (size_t)h * d.dk * d.dv;
+    TA* out = (TA*)d.out + h * d.dv + j;
+    const float skip = d.skip ? d.skip[h] : 0.f, ld = d.log_decay ? d.log_decay[h] : 0.f, fixed = d.decay ? d.decay[h] : 0.f;
+    float s[NR];
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const uint32_t i = warp + 8 * r;
+        s[r] = (!fresh && i < d.dk && live) ? S[(size_t)i * d.dv + j] : 0.f;
+    }
+    for (uint32_t t = 0; t < T; t++) {
+        const uint32_t b = t & 1;
+        const float dt = d.dt ? d.dt[(size_t)t * d.heads + h] : 1.f;
+        for (uint32_t i = tid; i < NR * 8; i += 256) {
+            qs[b][i] = i < d.dk ? to_f32(q[(size_t)t * d.ldq + i]) : 0.f;
+            ks[b][i] = i < d.dk ? to_f32(k[(size_t)t * d.ldk + i]) * dt : 0.f;
+        }
+        const float vv = live ? to_f32(v[(size_t)t * d.ldv]) : 0.f, decay = d.dt ? expf(ld * dt) : fixed;
+        __syncthreads();
+        float o = 0.f;
+#pragma unroll
+        for (int r = 0; r < NR; r++) {
+            s[r] = fmaf(ks[b][warp + 8 * r], vv, decay * s[r]);
+            o = fmaf(s[r], qs[b][warp + 8 * r], o);
+        }
+        red[b][warp][lane] = o;
+        __syncthreads();
+        if (warp == 0 && live) {
+            float sum = skip * vv;
+#pragma unroll
+            for (int w = 0; w < 8; w++) sum += red[b][w][lane];
+            put(out + (size_t)t * d.ldo, sum);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < NR; r++) {
+        const uint32_t i = warp + 8 * r;
+        if (i < d.dk && live) S[(size_t)i * d.dv + j] = s[r];
+    }
+}
+
+// ── many tokens: chunks ──
+constexpr uint32_t kChunk = 64;
+static inline uint32_t pad64(uint32_t n) { return (n + 63) & ~63u; }
+
+__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"(addr));
+}
+// Rows t0 .. t0+63 of a bf16 matrix (n of its columns) into shared rows of `pitch` elements, `cols` of them filled; rows from T
+// on and columns from n on become zero.  Asynchronous where the rows are 16-byte aligned (wide).
+__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, uint32_t pitch, const __nv_bfloat16* src, uint32_t ld, uint32_t n, uint32_t cols,
+                                            uint32_t t0, uint32_t T, bool wide, uint32_t threads) {
+    const uint32_t cpr = cols / 8;
+    for (uint32_t i = threadIdx.x; i < kChunk * cpr; i += threads) {
+        const uint32_t r = i / cpr, c = (i - r * cpr) * 8;
+        __nv_bfloat16* p = dst + r * pitch + c;
+        const __nv_bfloat16* s = src + (size_t)(t0 + r) * ld + c;
+        if (t0 + r >= T || c >= n) {
+            *reinterpret_cast<uint4*>(p) = make_uint4(0, 0, 0, 0);
+        } else if (wide) {
+            cp_async16(smem_u32(p), s);
+        } else {
+            for (uint32_t e = 0; e < 8; e++) p[e] = c + e < n ? s[e] : __float2bfloat16_rn(0.f);
+        }
+    }
+}
+__device__ __forceinline__ bool rows_aligned(const void* p, uint32_t ld, uint32_t n) {
+    return (reinterpret_cast<uintptr_t>(p) & 15u) == 0 && (ld & 7u) == 0 && (n & 7u) == 0;
+}
+// One warp: la[t] = sum of the log decays of tokens 0 .. t of the chunk (0 for the tokens past the end), w[t] = step size.
+__device__ __forceinline__ void chunk_decays(const LinearRows& d, uint32_t h, uint32_t t0, uint32_t T, float* la, float* w) {
+    const uint32_t lane = threadIdx.x & 31;
+    const float ld = d.log_decay[h];
+    float x[2];
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const uint32_t t = t0 + 2 * lane + i;
+        const float dt = t < T ? (d.dt ? d.dt[(size_t)t * d.heads + h] : 1.f) : 0.f;
+        w[2 * lane + i] = dt;
+        x[i] = ld * dt;
+    }
+    x[1] += x[0];
+    float s = x[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float n = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= (uint32_t)o) s += n;
+    }
+    const float before = s - x[1];
+    la[2 * lane] = before + x[0];
+    la[2 * lane + 1] = s;
+}
+
+// grid (heads, dvp / 32), 8 warps; warp w owns the 16-row tiles w, w + 8 of the state.  states: [chunk][head][2][dkp][dvp], the
+// high and the low bf16 part of the state at the start of a chunk.
+__global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, __nv_bfloat16* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T,
+                                                           uint32_t fresh) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    constexpr uint32_t LV = 40;
+    const uint32_t lk = dkp + 8;
+    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [2][64][lk]
+    __nv_bfloat16* vS = kS + 2 * kChunk * lk;                         // [2][64][LV]
+    __shared__ float la[2][kChunk], wt[2][kChunk];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const uint32_t h = blockIdx.x, j0 = blockIdx.y * 32, grp = h / (d.heads / d.groups);
+    const __nv_bfloat16 *k = (const __nv_bfloat16*)d.k + grp * d.dk, *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
+    float* S = d.state + (size_t)h * d.dk * d.dv;
+    const bool wide = rows_aligned(k, d.ldk, d.dk);
+    float acc[2][4][4];
+#pragma unroll
+    for (int m = 0; m < 2; m++)
+#pragma unroll
+        for (int n = 0; n < 4; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const uint32_t i = (warp + 8 * m) * 16 + g + (e >> 1) * 8, j = j0 + n * 8 + 2 * t4 + (e & 1);
+                acc[m][n][e] = (!fresh && i < d.dk && j < d.dv) ? S[(size_t)i * d.dv + j] : 0.f;
+            }
+    const uint32_t nc = (T + kChunk - 1) / kChunk;
+    // value rows: thread -> token tid / 4, columns 8 * (tid % 4) ..
+    const uint32_t vt = tid >> 2, vc = (tid & 3) * 8;
+    const bool vwide = rows_aligned(v, d.ldv, 8) && j0 + vc + 8 <= d.dv;
+    float vr[8];
+    auto load_v = [&](uint32_t c) {
+        const uint32_t t = c * kChunk + vt;
+        const __nv_bfloat16* p = v + (size_t)t * d.ldv + vc;
+        if (t < T && vwide) {
+            const uint4 u = *reinterpret_cast<const uint4*>(p);
+            const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                vr[2 * i] = __uint_as_float(w[i] << 16);
+                vr[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; i++) vr[i] = (t < T && j0 + vc + i < d.dv) ? __bfloat162float(p[i]) : 0.f;
+        }
+    };
+    stage_rows(kS, lk, k, d.ldk, d.dk, dkp, 0, T, wide, 256);
+    cp_async_commit();
+    load_v(0);
+    if (warp == 7) chunk_decays(d, h, 0, T, la[0], wt[0]);
+    __syncthreads();
+    for (uint32_t c = 0; c < nc; c++) {
+        const uint32_t b = c & 1;
+        const float total = la[b][kChunk - 1];
+        {
+            const float f = wt[b][vt] * expf(total - la[b][vt]);
+            uint4 u = make_uint4(pack_bf2(vr[0] * f, vr[1] * f), pack_bf2(vr[2] * f, vr[3] * f), pack_bf2(vr[4] * f, vr[5] * f), pack_bf2(vr[6] * f, vr[7] * f));
+            *reinterpret_cast<uint4*>(vS + (size_t)b * kChunk * LV + vt * LV + vc) = u;
+        }
+        if (c + 1 < nc) {
+            stage_rows(kS + (size_t)(b ^ 1) * kChunk * lk, lk, k, d.ldk, d.dk, dkp, (c + 1) * kChunk, T, wide, 256);
+            cp_async_commit();
+            load_v(c + 1);
+            if (warp == 7) chunk_decays(d, h, (c + 1) * kChunk, T, la[b ^ 1], wt[b ^ 1]);
+        }
+        // the state at the start of the chunk
+        __nv_bfloat16* hi = states + ((size_t)c * d.heads + h) * 2 * dkp * dvp;
+        __nv_bfloat16* lo = hi + (size_t)dkp * dvp;
+        const float e = expf(total);
+#pragma unroll
+        for (int m = 0; m < 2; m++) {
+            const uint32_t i0 = (warp + 8 * m) * 16 + g;
+            if ((warp + 8 * m) * 16 >= dkp) break;
+#pragma unroll
+            for (int n = 0; n < 4; n++)
+#pragma unroll
+                for (int half = 0; half < 2; half++) {
+                    float &x = acc[m][n][2 * half], &y = acc[m][n][2 * half + 1];
+                    const size_t at = (size_t)(i0 + 8 * half) * dvp + j0 + n * 8 + 2 * t4;
+                    const __nv_bfloat16 hx = __float2bfloat16_rn(x), hy = __float2bfloat16_rn(y);
+                    *reinterpret_cast<__nv_bfloat162*>(hi + at) = __halves2bfloat162(hx, hy);
+                    *reinterpret_cast<uint32_t*>(lo + at) = pack_bf2(x - __bfloat162float(hx), y - __bfloat162float(hy));
+                    x *= e;
+                    y *= e;
+                }
+        }
+        if (c + 1 < nc) cp_async_wait<1>();
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t k_u = smem_u32(kS + (size_t)b * kChunk * lk), v_u = smem_u32(vS + (size_t)b * kChunk * LV);
+#pragma unroll
+        for (int kk = 0; kk < 4; kk++) {
+            uint32_t vb[2][4];
+#pragma unroll
+            for (int n = 0; n < 2; n++) ldsm_x4_trans(vb[n], v_u + ((kk * 16 + (lane & 15)) * LV + n * 16 + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int m = 0; m < 2; m++) {
+                const uint32_t mt = (warp + 8 * m) * 16;
+                if (mt >= dkp) break;
+                uint32_t a[4];          // K^T: tiles (tokens 0-7 | 8-15) x (rows 0-7 | 8-15), transposed
+                ldsm_x4_trans(a, k_u + ((kk * 16 + (lane >> 4) * 8 + (lane & 7)) * lk + mt + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll
+                for (int n = 0; n < 4; n++) mma_bf16(acc[m][n], a, vb[n >> 1][(n & 1) * 2], vb[n >> 1][(n & 1) * 2 + 1]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int m = 0; m < 2; m++)
+#pragma unroll
+        for (int n = 0; n < 4; n++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const uint32_t i = (warp + 8 * m) * 16 + g + (e >> 1) * 8, j = j0 + n * 8 + 2 * t4 + (e & 1);
+                if (i < d.dk && j < d.dv) S[(size_t)i * d.dv + j] = acc[m][n][e];
+            }
+}
+
+// grid (chunks, heads, dvp / 64), 4 warps of 16 tokens.
+__global__ void __launch_bounds__(128) chunk_out_kernel(const LinearRows d, const __nv_bfloat16* __restrict__ states, uint32_t dkp, uint32_t dvp,
+                                                         uint32_t T) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    constexpr uint32_t LV = 72;
+    const uint32_t lk = dkp + 8;
+    __nv_bfloat16* qS = reinterpret_cast<__nv_bfloat16*>(smem);       // [64][lk]
+    __nv_bfloat16* kS = qS + kChunk * lk;                             // [64][lk]
+    __nv_bfloat16* vS = kS + kChunk * lk;                             // [64][LV]
+    __nv_bfloat16* hS = vS + kChunk * LV;                             // [2][dkp][LV]
+    __shared__ float la[kChunk], wt[kChunk];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const uint32_t c = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 64, grp = h / (d.heads / d.groups), t0 = c * kChunk;
+    const __nv_bfloat16 *q = (const __nv_bfloat16*)d.q + grp * d.dk, *k = (const __nv_bfloat16*)d.k + grp * d.dk,
+                        *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
+    const uint32_t nv = min(64u, d.dv - j0);
+    const bool wq = rows_aligned(q, d.ldq, d.dk), wk = rows_aligned(k, d.ldk, d.dk), wv = rows_aligned(v, d.ldv, nv);
+    stage_rows(qS, lk, q, d.ldq, d.dk, dkp, t0, T, wq, 128);
+    {
+        const __nv_bfloat16* hi = states + ((size_t)c * d.heads + h) * 2 * dkp * dvp + j0;
+        for (uint32_t i = tid; i < 2 * dkp * 8; i += 128) cp_async16(smem_u32(hS + (i >> 3) * LV + (i & 7) * 8), hi + (size_t)(i >> 3) * dvp + (i & 7) * 8);
+    }
+    cp_async_commit();
+    stage_rows(kS, lk, k, d.ldk, d.dk, dkp, t0, T, wk, 128);
+    stage_rows(vS, LV, v, d.ldv, nv, 64, t0, T, wv, 128);
+    cp_async_commit();
+    if (warp == 0) chunk_decays(d, h, t0, T, la, wt);
+    cp_async_wait<1>();
+    __syncthreads();
+    float o[8][4];
+#pragma unroll
+    for (int n = 0; n < 8; n++) { o[n][0] = 0.f; o[n][1] = 0.f; o[n][2] = 0.f; o[n][3] = 0.f; }
+    const uint32_t q_u = smem_u32(qS + (warp * 16 + (lane & 15)) * lk + (lane >> 4) * 8);
+    const uint32_t h_u = smem_u32(hS + (lane & 15) * LV + (lane >> 4) * 8), lo_off = dkp * LV * 2;
+#pragma unroll 2
+    for (uint32_t ks = 0; ks < dkp / 16; ks++) {
+        uint32_t a[4];
+        ldsm_x4(a, q_u + ks * 32);
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+            uint32_t b[4], bl[4];
+            ldsm_x4_trans(b, h_u + (ks * 16 * LV + n * 8) * 2);
+            ldsm_x4_trans(bl, h_u + lo_off + (ks * 16 * LV + n * 8) * 2);
+            mma_bf16(o[n], a, b[0], b[1]);
+            mma_bf16(o[n + 1], a, b[2], b[3]);
+            mma_bf16(o[n], a, bl[0], bl[1]);
+            mma_bf16(o[n + 1], a, bl[2], bl[3]);
+        }
+    }
+    const uint32_t ra = warp * 16 + g, rb = ra + 8;
+    const float la_a = la[ra], la_b = la[rb];
+    {
+        const float e_a = expf(la_a), e_b = expf(la_b);
+#pragma unroll
+        for (int n = 0; n < 8; n++) { o[n][0] *= e_a; o[n][1] *= e_a; o[n][2] *= e_b; o[n][3] *= e_b; }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    // products within the chunk: 16 tokens at a time up to this warp's own
+    const uint32_t k_u = smem_u32(kS + ((lane >> 4) * 8 + (lane & 7)) * lk + ((lane >> 3) & 1) * 8);
+    const uint32_t v_u = smem_u32(vS + (lane & 15) * LV + (lane >> 4) * 8);
+    for (uint32_t kk = 0; kk <= warp; kk++) {
+        float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (uint32_t ks = 0; ks < dkp / 16; ks++) {
+            uint32_t a[4], b[4];
+            ldsm_x4(a, q_u + ks * 32);
+            ldsm_x4(b, k_u + (kk * 16 * lk + ks * 16) * 2);
+            mma_bf16(s0, a, b[0], b[1]);
+            mma_bf16(s1, a, b[2], b[3]);
+        }
+        auto weigh = [&](float s, uint32_t i, float la_i, uint32_t j) { return j <= i ? s * wt[j] * expf(la_i - la[j]) : 0.f; };
+        const uint32_t ja = kk * 16 + 2 * t4;
+        const uint32_t p[4] = {pack_bf2(weigh(s0[0], ra, la_a, ja), weigh(s0[1], ra, la_a, ja + 1)),
+                               pack_bf2(weigh(s0[2], rb, la_b, ja), weigh(s0[3], rb, la_b, ja + 1)),
+                               pack_bf2(weigh(s1[0], ra, la_a, ja + 8), weigh(s1[1], ra, la_a, ja + 9)),
+                               pack_bf2(weigh(s1[2], rb, la_b, ja + 8), weigh(s1[3], rb, la_b, ja + 9))};
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+            uint32_t b[4];
+            ldsm_x4_trans(b, v_u + (kk * 16 * LV + n * 8) * 2);
+            mma_bf16(o[n], p, b[0], b[1]);
+            mma_bf16(o[n + 1], p, b[2], b[3]);
+        }
+    }
+    const float skip = d.skip ? d.skip[h] : 0.f;
+    const bool pairs = (d.dv & 1u) == 0 && (d.ldo & 1u) == 0;
+    __nv_bfloat16* out = (__nv_bfloat16*)d.out + h * d.dv + j0;
+#pragma unroll
+    for (int n = 0; n < 8; n++) {
+        const uint32_t j = n * 8 + 2 * t4;
+        if (j >= nv) continue;
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const uint32_t r = half ? rb : ra;
+            if (t0 + r >= T) continue;
+            const float x = fmaf(skip, __bfloat162float(vS[r * LV + j]), o[n][2 * half]), y = fmaf(skip, __bfloat162float(vS[r * LV + j + 1]), o[n][2 * half + 1]);
+            __nv_bfloat16* p = out + (size_t)(t0 + r) * d.ldo + j;
+            if (pairs) {
+                *reinterpret_cast<uint32_t*>(p) = pack_bf2(x, y);
+            } else {
+                p[0] = __float2bfloat16_rn(x);
+                if (j + 1 < nv) p[1] = __float2bfloat16_rn(y);
+            }
+        }
+    }
+}
+
+// ── gate and norm ──
+// grid (T), 256 threads; the row's values (and their factors) pass through shared memory.
+template <typename TA, bool BEFORE>
+__global__ void __launch_bounds__(256) gated_norm_kernel(TA* __restrict__ a, uint32_t lda, uint32_t n, uint32_t group, const TA* __restrict__ gate,
+                                                          uint32_t ldg, const float* __restrict__ weight, float out_scale, float eps) {
+    extern __shared__ __align__(16) float sm[];
+    float *v = sm, *fac = sm + n;
+    TA* row = a + (size_t)blockIdx.x * lda;
+    const TA* gr = gate + (size_t)blockIdx.x * ldg;
+    for (uint32_t i = threadIdx.x; i < n; i += 256) {
+        float x = to_f32(row[i]);
+        if (BEFORE) x *= silu(to_f32(gr[i]));
+        v[i] = x;
+    }
+    __syncthreads();
+    const uint32_t groups = n / group, wpg = groups >= 8 ? 1u : (groups >= 3 ? 2u : (groups == 2 ? 4u : 8u));
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = warp % wpg;
+    for (uint32_t g = warp / wpg; g < groups; g += 8 / wpg) {
+        float sq = 0.f;
+        for (uint32_t i = sub * 32 + lane; i < group; i += 32 * wpg) sq = fmaf(v[g * group + i], v[g * group + i], sq);
+        sq = wsum(sq);
+        if (lane == 0) fac[g * wpg + sub] = sq;
+    }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x; i < n; i += 256) {
+        const uint32_t g = i / group;
+        float sq = 0.f;
+        for (uint32_t k = 0; k < wpg; k++) sq += fac[g * wpg + k];
+        float x = v[i] * rsqrtf(sq / (float)group + eps);
+        if (BEFORE) x *= weight[i];
+        else x *= silu(to_f32(gr[i])) * out_scale;
+        put(row + i, x);
+    }
+}
+
+template <typename K>
+static int32_t allow_smem(runit_ctx* ctx, const char* name, K kern, size_t smem) {
+    RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 2048, "%s: the layer's sizes do not fit shared memory", name);
+    if (smem > 40 * 1024) RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return RUNIT_OK;
+}
+
+}  // namespace ls
+
+using namespace ls;
+
+int32_t ssm_step(runit_ctx* ctx, const Ssm& m, const float* proj, float* y, const int32_t* pos_ptr) {
+    RUNIT_REQUIRE(ctx, m.state <= kMaxKeyDim, "ssm_step: bad sizes");
+    runit_launch_chain_smem(ctx, ssm_step_kernel, dim3(m.heads, (m.vdim + 31) / 32), dim3(256), (size_t)m.state * 8, m, proj, y, pos_ptr);
+    return runit_after_launch(ctx, "ssm_step");
+}
+
+int32_t ssm_conv_rows(runit_ctx* ctx, const Ssm& m, bool exact, const void* proj, uint32_t ld, void* xbc, uint32_t ld_out, float* dt, uint32_t T,
+                      uint32_t start) {
+    RUNIT_REQUIRE(ctx, m.taps >= 1 && m.taps <= kConvTok, "ssm_conv: %u taps (1 .. %u)", m.taps, kConvTok);
+    const dim3 grid((m.channels() + 255) / 256 + 1, (T + kConvTok - 1) / kConvTok);
+    auto go = [&](auto kern, auto* p, auto* o) -> int32_t {
+        kern<<<grid, 256, 0, ctx->stream>>>(m, p, ld, o, ld_out, dt, T, start);
+        return runit_after_launch(ctx, "ssm_conv");
+    };
+    if (exact) return m.taps == 4 ? go(ssm_conv_kernel<float, 4>, (const float*)proj, (float*)xbc) : go(ssm_conv_kernel<float, 0>, (const float*)proj, (float*)xbc);
+    if (m.taps == 4) return go(ssm_conv_kernel<__nv_bfloat16, 4>, (const __nv_bfloat16*)proj, (__nv_bfloat16*)xbc);
+    return go(ssm_conv_kernel<__nv_bfloat16, 0>, (const __nv_bfloat16*)proj, (__nv_bfloat16*)xbc);
+}
+
+static bool chunk_sizes(uint32_t dk) { return ((dk + 15) & ~15u) <= 256; }
+size_t linear_chunk_bytes(uint32_t heads, uint32_t dk, uint32_t dv, uint32_t T) {
+    if (!chunk_sizes(dk)) return 0;
+    return (size_t)((T + kChunk - 1) / kChunk) * heads * pad16(dk) * pad64(dv) * 4;
+}
+
+int32_t linear_rows(runit_ctx* ctx, const LinearRows& d, bool exact, void* chunk_states, uint32_t T, uint32_t start) {
+    RUNIT_REQUIRE(ctx, d.heads > 0 && d.groups > 0 && d.heads % d.groups == 0 && d.dk > 0 && d.dk <= kMaxKeyDim && d.dv > 0, "linear_rows: bad sizes");
+    int32_t st;
+    if (!exact && T >= 16 && chunk_states && chunk_sizes(d.dk)) {
+        const uint32_t dkp = pad16(d.dk), dvp = pad64(d.dv), nc = (T + kChunk - 1) / kChunk;
+        const size_t sa = (size_t)2 * kChunk * (dkp + 8 + 40) * 2, sb = ((size_t)2 * kChunk * (dkp + 8) + kChunk * 72 + (size_t)2 * dkp * 72) * 2;
+        if ((st = allow_smem(ctx, "chunk_state", chunk_state_kernel, sa)) != RUNIT_OK) return st;
+        chunk_state_kernel<<<dim3(d.heads, dvp / 32), 256, sa, ctx->stream>>>(d, (__nv_bfloat16*)chunk_states, dkp, dvp, T, start == 0);
+        if ((st = runit_after_launch(ctx, "chunk_state")) != RUNIT_OK) return st;
+        if ((st = allow_smem(ctx, "chunk_out", chunk_out_kernel, sb)) != RUNIT_OK) return st;
+        chunk_out_kernel<<<dim3(nc, d.heads, dvp / 64), 128, sb, ctx->stream>>>(d, (const __nv_bfloat16*)chunk_states, dkp, dvp, T);
+        return runit_after_launch(ctx, "chunk_out");
+    }
+    const dim3 grid(d.heads, (d.dv + 31) / 32);
+#define RUNIT_SCAN(NR)                                                                                            \
+    do {                                                                                                          \
+        if (exact) linear_scan_kernel<float, NR><<<grid, 256, 0, ctx->stream>>>(d, T, start == 0);                 \
+        else linear_scan_kernel<__nv_bfloat16, NR><<<grid, 256, 0, ctx->stream>>>(d, T, start == 0);               \
+    } while (0)
+    if (d.dk <= 64) RUNIT_SCAN(8);
+    else if (d.dk <= 128) RUNIT_SCAN(16);
+    else if (d.dk <= 256) RUNIT_SCAN(32);
+    else RUNIT_SCAN(128);
+#undef RUNIT_SCAN
+    return runit_after_launch(ctx, "linear_scan");
+}
+
+int32_t gated_norm_rows(runit_ctx* ctx, bool exact, void* a, uint32_t lda, uint32_t n, uint32_t group, const void* gate, uint32_t ldg, bool before,
+                        const float* weight, float out_scale, float eps, uint32_t T) {
+    RUNIT_REQUIRE(ctx, group > 0 && n % group == 0 && (!before || weight), "gated_norm: bad groups");
+    const size_t smem = ((size_t)n + n / group + 8) * 4;
+    int32_t st;
+    auto go = [&](auto kern, auto* p, auto* g) -> int32_t {
+        if ((st = allow_smem(ctx, "gated_norm", kern, smem)) != RUNIT_OK) return st;
+        kern<<<T, 256, smem, ctx->stream>>>(p, lda, n, group, g, ldg, weight, out_scale, eps);
+        return runit_after_launch(ctx, "gated_norm");
+    };
+    if (exact) return before ? go(gated_norm_kernel<float, true>, (float*)a, (const float*)gate) : go(gated_norm_kernel<float, false>, (float*)a, (const float*)gate);
+    return before ? go(gated_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16*)a, (const __nv_bfloat16*)gate)
+                  : go(gated_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)a, (const __nv_bfloat16*)gate);
+}
+
+}  // namespace runit

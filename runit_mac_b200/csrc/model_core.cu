@@ -135,6 +135,8 @@ int32_t runit_model::forward(const int32_t*, uint32_t, uint32_t, const uint32_t*
     return runit_fail(ctx, RUNIT_ERR_UNSUPPORTED, "model_forward: not available on this decoder");
 }
 
+int32_t runit_model::check_start(uint32_t) { return RUNIT_OK; }
+
 extern "C" {
 
 int32_t runit_model_destroy(runit_model_t* m) {
@@ -183,7 +185,8 @@ int32_t runit_model_reset(runit_model_t* m, int32_t token, int32_t pos) {
 int32_t runit_model_forward_greedy(runit_model_t* m, int32_t token_id, int32_t pos, int32_t* next_token) {
     if (!m) return RUNIT_ERR_BAD_ARG;
     runit_ctx* ctx = m->ctx;
-    int32_t st = runit_model_reset(m, token_id, pos);
+    int32_t st = pos > 0 ? m->check_start((uint32_t)pos) : RUNIT_OK;
+    if (st == RUNIT_OK) st = runit_model_reset(m, token_id, pos);
     if (st != RUNIT_OK) return st;
     // step 0 must not be forced by a prompt left over from runit_model_generate_greedy
     RUNIT_CUDA_TRY(ctx, cudaMemsetAsync(m->forced, 0xFF, 4, ctx->stream));
@@ -250,6 +253,10 @@ static int32_t generate_impl(runit_model_t* m, const int32_t* prompt, uint32_t n
     RUNIT_REQUIRE(ctx, n_prompt <= m->forced_cap && n_steps <= m->out_cap, "model_generate_greedy: too many steps");
     for (uint32_t i = 0; i < n_prompt; i++)
         RUNIT_REQUIRE(ctx, prompt[i] >= 0 && prompt[i] < m->vocab, "model_generate_greedy: token id %d out of range", prompt[i]);
+    if (start_pos > 0) {
+        const int32_t ok = m->check_start((uint32_t)start_pos);
+        if (ok != RUNIT_OK) return ok;
+    }
     RUNIT_CUDA_TRY(ctx, cudaMemcpyAsync(m->forced, prompt, (size_t)n_prompt * 4, cudaMemcpyHostToDevice, ctx->stream));
     // the sampler's context range inside out_tokens: from the step that produces the first generated token to the current step
     const int32_t range[2] = {(int32_t)n_prompt - 1, 0};

@@ -36,6 +36,8 @@ struct runit_model {
     virtual int32_t forward(const int32_t* tokens, uint32_t n, uint32_t start_pos, const uint32_t* want, uint32_t n_want, float* logits_host);
     virtual uint64_t launches_per_token() = 0;
     virtual bool can_sample() const { return true; }
+    // Whether the cache and state allow a pass that starts at `pos` (0 always does).
+    virtual int32_t check_start(uint32_t pos);
 };
 
 namespace runit {

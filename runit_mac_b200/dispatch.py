@@ -415,6 +415,7 @@ class Model:
 
 
 FF_NONE, FF_DENSE, FF_MOE = 0, 1, 2
+MIX_LATENT, MIX_HEADS, MIX_SSM = 0, 1, 2
 ACT_SILU_GLU, ACT_RELU2 = 0, 1
 
 
@@ -432,12 +433,18 @@ class LayerDesc(C.Structure):
                 [(n, C.c_float) for n in ("scale", "rot_base")] +
                 [(n, C.c_int32) for n in ("ff_kind", "ff_act", "ff", "n_experts", "top_k", "score", "renorm", "shared_ff")] +
                 [(n, C.c_void_p) for n in ("norm1", "norm2", "w_q", "kv_norm", "w_ukv", "w_o", "ff_up", "ff_down", "router", "shared_up",
-                                           "shared_down")])
+                                           "shared_down")] +
+                [(n, C.c_int32) for n in ("mixer", "at_heads", "at_kv_heads", "at_dim", "at_vdim", "at_window", "at_unit_qk",
+                                          "rt_heads", "rt_dim", "rt_vdim", "rt_rot_dims",
+                                          "ss_heads", "ss_vdim", "ss_state", "ss_groups", "ss_taps", "ss_norm_groups")] +
+                [(n, C.c_float) for n in ("at_scale", "at_out_scale", "rt_rot_base", "rt_out_scale")] +
+                [(n, C.c_void_p) for n in ("at_slopes", "rt_decay", "ss_conv", "ss_conv_b", "ss_dt_bias", "ss_a", "ss_skip", "ss_norm")])
 
 
 class LayeredCfg(C.Structure):
     """runit_layered_cfg"""
-    _fields_ = [(n, C.c_int32) for n in ("n_layers", "width", "vocab", "max_seq", "exact")] + [("eps", C.c_float)]
+    _fields_ = ([(n, C.c_int32) for n in ("n_layers", "width", "vocab", "max_seq", "exact", "post_norm")] +
+                [(n, C.c_float) for n in ("eps", "embed_scale", "logit_cap")])
 
 
 class LayeredWeights(C.Structure):
@@ -519,5 +526,5 @@ def moe_layer_q4k_host(ctx: Context, router, gate, up, down, x, *, h, ff, E, top
 
 
 __all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc", "LatentCfg", "EPI_F32", "EPI_ADD", "EPI_CAST", "EPI_SILU_GLU", "EPI_RELU2",
-           "FF_NONE", "FF_DENSE", "FF_MOE", "ACT_SILU_GLU", "ACT_RELU2", "SCORE_SOFTMAX", "SCORE_SIGMOID", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
+           "FF_NONE", "FF_DENSE", "FF_MOE", "MIX_LATENT", "MIX_HEADS", "MIX_SSM", "ACT_SILU_GLU", "ACT_RELU2", "SCORE_SOFTMAX", "SCORE_SIGMOID", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
            "FMT_Q8_0", "FMT_Q4_0", "FMT_Q4K", "FMT_Q5_0", "FMT_Q5K", "FMT_Q6K"] + [n for n, _ in _TWINS]

@@ -92,6 +92,26 @@ class _Uploader:
             parts.append(a.reshape(-1))
         return self._put(np.concatenate(parts))
 
+    def beside(self, parts, rows: int) -> int:
+        """Matrices side by side, as one: parts = [(name, columns)], each [rows][columns]; rows padded to pad8 of the sum."""
+        out = np.zeros((rows, pad8(sum(c for _, c in parts))), np.uint16)
+        at = 0
+        for name, c in parts:
+            out[:, at:at + c] = self._rows(name, rows, c)
+            at += c
+        return self._put(out)
+
+    def gain_offset(self, name: str, n: int) -> int:
+        """f32 gains of a norm whose weight is stored as the distance from one."""
+        a = self.source.f32(name)
+        if a.shape != (n,):
+            raise ConfigError("tensor %s has shape %r, the configuration says %r" % (name, a.shape, (n,)))
+        return self._put(np.float32(1.0) + a)
+
+    def values(self, a) -> int:
+        """f32 values that are computed from the configuration or from tensors."""
+        return self._put(np.ascontiguousarray(a, np.float32))
+
 
 def _latent_mixer(up: _Uploader, d: D.LayerDesc, p: str, mix: dict, width: int):
     """Latent attention: mixer sizes and tensors of the layer with prefix p."""
@@ -132,6 +152,107 @@ def _moe_ff(up: _Uploader, d: D.LayerDesc, p: str, mlp: dict, width: int):
         rows.append(p + "shared.sg")
         shapes.append((1, width))
     d.router = up.f32(rows, shapes)
+
+
+def head_slopes(heads: int) -> np.ndarray:
+    """Distance slopes of a layer's heads: a geometric series that ends at 2^-8."""
+    return (2.0 ** (-8.0 * np.arange(1, heads + 1) / heads)).astype(np.float32)
+
+
+def _attention_heads(d: D.LayerDesc, up: _Uploader, mix: dict):
+    """Windowed attention with unit queries and keys and a distance bias per head."""
+    d.at_heads, d.at_kv_heads, d.at_dim, d.at_vdim = (int(mix[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+    d.at_window, d.at_unit_qk, d.at_scale = int(mix["mask"]["size"]), 1, float(mix["scale"])
+    d.at_slopes = up.values(head_slopes(d.at_heads))
+
+
+def _retention_heads(d: D.LayerDesc, up: _Uploader, mix: dict, p: str):
+    d.rt_heads, d.rt_dim, d.rt_vdim = (int(mix[k]) for k in ("heads", "dim", "vdim"))
+    d.rt_rot_dims, d.rt_rot_base = int(mix["rot"]["dims"]), float(mix["rot"]["base"])
+    decay = np.asarray(mix["decay"], np.float64)
+    if decay.shape != (d.rt_heads,) or (decay < 0).any():
+        raise ConfigError("%s: %d decays for %d heads, none of them negative" % (p, decay.size, d.rt_heads))
+    # a decay of 0 has no logarithm: e^-1000 is 0 in f32 and stays finite when it is summed over a chunk
+    d.rt_decay = up.values(np.stack([decay, np.log(np.maximum(decay, np.exp(-700.0))) - 300.0 * (decay == 0)]))
+
+
+def _parallel_mixer(up: _Uploader, d: D.LayerDesc, p: str, mix: dict, width: int):
+    """Attention and retention side by side on the same input; one projection in, one out."""
+    left, right = mix["left"], mix["right"]
+    d.mixer = D.MIX_HEADS
+    _attention_heads(d, up, left)
+    _retention_heads(d, up, right, p)
+    d.at_out_scale, d.rt_out_scale = float(mix["left_scale"]), float(mix["right_scale"])
+    L, R = p + "left.", p + "right."
+    lv, rk, rv = d.at_heads * d.at_vdim, d.rt_heads * d.rt_dim, d.rt_heads * d.rt_vdim
+    d.w_q = up.matrix([(L + "q", d.at_heads * d.at_dim), (L + "k", d.at_kv_heads * d.at_dim), (L + "v", d.at_kv_heads * d.at_vdim),
+                       (R + "q", rk), (R + "k", rk), (R + "v", rv), (R + "g", rv)], width)
+    d.w_o = up.beside([(L + "o", lv), (R + "o", rv)], width)
+
+
+def _mamba2_mixer(up: _Uploader, d: D.LayerDesc, p: str, mix: dict, width: int):
+    d.mixer = D.MIX_SSM
+    H, vdim, N, G, taps = (int(mix[k]) for k in ("heads", "vdim", "state", "groups", "conv"))
+    d.ss_heads, d.ss_vdim, d.ss_state, d.ss_groups, d.ss_taps, d.ss_norm_groups = H, vdim, N, G, taps, int(mix["norm_groups"])
+    inner, channels = H * vdim, H * vdim + 2 * G * N
+    d.w_q = up.matrix([(p + "in", inner + channels + H)], width)
+    d.w_o = up.matrix([(p + "o", width)], inner)
+    d.ss_conv, d.ss_conv_b = up.f32([p + "conv"], [(channels, taps)]), up.f32([p + "conv.b"], [(channels,)])
+    d.ss_dt_bias, d.ss_skip, d.ss_norm = up.f32([p + "dt_bias"], [(H,)]), up.f32([p + "D"], [(H,)]), up.f32([p + "norm"], [(inner,)])
+    a = up.source.f32(p + "A_log").astype(np.float64).reshape(-1)
+    if a.size != H:
+        raise ConfigError("tensor %sA_log has %d values, the configuration says %d" % (p, a.size, H))
+    d.ss_a = up.values(-np.exp(a))
+
+
+def _relu2_ff(up: _Uploader, d: D.LayerDesc, p: str, mlp: dict, width: int):
+    d.ff_kind, d.ff_act, d.ff = D.FF_DENSE, D.ACT_RELU2, int(mlp["ff"])
+    d.ff_up = up.matrix([(p + "up", d.ff)], width)
+    d.ff_down = up.matrix([(p + "down", width)], d.ff)
+
+
+_PAGAZEN_MIXERS = {"parallel": _parallel_mixer, "mamba2": _mamba2_mixer}
+
+
+@register("Pagazen")
+def build_pagazen(ctx: D.Context, cfg: dict, source, dtype: str, max_seq: int) -> D.LayeredModel:
+    """Attention beside retention, or state-space layers; norms on the sublayers' outputs; layers may use another layer's
+    tensors, with a cache and state of their own."""
+    width, vocab = int(cfg["width"]), int(cfg["vocab"])
+    up = _Uploader(ctx, source)
+    entries = cfg["layers"]
+    own = {}
+
+    def layer_of(i: int) -> D.LayerDesc:
+        if i in own:
+            return own[i]
+        layer, p, d = entries[i], "l%d." % i, D.LayerDesc()
+        if layer["type"] not in _PAGAZEN_MIXERS:
+            raise ConfigError("layer %d: unknown mixer %r" % (i, layer["type"]))
+        d.norm1 = up.gain_offset(p + "norm1", width)
+        _PAGAZEN_MIXERS[layer["type"]](up, d, p + "mix.", layer["mixer"], width)
+        mlp = layer.get("mlp")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise ConfigError("layer %d: unknown feed-forward %r" % (i, mlp["kind"]))
+            d.norm2 = up.gain_offset(p + "norm2", width)
+            _relu2_ff(up, d, p + "mlp.", mlp, width)
+        own[i] = d
+        return d
+
+    layers = []
+    for i, layer in enumerate(entries):
+        j = layer.get("weights_of")
+        j = i if j is None else int(j)
+        if not 0 <= j < len(entries) or (j != i and entries[j].get("weights_of") not in (None, j)):
+            raise ConfigError("layer %d: uses the tensors of layer %d, which has none" % (i, j))
+        if any(layer.get(k) != entries[j].get(k) for k in ("type", "mixer", "mlp")):
+            raise ConfigError("layer %d differs from layer %d, whose tensors it uses" % (i, j))
+        layers.append(layer_of(j))
+    w = {"embed": up.matrix([("embed", vocab)], width), "final_norm": up.gain_offset("final.norm", width), "head": up.matrix([("head", vocab)], width)}
+    c = D.LayeredCfg(n_layers=len(layers), width=width, vocab=vocab, max_seq=max_seq, exact=int(dtype == "float32"), post_norm=1,
+                     eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]), logit_cap=float(cfg["logit_softcap"] or 0.0))
+    return D.LayeredModel(ctx, c, layers, w, keep=up)
 
 
 @register("Nuvilorn")
