@@ -644,7 +644,7 @@ def build_layered(R, ctx, torch, size, max_seq):
             d.shared_up, d.shared_down = mat(ff, W), mat(W, ff)
         layers.append(d)
     w = {"embed": mat(V, W), "embed_norm": one, "final_norm": one, "head": mat(V, W)}
-    cfg = R.LayeredCfg(n_layers=L, width=W, vocab=V, max_seq=max_seq, exact=0, eps=1e-6)
+    cfg = R.LayeredCfg(n_layers=L, width=W, vocab=V, max_seq=max_seq, exact=0, post_norm=0, eps=1e-6, embed_scale=1.0, logit_cap=0.0)
     torch.cuda.synchronize()
     return R.LayeredModel(ctx, cfg, layers, w, keep=keep)
 
@@ -685,11 +685,34 @@ def time_model(model, vocab, contexts=(128, 2048), steps=64):
         pr = np.random.default_rng(n).integers(0, vocab, n).astype(np.int32)
         nxt = np.array([model.prefill(pr)], np.int32)
         model.generate_greedy(nxt, 3, start_pos=n)
+        nxt = np.array([model.prefill(pr)], np.int32)      # a recurrent state does not go back
         t0 = time.perf_counter()
         model.generate_greedy(nxt, steps - 1, start_pos=n)
         dt = (time.perf_counter() - t0) / steps
         out["decode"]["context%d" % n] = {"us_per_token": dt * 1e6, "tokens_per_s": 1 / dt}
     return out
+
+
+def timed_list(ctx, torch, stream, fns, reps=20):
+    """Microseconds per call of the functions in turn, replayed from a recorded list (the host's launch cost stays out of it)."""
+    for f in fns[:3]:
+        f()
+    ctx.flush()
+    n = max(reps, len(fns))
+    ctx.graph_begin()
+    for i in range(n):
+        fns[i % len(fns)]()
+    gr = ctx.graph_end()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    for _ in range(2):
+        gr.launch()
+    torch.cuda.synchronize()
+    a.record(stream)
+    gr.launch()
+    b.record(stream)
+    torch.cuda.synchronize()
+    gr.destroy()
+    return a.elapsed_time(b) / n * 1e3
 
 
 def time_layered_kernels(R, ctx, torch, stream, size, reps=20):
@@ -701,26 +724,7 @@ def time_layered_kernels(R, ctx, torch, stream, size, reps=20):
     tc, _ = measured_tensor_peak()
     rows = []
 
-    def timed(fns):
-        # recorded: the host's launch cost stays out of the time of small kernels
-        for f in fns[:3]:
-            f()
-        ctx.flush()
-        n = max(reps, len(fns))
-        ctx.graph_begin()
-        for i in range(n):
-            fns[i % len(fns)]()
-        gr = ctx.graph_end()
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        for _ in range(2):
-            gr.launch()
-        torch.cuda.synchronize()
-        a.record(stream)
-        gr.launch()
-        b.record(stream)
-        torch.cuda.synchronize()
-        gr.destroy()
-        return a.elapsed_time(b) / n * 1e3
+    timed = lambda fns: timed_list(ctx, torch, stream, fns, reps)
 
     def add(name, us, us_like, nbytes=0, flops=0, nbytes_like=0, flops_like=0):
         f = lambda t, by, fl: by / (t * 1e-6) / 1e9 / hbm if by else fl / (t * 1e-6) / 1e12 / tc
@@ -816,6 +820,233 @@ def run_layered(R, ctx, torch, stream, sizes):
         del m
         if name == "2048":
             res["kernels"] = time_layered_kernels(R, ctx, torch, stream, size)
+        out[name] = res
+        torch.cuda.empty_cache()
+    return out
+
+
+# ── attention beside retention, and state-space layers ──
+# (width, layers, ff, state-space groups, vocab): every third layer runs grouped-query attention over a window of 1024 beside
+# retention, the others are state-space layers with inner width 2 W.  Next to it a dense latent-attention decoder of equal width,
+# depth and vocabulary whose gated feed-forward has as many weights.
+PAGAZEN_SIZES = {"1024": (1024, 12, 4096, 1, 50304), "2048": (2048, 12, 8192, 2, 50304), "4096": (4096, 6, 16384, 4, 50304)}
+
+
+def pagazen_dims(W):
+    return {"H": W // 128, "G": max(1, W // 512), "d": 128, "dv": 128, "window": 1024, "rH": W // 256, "rd": 128, "rdv": 256,
+            "sH": W // 32, "sd": 64, "N": 128}
+
+
+def build_pagazen(R, ctx, torch, size, max_seq):
+    W, L, ff, G, V = size
+    p = pagazen_dims(W)
+    keep = []
+
+    def own(t):
+        keep.append(t)
+        return t.data_ptr()
+    mat = lambda rows, cols: own(torch.empty(rows, cols, dtype=torch.bfloat16, device="cuda").normal_(0, 1.0 / cols ** 0.5))
+    f32 = lambda a: own(torch.as_tensor(np.asarray(a, np.float32), device="cuda"))
+    ones = f32(np.ones(8 * W))
+    g = np.random.default_rng(0)
+    layers = []
+    for i in range(L):
+        d = R.LayerDesc(norm1=ones, norm2=ones, ff_kind=R.FF_DENSE, ff_act=R.ACT_RELU2, ff=ff, ff_up=mat(ff, W), ff_down=mat(W, ff))
+        if i % 3 == 0:
+            decay = 1 - 2.0 ** -np.linspace(5, 11, p["rH"])
+            d.mixer, d.at_heads, d.at_kv_heads, d.at_dim, d.at_vdim, d.at_window, d.at_unit_qk = (
+                R.MIX_HEADS, p["H"], p["G"], p["d"], p["dv"], p["window"], 1)
+            d.at_scale, d.at_out_scale, d.at_slopes = p["d"] ** -0.5, 0.7, f32(2.0 ** (-8 * np.arange(1, p["H"] + 1) / p["H"]))
+            d.rt_heads, d.rt_dim, d.rt_vdim, d.rt_rot_dims, d.rt_rot_base, d.rt_out_scale = p["rH"], p["rd"], p["rdv"], p["rd"], 10000.0, 0.8
+            d.rt_decay = f32(np.stack([decay, np.log(decay)]))
+            d.w_q = mat(p["H"] * p["d"] + p["G"] * (p["d"] + p["dv"]) + 2 * p["rH"] * (p["rd"] + p["rdv"]), W)
+            d.w_o = mat(W, p["H"] * p["dv"] + p["rH"] * p["rdv"])
+        else:
+            inner, ch = p["sH"] * p["sd"], p["sH"] * p["sd"] + 2 * G * p["N"]
+            d.mixer, d.ss_heads, d.ss_vdim, d.ss_state, d.ss_groups, d.ss_taps, d.ss_norm_groups = R.MIX_SSM, p["sH"], p["sd"], p["N"], G, 4, G
+            d.ss_conv, d.ss_conv_b, d.ss_norm = f32(g.normal(0, 0.5, (ch, 4))), f32(np.zeros(ch)), ones
+            d.ss_dt_bias, d.ss_a, d.ss_skip = f32(g.uniform(-4, -1, p["sH"])), f32(-g.uniform(1, 8, p["sH"])), ones
+            d.w_q, d.w_o = mat(inner + ch + p["sH"], W), mat(W, inner)
+        layers.append(d)
+    w = {"embed": mat(V, W), "embed_norm": None, "final_norm": ones, "head": mat(V, W)}
+    cfg = R.LayeredCfg(n_layers=L, width=W, vocab=V, max_seq=max_seq, exact=0, post_norm=1, eps=1e-6, embed_scale=W ** 0.5, logit_cap=30.0)
+    torch.cuda.synchronize()
+    return R.LayeredModel(ctx, cfg, layers, w, keep=keep)
+
+
+def build_dense_latent(R, ctx, torch, size, max_seq):
+    W, L, ff, _G, V = size
+    H, rank, ff = W // 128, W // 4, ff * 2 // 3 // 8 * 8
+    keep = []
+
+    def own(t):
+        keep.append(t)
+        return t.data_ptr()
+    mat = lambda rows, cols: own(torch.empty(rows, cols, dtype=torch.bfloat16, device="cuda").normal_(0, 1.0 / cols ** 0.5))
+    one, ones = own(torch.ones(1, device="cuda")), own(torch.ones(rank, device="cuda"))
+    layers = [R.LayerDesc(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=rank, kv_from=-1, scale=192 ** -0.5, rot_base=10000.0, norm1=one, norm2=one,
+                          kv_norm=ones, w_q=mat(H * 192 + rank + 64, W), w_ukv=mat(H * 256, rank), w_o=mat(W, H * 128), ff_kind=R.FF_DENSE,
+                          ff_act=R.ACT_SILU_GLU, ff=ff, ff_up=mat(2 * ff, W), ff_down=mat(W, ff)) for _ in range(L)]
+    w = {"embed": mat(V, W), "embed_norm": one, "final_norm": one, "head": mat(V, W)}
+    cfg = R.LayeredCfg(n_layers=L, width=W, vocab=V, max_seq=max_seq, exact=0, post_norm=0, eps=1e-6, embed_scale=1.0, logit_cap=0.0)
+    torch.cuda.synchronize()
+    return R.LayeredModel(ctx, cfg, layers, w, keep=keep)
+
+
+def time_pagazen_kernels(R, ctx, torch, stream, size, reps=20, T=2048):
+    """Every kernel of a layer beside the like kernel of the latent-attention decoder: fraction of its roofline, the larger of
+    bytes / measured bandwidth and multiply-adds / measured tensor peak.  Inputs rotate over sets larger than L2."""
+    import ctypes as C
+    W, _L, ff, G, V = size
+    p = pagazen_dims(W)
+    hbm, tc = measured_peak()[0] * 1e9, measured_tensor_peak()[0] * 1e12
+    timed = lambda fns: timed_list(ctx, torch, stream, fns, reps)
+    bf = lambda *s: torch.empty(*s, dtype=torch.bfloat16, device="cuda").normal_(0, 0.5)
+    rows, likes = [], {}
+
+    def frac(us, nbytes, flops):
+        return max(nbytes / hbm, flops / tc) * 1e6 / us
+
+    def like(key, us, nbytes=0, flops=0):
+        likes[key] = frac(us, nbytes, flops)
+        rows.append({"like": key, "us": round(us, 2), "frac": round(likes[key], 3)})
+
+    def add(name, key, us, nbytes=0, flops=0):
+        f = frac(us, nbytes, flops)
+        rows.append({"kernel": name, "us": round(us, 2), "frac": round(f, 3), "like": key, "like_frac": round(likes[key], 3), "ratio": round(likes[key] / f, 2)})
+    n_sets = lambda nbytes: max(2, min(64, int(300e6 // nbytes) + 1))
+    # ── one token ──
+    x, y, gains, xo = torch.randn(W, device="cuda"), torch.randn(W, device="cuda"), torch.rand(8 * W, device="cuda"), torch.empty(W, device="cuda")
+    out, one = torch.empty(max(V, ff, 8 * W), device="cuda"), torch.ones(1, device="cuda")
+    ml, kl = (W // 128) * 192 + W // 4 + 64, W // 4
+    in_h = p["H"] * p["d"] + p["G"] * (p["d"] + p["dv"]) + 2 * p["rH"] * (p["rd"] + p["rdv"])
+    k_h, inner, ch = p["H"] * p["dv"] + p["rH"] * p["rdv"], p["sH"] * p["sd"], p["sH"] * p["sd"] + 2 * G * p["N"]
+    in_s = inner + ch + p["sH"]
+    gff = ff * 2 // 3 // 8 * 8
+
+    def gemv(m, k, call):
+        ws = [bf(m, k) for _ in range(n_sets(m * k * 2))]
+        return timed([(lambda w=w: call(w)) for w in ws])
+    plain = lambda m, k: gemv(m, k, lambda w: R.gemv_bf16_f32(ctx, w, gains, None if k != W else one, 1e-6, out, None, m, k))
+    res = lambda m, k, act: gemv(m, k, lambda w: R.gemv_bf16_residual_f32(ctx, w, x, y, gains, None, xo, out, 1e-6, 0.0, act, m, k))
+    for key, m, k in (("norm + projection", ml, W), ("gate / up", 2 * gff, W), ("output projection", W, W), ("down", W, gff), ("norm + head", V, W)):
+        like(key, plain(m, k), m * k * 2)
+    add("norm + residual + projections, attention beside retention", "norm + projection", res(in_h, W, 0), in_h * W * 2)
+    add("norm + residual + projections, state space", "norm + projection", res(in_s, W, 0), in_s * W * 2)
+    add("norm + residual + up + relu2", "gate / up", res(ff, W, 1), ff * W * 2)
+    add("down", "down", plain(W, ff), W * ff * 2)
+    grp = lambda m, k, pl, gr: gemv(m, k, lambda w: R.gemv_bf16_groups_f32(ctx, w, gains, gains, out, 1e-6, pl, gr, m, k))
+    add("head norms + output projection, attention beside retention", "output projection", grp(W, k_h, p["H"] * p["dv"], p["rdv"]), W * k_h * 2)
+    add("group norms + output projection, state space", "output projection", grp(W, inner, 0, inner // G), W * inner * 2)
+    add("norm + residual + final norm + head + cap", "norm + head",
+        gemv(V, W, lambda w: R.gemv_bf16_residual_f32(ctx, w, x, y, gains, gains, None, out, 1e-6, 30.0, 0, V, W)), V * W * 2)
+    S, H = 1024, W // 128
+    pitch = kl + 64
+    lc = R.LatentCfg(H, 128, 64, 128, kl, 192 ** -0.5, 1e-6)
+    ns = max(1, min(64, 296 // ((H + 15) // 16)))
+    caches = [bf(S, pitch) for _ in range(64)]
+    qe, po, pm = bf(H * 2 * pitch), torch.empty(H * ns * kl, device="cuda"), torch.empty(H * ns * 2, device="cuda")
+    like("attention over 1024 cached rows", timed([(lambda c=c: R.latent_attention(ctx, C.byref(lc), 0, qe, c, po, pm, ns, 1, S - 1)) for c in caches]), S * pitch * 2)
+    del caches
+    slopes = torch.rand(p["H"], device="cuda")
+    decay = torch.rand(2, p["rH"], device="cuda") * 0.1 + 0.85
+    freq = torch.rand(p["rd"] // 2, device="cuda")
+    proj, tickets, pos = torch.randn(max(in_h, in_s), device="cuda"), torch.zeros(4096, dtype=torch.int32, device="cuda"), torch.tensor([S - 1], dtype=torch.int32, device="cuda")
+    part, ao = torch.empty(p["H"] * 64 * (p["dv"] + 2), device="cuda"), torch.empty(max(k_h, inner), device="cuda")
+    sets = []
+    for _ in range(48):
+        kc, vc, st = bf(p["G"], S, p["d"]), bf(p["G"], S, p["dv"]), torch.randn(p["rH"], p["rd"], p["rdv"], device="cuda")
+        sets.append((R.HeadsCfg(p["H"], p["G"], p["d"], p["dv"], p["window"], S, 1, p["d"] ** -0.5, 0.7, 1e-6, slopes.data_ptr(), kc.data_ptr(), vc.data_ptr()),
+                     R.RetentionCfg(p["rH"], p["rd"], p["rdv"], p["rd"], 0.8, freq.data_ptr(), decay.data_ptr(), st.data_ptr()), (kc, vc, st)))
+    nsp = min(16, max(1, -(-296 // p["G"])))
+    by_at, by_rt = p["G"] * S * (p["d"] + p["dv"]) * 2, p["rH"] * p["rd"] * p["rdv"] * 8
+    step = lambda a, r: timed([(lambda s=s: R.heads_step(ctx, C.byref(s[0]) if a else None, C.byref(s[1]) if r else None, 0, proj, ao, gains, part, tickets, nsp, pos)) for s in sets])
+    add("attention (window 1024) beside retention, one step", "attention over 1024 cached rows", step(1, 1), by_at + by_rt)
+    add("  the attention alone", "attention over 1024 cached rows", step(1, 0), by_at)
+    add("  the retention alone", "attention over 1024 cached rows", step(0, 1), by_rt)
+    del sets
+    f32s = lambda *s: torch.rand(*s, device="cuda")
+    cw, cb, dtb, sa, sk = f32s(ch, 4), f32s(ch), f32s(p["sH"]), -f32s(p["sH"]), f32s(p["sH"])
+    ring = f32s(4, ch)
+    sst = [f32s(p["sH"], p["N"], p["sd"]) for _ in range(max(2, int(300e6 // (p["sH"] * p["N"] * p["sd"] * 4))))]
+    ss = [R.SsmCfg(p["sH"], p["sd"], p["N"], G, 4, *(t.data_ptr() for t in (cw, cb, dtb, sa, sk, s, ring))) for s in sst]
+    add("state-space step", "attention over 1024 cached rows", timed([(lambda s=s: R.ssm_step(ctx, C.byref(s), proj, ao, pos)) for s in ss]), p["sH"] * p["N"] * p["sd"] * 8)
+    del sst
+    # ── many tokens ──
+    lat_kv, lat_c = bf(T, H * 256), bf(T, pitch)
+    q, o = torch.randn(T, H * 192, device="cuda"), bf(T, max(k_h, inner))
+    like("causal attention", timed([lambda: R.latent_prefill_attention(ctx, C.byref(lc), q, H * 192, lat_kv, H * 256, lat_c, o, H * 128, T, 0)]), flops=T * T * H * (192 + 128))
+    xs = [torch.randn(T, W, device="cuda") for _ in range(8)]
+    hs = [bf(T, W) for _ in range(8)]
+    like("norm rows", timed([(lambda a=a, b=b: R.norm_gain_rows(ctx, a, one, 1e-6, b, 0, T, W)) for a, b in zip(xs, hs)]), T * W * 6)
+    ql = [torch.randn(T, ml, device="cuda") for _ in range(4)]
+    like("cache rows + rotation", timed([(lambda a=a: R.latent_rows(ctx, C.byref(lc), 0, a, ml, gains, freq, lat_c, T, 0)) for a in ql]),
+         T * (H * 64 * 8 + pitch * 6))
+    del ql
+    ys = [torch.randn(T, W, device="cuda") for _ in range(8)]
+    add("norm + residual rows", "norm rows", timed([(lambda a=a, b=b, c=c: R.add_norm_rows(ctx, a, c, gains, 1e-6, None, b, 0, T, W)) for a, b, c in zip(xs, hs, ys)]), T * W * 14)
+    del xs, hs, ys
+
+    def gemm(m, k, epi):
+        ws, a = [bf(m, k) for _ in range(4)], bf(T, k)
+        c = torch.empty(T, m, device="cuda")
+        return timed([(lambda w=w: R.gemm_bf16_rows(ctx, w, a, c, m // 2 if epi == R.EPI_SILU_GLU else m, T, m, k, 0, epi, None, None)) for w in ws])
+    for key, m, k, epi in (("projection GEMM", ml, W, R.EPI_F32), ("output GEMM + residual", W, W, R.EPI_ADD), ("gate / up GEMM", 2 * gff, W, R.EPI_SILU_GLU),
+                           ("down GEMM + residual", W, gff, R.EPI_ADD)):
+        like(key, gemm(m, k, epi), flops=2.0 * T * m * k)
+    for name, key, m, k, epi in (("projections GEMM, attention beside retention", "projection GEMM", in_h, W, R.EPI_CAST), ("projections GEMM, state space", "projection GEMM", in_s, W, R.EPI_CAST),
+                                 ("output GEMM, attention beside retention", "output GEMM + residual", W, k_h, R.EPI_F32), ("output GEMM, state space", "output GEMM + residual", W, inner, R.EPI_F32),
+                                 ("up GEMM + relu2", "gate / up GEMM", ff, W, R.EPI_RELU2), ("down GEMM", "down GEMM + residual", W, ff, R.EPI_F32)):
+        add(name, key, gemm(m, k, epi), flops=2.0 * T * m * k)
+    kc, vc = bf(p["G"], T, p["d"]), bf(p["G"], T, p["dv"])
+    hc = R.HeadsCfg(p["H"], p["G"], p["d"], p["dv"], p["window"], T, 1, p["d"] ** -0.5, 0.7, 1e-6, slopes.data_ptr(), kc.data_ptr(), vc.data_ptr())
+    st = torch.zeros(p["rH"], p["rd"], p["rdv"], device="cuda")
+    rc = R.RetentionCfg(p["rH"], p["rd"], p["rdv"], p["rd"], 0.8, freq.data_ptr(), decay.data_ptr(), st.data_ptr())
+    prs = [bf(T, in_h) for _ in range(8)]
+    add("cache rows + rotation", "cache rows + rotation", timed([(lambda a=a: R.heads_rows(ctx, C.byref(hc), C.byref(rc), 0, a, in_h, T, 0)) for a in prs]),
+        T * (p["G"] * (p["d"] + p["dv"]) * 4 + 2 * p["rH"] * p["rd"] * 4))
+    wpairs = sum(min(i + 1, p["window"]) for i in range(T))
+    add("attention over a window of 1024", "causal attention",
+        timed([(lambda a=a: R.head_attention_rows(ctx, C.byref(hc), 0, a, in_h, o, k_h, T, 0, part, 0, tickets)) for a in prs]), flops=2 * wpairs * p["H"] * (p["d"] + p["dv"]))
+
+    def linear(heads, groups, dk, dv, bufs, ld, off, dt, skip, state):
+        scr = torch.empty(ctx.lib.runit_linear_scratch_bytes(heads, dk, dv, T) // 4, device="cuda")
+        cs = [R.LinearCfg(heads, groups, dk, dv, ld, ld, ld, heads * dv, b.data_ptr() + 2 * off[0], b.data_ptr() + 2 * off[1], b.data_ptr() + 2 * off[2], dt, ldec.data_ptr(),
+                          dec.data_ptr(), skip, state.data_ptr(), o.data_ptr()) for b in bufs]
+        us = timed([(lambda c=c: R.linear_rows(ctx, C.byref(c), 0, scr, T, 0)) for c in cs])
+        return us, T * (2 * groups * dk + 2 * heads * dv) * 2, T * heads * (4.0 * dk * dv + 64 * (dk + dv))
+    base = p["H"] * p["d"] + p["G"] * (p["d"] + p["dv"])
+    dec = torch.rand(256, device="cuda") * 0.1 + 0.9
+    ldec = torch.log(dec)
+    us, nb, fl = linear(p["rH"], p["rH"], p["rd"], p["rdv"], prs, in_h, (base, base + p["rH"] * p["rd"], base + 2 * p["rH"] * p["rd"]), None, None, st)
+    add("retention over chunks", "causal attention", us, nb, fl)
+    add("head norms + gate", "norm rows", timed([(lambda a=a: R.gated_norm_rows(ctx, 0, o, k_h, p["rH"] * p["rdv"], p["rdv"], a[:, base:], in_h, 0, None, 0.8, 1e-6, T)) for a in prs]),
+        T * p["rH"] * p["rdv"] * 6)
+    del prs
+    prs, xbc, dts = [bf(T, in_s) for _ in range(6)], [bf(T, ch) for _ in range(6)], torch.rand(T, p["sH"], device="cuda") * 0.1
+    dconv = torch.rand(T, p["sH"], device="cuda")
+    add("convolution + silu + step sizes", "norm rows", timed([(lambda a=a, b=b: R.ssm_conv_rows(ctx, C.byref(ss[0]), 0, a, in_s, b, ch, dconv, T, 0)) for a, b in zip(prs, xbc)]), T * ch * 4)
+    st2 = torch.zeros(p["sH"], p["N"], p["sd"], device="cuda")
+    us, nb, fl = linear(p["sH"], G, p["N"], p["sd"], xbc, ch, (inner + G * p["N"], inner, 0), dts.data_ptr(), sk.data_ptr(), st2)
+    add("state space over chunks", "causal attention", us, nb, fl)
+    add("gate + group norms", "norm rows", timed([(lambda a=a: R.gated_norm_rows(ctx, 0, o, inner, inner, inner // G, a, in_s, 1, gains, 1.0, 1e-6, T)) for a in prs]), T * inner * 6)
+    return rows
+
+
+def run_pagazen(R, ctx, torch, stream, sizes):
+    out = {"note": "random weights; the closest model is the latent-attention decoder with a dense feed-forward at equal width, depth, "
+                   "vocabulary and feed-forward weights"}
+    for name in sizes:
+        size = PAGAZEN_SIZES[name]
+        res = {"size": dict(zip(("width", "layers", "ff", "groups", "vocab"), size))}
+        for key, make in (("pagazen_bf16", build_pagazen), ("nuvilorn_dense_bf16", build_dense_latent)):
+            m = make(R, ctx, torch, size, 2304)
+            res[key] = time_model(m, size[-1])
+            m.close()
+            del m
+            torch.cuda.empty_cache()
+        if name == "2048":
+            res["kernels"] = time_pagazen_kernels(R, ctx, torch, stream, size)
         out[name] = res
         torch.cuda.empty_cache()
     return out
@@ -1153,6 +1384,8 @@ def main():
     ap.add_argument("--shapes", action="store_true", help="per-shape GEMV table (one JSON line per shape) instead of the headline run")
     ap.add_argument("--layered", nargs="?", const="1024,2048,4096", default="",
                     help="prefill and decode throughput of the layered (latent attention) decoder at these widths beside the Q4_K decoder, then exit")
+    ap.add_argument("--layered-design", default="nuvilorn", choices=("nuvilorn", "pagazen"),
+                    help="design of the --layered run; pagazen: beside a latent-attention decoder with a dense feed-forward")
     args = ap.parse_args()
     if args.impl == "reference":
         return run_reference(args)
@@ -1200,7 +1433,8 @@ def main():
         print(json.dumps({"one": args.one, "launches": ctx.launches}))
         return
     if args.layered:
-        print(json.dumps(run_layered(R, ctx, torch, stream, args.layered.split(","))))
+        run = run_pagazen if args.layered_design == "pagazen" else run_layered
+        print(json.dumps(run(R, ctx, torch, stream, args.layered.split(","))))
         return
     if args.ffn:
         T = int(args.ffn)

@@ -516,6 +516,89 @@ int32_t runit_latent_rows(runit_ctx_t*, const runit_latent_cfg* cfg, int32_t cac
 int32_t runit_latent_prefill_attention(runit_ctx_t*, const runit_latent_cfg* cfg, const void* q, uint32_t ldq, const void* kv, uint32_t ldkv,
                                        const void* cache, void* out, uint32_t ldo, uint32_t T, uint32_t start);
 
+/* Attention over cached keys and values per head.  A projected row holds [q: heads x dim | k: kv_heads x dim | v: kv_heads x
+ * vdim]; query head h uses key head h / (heads / kv_heads).  Score (q . k) * scale - slopes[h] * (i - j) (slopes f32 [heads] or
+ * NULL); window 0: all earlier positions, else a position sees itself and the window - 1 before it; unit_qk: q and k are divided by
+ * their root mean square.  Caches: bf16 or f32 (cache_f32), [kv_heads][cap][dim, vdim padded to 8], position p in row p % cap. */
+typedef struct {
+    uint32_t heads, kv_heads, dim, vdim, window, cap, unit_qk;
+    float    scale, out_scale, eps;
+    const void* slopes;
+    void*    k_cache;
+    void*    v_cache;
+} runit_heads_cfg;
+/* Retention, S <- decay_h S + k v^T, o = S^T q.  A projected row holds [q, k: heads x dim | v, gate: heads x vdim]; the first
+ * rot_dims coordinates of q and k rotate (pairs (i, i + rot_dims/2), angle position * freq[i]), k is multiplied by dim^(-1/2).
+ * decay f32 [2][heads]: the decays, then their logarithms; state f32 [heads][dim][vdim]. */
+typedef struct {
+    uint32_t heads, dim, vdim, rot_dims;
+    float    out_scale;
+    const void* freq;
+    const void* decay;
+    void*    state;
+} runit_retention_cfg;
+/* State-space layer.  A projected row holds [z: heads x vdim | x: heads x vdim | B, C: groups x state_dim | dt: heads]; the other
+ * fields are those of runit_layer_desc; state f32 [heads][state_dim][vdim]; ring f32 [taps][channels]: the inputs of the
+ * convolution at position p in row p % taps. */
+typedef struct {
+    uint32_t heads, vdim, state_dim, groups, taps;
+    const void* conv;
+    const void* conv_b;
+    const void* dt_bias;
+    const void* a;
+    const void* skip;
+    void*    state;
+    void*    ring;
+} runit_ssm_cfg;
+/* One token at position *pos (device int32): attention and / or retention (either NULL) on one f32 projected row; writes the
+ * position's cache row and the state.  ao f32 = [attention * out_scale | retention o], factor f32 = silu(gate) * out_scale of the
+ * retention.  part f32 [heads * nsplit * (vdim + 2)], tickets uint32 [4096], zero (zero again afterwards); nsplit <= 64. */
+int32_t runit_heads_step(runit_ctx_t*, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, const void* proj, void* ao,
+                         void* factor, void* part, void* tickets, uint32_t nsplit, const void* pos);
+/* T tokens, projected rows of ld elements (bf16, or f32 with an f32 cache): cache rows of their positions, rotated q and k of the
+ * retention in place (k scaled); then attention over them: out rows of ldo, the same type.  part: part_floats f32 (any number). */
+int32_t runit_heads_rows(runit_ctx_t*, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, void* proj, uint32_t ld,
+                         uint32_t T, uint32_t start);
+int32_t runit_head_attention_rows(runit_ctx_t*, const runit_heads_cfg* attn, int32_t cache_f32, const void* proj, uint32_t ld, void* out,
+                                  uint32_t ldo, uint32_t T, uint32_t start, void* part, size_t part_floats, void* tickets);
+/* One token of a state-space layer: y f32 [heads * vdim] = (S^T C + skip x) * silu(z). */
+int32_t runit_ssm_step(runit_ctx_t*, const runit_ssm_cfg* cfg, const void* proj, void* y, const void* pos);
+/* T tokens: x, B, C convolved and activated into rows of ldx (bf16 or f32); dt f32 [T][heads] becomes softplus(dt + dt_bias). */
+int32_t runit_ssm_conv_rows(runit_ctx_t*, const runit_ssm_cfg* cfg, int32_t f32, const void* proj, uint32_t ld, void* xbc, uint32_t ldx, void* dt,
+                            uint32_t T, uint32_t start);
+/* The recurrence over T tokens: q, k [groups][dk] and v [heads][dv] per token (rows of ldq, ldk, ldv, bf16 or f32), head h uses group
+ * h / (heads / groups).  dt f32 [T][heads]: decay exp(log_decay[h] * dt), k times dt; dt NULL: decay[h] (and its logarithm).  skip
+ * f32 [heads] or NULL: o += skip[h] v.  start 0: from a zero state.  scratch: runit_linear_scratch_bytes (NULL: token by token). */
+typedef struct {
+    uint32_t heads, groups, dk, dv, ldq, ldk, ldv, ldo;
+    const void* q;
+    const void* k;
+    const void* v;
+    const void* dt;
+    const void* log_decay;
+    const void* decay;
+    const void* skip;
+    void*    state;
+    void*    out;
+} runit_linear_cfg;
+size_t  runit_linear_scratch_bytes(uint32_t heads, uint32_t dk, uint32_t dv, uint32_t T);
+int32_t runit_linear_rows(runit_ctx_t*, const runit_linear_cfg* cfg, int32_t f32, void* scratch, uint32_t T, uint32_t start);
+/* Groups of `group` values of the n in every row of a (in place): before: a * silu(gate), normed, times weight (f32 [n]); else a
+ * normed, times silu(gate) * out_scale. */
+int32_t runit_gated_norm_rows(runit_ctx_t*, int32_t f32, void* a, uint32_t lda, uint32_t n, uint32_t group, const void* gate, uint32_t ldg,
+                              int32_t before, const void* weight, float out_scale, float eps, uint32_t T);
+/* x[t] += norm(y[t]) (y NULL: x stays), a gain per coordinate; out (may be NULL) = x in rows of pad8(width), or norm(x) with
+ * out_gain when that is not NULL */
+int32_t runit_add_norm_rows(runit_ctx_t*, void* x, const void* y, const void* gain, float eps, const void* out_gain, void* out, int32_t out_f32,
+                            uint32_t T, uint32_t width);
+/* out[m] = W . v (cap != 0: cap * tanh(. / cap)) with v = x + norm(y) (gain y_gain per coordinate; y NULL: v = x), stored in x_out,
+ * and then norm(v) with `gain` when that is not NULL.  relu2: max(., 0)^2 instead of cap. */
+int32_t runit_gemv_bf16_residual_f32(runit_ctx_t*, const void* weight, const void* x, const void* y, const void* y_gain, const void* gain, void* x_out,
+                                     void* out, float eps, float cap, int32_t relu2, uint32_t m, uint32_t k);
+/* out[m] = W . v: the first `plain` values of v are x, the others groups of `group` values of x, normed, times factor [k - plain] */
+int32_t runit_gemv_bf16_groups_f32(runit_ctx_t*, const void* weight, const void* x, const void* factor, void* out, float eps, uint32_t plain,
+                                   uint32_t group, uint32_t m, uint32_t k);
+
 /* ── decoders described layer by layer (no twin), weights in bf16 ──
  * Every matrix is row-major [rows][pad8(columns)] bf16 with zero padding; norms and router are f32.  Linear maps W x.
  * Residual stream, norms, scores, softmax, router, angles and recurrent state are f32.  norm(x) = x / sqrt(mean(x^2) + eps) * gain.

@@ -23,6 +23,7 @@ _CTYPES = {
     "const runit_model_cfg*": C.c_void_p, "const runit_sampler_cfg*": C.c_void_p, "const runit_model_weights*": C.c_void_p, "runit_model_t*": C.c_void_p,
     "int32_t*": C.POINTER(C.c_int32),
     "const runit_layered_cfg*": C.c_void_p, "const runit_layer_desc*": C.c_void_p, "const runit_layered_weights*": C.c_void_p, "const runit_latent_cfg*": C.c_void_p,
+    "const runit_heads_cfg*": C.c_void_p, "const runit_retention_cfg*": C.c_void_p, "const runit_ssm_cfg*": C.c_void_p, "const runit_linear_cfg*": C.c_void_p,
     "runit_model_t**": C.POINTER(C.c_void_p), "const void* const*": C.POINTER(C.c_void_p),
     "void* const*": C.POINTER(C.c_void_p), "float*": C.POINTER(C.c_float),
     "uint64_t*": C.POINTER(C.c_uint64), "runit_graph_t*": C.c_void_p, "runit_graph_t**": C.POINTER(C.c_void_p),

@@ -644,4 +644,33 @@ int32_t runit_norm_gain_rows(runit_ctx_t* ctx, const void* x, const void* gain, 
     return norm_rows(ctx, (const float*)x, nullptr, (const float*)gain, eps, y, y_f32 != 0, pad8(width), nullptr, T, width);
 }
 
+int32_t runit_add_norm_rows(runit_ctx_t* ctx, void* x, const void* y, const void* gain, float eps, const void* out_gain, void* out, int32_t out_f32,
+                            uint32_t T, uint32_t width) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, x && (!y || gain) && T > 0 && width > 0, "add_norm_rows: bad argument");
+    return add_norm_rows(ctx, (float*)x, (const float*)y, (const float*)gain, eps, nullptr, (const float*)out_gain, out, out_f32 != 0, pad8(width), T, width);
+}
+
+int32_t runit_gemv_bf16_residual_f32(runit_ctx_t* ctx, const void* weight, const void* x, const void* y, const void* y_gain, const void* gain, void* x_out,
+                                     void* out, float eps, float cap, int32_t relu2, uint32_t m, uint32_t k) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, weight && x && out && m > 0 && k > 0 && runit_aligned(weight, 16) && x_out != x, "gemv_bf16_residual_f32: bad argument");
+    GemvDesc d;
+    d.w = weight; d.rows = m; d.K = k; d.ldw = pad8(k); d.x = (const float*)x; d.eps = eps; d.out = (float*)out; d.cap = cap;
+    d.epi = relu2 ? EPI_RELU2 : EPI_F32;
+    d.pro.kind = GEMV_PRO_RESIDUAL; d.pro.y = (const float*)y; d.pro.y_gain = (const float*)y_gain; d.pro.gain = (const float*)gain;
+    d.pro.x_out = (float*)x_out;
+    return gemv_bf16(ctx, "gemv_bf16_residual_f32", d);
+}
+
+int32_t runit_gemv_bf16_groups_f32(runit_ctx_t* ctx, const void* weight, const void* x, const void* factor, void* out, float eps, uint32_t plain,
+                                   uint32_t group, uint32_t m, uint32_t k) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, weight && x && out && m > 0 && k > 0 && runit_aligned(weight, 16), "gemv_bf16_groups_f32: bad argument");
+    GemvDesc d;
+    d.w = weight; d.rows = m; d.K = k; d.ldw = pad8(k); d.x = (const float*)x; d.eps = eps; d.out = (float*)out;
+    d.pro.kind = GEMV_PRO_GROUPS; d.pro.plain = plain; d.pro.group = group; d.pro.factor = (const float*)factor;
+    return gemv_bf16(ctx, "gemv_bf16_groups_f32", d);
+}
+
 }  // extern "C"

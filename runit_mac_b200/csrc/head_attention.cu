@@ -8,6 +8,8 @@
 //     of 64, split over CTAs; the last CTA of a head block to finish merges the splits.  Decoding, short portions, 32-bit runs.
 //   * window_prefill_kernel: long portions in bf16, 64 queries of a head per CTA, blocks of 64 keys, mma.sync (the arrangement of
 //     latent_prefill_kernel); blocks outside of the window are not visited.
+#include <cmath>
+
 #include "bf16_ops.cuh"
 #include "gemv_common.cuh"
 #include "linear_state.cuh"
@@ -613,3 +615,64 @@ int32_t head_attention_rows(runit_ctx* ctx, const HeadAttn& a, bool exact, const
 }
 
 }  // namespace runit
+
+using namespace runit;
+
+namespace {
+int32_t heads_of(runit_ctx* ctx, const char* who, const runit_heads_cfg* c, HeadAttn* a) {
+    RUNIT_REQUIRE(ctx, c->heads > 0 && c->kv_heads > 0 && c->heads % c->kv_heads == 0 && c->dim > 0 && c->dim <= 1024 && c->vdim > 0 && c->vdim <= 1024 &&
+                           c->cap > 0 && c->k_cache && c->v_cache, "%s: bad attention sizes", who);
+    a->heads = c->heads; a->kv_heads = c->kv_heads; a->dim = c->dim; a->vdim = c->vdim; a->window = c->window; a->cap = c->cap; a->unit_qk = c->unit_qk;
+    a->scale = c->scale; a->out_scale = c->out_scale; a->eps = c->eps; a->slopes = (const float*)c->slopes; a->kc = c->k_cache; a->vc = c->v_cache;
+    return RUNIT_OK;
+}
+int32_t retention_of(runit_ctx* ctx, const char* who, const runit_retention_cfg* c, Retention* r) {
+    RUNIT_REQUIRE(ctx, c->heads > 0 && c->dim > 0 && c->dim <= 1024 && c->vdim > 0 && c->rot_dims <= c->dim && c->rot_dims % 2 == 0 && c->decay && c->state &&
+                           (c->freq || c->rot_dims == 0), "%s: bad retention", who);
+    r->heads = c->heads; r->dim = c->dim; r->vdim = c->vdim; r->rot_dims = c->rot_dims; r->out_scale = c->out_scale;
+    r->k_scale = (float)(1.0 / std::sqrt((double)c->dim)); r->freq = (const float*)c->freq; r->decay = (const float*)c->decay; r->state = (float*)c->state;
+    return RUNIT_OK;
+}
+}  // namespace
+
+extern "C" {
+
+int32_t runit_heads_step(runit_ctx_t* ctx, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, const void* proj, void* ao,
+                         void* factor, void* part, void* tickets, uint32_t nsplit, const void* pos) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    HeadAttn a;
+    Retention r;
+    int32_t st;
+    if (attn && (st = heads_of(ctx, "heads_step", attn, &a))) return st;
+    if (ret && (st = retention_of(ctx, "heads_step", ret, &r))) return st;
+    RUNIT_REQUIRE(ctx, proj && ao && pos && (!attn || (part && tickets)) && (!ret || factor), "heads_step: null argument");
+    return heads_step(ctx, attn ? &a : nullptr, ret ? &r : nullptr, cache_f32 != 0, (const float*)proj, (float*)ao, (float*)factor, (float*)part,
+                      (uint32_t*)tickets, nsplit, (const int32_t*)pos);
+}
+
+int32_t runit_heads_rows(runit_ctx_t* ctx, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, void* proj, uint32_t ld,
+                         uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    HeadAttn a;
+    Retention r;
+    int32_t st;
+    if (attn && (st = heads_of(ctx, "heads_rows", attn, &a))) return st;
+    if (ret && (st = retention_of(ctx, "heads_rows", ret, &r))) return st;
+    RUNIT_REQUIRE(ctx, proj && (attn || ret) && T > 0 && ld >= a.in_rows() + r.in_rows(), "heads_rows: bad argument");
+    return heads_rows(ctx, attn ? &a : nullptr, ret ? &r : nullptr, cache_f32 != 0, proj, ld, T, start);
+}
+
+int32_t runit_head_attention_rows(runit_ctx_t* ctx, const runit_heads_cfg* attn, int32_t cache_f32, const void* proj, uint32_t ld, void* out,
+                                  uint32_t ldo, uint32_t T, uint32_t start, void* part, size_t part_floats, void* tickets) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    HeadAttn a;
+    int32_t st;
+    RUNIT_REQUIRE(ctx, attn, "head_attention_rows: null argument");
+    if ((st = heads_of(ctx, "head_attention_rows", attn, &a))) return st;
+    const uint32_t reach = T + (a.window ? a.window - 1 : start);
+    RUNIT_REQUIRE(ctx, proj && out && T > 0 && T <= 65535 && ld >= a.in_rows() && ldo >= a.out_rows() && (a.cap >= reach || a.cap >= start + T) && tickets &&
+                           (part || part_floats == 0), "head_attention_rows: bad argument");
+    return head_attention_rows(ctx, a, cache_f32 != 0, proj, ld, out, ldo, T, start, (float*)part, part_floats, (uint32_t*)tickets);
+}
+
+}  // extern "C"

@@ -577,3 +577,61 @@ int32_t gated_norm_rows(runit_ctx* ctx, bool exact, void* a, uint32_t lda, uint3
 }
 
 }  // namespace runit
+
+using namespace runit;
+
+namespace {
+int32_t ssm_of(runit_ctx* ctx, const char* who, const runit_ssm_cfg* c, Ssm* m) {
+    RUNIT_REQUIRE(ctx, c && c->heads > 0 && c->vdim > 0 && c->state_dim > 0 && c->state_dim <= kMaxKeyDim && c->groups > 0 && c->heads % c->groups == 0 &&
+                           c->taps > 0 && c->taps <= kConvTok && c->conv && c->conv_b && c->dt_bias && c->a && c->skip && c->state && c->ring,
+                  "%s: bad state-space layer", who);
+    m->heads = c->heads; m->vdim = c->vdim; m->state = c->state_dim; m->groups = c->groups; m->taps = c->taps;
+    m->conv_w = (const float*)c->conv; m->conv_b = (const float*)c->conv_b; m->dt_bias = (const float*)c->dt_bias; m->a = (const float*)c->a;
+    m->skip = (const float*)c->skip; m->s = (float*)c->state; m->ring = (float*)c->ring;
+    return RUNIT_OK;
+}
+}  // namespace
+
+extern "C" {
+
+int32_t runit_ssm_step(runit_ctx_t* ctx, const runit_ssm_cfg* cfg, const void* proj, void* y, const void* pos) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    Ssm m;
+    int32_t st = ssm_of(ctx, "ssm_step", cfg, &m);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, proj && y && pos, "ssm_step: null argument");
+    return ssm_step(ctx, m, (const float*)proj, (float*)y, (const int32_t*)pos);
+}
+
+int32_t runit_ssm_conv_rows(runit_ctx_t* ctx, const runit_ssm_cfg* cfg, int32_t f32, const void* proj, uint32_t ld, void* xbc, uint32_t ldx, void* dt,
+                            uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    Ssm m;
+    int32_t st = ssm_of(ctx, "ssm_conv_rows", cfg, &m);
+    if (st != RUNIT_OK) return st;
+    RUNIT_REQUIRE(ctx, proj && xbc && dt && T > 0 && ld >= m.inner() + m.channels() && ldx >= m.channels(), "ssm_conv_rows: bad argument");
+    return ssm_conv_rows(ctx, m, f32 != 0, proj, ld, xbc, ldx, (float*)dt, T, start);
+}
+
+size_t runit_linear_scratch_bytes(uint32_t heads, uint32_t dk, uint32_t dv, uint32_t T) { return linear_chunk_bytes(heads, dk, dv, T); }
+
+int32_t runit_linear_rows(runit_ctx_t* ctx, const runit_linear_cfg* c, int32_t f32, void* scratch, uint32_t T, uint32_t start) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, c && c->q && c->k && c->v && c->log_decay && (c->dt || c->decay) && c->state && c->out && T > 0 && c->groups > 0 &&
+                           c->ldq >= c->groups * c->dk && c->ldk >= c->groups * c->dk && c->ldv >= c->heads * c->dv && c->ldo >= c->heads * c->dv &&
+                           runit_aligned(scratch, 16), "linear_rows: bad argument");
+    LinearRows d;
+    d.heads = c->heads; d.groups = c->groups; d.dk = c->dk; d.dv = c->dv; d.q = c->q; d.k = c->k; d.v = c->v; d.ldq = c->ldq; d.ldk = c->ldk; d.ldv = c->ldv;
+    d.dt = (const float*)c->dt; d.log_decay = (const float*)c->log_decay; d.decay = (const float*)c->decay; d.skip = (const float*)c->skip;
+    d.state = (float*)c->state; d.out = c->out; d.ldo = c->ldo;
+    return linear_rows(ctx, d, f32 != 0, scratch, T, start);
+}
+
+int32_t runit_gated_norm_rows(runit_ctx_t* ctx, int32_t f32, void* a, uint32_t lda, uint32_t n, uint32_t group, const void* gate, uint32_t ldg,
+                              int32_t before, const void* weight, float out_scale, float eps, uint32_t T) {
+    if (!ctx) return RUNIT_ERR_BAD_ARG;
+    RUNIT_REQUIRE(ctx, a && gate && n > 0 && lda >= n && ldg >= n && T > 0, "gated_norm_rows: bad argument");
+    return gated_norm_rows(ctx, f32 != 0, a, lda, n, group, gate, ldg, before != 0, (const float*)weight, out_scale, eps, T);
+}
+
+}  // extern "C"

@@ -285,6 +285,16 @@ _TWINS = [
     ("latent_value", "no twin: (LatentCfg ref, part_o, part_ml, nsplit, w_uv, out, T)"),
     ("latent_rows", "no twin: (LatentCfg ref, cache_f32, qkv, ldq, kv_norm or None, freq, cache, T, start)"),
     ("latent_prefill_attention", "no twin: (LatentCfg ref, q, ldq, kv, ldkv, cache, out, ldo, T, start)"),
+    ("heads_step", "no twin: (HeadsCfg ref or None, RetentionCfg ref or None, cache_f32, proj, ao, factor, part, tickets, nsplit, pos)"),
+    ("heads_rows", "no twin: (HeadsCfg ref or None, RetentionCfg ref or None, cache_f32, proj, ld, T, start)"),
+    ("head_attention_rows", "no twin: (HeadsCfg ref, cache_f32, proj, ld, out, ldo, T, start, part, part_floats, tickets)"),
+    ("ssm_step", "no twin: (SsmCfg ref, proj, y, pos)"),
+    ("ssm_conv_rows", "no twin: (SsmCfg ref, f32, proj, ld, xbc, ldx, dt, T, start)"),
+    ("linear_rows", "no twin: (LinearCfg ref, f32, scratch or None, T, start)"),
+    ("gated_norm_rows", "no twin: (f32, a, lda, n, group, gate, ldg, before, weight or None, out_scale, eps, T)"),
+    ("add_norm_rows", "no twin: (x, y or None, gain, eps, out_gain or None, out or None, out_f32, T, width)"),
+    ("gemv_bf16_residual_f32", "no twin: (weight, x, y or None, y_gain, gain or None, x_out or None, out, eps, cap, relu2, m, k)"),
+    ("gemv_bf16_groups_f32", "no twin: (weight, x, factor, out, eps, plain, group, m, k)"),
     ("fill_weights", "no twin: (fmt, dst, n_blocks, seed, sigma)"),
     ("fill_weights_q4k_zero_mean", "no twin: (dst, n_blocks, seed, sigma), Q4_K blocks with zero-mean weights"),
     ("fill_normal_f32", "no twin: (dst, n, seed, sigma)"),
@@ -427,6 +437,30 @@ class LatentCfg(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank")] + [("scale", C.c_float), ("eps", C.c_float)]
 
 
+class HeadsCfg(C.Structure):
+    """runit_heads_cfg; pass ``ctypes.byref(cfg)``."""
+    _fields_ = ([(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "window", "cap", "unit_qk")] +
+                [(n, C.c_float) for n in ("scale", "out_scale", "eps")] + [(n, C.c_void_p) for n in ("slopes", "k_cache", "v_cache")])
+
+
+class RetentionCfg(C.Structure):
+    """runit_retention_cfg"""
+    _fields_ = ([(n, C.c_uint32) for n in ("heads", "dim", "vdim", "rot_dims")] + [("out_scale", C.c_float)] +
+                [(n, C.c_void_p) for n in ("freq", "decay", "state")])
+
+
+class SsmCfg(C.Structure):
+    """runit_ssm_cfg"""
+    _fields_ = ([(n, C.c_uint32) for n in ("heads", "vdim", "state_dim", "groups", "taps")] +
+                [(n, C.c_void_p) for n in ("conv", "conv_b", "dt_bias", "a", "skip", "state", "ring")])
+
+
+class LinearCfg(C.Structure):
+    """runit_linear_cfg"""
+    _fields_ = ([(n, C.c_uint32) for n in ("heads", "groups", "dk", "dv", "ldq", "ldk", "ldv", "ldo")] +
+                [(n, C.c_void_p) for n in ("q", "k", "v", "dt", "log_decay", "decay", "skip", "state", "out")])
+
+
 class LayerDesc(C.Structure):
     """runit_layer_desc: mixer and feed-forward of one layer, sizes, constants and device pointers."""
     _fields_ = ([(n, C.c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "kv_from")] +
@@ -525,6 +559,6 @@ def moe_layer_q4k_host(ctx: Context, router, gate, up, down, x, *, h, ff, E, top
             w.download(np.float32, T * top_k).reshape(T, top_k))
 
 
-__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc", "LatentCfg", "EPI_F32", "EPI_ADD", "EPI_CAST", "EPI_SILU_GLU", "EPI_RELU2",
+__all__ = ["Context", "DeviceBuffer", "Graph", "KernelError", "Model", "ModelCfg", "ModelWeights", "LayeredModel", "LayeredCfg", "LayeredWeights", "LayerDesc", "LatentCfg", "HeadsCfg", "RetentionCfg", "SsmCfg", "LinearCfg", "EPI_F32", "EPI_ADD", "EPI_CAST", "EPI_SILU_GLU", "EPI_RELU2",
            "FF_NONE", "FF_DENSE", "FF_MOE", "MIX_LATENT", "MIX_HEADS", "MIX_SSM", "ACT_SILU_GLU", "ACT_RELU2", "SCORE_SOFTMAX", "SCORE_SIGMOID", "SamplerCfg", "sample_f32", "sampler_seed_state", "gemv_batched_multi_f32", "moe_scratch_bytes", "moe_layer_q4k_host", "moe_grouped_scratch_bytes", "moe_layer_q4k_bf16_host", "row_bytes", "BLOCK_ELEMS", "BLOCK_BYTES",
            "FMT_Q8_0", "FMT_Q4_0", "FMT_Q4K", "FMT_Q5_0", "FMT_Q5K", "FMT_Q6K"] + [n for n, _ in _TWINS]
