@@ -935,7 +935,8 @@ def time_pagazen_kernels(R, ctx, torch, stream, size, reps=20, T=2048):
     add("norm + residual + projections, state space", "norm + projection", res(in_s, W, 0), in_s * W * 2)
     add("norm + residual + up + relu2", "gate / up", res(ff, W, 1), ff * W * 2)
     add("down", "down", plain(W, ff), W * ff * 2)
-    grp = lambda m, k, pl, gr: gemv(m, k, lambda w: R.gemv_bf16_groups_f32(ctx, w, gains, gains, out, 1e-6, pl, gr, m, k))
+    sqs = torch.rand(8 * W, device="cuda")
+    grp = lambda m, k, pl, gr: gemv(m, k, lambda w: R.gemv_bf16_groups_f32(ctx, w, gains, gains, sqs, gr // 32, out, 1e-6, pl, gr, m, k))
     add("head norms + output projection, attention beside retention", "output projection", grp(W, k_h, p["H"] * p["dv"], p["rdv"]), W * k_h * 2)
     add("group norms + output projection, state space", "output projection", grp(W, inner, 0, inner // G), W * inner * 2)
     add("norm + residual + final norm + head + cap", "norm + head",
@@ -960,7 +961,7 @@ def time_pagazen_kernels(R, ctx, torch, stream, size, reps=20, T=2048):
                      R.RetentionCfg(p["rH"], p["rd"], p["rdv"], p["rd"], 0.8, freq.data_ptr(), decay.data_ptr(), st.data_ptr()), (kc, vc, st)))
     nsp = min(16, max(1, -(-296 // p["G"])))
     by_at, by_rt = p["G"] * S * (p["d"] + p["dv"]) * 2, p["rH"] * p["rd"] * p["rdv"] * 8
-    step = lambda a, r: timed([(lambda s=s: R.heads_step(ctx, C.byref(s[0]) if a else None, C.byref(s[1]) if r else None, 0, proj, ao, gains, part, tickets, nsp, pos)) for s in sets])
+    step = lambda a, r: timed([(lambda s=s: R.heads_step(ctx, C.byref(s[0]) if a else None, C.byref(s[1]) if r else None, 0, proj, ao, gains, sqs, part, tickets, nsp, pos)) for s in sets])
     add("attention (window 1024) beside retention, one step", "attention over 1024 cached rows", step(1, 1), by_at + by_rt)
     add("  the attention alone", "attention over 1024 cached rows", step(1, 0), by_at)
     add("  the retention alone", "attention over 1024 cached rows", step(0, 1), by_rt)
@@ -970,7 +971,7 @@ def time_pagazen_kernels(R, ctx, torch, stream, size, reps=20, T=2048):
     ring = f32s(4, ch)
     sst = [f32s(p["sH"], p["N"], p["sd"]) for _ in range(max(2, int(300e6 // (p["sH"] * p["N"] * p["sd"] * 4))))]
     ss = [R.SsmCfg(p["sH"], p["sd"], p["N"], G, 4, *(t.data_ptr() for t in (cw, cb, dtb, sa, sk, s, ring))) for s in sst]
-    add("state-space step", "attention over 1024 cached rows", timed([(lambda s=s: R.ssm_step(ctx, C.byref(s), proj, ao, pos)) for s in ss]), p["sH"] * p["N"] * p["sd"] * 8)
+    add("state-space step", "attention over 1024 cached rows", timed([(lambda s=s: R.ssm_step(ctx, C.byref(s), proj, ao, sqs, pos)) for s in ss]), p["sH"] * p["N"] * p["sd"] * 8)
     del sst
     # ── many tokens ──
     lat_kv, lat_c = bf(T, H * 256), bf(T, pitch)

@@ -552,17 +552,20 @@ typedef struct {
 } runit_ssm_cfg;
 /* One token at position *pos (device int32): attention and / or retention (either NULL) on one f32 projected row; writes the
  * position's cache row and the state.  ao f32 = [attention * out_scale | retention o], factor f32 = silu(gate) * out_scale of the
- * retention.  part f32 [heads * nsplit * (vdim + 2)], tickets uint32 [4096], zero (zero again afterwards); nsplit <= 64. */
+ * retention, squares f32 [heads][ceil(vdim / 32)] = sums of o^2 over slices of 32 columns.  part f32 [heads * nsplit * (vdim + 2)],
+ * tickets uint32 [4096], zero (zero again afterwards); nsplit <= 64.  Cache, state and pos must not be outputs of the launch in
+ * front of this one (they are read before it has ended). */
 int32_t runit_heads_step(runit_ctx_t*, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, const void* proj, void* ao,
-                         void* factor, void* part, void* tickets, uint32_t nsplit, const void* pos);
+                         void* factor, void* squares, void* part, void* tickets, uint32_t nsplit, const void* pos);
 /* T tokens, projected rows of ld elements (bf16, or f32 with an f32 cache): cache rows of their positions, rotated q and k of the
  * retention in place (k scaled); then attention over them: out rows of ldo, the same type.  part: part_floats f32 (any number). */
 int32_t runit_heads_rows(runit_ctx_t*, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, void* proj, uint32_t ld,
                          uint32_t T, uint32_t start);
 int32_t runit_head_attention_rows(runit_ctx_t*, const runit_heads_cfg* attn, int32_t cache_f32, const void* proj, uint32_t ld, void* out,
                                   uint32_t ldo, uint32_t T, uint32_t start, void* part, size_t part_floats, void* tickets);
-/* One token of a state-space layer: y f32 [heads * vdim] = (S^T C + skip x) * silu(z). */
-int32_t runit_ssm_step(runit_ctx_t*, const runit_ssm_cfg* cfg, const void* proj, void* y, const void* pos);
+/* One token of a state-space layer: y f32 [heads * vdim] = (S^T C + skip x) * silu(z), squares f32 [heads][ceil(vdim / 32)] its sums
+ * of squares over slices of 32 columns.  The state must not be an output of the launch in front of this one. */
+int32_t runit_ssm_step(runit_ctx_t*, const runit_ssm_cfg* cfg, const void* proj, void* y, void* squares, const void* pos);
 /* T tokens: x, B, C convolved and activated into rows of ldx (bf16 or f32); dt f32 [T][heads] becomes softplus(dt + dt_bias). */
 int32_t runit_ssm_conv_rows(runit_ctx_t*, const runit_ssm_cfg* cfg, int32_t f32, const void* proj, uint32_t ld, void* xbc, uint32_t ldx, void* dt,
                             uint32_t T, uint32_t start);
@@ -595,9 +598,10 @@ int32_t runit_add_norm_rows(runit_ctx_t*, void* x, const void* y, const void* ga
  * and then norm(v) with `gain` when that is not NULL.  relu2: max(., 0)^2 instead of cap. */
 int32_t runit_gemv_bf16_residual_f32(runit_ctx_t*, const void* weight, const void* x, const void* y, const void* y_gain, const void* gain, void* x_out,
                                      void* out, float eps, float cap, int32_t relu2, uint32_t m, uint32_t k);
-/* out[m] = W . v: the first `plain` values of v are x, the others groups of `group` values of x, normed, times factor [k - plain] */
-int32_t runit_gemv_bf16_groups_f32(runit_ctx_t*, const void* weight, const void* x, const void* factor, void* out, float eps, uint32_t plain,
-                                   uint32_t group, uint32_t m, uint32_t k);
+/* out[m] = W . v: the first `plain` values of v are x, the others groups of `group` values of x, normed, times factor [k - plain];
+ * squares (may be NULL): f32 [groups][squares_n], sums of squares that add up to those of the groups */
+int32_t runit_gemv_bf16_groups_f32(runit_ctx_t*, const void* weight, const void* x, const void* factor, const void* squares, uint32_t squares_n,
+                                   void* out, float eps, uint32_t plain, uint32_t group, uint32_t m, uint32_t k);
 
 /* ── decoders described layer by layer (no twin), weights in bf16 ──
  * Every matrix is row-major [rows][pad8(columns)] bf16 with zero padding; norms and router are f32.  Linear maps W x.

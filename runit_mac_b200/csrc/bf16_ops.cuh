@@ -32,8 +32,14 @@ struct GemvPrologue {
     int kind = GEMV_PRO_NONE;
     const float *y = nullptr, *y_gain = nullptr, *gain = nullptr;
     float* x_out = nullptr;
+    // the caller vouches that x and y_gain (RESIDUAL) are final before the launch in front of this one starts: they are read
+    // before the dependency wait
+    bool early = false;
     const float* factor = nullptr;
+    bool factor_early = false;          // the same for factor
     uint32_t plain = 0, group = 0;
+    const float* squares = nullptr;     // GROUPS, not null: [groups][squares_n] partial sums of squares of the groups
+    uint32_t squares_n = 0;
 };
 struct GemvDesc {
     const void* w = nullptr;
@@ -190,20 +196,23 @@ struct Ssm {
     __host__ __device__ uint32_t in_rows() const { return 2 * heads * vdim + 2 * groups * state + heads; }
 };
 // One token.  Attention and / or retention on one projected row (a null one is left out): ao = [attention output * out_scale |
-// retention o as it is], factor = silu(g) * out_scale of the retention.  Writes this position's cache row, updates the state.
+// retention o as it is], factor = silu(g) * out_scale of the retention, squares = sums of o^2 over the 32-column slices of every
+// head ([heads][ceil(vdim / 32)]).  Writes this position's cache row, updates the state.  *pos_ptr, the cache and the state are
+// read before the dependency wait: they must be final before the launch in front of this one starts.
 // part / tickets: heads_step_scratch() floats and kv_heads * ceil(rep / 8) zeroed words (zero again afterwards).
 uint32_t heads_step_splits(const runit_ctx* ctx, const HeadAttn& a, uint32_t T);
 size_t heads_part_floats(const HeadAttn& a, uint32_t nsplit, uint32_t T);
-int32_t heads_step(runit_ctx* ctx, const HeadAttn* a, const Retention* r, bool exact, const float* proj, float* ao, float* factor, float* part,
-                   uint32_t* tickets, uint32_t nsplit, const int32_t* pos_ptr);
+int32_t heads_step(runit_ctx* ctx, const HeadAttn* a, const Retention* r, bool exact, const float* proj, float* ao, float* factor, float* squares,
+                   float* part, uint32_t* tickets, uint32_t nsplit, const int32_t* pos_ptr);
 // Many tokens: cache rows of their positions; rotated q and k of the retention in place.
 int32_t heads_rows(runit_ctx* ctx, const HeadAttn* a, const Retention* r, bool exact, void* proj, uint32_t ld, uint32_t T, uint32_t start);
 // Attention of T tokens whose cache rows are written: out rows of ldo.  part / tickets (see heads_step) serve few tokens; the
 // number of splits is lowered until part_cap floats and 4096 tickets suffice.
 int32_t head_attention_rows(runit_ctx* ctx, const HeadAttn& a, bool exact, const void* proj, uint32_t ld, void* out, uint32_t ldo, uint32_t T,
                             uint32_t start, float* part, size_t part_cap, uint32_t* tickets);
-// One token of a state-space layer: y = (S^T C + skip x) * silu(z), state and ring updated.
-int32_t ssm_step(runit_ctx* ctx, const Ssm& m, const float* proj, float* y, const int32_t* pos_ptr);
+// One token of a state-space layer: y = (S^T C + skip x) * silu(z), squares as above; state and ring updated.  The state is
+// read before the dependency wait.
+int32_t ssm_step(runit_ctx* ctx, const Ssm& m, const float* proj, float* y, float* squares, const int32_t* pos_ptr);
 // Many tokens: convolution, silu and softplus.  xbc rows of ld_out in the operand type, dt f32 [T][heads] in place.
 int32_t ssm_conv_rows(runit_ctx* ctx, const Ssm& m, bool exact, const void* proj, uint32_t ld, void* xbc, uint32_t ld_out, float* dt, uint32_t T,
                       uint32_t start);

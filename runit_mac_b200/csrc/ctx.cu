@@ -210,6 +210,7 @@ int32_t runit_set_tuning(runit_ctx_t* ctx, const char* key, int32_t value) {
     if (!strcmp(key, "gemv_variant")) ctx->tune.gemv_variant = value;
     else if (!strcmp(key, "gemv_stages")) ctx->tune.gemv_stages = value;
     else if (!strcmp(key, "pdl")) ctx->tune.pdl = value;
+    else if (!strcmp(key, "gemv_pro_ctas")) ctx->tune.gemv_pro_ctas = value;
     else if (!strcmp(key, "gemv_load")) ctx->tune.gemv_load = value;
     else if (!strcmp(key, "gemv_ksl")) ctx->tune.gemv_ksl = value;
     else if (!strcmp(key, "gemv_csplit")) ctx->tune.gemv_csplit = value;

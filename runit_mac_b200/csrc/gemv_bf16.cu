@@ -81,21 +81,49 @@ __device__ __forceinline__ float4 load4(const float* p, uint32_t e, uint32_t n, 
 }
 __device__ __forceinline__ bool aligned4(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
-// GEMV_PRO_RESIDUAL: returns the factor of the products (that of the second norm).  A thread handles the same pieces in every
-// pass; ya / yb are two more planes like xa / xb.
+// The prologues work on two pairs of planes, xa / xb and ya / yb (four neighbouring values each, see stage_x); a thread handles
+// the same pieces in every pass.  stage_early runs before the dependency wait.
+__device__ __forceinline__ float4 group_factors(const GemvPrologue& p, uint32_t e, uint32_t K, bool vec) {
+    if (vec) return e >= p.plain ? load4(p.factor, e - p.plain, K - p.plain, true) : make_float4(1.f, 1.f, 1.f, 1.f);
+    auto one = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? p.factor[j - p.plain] : 0.f); };
+    return make_float4(one(e), one(e + 1), one(e + 2), one(e + 3));
+}
+__device__ __forceinline__ bool pro_vec(const float* x, const GemvPrologue& p, uint32_t K) {
+    return (K & 3u) == 0 && (p.plain & 3u) == 0 && aligned4(x) && aligned4(p.y) && aligned4(p.y_gain) && aligned4(p.gain) && aligned4(p.x_out) && aligned4(p.factor);
+}
+__device__ __forceinline__ void stage_early(const float* x, const GemvPrologue& p, uint32_t K, uint32_t nch, float4* xa, float4* xb, float4* ya,
+                                             float4* yb) {
+    const bool vec = pro_vec(x, p, K);
+    if (p.kind == GEMV_PRO_RESIDUAL && p.y && p.early) {
+        for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+            const float4 xv = load4(x, 4 * i, K, vec), g = load4(p.y_gain, 4 * i, K, vec);
+            ((i & 1u) ? xb : xa)[i >> 1] = xv;
+            ((i & 1u) ? yb : ya)[i >> 1] = g;
+        }
+    } else if (p.kind == GEMV_PRO_GROUPS && p.factor_early) {
+        for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) ((i & 1u) ? yb : ya)[i >> 1] = group_factors(p, 4 * i, K, vec);
+    }
+}
+
+// GEMV_PRO_RESIDUAL: returns the factor of the products (that of the second norm).
 __device__ __forceinline__ float stage_residual(const float* x, const GemvPrologue& p, float eps, uint32_t K, uint32_t nch, float4* xa, float4* xb,
                                                  float4* ya, float4* yb, float* part) {
-    const bool vec = (K & 3u) == 0 && aligned4(x) && aligned4(p.y) && aligned4(p.y_gain) && aligned4(p.gain) && aligned4(p.x_out);
+    const bool vec = pro_vec(x, p, K);
     float r = 0.f;
     if (p.y) {
         float sq = 0.f;
         for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
-            const float4 xv = load4(x, 4 * i, K, vec), g = load4(p.y_gain, 4 * i, K, vec);
-            float4 y = load4(p.y, 4 * i, K, vec);
+            float4& gs = ((i & 1u) ? yb : ya)[i >> 1];
+            float4 y = load4(p.y, 4 * i, K, vec), g;
+            if (p.early) {
+                g = gs;
+            } else {
+                g = load4(p.y_gain, 4 * i, K, vec);
+                ((i & 1u) ? xb : xa)[i >> 1] = load4(x, 4 * i, K, vec);
+            }
             sq = fmaf(y.x, y.x, sq); sq = fmaf(y.y, y.y, sq); sq = fmaf(y.z, y.z, sq); sq = fmaf(y.w, y.w, sq);
             y.x *= g.x; y.y *= g.y; y.z *= g.z; y.w *= g.w;
-            ((i & 1u) ? xb : xa)[i >> 1] = xv;
-            ((i & 1u) ? yb : ya)[i >> 1] = y;
+            gs = y;
         }
         r = rsqrtf(cta_sum(sq, part) / (float)K + eps);
     }
@@ -133,51 +161,60 @@ __device__ __forceinline__ float stage_residual(const float* x, const GemvProlog
     return rsqrtf(cta_sum(sq, part) / (float)K + eps);
 }
 
-// GEMV_PRO_GROUPS: the values and their factors go to shared memory first, then the groups are summed there.  fac: one word per
-// group and warp of it.
-__device__ __forceinline__ void stage_groups(const float* x, const GemvPrologue& p, float eps, uint32_t K, uint32_t nch, float4* xa, float4* xb,
-                                             float4* ya, float4* yb, float* fac) {
-    const bool vec = (K & 3u) == 0 && (p.plain & 3u) == 0 && aligned4(x) && aligned4(p.factor);
-    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
-        const uint32_t e = 4 * i;
-        ((i & 1u) ? xb : xa)[i >> 1] = load4(x, e, K, vec);
-        float4 f;
-        if (vec) {
-            f = e >= p.plain ? load4(p.factor, e - p.plain, K - p.plain, true) : make_float4(1.f, 1.f, 1.f, 1.f);
-        } else {
-            auto one = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? p.factor[j - p.plain] : 0.f); };
-            f = make_float4(one(e), one(e + 1), one(e + 2), one(e + 3));
-        }
-        ((i & 1u) ? yb : ya)[i >> 1] = f;
-    }
-    __syncthreads();
+// GEMV_PRO_GROUPS: the sums of squares of the groups come from the launch that made x (squares), or are formed from the staged
+// values.  fac: one word per group and warp of it.  Returns the factor of the products.
+__device__ __forceinline__ float stage_groups(const float* x, const GemvPrologue& p, float eps, uint32_t K, uint32_t nch, float4* xa, float4* xb,
+                                              float4* ya, float4* yb, float* fac) {
+    const bool vec = pro_vec(x, p, K);
     const uint32_t groups = (K - p.plain) / p.group, wpg = groups >= 8 ? 1u : (groups >= 3 ? 2u : (groups == 2 ? 4u : 8u));
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = warp % wpg;
+    for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
+        float4 v = load4(x, 4 * i, K, vec);
+        if (p.squares) {
+            const float4 f = p.factor_early ? ((i & 1u) ? yb : ya)[i >> 1] : group_factors(p, 4 * i, K, vec);
+            v.x *= f.x; v.y *= f.y; v.z *= f.z; v.w *= f.w;
+        } else if (!p.factor_early) {
+            ((i & 1u) ? yb : ya)[i >> 1] = group_factors(p, 4 * i, K, vec);
+        }
+        ((i & 1u) ? xb : xa)[i >> 1] = v;
+    }
+    if (!p.squares) __syncthreads();
     auto at = [&](uint32_t e) -> float { return reinterpret_cast<const float*>(((e >> 2) & 1u) ? xb : xa)[(e >> 3) * 4 + (e & 3u)]; };
     for (uint32_t g = warp / wpg; g < groups; g += kWarps / wpg) {
-        const uint32_t lo = p.plain + g * p.group;
         float sq = 0.f;
-        for (uint32_t i = sub * 32 + lane; i < p.group; i += 32 * wpg) {
-            const float v = at(lo + i);
-            sq = fmaf(v, v, sq);
+        if (p.squares) {
+            for (uint32_t i = sub * 32 + lane; i < p.squares_n; i += 32 * wpg) sq += p.squares[(size_t)g * p.squares_n + i];
+        } else {
+            const uint32_t lo = p.plain + g * p.group;
+            for (uint32_t i = sub * 32 + lane; i < p.group; i += 32 * wpg) {
+                const float v = at(lo + i);
+                sq = fmaf(v, v, sq);
+            }
         }
         sq = warp_add(sq);
         if (lane == 0) fac[g * wpg + sub] = sq;
     }
     __syncthreads();
-    for (uint32_t g = threadIdx.x; g < groups; g += kWarps * 32) {
+    auto group_factor = [&](uint32_t g) {
         float sq = 0.f;
         for (uint32_t i = 0; i < wpg; i++) sq += fac[g * wpg + i];
-        fac[g * wpg] = rsqrtf(sq / (float)p.group + eps);
-    }
-    __syncthreads();
+        return rsqrtf(sq / (float)p.group + eps);
+    };
+    if (p.squares && p.plain == 0 && groups == 1) return group_factor(0);
+    const bool whole = (p.group & 3u) == 0 && (p.plain & 3u) == 0;       // four neighbours share a group
     for (uint32_t i = threadIdx.x; i < 2 * nch; i += kWarps * 32) {
         const uint32_t e = 4 * i;
         float4& v = ((i & 1u) ? xb : xa)[i >> 1];
-        const float4 f = ((i & 1u) ? yb : ya)[i >> 1];
-        auto r = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? fac[(j - p.plain) / p.group * wpg] : 0.f); };
-        v.x *= f.x * r(e); v.y *= f.y * r(e + 1); v.z *= f.z * r(e + 2); v.w *= f.w * r(e + 3);
+        const float4 f = p.squares ? make_float4(1.f, 1.f, 1.f, 1.f) : ((i & 1u) ? yb : ya)[i >> 1];
+        auto r = [&](uint32_t j) { return j < p.plain ? 1.f : (j < K ? group_factor((j - p.plain) / p.group) : 0.f); };
+        if (whole) {
+            const float s = r(e);
+            v.x *= f.x * s; v.y *= f.y * s; v.z *= f.z * s; v.w *= f.w * s;
+        } else {
+            v.x *= f.x * r(e); v.y *= f.y * r(e + 1); v.z *= f.z * r(e + 2); v.w *= f.w * r(e + 3);
+        }
     }
+    return 1.f;
 }
 
 struct Args {
@@ -202,7 +239,7 @@ struct Args {
 
 // RPU: rows of a warp's unit; U: 16-byte loads per lane, row and group
 template <int EPI, int RPU, int U, bool SLOTS, bool PRO = false>
-__global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
+__global__ void __launch_bounds__(kWarps * 32, PRO && RPU * U <= 8 ? 4 : 1) gemv_bf16_kernel(const Args a) {
     extern __shared__ __align__(16) float4 smem4[];
     __shared__ float part[kWarps];
     __shared__ unsigned long long best_s[kWarps];
@@ -230,6 +267,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
     };
     const bool early = !SLOTS || extra;
     if (early && unit < units) load(unit, 0);
+    if constexpr (PRO) stage_early(a.x, a.pro, a.K, nch, xa, xb, xb + nch, xb + 2 * nch);
     grid_dependency_wait();
     grid_launch_dependents();
     float pre = 1.f, post = 1.f;
@@ -248,7 +286,7 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
     if constexpr (PRO) {
         float4 *ya = xb + nch, *yb = ya + nch;
         if (a.pro.kind == GEMV_PRO_RESIDUAL) scale = stage_residual(a.x, a.pro, a.eps, a.K, nch, xa, xb, ya, yb, part);
-        else stage_groups(a.x, a.pro, a.eps, a.K, nch, xa, xb, ya, yb, reinterpret_cast<float*>(yb + nch));
+        else scale = stage_groups(a.x, a.pro, a.eps, a.K, nch, xa, xb, ya, yb, reinterpret_cast<float*>(yb + nch));
         __syncthreads();
     } else {
         scale = stage_x(a.x, a.K, nch, xa, xb);
@@ -283,6 +321,10 @@ __global__ void __launch_bounds__(kWarps * 32) gemv_bf16_kernel(const Args a) {
                     for (int r = 0; r < RPU; r++) acc[r] = dot8(v[r][i], p, q, acc[r]);
                 }
             }
+        }
+        if (PRO && unit + gridDim.x * kWarps < units) {       // the next unit's first loads go out before this one's sums
+            load(unit + gridDim.x * kWarps, 0);
+            first = true;
         }
 #pragma unroll
         for (int r = 0; r < RPU; r++) acc[r] = warp_add(acc[r]) * scale;
@@ -543,8 +585,9 @@ static int32_t launch(runit_ctx* ctx, const char* name, const Args& a, uint32_t 
     if (smem > 48 * 1024)
         RUNIT_CUDA_TRY(ctx, cudaFuncSetAttribute(gemv_bf16_kernel<EPI, RPU, U, SLOTS, PRO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     // every CTA forms the whole vector: with a prologue that reads several vectors, fewer and longer-lived ones
-    const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * (PRO ? 3 : 8);
-    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, U, SLOTS, PRO>, dim3(want < cap ? want : cap, slots), dim3(kWarps * 32), smem, a);
+    const uint32_t units = (max_rows + RPU - 1) / RPU, want = (units + kWarps - 1) / kWarps, cap = (uint32_t)ctx->sm_count * (PRO ? (ctx->tune.gemv_pro_ctas > 0 ? ctx->tune.gemv_pro_ctas : (RPU * U <= 8 ? 4 : 2)) : 8);
+    const uint32_t rounds = PRO ? (want + cap - 1) / cap : 1;
+    runit_launch_chain_smem(ctx, gemv_bf16_kernel<EPI, RPU, U, SLOTS, PRO>, dim3(PRO ? (want + rounds - 1) / rounds : (want < cap ? want : cap), slots), dim3(kWarps * 32), smem, a);
     return runit_after_launch(ctx, name);
 }
 
@@ -563,7 +606,8 @@ int32_t gemv_bf16(runit_ctx* ctx, const char* name, const GemvDesc& d) {
 #define RUNIT_GVP(E, R, U) gv::launch<E, R, U, false, true>(ctx, name, a, d.rows, 1)
         if (d.epi == EPI_SILU_GLU) return d.K <= 512 ? RUNIT_GVP(EPI_SILU_GLU, 4, 2) : RUNIT_GVP(EPI_SILU_GLU, 2, 8);
         if (d.epi == EPI_RELU2) return d.K <= 512 ? RUNIT_GVP(EPI_RELU2, 4, 2) : (d.K <= 1024 ? RUNIT_GVP(EPI_RELU2, 2, 4) : RUNIT_GVP(EPI_RELU2, 1, 8));
-        return d.K <= 512 ? RUNIT_GVP(EPI_F32, 4, 2) : (d.K <= 1024 ? RUNIT_GVP(EPI_F32, 2, 4) : RUNIT_GVP(EPI_F32, 1, 8));
+        if (d.K <= 512) return RUNIT_GVP(EPI_F32, 4, 2);
+        return d.K <= 1024 ? RUNIT_GVP(EPI_F32, 2, 4) : (d.K <= 2048 ? RUNIT_GVP(EPI_F32, 1, 8) : RUNIT_GVP(EPI_F32, 1, 16));
 #undef RUNIT_GVP
     }
     const bool slots = d.slot_expert != nullptr;
@@ -663,13 +707,14 @@ int32_t runit_gemv_bf16_residual_f32(runit_ctx_t* ctx, const void* weight, const
     return gemv_bf16(ctx, "gemv_bf16_residual_f32", d);
 }
 
-int32_t runit_gemv_bf16_groups_f32(runit_ctx_t* ctx, const void* weight, const void* x, const void* factor, void* out, float eps, uint32_t plain,
-                                   uint32_t group, uint32_t m, uint32_t k) {
+int32_t runit_gemv_bf16_groups_f32(runit_ctx_t* ctx, const void* weight, const void* x, const void* factor, const void* squares, uint32_t squares_n,
+                                   void* out, float eps, uint32_t plain, uint32_t group, uint32_t m, uint32_t k) {
     if (!ctx) return RUNIT_ERR_BAD_ARG;
     RUNIT_REQUIRE(ctx, weight && x && out && m > 0 && k > 0 && runit_aligned(weight, 16), "gemv_bf16_groups_f32: bad argument");
     GemvDesc d;
     d.w = weight; d.rows = m; d.K = k; d.ldw = pad8(k); d.x = (const float*)x; d.eps = eps; d.out = (float*)out;
     d.pro.kind = GEMV_PRO_GROUPS; d.pro.plain = plain; d.pro.group = group; d.pro.factor = (const float*)factor;
+    d.pro.squares = (const float*)squares; d.pro.squares_n = squares_n;
     return gemv_bf16(ctx, "gemv_bf16_groups_f32", d);
 }
 

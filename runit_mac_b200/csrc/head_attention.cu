@@ -40,6 +40,16 @@ __device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
         v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
     }
 }
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+// element i of a small array in registers
+__device__ __forceinline__ uint4 pick(const uint4 (&x)[4], uint32_t i) { return i == 0 ? x[0] : (i == 1 ? x[1] : (i == 2 ? x[2] : x[3])); }
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
@@ -55,13 +65,39 @@ __device__ __forceinline__ float unit_factor(const HeadAttn& a, const T* p) {
     }
     return rsqrtf(wsum(s) / (float)a.dim + a.eps);
 }
-// one warp writes the cache row of key head g (padding zero)
+// one warp writes the cache row of key head g (padding zero); wide: bf16 rows whose heads start at multiples of 4 elements
 template <typename TC, typename T>
-__device__ __forceinline__ void write_row(const HeadAttn& a, const T* row, uint32_t g, uint32_t pos) {
+__device__ __forceinline__ void write_row(const HeadAttn& a, const T* row, uint32_t g, uint32_t pos, bool wide = false) {
     const uint32_t lane = threadIdx.x & 31, slot = pos % a.cap;
     const T *k = row + a.heads * a.dim + g * a.dim, *v = row + (a.heads + a.kv_heads) * a.dim + g * a.vdim;
     TC* kd = reinterpret_cast<TC*>(a.kc) + ((size_t)g * a.cap + slot) * a.kd();
     TC* vd = reinterpret_cast<TC*>(a.vc) + ((size_t)g * a.cap + slot) * a.vd();
+    if constexpr (sizeof(T) == 2 && sizeof(TC) == 2) {
+        if (wide && a.kd() == a.dim && a.vd() == a.vdim && a.dim <= 256) {
+            uint2 u[2];
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const uint32_t c = (lane + 32 * i) * 4;
+                u[i] = c < a.dim ? *reinterpret_cast<const uint2*>(k + c) : make_uint2(0, 0);
+                const float x[4] = {__uint_as_float(u[i].x << 16), __uint_as_float(u[i].x & 0xffff0000u), __uint_as_float(u[i].y << 16),
+                                    __uint_as_float(u[i].y & 0xffff0000u)};
+#pragma unroll
+                for (int e = 0; e < 4; e++) s = fmaf(x[e], x[e], s);
+            }
+            for (uint32_t c = lane * 4; c < a.vdim; c += 128) *reinterpret_cast<uint2*>(vd + c) = *reinterpret_cast<const uint2*>(v + c);
+            const float f = a.unit_qk ? rsqrtf(wsum(s) / (float)a.dim + a.eps) : 1.f;
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const uint32_t c = (lane + 32 * i) * 4;
+                if (c >= a.dim) break;
+                const __nv_bfloat162 p = __floats2bfloat162_rn(__uint_as_float(u[i].x << 16) * f, __uint_as_float(u[i].x & 0xffff0000u) * f);
+                const __nv_bfloat162 q = __floats2bfloat162_rn(__uint_as_float(u[i].y << 16) * f, __uint_as_float(u[i].y & 0xffff0000u) * f);
+                *reinterpret_cast<uint2*>(kd + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&p), *reinterpret_cast<const uint32_t*>(&q));
+            }
+            return;
+        }
+    }
     const float f = unit_factor(a, k);
     for (uint32_t i = lane; i < a.kd(); i += 32) put(kd + i, i < a.dim ? to_f32(k[i]) * f : 0.f);
     for (uint32_t i = lane; i < a.vd(); i += 32) put(vd + i, i < a.vdim ? to_f32(v[i]) : 0.f);
@@ -78,17 +114,49 @@ static size_t cta_smem(const HeadAttn& a, int RB) {
     return ((size_t)RB * a.kd() + RB * kTile + 4 * 8 + (red > wts ? red : wts)) * 4;
 }
 
-// RAW: the token's own key and value are still in the projected row; the CTA whose keys end with it writes the cache row.
+// Cached rows of a CTA's first tile, requested before its inputs are known: a thread's pieces of a key row and of the value rows
+// it adds up (at most P of each).  bf16 caches only.
+constexpr int kPre = 4;
+struct FirstTile {
+    uint4 k[kPre], v[kPre];
+};
+
+// RAW: the token's own key and value are still in the projected row; the CTA whose keys end with it writes the cache row.  With a
+// bf16 cache the first tile is requested before the dependency wait (which this function then does).
 template <typename TC, typename TQ, typename TO, int RB, bool RAW>
 __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* out, uint32_t pos, uint32_t g, uint32_t hb, uint32_t nhb,
                                           uint32_t split, uint32_t t, const Parts& pt, float* sm) {
+    constexpr bool EARLY = RAW && sizeof(TC) == 2;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t rep = a.heads / a.kv_heads, h0 = g * rep + hb * RB, nr = min((uint32_t)RB, rep - hb * RB), kd = a.kd(), vd = a.vd();
     __shared__ uint32_t last_s;
+    __shared__ float slope_s[8];
     float* qs = sm;
     float* ss = qs + RB * kd;
     float *ms = ss + RB * kTile, *lsum = ms + 8, *fs = lsum + 8;
     float* red = fs + 16;
+    const uint32_t lo = a.window && pos + 1 > a.window ? pos + 1 - a.window : 0, len = pos + 1 - lo;
+    const uint32_t chunk = max(16u, ((len + pt.nsplit - 1) / pt.nsplit + 15) / 16 * 16);
+    const uint32_t beg = lo + min(len, split * chunk), end = min(lo + len, beg + chunk);
+    const TC* kc = reinterpret_cast<const TC*>(a.kc) + (size_t)g * a.cap * kd;
+    const TC* vc = reinterpret_cast<const TC*>(a.vc) + (size_t)g * a.cap * vd;
+    const uint32_t nv = vd / 8, ng = 256 / nv, cv = tid % nv, gp = tid / nv;
+    const uint32_t fkey = beg + (tid >> 2);
+    FirstTile ft;
+    if constexpr (EARLY) {
+#pragma unroll
+        for (int i = 0; i < kPre; i++) {
+            const uint32_t ch = (tid & 3) + 4 * i, kk = gp + ng * i;
+            if (fkey < end && fkey != pos && ch < kd / 8) ft.k[i] = *reinterpret_cast<const uint4*>(kc + (size_t)(fkey % a.cap) * kd + ch * 8);
+            if (gp < ng && kk < (uint32_t)kTile && beg + kk < end && beg + kk != pos)
+                ft.v[i] = *reinterpret_cast<const uint4*>(vc + (size_t)((beg + kk) % a.cap) * vd + cv * 8);
+        }
+    }
+    if (tid < nr) slope_s[tid] = a.slopes ? a.slopes[h0 + tid] : 0.f;
+    if constexpr (RAW) {
+        grid_dependency_wait();
+        grid_launch_dependents();
+    }
     for (uint32_t r = warp; r < RB; r += 8) {
         if (r < nr) {
             const TQ* q = row + (size_t)(h0 + r) * a.dim;
@@ -102,14 +170,8 @@ __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* o
             lsum[r] = 0.f;
         }
     }
-    const uint32_t lo = a.window && pos + 1 > a.window ? pos + 1 - a.window : 0, len = pos + 1 - lo;
-    const uint32_t chunk = max(16u, ((len + pt.nsplit - 1) / pt.nsplit + 15) / 16 * 16);
-    const uint32_t beg = lo + min(len, split * chunk), end = min(lo + len, beg + chunk);
     if (RAW && beg < end && end == pos + 1 && warp == 7) write_row<TC>(a, row, g, pos);
     __syncthreads();
-    const TC* kc = reinterpret_cast<const TC*>(a.kc) + (size_t)g * a.cap * kd;
-    const TC* vc = reinterpret_cast<const TC*>(a.vc) + (size_t)g * a.cap * vd;
-    const uint32_t nv = vd / 8, ng = 256 / nv, cv = tid % nv, gp = tid / nv;
     float acc[RB][8];
 #pragma unroll
     for (int r = 0; r < RB; r++)
@@ -123,10 +185,13 @@ __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* o
             for (int r = 0; r < RB; r++) s[r] = 0.f;
             if (key < end) {
                 const TC* kr = kc + (size_t)(key % a.cap) * kd;
+                const bool have = EARLY && k0 == beg && key != pos;      // the pieces requested early
 #pragma unroll 4
-                for (uint32_t ch = c; ch < kd / 8; ch += 4) {
+                for (uint32_t i = 0; 4 * i + c < kd / 8; i++) {
+                    const uint32_t ch = 4 * i + c;
                     float kv[8];
-                    load8(kr + ch * 8, kv);
+                    if (EARLY && have && i < kPre) unpack8(pick(ft.k, i), kv);
+                    else load8(kr + ch * 8, kv);
 #pragma unroll
                     for (int r = 0; r < RB; r++) {
                         const float4 x = *reinterpret_cast<const float4*>(qs + r * kd + ch * 8), y = *reinterpret_cast<const float4*>(qs + r * kd + ch * 8 + 4);
@@ -140,8 +205,7 @@ __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* o
                 s[r] += __shfl_xor_sync(0xffffffffu, s[r], 1);
                 s[r] += __shfl_xor_sync(0xffffffffu, s[r], 2);
                 if (c == (uint32_t)(r & 3) && (uint32_t)r < nr) {
-                    const float bias = a.slopes ? a.slopes[h0 + r] * (float)(pos - min(key, pos)) : 0.f;
-                    ss[r * kTile + (tid >> 2)] = key < end ? s[r] - bias : -INFINITY;
+                    ss[r * kTile + (tid >> 2)] = key < end ? s[r] - slope_s[r] * (float)(pos - key) : -INFINITY;
                 }
             }
         }
@@ -169,9 +233,11 @@ __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* o
             }
             const uint32_t n = min((uint32_t)kTile, end - k0);
 #pragma unroll 4
-            for (uint32_t kk = gp; kk < n; kk += ng) {
+            for (uint32_t i = 0; gp + ng * i < n; i++) {
+                const uint32_t kk = gp + ng * i;
                 float v[8];
-                load8(vc + (size_t)((k0 + kk) % a.cap) * vd + cv * 8, v);
+                if (EARLY && k0 == beg && i < kPre && k0 + kk != pos) unpack8(pick(ft.v, i), v);
+                else load8(vc + (size_t)((k0 + kk) % a.cap) * vd + cv * 8, v);
 #pragma unroll
                 for (int r = 0; r < RB; r++) {
                     const float p = (uint32_t)r < nr ? ss[r * kTile + kk] : 0.f;
@@ -235,7 +301,7 @@ __device__ __forceinline__ void attn_cta(const HeadAttn& a, const TQ* row, TO* o
 }
 
 // One retention step for columns 32 * jb .. of head h; row: [q | k | v | g] of all heads.
-__device__ __forceinline__ void retention_cta(const Retention& r, const float* row, float* out, float* factor, uint32_t h, uint32_t jb,
+__device__ __forceinline__ void retention_cta(const Retention& r, const float* row, float* out, float* factor, float* squares, uint32_t h, uint32_t jb,
                                                const int32_t* pos_ptr, float* sm) {
     __shared__ float red[8][33];
     const uint32_t tid = threadIdx.x, lane = tid & 31, j = jb * 32 + lane, half = r.rot_dims / 2;
@@ -267,24 +333,25 @@ __device__ __forceinline__ void retention_cta(const Retention& r, const float* r
     const float v = j < r.vdim ? vrow[at] : 0.f;
     __syncthreads();
     const float o = ls::state_step(st, S, r.dim, r.vdim, j, qs, ks, v, decay, pos == 0, red);
-    if (tid < 32 && j < r.vdim) {
+    if (tid >= 32) return;
+    if (j < r.vdim) {
         out[at] = o;
         factor[at] = ls::silu(vrow[(size_t)r.heads * r.vdim + at]) * r.out_scale;
     }
+    const float sq = wsum(j < r.vdim ? o * o : 0.f);
+    if (tid == 0) squares[h * ((r.vdim + 31) / 32) + jb] = sq;
 }
 
 // grid: attention CTAs (kv_heads x head blocks x splits), then retention CTAs (heads x 32-column slices)
 template <typename TC, int RB>
-__global__ void __launch_bounds__(256) heads_step_kernel(const HeadAttn a, const Retention r, const float* proj, float* ao, float* factor, const Parts pt,
+__global__ void __launch_bounds__(256) heads_step_kernel(const HeadAttn a, const Retention r, const float* proj, float* ao, float* factor, float* squares, const Parts pt,
                                                           uint32_t n_attn, uint32_t nhb, const int32_t* pos_ptr) {
     extern __shared__ __align__(16) float sm[];
     if (blockIdx.x >= n_attn) {
         const uint32_t i = blockIdx.x - n_attn, nj = (r.vdim + 31) / 32;
-        retention_cta(r, proj + (n_attn ? a.in_rows() : 0), ao + (n_attn ? a.out_rows() : 0), factor, i / nj, i % nj, pos_ptr, sm);
+        retention_cta(r, proj + (n_attn ? a.in_rows() : 0), ao + (n_attn ? a.out_rows() : 0), factor, squares, i / nj, i % nj, pos_ptr, sm);
         return;
     }
-    grid_dependency_wait();
-    grid_launch_dependents();
     const uint32_t split = blockIdx.x % pt.nsplit, b = blockIdx.x / pt.nsplit;
     attn_cta<TC, float, float, RB, true>(a, proj, ao, (uint32_t)*pos_ptr, b / nhb, b % nhb, nhb, split, 0, pt, sm);
 }
@@ -308,15 +375,26 @@ __global__ void __launch_bounds__(256) heads_rows_kernel(const HeadAttn a, const
     TC* row = proj + (size_t)t * ld;
     for (uint32_t i = threadIdx.x; i < (r.heads ? half : 0); i += 256) sincosf((float)pos * r.freq[i], &cs[i].y, &cs[i].x);
     __syncthreads();
+    const bool wide = (ld & 3u) == 0 && (a.dim & 3u) == 0 && (a.vdim & 3u) == 0 && (reinterpret_cast<uintptr_t>(proj) & 7u) == 0;
+    const bool pairs = sizeof(TC) == 2 && (ld & 1u) == 0 && (r.dim & 1u) == 0 && (half & 1u) == 0 && (a.in_rows() & 1u) == 0 &&
+                       (reinterpret_cast<uintptr_t>(proj) & 3u) == 0;
     for (uint32_t item = warp; item < a.kv_heads + 2 * r.heads; item += 8) {
         if (item < a.kv_heads) {
-            write_row<TC>(a, row, item, pos);
+            write_row<TC>(a, row, item, pos, wide);
             continue;
         }
         const uint32_t i0 = item - a.kv_heads;
         TC* p = row + (a.heads ? a.in_rows() : 0) + (size_t)i0 * r.dim;          // q of all heads, then k of all heads
         const float f = i0 < r.heads ? 1.f : r.k_scale;
-        for (uint32_t i = lane; i < half; i += 32) {
+        if constexpr (sizeof(TC) == 2) {
+            for (uint32_t i = 2 * lane; i < (pairs ? half : 0); i += 64) {
+                __nv_bfloat162 *pu = reinterpret_cast<__nv_bfloat162*>(p + i), *pv = reinterpret_cast<__nv_bfloat162*>(p + i + half);
+                const float2 u = __bfloat1622float2(*pu), v = __bfloat1622float2(*pv), a0 = cs[i], a1 = cs[i + 1];
+                *pu = __floats2bfloat162_rn(fmaf(u.x, a0.x, -(v.x * a0.y)) * f, fmaf(u.y, a1.x, -(v.y * a1.y)) * f);
+                *pv = __floats2bfloat162_rn(fmaf(v.x, a0.x, u.x * a0.y) * f, fmaf(v.y, a1.x, u.y * a1.y) * f);
+            }
+        }
+        for (uint32_t i = pairs ? half : lane; i < half; i += 32) {
             const float u = to_f32(p[i]), v = to_f32(p[i + half]), c = cs[i].x, s = cs[i].y;
             put(p + i, fmaf(u, c, -(v * s)) * f);
             put(p + i + half, fmaf(v, c, u * s) * f);
@@ -542,8 +620,8 @@ uint32_t heads_step_splits(const runit_ctx* ctx, const HeadAttn& a, uint32_t T) 
 }
 size_t heads_part_floats(const HeadAttn& a, uint32_t nsplit, uint32_t T) { return (size_t)T * a.heads * nsplit * (a.vdim + 2); }
 
-int32_t heads_step(runit_ctx* ctx, const HeadAttn* ap, const Retention* rp, bool exact, const float* proj, float* ao, float* factor, float* part,
-                   uint32_t* tickets, uint32_t nsplit, const int32_t* pos_ptr) {
+int32_t heads_step(runit_ctx* ctx, const HeadAttn* ap, const Retention* rp, bool exact, const float* proj, float* ao, float* factor, float* squares,
+                   float* part, uint32_t* tickets, uint32_t nsplit, const int32_t* pos_ptr) {
     const HeadAttn a = ap ? *ap : HeadAttn();
     const Retention r = rp ? *rp : Retention();
     RUNIT_REQUIRE(ctx, nsplit > 0 && nsplit <= 64 && (a.heads || r.heads) && r.dim <= ls::kMaxKeyDim && a.vd() <= 2048, "heads_step: bad sizes");
@@ -554,7 +632,7 @@ int32_t heads_step(runit_ctx* ctx, const HeadAttn* ap, const Retention* rp, bool
         smem = smem > (size_t)r.dim * 8 ? smem : (size_t)r.dim * 8;
         int32_t st = allow_smem(ctx, "heads_step", kern, smem);
         if (st != RUNIT_OK) return st;
-        runit_launch_chain_smem(ctx, kern, dim3(n_attn + n_ret), dim3(256), smem, a, r, proj, ao, factor, pt, n_attn, nhb, pos_ptr);
+        runit_launch_chain_smem(ctx, kern, dim3(n_attn + n_ret), dim3(256), smem, a, r, proj, ao, factor, squares, pt, n_attn, nhb, pos_ptr);
         return runit_after_launch(ctx, "heads_step");
     };
 #define RUNIT_HS(RB) (exact ? go(heads_step_kernel<float, RB>, RB) : go(heads_step_kernel<__nv_bfloat16, RB>, RB))
@@ -638,15 +716,15 @@ int32_t retention_of(runit_ctx* ctx, const char* who, const runit_retention_cfg*
 extern "C" {
 
 int32_t runit_heads_step(runit_ctx_t* ctx, const runit_heads_cfg* attn, const runit_retention_cfg* ret, int32_t cache_f32, const void* proj, void* ao,
-                         void* factor, void* part, void* tickets, uint32_t nsplit, const void* pos) {
+                         void* factor, void* squares, void* part, void* tickets, uint32_t nsplit, const void* pos) {
     if (!ctx) return RUNIT_ERR_BAD_ARG;
     HeadAttn a;
     Retention r;
     int32_t st;
     if (attn && (st = heads_of(ctx, "heads_step", attn, &a))) return st;
     if (ret && (st = retention_of(ctx, "heads_step", ret, &r))) return st;
-    RUNIT_REQUIRE(ctx, proj && ao && pos && (!attn || (part && tickets)) && (!ret || factor), "heads_step: null argument");
-    return heads_step(ctx, attn ? &a : nullptr, ret ? &r : nullptr, cache_f32 != 0, (const float*)proj, (float*)ao, (float*)factor, (float*)part,
+    RUNIT_REQUIRE(ctx, proj && ao && pos && (!attn || (part && tickets)) && (!ret || (factor && squares)), "heads_step: null argument");
+    return heads_step(ctx, attn ? &a : nullptr, ret ? &r : nullptr, cache_f32 != 0, (const float*)proj, (float*)ao, (float*)factor, (float*)squares, (float*)part,
                       (uint32_t*)tickets, nsplit, (const int32_t*)pos);
 }
 

@@ -61,7 +61,7 @@ struct LayeredModel : runit_model {
     uint32_t* counter = nullptr;    // ticket word of the routing launch
     // one token (f32)
     float *x1 = nullptr, *xn1 = nullptr, *qkv1 = nullptr, *qeff1 = nullptr, *po1 = nullptr, *pml1 = nullptr, *ao1 = nullptr, *act1 = nullptr,
-          *rl1 = nullptr, *rw1 = nullptr, *gate1 = nullptr, *x2 = nullptr, *y1 = nullptr, *factor1 = nullptr, *part1 = nullptr;
+          *rl1 = nullptr, *rw1 = nullptr, *gate1 = nullptr, *x2 = nullptr, *y1 = nullptr, *factor1 = nullptr, *squares1 = nullptr, *part1 = nullptr;
     int32_t* idx1 = nullptr;
     uint32_t act_stride = 0;
     // portions (allocated on first use)
@@ -115,7 +115,8 @@ int32_t LayeredModel::issue_step(bool with_logits, uint32_t n_forced, bool sampl
             g.gain = (const float*)gain;
         } else if (y) {
             g.pro.kind = GEMV_PRO_RESIDUAL;
-            g.pro.y = y; g.pro.y_gain = y_gain; g.pro.x_out = x_other;
+            // the stream was last written two launches or more before this one (by the matrix that entered the sublayer)
+            g.pro.y = y; g.pro.y_gain = y_gain; g.pro.x_out = x_other; g.pro.early = true;
             std::swap(x, x_other);
             y = nullptr;
         }
@@ -144,17 +145,21 @@ int32_t LayeredModel::issue_step(bool with_logits, uint32_t n_forced, bool sampl
         g = GemvDesc();
         g.w = d.w_o; g.rows = wd; g.K = l.out_k; g.ldw = pad8(l.out_k); g.x = ao1; g.eps = cfg.eps;
         if (d.mixer == RUNIT_MIX_HEADS) {
-            if ((st = heads_step(ctx, l.attn(), l.ret(), exact, qkv1, ao1, factor1, part1, tickets, l.at.heads ? heads_step_splits(ctx, l.at, 1) : 1,
+            if ((st = heads_step(ctx, l.attn(), l.ret(), exact, qkv1, ao1, factor1, squares1, part1, tickets, l.at.heads ? heads_step_splits(ctx, l.at, 1) : 1,
                                  state + 1)))
                 return st;
             if (l.rt.heads) {
                 g.pro.kind = GEMV_PRO_GROUPS;
                 g.pro.plain = l.at.out_rows(); g.pro.group = l.rt.vdim; g.pro.factor = factor1;
+                g.pro.squares = squares1; g.pro.squares_n = (l.rt.vdim + 31) / 32;
             }
         } else if (d.mixer == RUNIT_MIX_SSM) {
-            if ((st = ssm_step(ctx, l.ss, qkv1, ao1, state + 1))) return st;
+            if ((st = ssm_step(ctx, l.ss, qkv1, ao1, squares1, state + 1))) return st;
             g.pro.kind = GEMV_PRO_GROUPS;
-            g.pro.group = l.ss.inner() / l.ss.norm_groups; g.pro.factor = l.ss.norm;
+            g.pro.group = l.ss.inner() / l.ss.norm_groups; g.pro.factor = l.ss.norm; g.pro.factor_early = true;
+            if (g.pro.group % l.ss.vdim == 0) {       // whole heads
+                g.pro.squares = squares1; g.pro.squares_n = g.pro.group / l.ss.vdim * ((l.ss.vdim + 31) / 32);
+            }
         } else {
             const uint32_t ldk = pad8(l.lat.kv_rank);
             if ((st = latent_query(ctx, l.lat, exact, qkv1, 0, d.w_ukv, ldk, (const float*)d.kv_norm, l.freq, l.cache, qeff1, 1, pos))) return st;
@@ -191,7 +196,7 @@ int32_t LayeredModel::issue_step(bool with_logits, uint32_t n_forced, bool sampl
     }
     if (with_logits) {
         GemvDesc g = head_product(x);
-        if (cfg.post_norm) { g.pro.y = y; g.pro.y_gain = y_gain; }
+        if (cfg.post_norm) { g.pro.y = y; g.pro.y_gain = y_gain; g.pro.early = true; }
         if (!sampled) { g.argmax = state + 3; g.argmax_ctl = argmax_ctl; }
         if ((st = gemv_bf16(ctx, "layer_head", g))) return st;
         // the context of the draw: what has been generated so far, out_tokens[state[4] .. state[5])
@@ -667,7 +672,7 @@ int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cf
     A((void**)&m->po1, po * splits * 4); A((void**)&m->pml1, rows * splits * 8); A((void**)&m->ao1, hv * 4); A((void**)&m->act1, (act + 8) * 4);
     A((void**)&m->rl1, (routers + 1) * 4); A((void**)&m->rw1, 128); A((void**)&m->gate1, 16); A((void**)&m->idx1, 128); A((void**)&m->counter, 16);
     A((void**)&m->argmax_ctl, 16);
-    A((void**)&m->x2, (size_t)c.width * 4); A((void**)&m->y1, (size_t)c.width * 4); A((void**)&m->factor1, hv * 4);
+    A((void**)&m->x2, (size_t)c.width * 4); A((void**)&m->y1, (size_t)c.width * 4); A((void**)&m->factor1, hv * 4); A((void**)&m->squares1, hv * 4);
     A((void**)&m->part1, m->part_cap * 4); A((void**)&m->tickets, 4096 * 4);
     if (st == RUNIT_OK) st = model_record(m);
     if (st != RUNIT_OK) {

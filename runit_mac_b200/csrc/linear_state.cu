@@ -5,7 +5,7 @@
 //   * ssm_step_kernel: one token, convolution to gate (the retention's step is in head_attention.cu, beside the attention).
 //   * ssm_conv_kernel: convolution, silu and softplus of a portion.
 //   * linear_scan_kernel: the recurrence token by token, state in registers.  32-bit runs, short portions, odd sizes.
-//   * chunk_state_kernel + chunk_out_kernel: long portions in bf16, in chunks of 64 tokens on tensor cores.  The first walks the
+//   * chunk_state_kernel + chunk_out_kernel: long portions in bf16, in chunks of 128 tokens on tensor cores.  The first walks the
 //     chunks of one head and 32 value columns with the state in accumulators and leaves the state at the start of every chunk
 //     (as the sum of two bf16 numbers); the second forms all chunks at once: what the starting state contributes, and the masked
 //     products within the chunk, weighted by decays in f32.
@@ -37,7 +37,7 @@ __device__ __forceinline__ float conv_step(const Ssm& m, uint32_t c, float raw, 
 }
 
 // grid (heads, ceil(vdim / 32)).  The ring row of this position is not read by anyone in this launch.
-__global__ void __launch_bounds__(256) ssm_step_kernel(const Ssm m, const float* proj, float* y, const int32_t* pos_ptr) {
+__global__ void __launch_bounds__(256) ssm_step_kernel(const Ssm m, const float* proj, float* y, float* squares, const int32_t* pos_ptr) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[8][33];
     float *qs = sm, *ks = sm + m.state;
@@ -72,55 +72,119 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const Ssm m, const float*
     }
     __syncthreads();
     const float o = state_step(st, S, m.state, m.vdim, j, qs, ks, v, expf(a * dt), pos == 0, red);
-    if (tid < 32 && j < m.vdim) y[h * m.vdim + j] = fmaf(skip, v, o) * silu(z);
+    if (tid < 32) {
+        const float r = j < m.vdim ? fmaf(skip, v, o) * silu(z) : 0.f;
+        if (j < m.vdim) y[h * m.vdim + j] = r;
+        const float sq = wsum(r * r);
+        if (tid == 0) squares[h * gridDim.y + blockIdx.y] = sq;
+    }
 }
 
 // ── many tokens: convolution ──
-// grid (channel blocks + 1, token blocks of kConvTok), a thread walks one channel; the last column of blocks does the step
-// sizes.  Only the first token block reads the ring, and each of its threads rewrites it for its channel afterwards.
-constexpr uint32_t kConvTok = 32;
-template <typename TA, int TAPS>
-__global__ void __launch_bounds__(256) ssm_conv_kernel(const Ssm m, const TA* __restrict__ proj, uint32_t ld, TA* __restrict__ out, uint32_t ld_out,
-                                                        float* __restrict__ dt, uint32_t T, uint32_t start) {
+// grid (channel blocks + 1, token blocks of kConvTok), a thread walks VEC neighbouring channels; the last column of blocks does the
+// step sizes.  Only the first token block reads the ring, and each of its threads rewrites it for its channels afterwards.
+// TAPS > 0: the window stays in registers.
+constexpr uint32_t kConvTok = 32, kConvThreads = 128;
+template <int VEC, typename TA>
+__device__ __forceinline__ void load_vec(const TA* p, float (&v)[VEC]) {
+    if constexpr (VEC == 1) {
+        v[0] = to_f32(*p);
+    } else if constexpr (sizeof(TA) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        v[0] = __uint_as_float(u.x << 16); v[1] = __uint_as_float(u.x & 0xffff0000u);
+        v[2] = __uint_as_float(u.y << 16); v[3] = __uint_as_float(u.y & 0xffff0000u);
+    } else {
+        const float4 u = *reinterpret_cast<const float4*>(p);
+        v[0] = u.x; v[1] = u.y; v[2] = u.z; v[3] = u.w;
+    }
+}
+template <int VEC, typename TA>
+__device__ __forceinline__ void store_vec(TA* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 1) {
+        put(p, v[0]);
+    } else if constexpr (sizeof(TA) == 2) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+}
+template <typename TA, int TAPS, int VEC>
+__global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const Ssm m, const TA* __restrict__ proj, uint32_t ld, TA* __restrict__ out,
+                                                                 uint32_t ld_out, float* __restrict__ dt, uint32_t T, uint32_t start) {
     const uint32_t t0 = blockIdx.y * kConvTok, t1 = min(T, t0 + kConvTok);
     if (blockIdx.x == gridDim.x - 1) {
-        for (uint32_t i = t0 * m.heads + threadIdx.x; i < t1 * m.heads; i += 256) dt[i] = softplus(dt[i] + m.dt_bias[i % m.heads]);
+        for (uint32_t i = t0 * m.heads + threadIdx.x; i < t1 * m.heads; i += kConvThreads) dt[i] = softplus(dt[i] + m.dt_bias[i % m.heads]);
         return;
     }
-    const uint32_t c = blockIdx.x * 256 + threadIdx.x, ch = m.channels(), taps = TAPS ? TAPS : m.taps;
+    const uint32_t c = (blockIdx.x * kConvThreads + threadIdx.x) * VEC, ch = m.channels(), taps = TAPS ? TAPS : m.taps;
     if (c >= ch) return;
     const TA* x = proj + m.inner() + c;
-    const float* w = m.conv_w + (size_t)c * taps;
-    const float b = m.conv_b[c];
-    auto input = [&](int32_t t) -> float {           // t relative to the portion
-        if (t >= 0) return to_f32(x[(size_t)t * ld]);
-        return (int32_t)start + t >= 0 ? m.ring[(size_t)((start + t) % taps) * ch + c] : 0.f;
+    float b[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; e++) b[e] = m.conv_b[c + e];
+    auto input = [&](int32_t t, float (&v)[VEC]) {           // t relative to the portion
+        if (t >= 0) {
+            load_vec<VEC>(x + (size_t)t * ld, v);
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; e++) v[e] = (int32_t)start + t >= 0 ? m.ring[(size_t)((start + t) % taps) * ch + c + e] : 0.f;
+        }
     };
     if constexpr (TAPS > 0) {
-        float win[TAPS], wr[TAPS];
+        float win[TAPS][VEC], wr[TAPS][VEC];
 #pragma unroll
-        for (int j = 0; j < TAPS; j++) wr[j] = w[j];
+        for (int j = 0; j < TAPS; j++)
 #pragma unroll
-        for (int j = 0; j + 1 < TAPS; j++) win[j + 1] = input((int32_t)t0 - (TAPS - 1 - j));
-#pragma unroll 4
-        for (uint32_t t = t0; t < t1; t++) {
+            for (int e = 0; e < VEC; e++) wr[j][e] = m.conv_w[(size_t)(c + e) * TAPS + j];
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; j++) win[j] = win[j + 1];
-            win[TAPS - 1] = to_f32(x[(size_t)t * ld]);
-            float s = b;
+        for (int j = 0; j + 1 < TAPS; j++) input((int32_t)t0 - (TAPS - 1 - j), win[j + 1]);
+        constexpr uint32_t B = 8;                            // tokens requested together
+        for (uint32_t tb = t0; tb < t1; tb += B) {
+            float in[B][VEC];
 #pragma unroll
-            for (int j = 0; j < TAPS; j++) s = fmaf(wr[j], win[j], s);
-            put(out + (size_t)t * ld_out + c, silu(s));
+            for (uint32_t i = 0; i < B; i++)
+                if (tb + i < t1) load_vec<VEC>(x + (size_t)(tb + i) * ld, in[i]);
+#pragma unroll
+            for (uint32_t i = 0; i < B; i++) {
+                if (tb + i >= t1) break;
+                float y[VEC];
+#pragma unroll
+                for (int e = 0; e < VEC; e++) {
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; j++) win[j][e] = win[j + 1][e];
+                    win[TAPS - 1][e] = in[i][e];
+                    float s = b[e];
+#pragma unroll
+                    for (int j = 0; j < TAPS; j++) s = fmaf(wr[j][e], win[j][e], s);
+                    y[e] = silu_for<TA>(s);
+                }
+                store_vec<VEC>(out + (size_t)(tb + i) * ld_out + c, y);
+            }
         }
     } else {
         for (uint32_t t = t0; t < t1; t++) {
-            float s = b;
-            for (uint32_t j = 0; j < taps; j++) s = fmaf(w[j], input((int32_t)t - (int32_t)(taps - 1 - j)), s);
-            put(out + (size_t)t * ld_out + c, silu(s));
+            float s[VEC];
+#pragma unroll
+            for (int e = 0; e < VEC; e++) s[e] = b[e];
+            for (uint32_t j = 0; j < taps; j++) {
+                float v[VEC];
+                input((int32_t)t - (int32_t)(taps - 1 - j), v);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) s[e] = fmaf(m.conv_w[(size_t)(c + e) * taps + j], v[e], s[e]);
+            }
+#pragma unroll
+            for (int e = 0; e < VEC; e++) s[e] = silu_for<TA>(s[e]);
+            store_vec<VEC>(out + (size_t)t * ld_out + c, s);
         }
     }
     if (blockIdx.y == 0)
-        for (uint32_t t = T > taps ? T - taps : 0; t < T; t++) m.ring[(size_t)((start + t) % taps) * ch + c] = to_f32(x[(size_t)t * ld]);
+        for (uint32_t t = T > taps ? T - taps : 0; t < T; t++) {
+            float v[VEC];
+            load_vec<VEC>(x + (size_t)t * ld, v);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) m.ring[(size_t)((start + t) % taps) * ch + c + e] = v[e];
+        }
 }
 
 // ── many tokens: the recurrence token by token ──
@@ -172,13 +236,15 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const LinearRows d, ui
 }
 
 // ── many tokens: chunks ──
-constexpr uint32_t kChunk = 64;
+constexpr uint32_t kChunk = 128;
 static inline uint32_t pad64(uint32_t n) { return (n + 63) & ~63u; }
 
 __device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
     return *reinterpret_cast<const uint32_t*>(&h);
 }
+__device__ __forceinline__ float bf_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -192,219 +258,252 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                  : "r"(addr));
 }
-// Rows t0 .. t0+63 of a bf16 matrix (n of its columns) into shared rows of `pitch` elements, `cols` of them filled; rows from T
-// on and columns from n on become zero.  Asynchronous where the rows are 16-byte aligned (wide).
+// Rows t0 .. t0 + ROWS - 1 of a bf16 matrix (n of its columns) into shared rows of `pitch` elements, `cols` of them filled; rows
+// from T on and columns from n on become zero.  Asynchronous where the rows are 16-byte aligned (wide).  256 threads.
+template <int ROWS>
 __device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, uint32_t pitch, const __nv_bfloat16* src, uint32_t ld, uint32_t n, uint32_t cols,
-                                            uint32_t t0, uint32_t T, bool wide, uint32_t threads) {
+                                            uint32_t t0, uint32_t T, bool wide) {
     const uint32_t cpr = cols / 8;
-    for (uint32_t i = threadIdx.x; i < kChunk * cpr; i += threads) {
-        const uint32_t r = i / cpr, c = (i - r * cpr) * 8;
-        __nv_bfloat16* p = dst + r * pitch + c;
-        const __nv_bfloat16* s = src + (size_t)(t0 + r) * ld + c;
-        if (t0 + r >= T || c >= n) {
+    uint32_t r = threadIdx.x / cpr, c = threadIdx.x - r * cpr;
+    const uint32_t dr = 256 / cpr, dc = 256 - dr * cpr;
+    for (; r < (uint32_t)ROWS;) {
+        __nv_bfloat16* p = dst + r * pitch + c * 8;
+        const __nv_bfloat16* s = src + (size_t)(t0 + r) * ld + c * 8;
+        if (t0 + r >= T || c * 8 >= n) {
             *reinterpret_cast<uint4*>(p) = make_uint4(0, 0, 0, 0);
         } else if (wide) {
             cp_async16(smem_u32(p), s);
         } else {
-            for (uint32_t e = 0; e < 8; e++) p[e] = c + e < n ? s[e] : __float2bfloat16_rn(0.f);
+            for (uint32_t e = 0; e < 8; e++) p[e] = c * 8 + e < n ? s[e] : __float2bfloat16_rn(0.f);
         }
+        r += dr;
+        c += dc;
+        if (c >= cpr) { c -= cpr; r++; }
     }
 }
 __device__ __forceinline__ bool rows_aligned(const void* p, uint32_t ld, uint32_t n) {
     return (reinterpret_cast<uintptr_t>(p) & 15u) == 0 && (ld & 7u) == 0 && (n & 7u) == 0;
 }
-// One warp: la[t] = sum of the log decays of tokens 0 .. t of the chunk (0 for the tokens past the end), w[t] = step size.
+// One warp: la[t] = sum of the log decays of tokens 0 .. t of the chunk (nothing for the tokens past the end), w[t] = step size.
 __device__ __forceinline__ void chunk_decays(const LinearRows& d, uint32_t h, uint32_t t0, uint32_t T, float* la, float* w) {
+    constexpr int P = kChunk / 32;
     const uint32_t lane = threadIdx.x & 31;
     const float ld = d.log_decay[h];
-    float x[2];
+    float x[P];
 #pragma unroll
-    for (int i = 0; i < 2; i++) {
-        const uint32_t t = t0 + 2 * lane + i;
+    for (int i = 0; i < P; i++) {
+        const uint32_t t = t0 + P * lane + i;
         const float dt = t < T ? (d.dt ? d.dt[(size_t)t * d.heads + h] : 1.f) : 0.f;
-        w[2 * lane + i] = dt;
-        x[i] = ld * dt;
+        w[P * lane + i] = dt;
+        x[i] = ld * dt + (i ? x[i - 1] : 0.f);
     }
-    x[1] += x[0];
-    float s = x[1];
+    float s = x[P - 1];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
         const float n = __shfl_up_sync(0xffffffffu, s, o);
         if (lane >= (uint32_t)o) s += n;
     }
-    const float before = s - x[1];
-    la[2 * lane] = before + x[0];
-    la[2 * lane + 1] = s;
+    const float before = s - x[P - 1];
+#pragma unroll
+    for (int i = 0; i < P; i++) la[P * lane + i] = before + x[i];
 }
 
-// grid (heads, dvp / 32), 8 warps; warp w owns the 16-row tiles w, w + 8 of the state.  states: [chunk][head][2][dkp][dvp], the
-// high and the low bf16 part of the state at the start of a chunk.
-__global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, __nv_bfloat16* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T,
+// The state of one head at the start of a chunk, as the operand fragments the second kernel multiplies: [16 value columns]
+// [16 key rows][high, low part][lane] 16 bytes.  A lane's 16 bytes: value column lane / 4, key rows 2 (lane % 4), + 1 and + 8, + 9;
+// then the same of value column lane / 4 + 8.
+__device__ __forceinline__ size_t state_fragments(uint32_t chunk, uint32_t heads, uint32_t h, uint32_t dkp, uint32_t dvp) {
+    return ((size_t)chunk * heads + h) * (dvp / 16) * (dkp / 16) * 64;
+}
+
+// The state is carried as its transpose, 16 value columns x 8 key rows per accumulator tile, which is the layout of those
+// fragments.  grid (heads, dvp / 32), 8 warps: warp = 16 of the CTA's 32 value columns x every fourth block of 16 key rows.  Keys
+// arrive in steps of 64 tokens, three steps deep; the values are weighted on their way into shared memory.  The decays of all
+// chunks are summed up before the walk.
+constexpr uint32_t kStep = 64;
+static size_t chunk_state_smem(uint32_t dkp, uint32_t nc) {
+    return (size_t)3 * kStep * (dkp + 8) * 2 + (size_t)2 * kStep * 40 * 2 + (size_t)nc * kChunk * 8;
+}
+__global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, uint4* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T,
                                                            uint32_t fresh) {
     extern __shared__ __align__(16) uint8_t smem[];
     constexpr uint32_t LV = 40;
-    const uint32_t lk = dkp + 8;
-    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [2][64][lk]
-    __nv_bfloat16* vS = kS + 2 * kChunk * lk;                         // [2][64][LV]
-    __shared__ float la[2][kChunk], wt[2][kChunk];
-    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const uint32_t lk = dkp + 8, nb = dkp / 16, nc = (T + kChunk - 1) / kChunk, ns = (T + kStep - 1) / kStep;
+    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [3][kStep][lk]
+    __nv_bfloat16* vS = kS + 3 * kStep * lk;                          // [2][kStep][LV]
+    float* la = reinterpret_cast<float*>(vS + 2 * kStep * LV);        // [nc][kChunk]
+    float* wt = la + nc * kChunk;                                     // [nc][kChunk]
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mt = warp & 1, quarter = warp >> 1;
     const uint32_t h = blockIdx.x, j0 = blockIdx.y * 32, grp = h / (d.heads / d.groups);
     const __nv_bfloat16 *k = (const __nv_bfloat16*)d.k + grp * d.dk, *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
     float* S = d.state + (size_t)h * d.dk * d.dv;
     const bool wide = rows_aligned(k, d.ldk, d.dk);
-    float acc[2][4][4];
-#pragma unroll
-    for (int m = 0; m < 2; m++)
-#pragma unroll
-        for (int n = 0; n < 4; n++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const uint32_t i = (warp + 8 * m) * 16 + g + (e >> 1) * 8, j = j0 + n * 8 + 2 * t4 + (e & 1);
-                acc[m][n][e] = (!fresh && i < d.dk && j < d.dv) ? S[(size_t)i * d.dv + j] : 0.f;
-            }
-    const uint32_t nc = (T + kChunk - 1) / kChunk;
-    // value rows: thread -> token tid / 4, columns 8 * (tid % 4) ..
+    // value rows: thread -> token tid / 4 of a step, columns 8 * (tid % 4) ..
     const uint32_t vt = tid >> 2, vc = (tid & 3) * 8;
     const bool vwide = rows_aligned(v, d.ldv, 8) && j0 + vc + 8 <= d.dv;
-    float vr[8];
-    auto load_v = [&](uint32_t c) {
-        const uint32_t t = c * kChunk + vt;
+    uint4 vr;
+    auto load_v = [&](uint32_t s) {
+        const uint32_t t = s * kStep + vt;
         const __nv_bfloat16* p = v + (size_t)t * d.ldv + vc;
         if (t < T && vwide) {
-            const uint4 u = *reinterpret_cast<const uint4*>(p);
-            const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+            vr = *reinterpret_cast<const uint4*>(p);
+        } else {
+            uint32_t w[4];
 #pragma unroll
             for (int i = 0; i < 4; i++) {
-                vr[2 * i] = __uint_as_float(w[i] << 16);
-                vr[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+                const float x = (t < T && j0 + vc + 2 * i < d.dv) ? __bfloat162float(p[2 * i]) : 0.f;
+                const float y = (t < T && j0 + vc + 2 * i + 1 < d.dv) ? __bfloat162float(p[2 * i + 1]) : 0.f;
+                w[i] = pack_bf2(x, y);
             }
-        } else {
-#pragma unroll
-            for (int i = 0; i < 8; i++) vr[i] = (t < T && j0 + vc + i < d.dv) ? __bfloat162float(p[i]) : 0.f;
+            vr = make_uint4(w[0], w[1], w[2], w[3]);
         }
     };
-    stage_rows(kS, lk, k, d.ldk, d.dk, dkp, 0, T, wide, 256);
-    cp_async_commit();
+    auto put_v = [&](uint32_t s) {         // weighted by what is left of it at the end of its chunk
+        const uint32_t c = s / (kChunk / kStep), t = s * kStep + vt;
+        const float f = wt[t] * expf(la[c * kChunk + kChunk - 1] - la[t]);
+        const uint32_t w[4] = {vr.x, vr.y, vr.z, vr.w};
+        uint32_t p[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) p[i] = pack_bf2(bf_lo(w[i]) * f, bf_hi(w[i]) * f);
+        *reinterpret_cast<uint4*>(vS + (size_t)(s & 1) * kStep * LV + vt * LV + vc) = make_uint4(p[0], p[1], p[2], p[3]);
+    };
+    auto stage_k = [&](uint32_t s) {
+        if (s < ns) stage_rows<kStep>(kS + (size_t)(s % 3) * kStep * lk, lk, k, d.ldk, d.dk, dkp, s * kStep, T, wide);
+        cp_async_commit();
+    };
+    stage_k(0);
+    stage_k(1);
     load_v(0);
-    if (warp == 7) chunk_decays(d, h, 0, T, la[0], wt[0]);
+    for (uint32_t c = warp; c < nc; c += 8) chunk_decays(d, h, c * kChunk, T, la + c * kChunk, wt + c * kChunk);
+    float acc[4][2][4];                                               // blocks quarter, quarter + 4, ...: two tiles of 8 key rows
+    auto each = [&](auto f) {
+#pragma unroll
+        for (int b = 0; b < 4; b++)
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const uint32_t i = (quarter + 4 * b) * 16 + n * 8 + 2 * t4 + (e & 1), j = j0 + mt * 16 + g + 8 * (e >> 1);
+                    f(acc[b][n][e], i < d.dk && j < d.dv, (size_t)i * d.dv + j);
+                }
+    };
+    each([&](float& x, bool in, size_t at) { x = in && !fresh ? S[at] : 0.f; });
     __syncthreads();
-    for (uint32_t c = 0; c < nc; c++) {
-        const uint32_t b = c & 1;
-        const float total = la[b][kChunk - 1];
-        {
-            const float f = wt[b][vt] * expf(total - la[b][vt]);
-            uint4 u = make_uint4(pack_bf2(vr[0] * f, vr[1] * f), pack_bf2(vr[2] * f, vr[3] * f), pack_bf2(vr[4] * f, vr[5] * f), pack_bf2(vr[6] * f, vr[7] * f));
-            *reinterpret_cast<uint4*>(vS + (size_t)b * kChunk * LV + vt * LV + vc) = u;
-        }
-        if (c + 1 < nc) {
-            stage_rows(kS + (size_t)(b ^ 1) * kChunk * lk, lk, k, d.ldk, d.dk, dkp, (c + 1) * kChunk, T, wide, 256);
-            cp_async_commit();
-            load_v(c + 1);
-            if (warp == 7) chunk_decays(d, h, (c + 1) * kChunk, T, la[b ^ 1], wt[b ^ 1]);
-        }
-        // the state at the start of the chunk
-        __nv_bfloat16* hi = states + ((size_t)c * d.heads + h) * 2 * dkp * dvp;
-        __nv_bfloat16* lo = hi + (size_t)dkp * dvp;
-        const float e = expf(total);
+    put_v(0);
+    if (ns > 1) load_v(1);
+    for (uint32_t s = 0; s < ns; s++) {
+        if (s % (kChunk / kStep) == 0) {
+            // the state at the start of the chunk
+            const uint32_t c = s / (kChunk / kStep);
+            uint4* fr = states + state_fragments(c, d.heads, h, dkp, dvp) + (size_t)(j0 / 16 + mt) * nb * 64 + lane;
+            const float e = expf(la[c * kChunk + kChunk - 1]);
 #pragma unroll
-        for (int m = 0; m < 2; m++) {
-            const uint32_t i0 = (warp + 8 * m) * 16 + g;
-            if ((warp + 8 * m) * 16 >= dkp) break;
+            for (int blk = 0; blk < 4; blk++) {
+                const uint32_t kb = quarter + 4 * blk;
+                if (kb >= nb) break;
+                uint32_t hi[4], lo[4];
 #pragma unroll
-            for (int n = 0; n < 4; n++)
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    float &x = acc[m][n][2 * half], &y = acc[m][n][2 * half + 1];
-                    const size_t at = (size_t)(i0 + 8 * half) * dvp + j0 + n * 8 + 2 * t4;
-                    const __nv_bfloat16 hx = __float2bfloat16_rn(x), hy = __float2bfloat16_rn(y);
-                    *reinterpret_cast<__nv_bfloat162*>(hi + at) = __halves2bfloat162(hx, hy);
-                    *reinterpret_cast<uint32_t*>(lo + at) = pack_bf2(x - __bfloat162float(hx), y - __bfloat162float(hy));
+                for (int i = 0; i < 4; i++) {          // i: value column half (i >> 1), tile (i & 1)
+                    float &x = acc[blk][i & 1][(i >> 1) * 2], &y = acc[blk][i & 1][(i >> 1) * 2 + 1];
+                    hi[i] = pack_bf2(x, y);
+                    lo[i] = pack_bf2(x - bf_lo(hi[i]), y - bf_hi(hi[i]));
                     x *= e;
                     y *= e;
                 }
-        }
-        if (c + 1 < nc) cp_async_wait<1>();
-        else cp_async_wait<0>();
-        __syncthreads();
-        const uint32_t k_u = smem_u32(kS + (size_t)b * kChunk * lk), v_u = smem_u32(vS + (size_t)b * kChunk * LV);
-#pragma unroll
-        for (int kk = 0; kk < 4; kk++) {
-            uint32_t vb[2][4];
-#pragma unroll
-            for (int n = 0; n < 2; n++) ldsm_x4_trans(vb[n], v_u + ((kk * 16 + (lane & 15)) * LV + n * 16 + (lane >> 4) * 8) * 2);
-#pragma unroll
-            for (int m = 0; m < 2; m++) {
-                const uint32_t mt = (warp + 8 * m) * 16;
-                if (mt >= dkp) break;
-                uint32_t a[4];          // K^T: tiles (tokens 0-7 | 8-15) x (rows 0-7 | 8-15), transposed
-                ldsm_x4_trans(a, k_u + ((kk * 16 + (lane >> 4) * 8 + (lane & 7)) * lk + mt + ((lane >> 3) & 1) * 8) * 2);
-#pragma unroll
-                for (int n = 0; n < 4; n++) mma_bf16(acc[m][n], a, vb[n >> 1][(n & 1) * 2], vb[n >> 1][(n & 1) * 2 + 1]);
+                fr[kb * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                fr[kb * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
             }
         }
-        __syncthreads();
+        cp_async_wait<1>();
+        __syncthreads();          // step s has arrived for everyone, step s - 1 has been read by everyone
+        stage_k(s + 2);
+        const uint32_t k_u = smem_u32(kS + (size_t)(s % 3) * kStep * lk + (lane & 15) * lk + (lane >> 4) * 8);
+        // V^T: tiles (tokens 0-7 | 8-15) x (columns 0-7 | 8-15), transposed
+        const uint32_t v_u = smem_u32(vS + (size_t)(s & 1) * kStep * LV + ((lane >> 4) * 8 + (lane & 7)) * LV + mt * 16 + ((lane >> 3) & 1) * 8);
+        uint32_t a[kStep / 16][4];
+#pragma unroll
+        for (uint32_t kk = 0; kk < kStep / 16; kk++) ldsm_x4_trans(a[kk], v_u + kk * 16 * LV * 2);
+#pragma unroll
+        for (int blk = 0; blk < 4; blk++) {
+            const uint32_t kb = quarter + 4 * blk;
+            if (kb >= nb) break;
+#pragma unroll
+            for (uint32_t kk = 0; kk < kStep / 16; kk++) {
+                uint32_t bk[4];
+                ldsm_x4_trans(bk, k_u + (kk * 16 * lk + kb * 16) * 2);
+                mma_bf16(acc[blk][0], a[kk], bk[0], bk[1]);
+                mma_bf16(acc[blk][1], a[kk], bk[2], bk[3]);
+            }
+        }
+        if (s + 1 < ns) put_v(s + 1);
+        if (s + 2 < ns) load_v(s + 2);
     }
-#pragma unroll
-    for (int m = 0; m < 2; m++)
-#pragma unroll
-        for (int n = 0; n < 4; n++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const uint32_t i = (warp + 8 * m) * 16 + g + (e >> 1) * 8, j = j0 + n * 8 + 2 * t4 + (e & 1);
-                if (i < d.dk && j < d.dv) S[(size_t)i * d.dv + j] = acc[m][n][e];
-            }
+    each([&](float& x, bool in, size_t at) { if (in) S[at] = x; });
 }
 
-// grid (chunks, heads, dvp / 64), 4 warps of 16 tokens.
-__global__ void __launch_bounds__(128) chunk_out_kernel(const LinearRows d, const __nv_bfloat16* __restrict__ states, uint32_t dkp, uint32_t dvp,
-                                                         uint32_t T) {
+// grid (chunks, heads, dvp / 64), 8 warps of 16 tokens; KS blocks of 16 key rows (the rest of the last ones is zero).
+template <int KS>
+__global__ void __launch_bounds__(256) chunk_out_kernel(const LinearRows d, const uint4* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T) {
     extern __shared__ __align__(16) uint8_t smem[];
     constexpr uint32_t LV = 72;
-    const uint32_t lk = dkp + 8;
-    __nv_bfloat16* qS = reinterpret_cast<__nv_bfloat16*>(smem);       // [64][lk]
-    __nv_bfloat16* kS = qS + kChunk * lk;                             // [64][lk]
-    __nv_bfloat16* vS = kS + kChunk * lk;                             // [64][LV]
-    __nv_bfloat16* hS = vS + kChunk * LV;                             // [2][dkp][LV]
+    const uint32_t lk = dkp + 8, nb = dkp / 16;
+    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [kChunk][lk]: first the queries, then the keys
+    __nv_bfloat16* vS = kS + kChunk * lk;                             // [kChunk][LV]
+    uint4* fS = reinterpret_cast<uint4*>(vS + kChunk * LV);           // [4 column blocks][nb][2][32]: the starting state
     __shared__ float la[kChunk], wt[kChunk];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const uint32_t c = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 64, grp = h / (d.heads / d.groups), t0 = c * kChunk;
     const __nv_bfloat16 *q = (const __nv_bfloat16*)d.q + grp * d.dk, *k = (const __nv_bfloat16*)d.k + grp * d.dk,
                         *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
     const uint32_t nv = min(64u, d.dv - j0);
-    const bool wq = rows_aligned(q, d.ldq, d.dk), wk = rows_aligned(k, d.ldk, d.dk), wv = rows_aligned(v, d.ldv, nv);
-    stage_rows(qS, lk, q, d.ldq, d.dk, dkp, t0, T, wq, 128);
+    stage_rows<kChunk>(kS, lk, q, d.ldq, d.dk, dkp, t0, T, rows_aligned(q, d.ldq, d.dk));
+    cp_async_commit();
     {
-        const __nv_bfloat16* hi = states + ((size_t)c * d.heads + h) * 2 * dkp * dvp + j0;
-        for (uint32_t i = tid; i < 2 * dkp * 8; i += 128) cp_async16(smem_u32(hS + (i >> 3) * LV + (i & 7) * 8), hi + (size_t)(i >> 3) * dvp + (i & 7) * 8);
+        const uint4* fr = states + state_fragments(c, d.heads, h, dkp, dvp) + (size_t)(j0 / 16) * nb * 64;
+        for (uint32_t i = tid; i < 4 * nb * 64; i += 256) cp_async16(smem_u32(fS + i), fr + i);
     }
     cp_async_commit();
-    stage_rows(kS, lk, k, d.ldk, d.dk, dkp, t0, T, wk, 128);
-    stage_rows(vS, LV, v, d.ldv, nv, 64, t0, T, wv, 128);
-    cp_async_commit();
+    stage_rows<kChunk>(vS, LV, v, d.ldv, nv, 64, t0, T, rows_aligned(v, d.ldv, nv));
     if (warp == 0) chunk_decays(d, h, t0, T, la, wt);
     cp_async_wait<1>();
     __syncthreads();
+    // a scheduler's two warps: one with many earlier tokens in the chunk, one with few
+    const uint32_t rblk = warp < 4 ? warp : 11 - warp;
+    uint32_t qa[KS][4];
+    {
+        const uint32_t q_u = smem_u32(kS + (rblk * 16 + (lane & 15)) * lk + (lane >> 4) * 8);
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++) {
+            if ((uint32_t)ks < nb) ldsm_x4(qa[ks], q_u + ks * 32);
+            else qa[ks][0] = qa[ks][1] = qa[ks][2] = qa[ks][3] = 0;
+        }
+    }
     float o[8][4];
 #pragma unroll
     for (int n = 0; n < 8; n++) { o[n][0] = 0.f; o[n][1] = 0.f; o[n][2] = 0.f; o[n][3] = 0.f; }
-    const uint32_t q_u = smem_u32(qS + (warp * 16 + (lane & 15)) * lk + (lane >> 4) * 8);
-    const uint32_t h_u = smem_u32(hS + (lane & 15) * LV + (lane >> 4) * 8), lo_off = dkp * LV * 2;
-#pragma unroll 2
-    for (uint32_t ks = 0; ks < dkp / 16; ks++) {
-        uint32_t a[4];
-        ldsm_x4(a, q_u + ks * 32);
+    __syncthreads();              // everyone has its queries
+    stage_rows<kChunk>(kS, lk, k, d.ldk, d.dk, dkp, t0, T, rows_aligned(k, d.ldk, d.dk));
+    cp_async_commit();
+    cp_async_wait<1>();
+    __syncthreads();
+    const uint4* fr = fS + lane;
 #pragma unroll
-        for (int n = 0; n < 8; n += 2) {
-            uint32_t b[4], bl[4];
-            ldsm_x4_trans(b, h_u + (ks * 16 * LV + n * 8) * 2);
-            ldsm_x4_trans(bl, h_u + lo_off + (ks * 16 * LV + n * 8) * 2);
-            mma_bf16(o[n], a, b[0], b[1]);
-            mma_bf16(o[n + 1], a, b[2], b[3]);
-            mma_bf16(o[n], a, bl[0], bl[1]);
-            mma_bf16(o[n + 1], a, bl[2], bl[3]);
+    for (int ks = 0; ks < KS; ks++) {
+        if ((uint32_t)ks >= nb) break;
+        uint4 hi[4], lo[4];
+#pragma unroll
+        for (int n = 0; n < 4; n++) {
+            hi[n] = fr[((size_t)n * nb + ks) * 64];
+            lo[n] = fr[((size_t)n * nb + ks) * 64 + 32];
+        }
+#pragma unroll
+        for (int n = 0; n < 4; n++) {
+            mma_bf16(o[2 * n], qa[ks], hi[n].x, hi[n].y);
+            mma_bf16(o[2 * n + 1], qa[ks], hi[n].z, hi[n].w);
+            mma_bf16(o[2 * n], qa[ks], lo[n].x, lo[n].y);
+            mma_bf16(o[2 * n + 1], qa[ks], lo[n].z, lo[n].w);
         }
     }
-    const uint32_t ra = warp * 16 + g, rb = ra + 8;
+    const uint32_t ra = rblk * 16 + g, rb = ra + 8;
     const float la_a = la[ra], la_b = la[rb];
     {
         const float e_a = expf(la_a), e_b = expf(la_b);
@@ -416,15 +515,15 @@ __global__ void __launch_bounds__(128) chunk_out_kernel(const LinearRows d, cons
     // products within the chunk: 16 tokens at a time up to this warp's own
     const uint32_t k_u = smem_u32(kS + ((lane >> 4) * 8 + (lane & 7)) * lk + ((lane >> 3) & 1) * 8);
     const uint32_t v_u = smem_u32(vS + (lane & 15) * LV + (lane >> 4) * 8);
-    for (uint32_t kk = 0; kk <= warp; kk++) {
+    for (uint32_t kk = 0; kk <= rblk; kk++) {
         float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-        for (uint32_t ks = 0; ks < dkp / 16; ks++) {
-            uint32_t a[4], b[4];
-            ldsm_x4(a, q_u + ks * 32);
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++) {
+            if ((uint32_t)ks >= nb) break;
+            uint32_t b[4];
             ldsm_x4(b, k_u + (kk * 16 * lk + ks * 16) * 2);
-            mma_bf16(s0, a, b[0], b[1]);
-            mma_bf16(s1, a, b[2], b[3]);
+            mma_bf16(s0, qa[ks], b[0], b[1]);
+            mma_bf16(s1, qa[ks], b[2], b[3]);
         }
         auto weigh = [&](float s, uint32_t i, float la_i, uint32_t j) { return j <= i ? s * wt[j] * expf(la_i - la[j]) : 0.f; };
         const uint32_t ja = kk * 16 + 2 * t4;
@@ -498,6 +597,72 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(TA* __restrict__ a, uin
     }
 }
 
+// The same for bf16 rows of 16-byte pieces: a thread keeps its (at most NC) pieces in registers, only their sums of squares pass
+// through shared memory.
+template <bool BEFORE, int NC>
+__global__ void __launch_bounds__(256) gated_norm_vec_kernel(__nv_bfloat16* __restrict__ a, uint32_t lda, uint32_t n, uint32_t group,
+                                                              const __nv_bfloat16* __restrict__ gate, uint32_t ldg, const float* __restrict__ weight,
+                                                              float out_scale, float eps) {
+    extern __shared__ __align__(16) float sm[];
+    const uint32_t pieces = n / 8, per = group / 8, groups = n / group;
+    float *sums = sm, *fac = sm + pieces;
+    uint4* row = reinterpret_cast<uint4*>(a + (size_t)blockIdx.x * lda);
+    const uint4* gr = reinterpret_cast<const uint4*>(gate + (size_t)blockIdx.x * ldg);
+    uint4 av[NC], gv[NC];
+#pragma unroll
+    for (int c = 0; c < NC; c++) {
+        const uint32_t i = threadIdx.x + 256 * c;
+        if (i < pieces) {
+            av[c] = row[i];
+            gv[c] = gr[i];
+        }
+    }
+    float v[NC][8];
+#pragma unroll
+    for (int c = 0; c < NC; c++) {
+        const uint32_t i = threadIdx.x + 256 * c;
+        if (i >= pieces) break;
+        const uint32_t w[4] = {av[c].x, av[c].y, av[c].z, av[c].w}, z[4] = {gv[c].x, gv[c].y, gv[c].z, gv[c].w};
+        float sq = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+            v[c][e] = (e & 1) ? bf_hi(w[e / 2]) : bf_lo(w[e / 2]);
+            if (BEFORE) v[c][e] *= silu_for<__nv_bfloat16>((e & 1) ? bf_hi(z[e / 2]) : bf_lo(z[e / 2]));
+            sq = fmaf(v[c][e], v[c][e], sq);
+        }
+        sums[i] = sq;
+    }
+    __syncthreads();
+    const uint32_t wpg = groups >= 8 ? 1u : (groups >= 3 ? 2u : (groups == 2 ? 4u : 8u));
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = warp % wpg;
+    for (uint32_t g = warp / wpg; g < groups; g += 8 / wpg) {
+        float sq = 0.f;
+        for (uint32_t i = sub * 32 + lane; i < per; i += 32 * wpg) sq += sums[g * per + i];
+        sq = wsum(sq);
+        if (lane == 0) fac[g * wpg + sub] = sq;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < NC; c++) {
+        const uint32_t i = threadIdx.x + 256 * c;
+        if (i >= pieces) break;
+        const uint32_t g = i / per, z[4] = {gv[c].x, gv[c].y, gv[c].z, gv[c].w};
+        float sq = 0.f;
+        for (uint32_t k = 0; k < wpg; k++) sq += fac[g * wpg + k];
+        const float r = rsqrtf(sq / (float)group + eps);
+        if (BEFORE) {
+            const float4 w0 = *reinterpret_cast<const float4*>(weight + 8 * i), w1 = *reinterpret_cast<const float4*>(weight + 8 * i + 4);
+            const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+            for (int e = 0; e < 8; e++) v[c][e] *= r * w[e];
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; e++) v[c][e] *= r * silu_for<__nv_bfloat16>((e & 1) ? bf_hi(z[e / 2]) : bf_lo(z[e / 2])) * out_scale;
+        }
+        row[i] = make_uint4(pack_bf2(v[c][0], v[c][1]), pack_bf2(v[c][2], v[c][3]), pack_bf2(v[c][4], v[c][5]), pack_bf2(v[c][6], v[c][7]));
+    }
+}
+
 template <typename K>
 static int32_t allow_smem(runit_ctx* ctx, const char* name, K kern, size_t smem) {
     RUNIT_REQUIRE(ctx, smem <= (size_t)ctx->max_smem_optin - 2048, "%s: the layer's sizes do not fit shared memory", name);
@@ -509,23 +674,27 @@ static int32_t allow_smem(runit_ctx* ctx, const char* name, K kern, size_t smem)
 
 using namespace ls;
 
-int32_t ssm_step(runit_ctx* ctx, const Ssm& m, const float* proj, float* y, const int32_t* pos_ptr) {
+int32_t ssm_step(runit_ctx* ctx, const Ssm& m, const float* proj, float* y, float* squares, const int32_t* pos_ptr) {
     RUNIT_REQUIRE(ctx, m.state <= kMaxKeyDim, "ssm_step: bad sizes");
-    runit_launch_chain_smem(ctx, ssm_step_kernel, dim3(m.heads, (m.vdim + 31) / 32), dim3(256), (size_t)m.state * 8, m, proj, y, pos_ptr);
+    runit_launch_chain_smem(ctx, ssm_step_kernel, dim3(m.heads, (m.vdim + 31) / 32), dim3(256), (size_t)m.state * 8, m, proj, y, squares, pos_ptr);
     return runit_after_launch(ctx, "ssm_step");
 }
 
 int32_t ssm_conv_rows(runit_ctx* ctx, const Ssm& m, bool exact, const void* proj, uint32_t ld, void* xbc, uint32_t ld_out, float* dt, uint32_t T,
                       uint32_t start) {
     RUNIT_REQUIRE(ctx, m.taps >= 1 && m.taps <= kConvTok, "ssm_conv: %u taps (1 .. %u)", m.taps, kConvTok);
-    const dim3 grid((m.channels() + 255) / 256 + 1, (T + kConvTok - 1) / kConvTok);
+    const size_t es = exact ? 4 : 2;
+    const bool wide = m.channels() % 4 == 0 && m.inner() % 4 == 0 && ld % 4 == 0 && ld_out % 4 == 0 && runit_aligned(proj, 4 * es) && runit_aligned(xbc, 4 * es);
+    const uint32_t vec = wide ? 4 : 1, per = kConvThreads * vec;
+    const dim3 grid((m.channels() + per - 1) / per + 1, (T + kConvTok - 1) / kConvTok);
     auto go = [&](auto kern, auto* p, auto* o) -> int32_t {
-        kern<<<grid, 256, 0, ctx->stream>>>(m, p, ld, o, ld_out, dt, T, start);
+        kern<<<grid, kConvThreads, 0, ctx->stream>>>(m, p, ld, o, ld_out, dt, T, start);
         return runit_after_launch(ctx, "ssm_conv");
     };
-    if (exact) return m.taps == 4 ? go(ssm_conv_kernel<float, 4>, (const float*)proj, (float*)xbc) : go(ssm_conv_kernel<float, 0>, (const float*)proj, (float*)xbc);
-    if (m.taps == 4) return go(ssm_conv_kernel<__nv_bfloat16, 4>, (const __nv_bfloat16*)proj, (__nv_bfloat16*)xbc);
-    return go(ssm_conv_kernel<__nv_bfloat16, 0>, (const __nv_bfloat16*)proj, (__nv_bfloat16*)xbc);
+#define RUNIT_CONV(TA, TAPS) (wide ? go(ssm_conv_kernel<TA, TAPS, 4>, (const TA*)proj, (TA*)xbc) : go(ssm_conv_kernel<TA, TAPS, 1>, (const TA*)proj, (TA*)xbc))
+    if (exact) return m.taps == 4 ? RUNIT_CONV(float, 4) : RUNIT_CONV(float, 0);
+    return m.taps == 4 ? RUNIT_CONV(__nv_bfloat16, 4) : RUNIT_CONV(__nv_bfloat16, 0);
+#undef RUNIT_CONV
 }
 
 static bool chunk_sizes(uint32_t dk) { return ((dk + 15) & ~15u) <= 256; }
@@ -539,13 +708,16 @@ int32_t linear_rows(runit_ctx* ctx, const LinearRows& d, bool exact, void* chunk
     int32_t st;
     if (!exact && T >= 16 && chunk_states && chunk_sizes(d.dk)) {
         const uint32_t dkp = pad16(d.dk), dvp = pad64(d.dv), nc = (T + kChunk - 1) / kChunk;
-        const size_t sa = (size_t)2 * kChunk * (dkp + 8 + 40) * 2, sb = ((size_t)2 * kChunk * (dkp + 8) + kChunk * 72 + (size_t)2 * dkp * 72) * 2;
+        const size_t sa = chunk_state_smem(dkp, nc), sb = (size_t)kChunk * (dkp + 8 + 72) * 2 + (size_t)dkp * 64 * 4;
         if ((st = allow_smem(ctx, "chunk_state", chunk_state_kernel, sa)) != RUNIT_OK) return st;
-        chunk_state_kernel<<<dim3(d.heads, dvp / 32), 256, sa, ctx->stream>>>(d, (__nv_bfloat16*)chunk_states, dkp, dvp, T, start == 0);
+        chunk_state_kernel<<<dim3(d.heads, dvp / 32), 256, sa, ctx->stream>>>(d, (uint4*)chunk_states, dkp, dvp, T, start == 0);
         if ((st = runit_after_launch(ctx, "chunk_state")) != RUNIT_OK) return st;
-        if ((st = allow_smem(ctx, "chunk_out", chunk_out_kernel, sb)) != RUNIT_OK) return st;
-        chunk_out_kernel<<<dim3(nc, d.heads, dvp / 64), 128, sb, ctx->stream>>>(d, (const __nv_bfloat16*)chunk_states, dkp, dvp, T);
-        return runit_after_launch(ctx, "chunk_out");
+        auto go = [&](auto kern) -> int32_t {
+            if ((st = allow_smem(ctx, "chunk_out", kern, sb)) != RUNIT_OK) return st;
+            kern<<<dim3(nc, d.heads, dvp / 64), 256, sb, ctx->stream>>>(d, (const uint4*)chunk_states, dkp, dvp, T);
+            return runit_after_launch(ctx, "chunk_out");
+        };
+        return dkp <= 64 ? go(chunk_out_kernel<4>) : (dkp <= 128 ? go(chunk_out_kernel<8>) : go(chunk_out_kernel<16>));
     }
     const dim3 grid(d.heads, (d.dv + 31) / 32);
 #define RUNIT_SCAN(NR)                                                                                            \
@@ -571,6 +743,16 @@ int32_t gated_norm_rows(runit_ctx* ctx, bool exact, void* a, uint32_t lda, uint3
         kern<<<T, 256, smem, ctx->stream>>>(p, lda, n, group, g, ldg, weight, out_scale, eps);
         return runit_after_launch(ctx, "gated_norm");
     };
+    if (!exact && n <= 8192 && group % 8 == 0 && lda % 8 == 0 && ldg % 8 == 0 && runit_aligned(a, 16) && runit_aligned(gate, 16) && runit_aligned(weight, 16)) {
+        const size_t small = ((size_t)n / 8 + n / group + 8) * 4;
+        auto vec = [&](auto kern) -> int32_t {
+            kern<<<T, 256, small, ctx->stream>>>((__nv_bfloat16*)a, lda, n, group, (const __nv_bfloat16*)gate, ldg, weight, out_scale, eps);
+            return runit_after_launch(ctx, "gated_norm");
+        };
+        if (n <= 2048) return before ? vec(gated_norm_vec_kernel<true, 1>) : vec(gated_norm_vec_kernel<false, 1>);
+        if (n <= 4096) return before ? vec(gated_norm_vec_kernel<true, 2>) : vec(gated_norm_vec_kernel<false, 2>);
+        return before ? vec(gated_norm_vec_kernel<true, 4>) : vec(gated_norm_vec_kernel<false, 4>);
+    }
     if (exact) return before ? go(gated_norm_kernel<float, true>, (float*)a, (const float*)gate) : go(gated_norm_kernel<float, false>, (float*)a, (const float*)gate);
     return before ? go(gated_norm_kernel<__nv_bfloat16, true>, (__nv_bfloat16*)a, (const __nv_bfloat16*)gate)
                   : go(gated_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)a, (const __nv_bfloat16*)gate);
@@ -594,13 +776,13 @@ int32_t ssm_of(runit_ctx* ctx, const char* who, const runit_ssm_cfg* c, Ssm* m) 
 
 extern "C" {
 
-int32_t runit_ssm_step(runit_ctx_t* ctx, const runit_ssm_cfg* cfg, const void* proj, void* y, const void* pos) {
+int32_t runit_ssm_step(runit_ctx_t* ctx, const runit_ssm_cfg* cfg, const void* proj, void* y, void* squares, const void* pos) {
     if (!ctx) return RUNIT_ERR_BAD_ARG;
     Ssm m;
     int32_t st = ssm_of(ctx, "ssm_step", cfg, &m);
     if (st != RUNIT_OK) return st;
-    RUNIT_REQUIRE(ctx, proj && y && pos, "ssm_step: null argument");
-    return ssm_step(ctx, m, (const float*)proj, (float*)y, (const int32_t*)pos);
+    RUNIT_REQUIRE(ctx, proj && y && squares && pos, "ssm_step: null argument");
+    return ssm_step(ctx, m, (const float*)proj, (float*)y, (float*)squares, (const int32_t*)pos);
 }
 
 int32_t runit_ssm_conv_rows(runit_ctx_t* ctx, const runit_ssm_cfg* cfg, int32_t f32, const void* proj, uint32_t ld, void* xbc, uint32_t ldx, void* dt,

@@ -47,6 +47,12 @@ __device__ __forceinline__ float state_step(StateRows& st, float* S, uint32_t dk
     return o;
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+// where the result is rounded to bf16 anyway (rows of a portion in the operand type TA)
+template <typename TA>
+__device__ __forceinline__ float silu_for(float x) {
+    if constexpr (sizeof(TA) == 2) return __fdividef(x, 1.0f + __expf(-x));
+    else return silu(x);
+}
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }

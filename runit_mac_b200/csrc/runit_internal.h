@@ -30,6 +30,7 @@ struct runit_tuning {
     int32_t imma_fold = 0;           // batched 4-bit GEMV: 1 = activation pre-pass inside the GEMV launch where the grid allows (measured slower:
                                      // 950 against 1331 GB/s over the 7B set at batch 8), 0 = a launch of its own
     int32_t ep_fused_exchange = 0;   // expert-parallel decoder: 1 = exchange inside the GEMVs (no launches of its own; measured slower)
+    int32_t gemv_pro_ctas = 0;    // bf16 GEMV with a prologue of several vectors: CTAs per SM at most (0 = default)
     int32_t router_variant = 0;   // batched f32 router: 0 = by size, 1 = one warp per expert, 2 = tiled GEMM, 3 = GEMM with K split over the warps of a CTA (tests force each)
 };
 

@@ -285,16 +285,16 @@ _TWINS = [
     ("latent_value", "no twin: (LatentCfg ref, part_o, part_ml, nsplit, w_uv, out, T)"),
     ("latent_rows", "no twin: (LatentCfg ref, cache_f32, qkv, ldq, kv_norm or None, freq, cache, T, start)"),
     ("latent_prefill_attention", "no twin: (LatentCfg ref, q, ldq, kv, ldkv, cache, out, ldo, T, start)"),
-    ("heads_step", "no twin: (HeadsCfg ref or None, RetentionCfg ref or None, cache_f32, proj, ao, factor, part, tickets, nsplit, pos)"),
+    ("heads_step", "no twin: (HeadsCfg ref or None, RetentionCfg ref or None, cache_f32, proj, ao, factor, squares, part, tickets, nsplit, pos)"),
     ("heads_rows", "no twin: (HeadsCfg ref or None, RetentionCfg ref or None, cache_f32, proj, ld, T, start)"),
     ("head_attention_rows", "no twin: (HeadsCfg ref, cache_f32, proj, ld, out, ldo, T, start, part, part_floats, tickets)"),
-    ("ssm_step", "no twin: (SsmCfg ref, proj, y, pos)"),
+    ("ssm_step", "no twin: (SsmCfg ref, proj, y, squares, pos)"),
     ("ssm_conv_rows", "no twin: (SsmCfg ref, f32, proj, ld, xbc, ldx, dt, T, start)"),
     ("linear_rows", "no twin: (LinearCfg ref, f32, scratch or None, T, start)"),
     ("gated_norm_rows", "no twin: (f32, a, lda, n, group, gate, ldg, before, weight or None, out_scale, eps, T)"),
     ("add_norm_rows", "no twin: (x, y or None, gain, eps, out_gain or None, out or None, out_f32, T, width)"),
     ("gemv_bf16_residual_f32", "no twin: (weight, x, y or None, y_gain, gain or None, x_out or None, out, eps, cap, relu2, m, k)"),
-    ("gemv_bf16_groups_f32", "no twin: (weight, x, factor, out, eps, plain, group, m, k)"),
+    ("gemv_bf16_groups_f32", "no twin: (weight, x, factor, squares or None, squares_n, out, eps, plain, group, m, k)"),
     ("fill_weights", "no twin: (fmt, dst, n_blocks, seed, sigma)"),
     ("fill_weights_q4k_zero_mean", "no twin: (dst, n_blocks, seed, sigma), Q4_K blocks with zero-mean weights"),
     ("fill_normal_f32", "no twin: (dst, n, seed, sigma)"),
