@@ -113,7 +113,8 @@ def causal_conv(x, w, b):
     y = np.zeros_like(x)
     for j in range(taps):
         back = taps - 1 - j
-        y[back:] += w[:, j] * x[:len(x) - back]
+        if back < len(x):
+            y[back:] += w[:, j] * x[:len(x) - back]
     return y + b
 
 
