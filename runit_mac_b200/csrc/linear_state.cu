@@ -85,6 +85,7 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const Ssm m, const float*
 // step sizes.  Only the first token block reads the ring, and each of its threads rewrites it for its channels afterwards.
 // TAPS > 0: the window stays in registers.
 constexpr uint32_t kConvTok = 32, kConvThreads = 128;
+static_assert(kConvTok == 32, "four groups of eight tokens");
 template <int VEC, typename TA>
 __device__ __forceinline__ void load_vec(const TA* p, float (&v)[VEC]) {
     if constexpr (VEC == 1) {
@@ -107,6 +108,21 @@ __device__ __forceinline__ void store_vec(TA* p, const float (&v)[VEC]) {
         *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
     } else {
         *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+}
+// One token of the window kernel: the window moves on by `in`, y = silu(taps . window + b).
+template <typename TA, int TAPS, int VEC>
+__device__ __forceinline__ void conv_token(float (&win)[TAPS][VEC], const float (&wr)[TAPS][VEC], const float (&b)[VEC], const float (&in)[VEC],
+                                           float (&y)[VEC]) {
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; j++) win[j][e] = win[j + 1][e];
+        win[TAPS - 1][e] = in[e];
+        float s = b[e];
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) s = fmaf(wr[j][e], win[j][e], s);
+        y[e] = silu_for<TA>(s);
     }
 }
 template <typename TA, int TAPS, int VEC>
@@ -132,6 +148,16 @@ __global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const Ssm m, con
         }
     };
     if constexpr (TAPS > 0) {
+        constexpr uint32_t B = 8;                            // tokens requested together
+        constexpr bool ASYNC = sizeof(TA) == 2 && VEC == 4;  // all of the block's tokens on their way at once, through shared memory
+        extern __shared__ __align__(16) uint2 own[];         // [kConvTok][kConvThreads]: a thread reads what it has requested itself
+        if constexpr (ASYNC) {
+#pragma unroll
+            for (uint32_t i = 0; i < kConvTok; i++) {
+                if (t0 + i < t1) cp_async8(smem_u32(own + i * kConvThreads + threadIdx.x), x + (size_t)(t0 + i) * ld);
+                if (i % B == B - 1) cp_async_commit();
+            }
+        }
         float win[TAPS][VEC], wr[TAPS][VEC];
 #pragma unroll
         for (int j = 0; j < TAPS; j++)
@@ -139,27 +165,35 @@ __global__ void __launch_bounds__(kConvThreads) ssm_conv_kernel(const Ssm m, con
             for (int e = 0; e < VEC; e++) wr[j][e] = m.conv_w[(size_t)(c + e) * TAPS + j];
 #pragma unroll
         for (int j = 0; j + 1 < TAPS; j++) input((int32_t)t0 - (TAPS - 1 - j), win[j + 1]);
-        constexpr uint32_t B = 8;                            // tokens requested together
-        for (uint32_t tb = t0; tb < t1; tb += B) {
-            float in[B][VEC];
+        if constexpr (ASYNC) {
 #pragma unroll
-            for (uint32_t i = 0; i < B; i++)
-                if (tb + i < t1) load_vec<VEC>(x + (size_t)(tb + i) * ld, in[i]);
+            for (uint32_t q = 0; q < kConvTok / B; q++) {
+                if (q == 0) cp_async_wait<3>();
+                else if (q == 1) cp_async_wait<2>();
+                else if (q == 2) cp_async_wait<1>();
+                else cp_async_wait<0>();
 #pragma unroll
-            for (uint32_t i = 0; i < B; i++) {
-                if (tb + i >= t1) break;
-                float y[VEC];
-#pragma unroll
-                for (int e = 0; e < VEC; e++) {
-#pragma unroll
-                    for (int j = 0; j + 1 < TAPS; j++) win[j][e] = win[j + 1][e];
-                    win[TAPS - 1][e] = in[i][e];
-                    float s = b[e];
-#pragma unroll
-                    for (int j = 0; j < TAPS; j++) s = fmaf(wr[j][e], win[j][e], s);
-                    y[e] = silu_for<TA>(s);
+                for (uint32_t i = q * B; i < q * B + B; i++) {
+                    if (t0 + i >= t1) break;
+                    float in[VEC], y[VEC];
+                    load_vec<VEC>(reinterpret_cast<const TA*>(own + i * kConvThreads + threadIdx.x), in);
+                    conv_token<TA, TAPS, VEC>(win, wr, b, in, y);
+                    store_vec<VEC>(out + (size_t)(t0 + i) * ld_out + c, y);
                 }
-                store_vec<VEC>(out + (size_t)(tb + i) * ld_out + c, y);
+            }
+        } else {
+            for (uint32_t tb = t0; tb < t1; tb += B) {
+                float in[B][VEC];
+#pragma unroll
+                for (uint32_t i = 0; i < B; i++)
+                    if (tb + i < t1) load_vec<VEC>(x + (size_t)(tb + i) * ld, in[i]);
+#pragma unroll
+                for (uint32_t i = 0; i < B; i++) {
+                    if (tb + i >= t1) break;
+                    float y[VEC];
+                    conv_token<TA, TAPS, VEC>(win, wr, b, in[i], y);
+                    store_vec<VEC>(out + (size_t)(tb + i) * ld_out + c, y);
+                }
             }
         }
     } else {
@@ -258,37 +292,45 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                  : "r"(addr));
 }
-// Rows t0 .. t0 + ROWS - 1 of a bf16 matrix (n of its columns) into shared rows of `pitch` elements, `cols` of them filled; rows
+// Rows t0 .. t0 + ROWS - 1 of a bf16 matrix (n of its columns) into shared rows of COLS + 8 elements; rows
 // from T on and columns from n on become zero.  Asynchronous where the rows are 16-byte aligned (wide).  256 threads.
-template <int ROWS>
-__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, uint32_t pitch, const __nv_bfloat16* src, uint32_t ld, uint32_t n, uint32_t cols,
-                                            uint32_t t0, uint32_t T, bool wide) {
-    const uint32_t cpr = cols / 8;
-    uint32_t r = threadIdx.x / cpr, c = threadIdx.x - r * cpr;
-    const uint32_t dr = 256 / cpr, dc = 256 - dr * cpr;
-    for (; r < (uint32_t)ROWS;) {
-        __nv_bfloat16* p = dst + r * pitch + c * 8;
-        const __nv_bfloat16* s = src + (size_t)(t0 + r) * ld + c * 8;
-        if (t0 + r >= T || c * 8 >= n) {
-            *reinterpret_cast<uint4*>(p) = make_uint4(0, 0, 0, 0);
+template <int ROWS, int COLS>
+__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat16* src, uint32_t ld, uint32_t n, uint32_t t0, uint32_t T, bool wide) {
+    constexpr uint32_t CPR = COLS / 8, STEP = 256 / CPR, PITCH = COLS + 8;
+    static_assert(256 % CPR == 0 && ROWS % STEP == 0, "whole passes");
+    const uint32_t r0 = threadIdx.x / CPR, c = (threadIdx.x % CPR) * 8;
+    const __nv_bfloat16* s = src + (size_t)(t0 + r0) * ld + c;
+    __nv_bfloat16* p = dst + r0 * PITCH + c;
+    const uint32_t rows = t0 + r0 < T ? T - t0 - r0 : 0;       // rows left from this thread's first one
+    const bool in = c < n;
+#pragma unroll
+    for (uint32_t r = 0; r < (uint32_t)ROWS; r += STEP) {
+        if (!in || r >= rows) {
+            *reinterpret_cast<uint4*>(p + r * PITCH) = make_uint4(0, 0, 0, 0);
         } else if (wide) {
-            cp_async16(smem_u32(p), s);
+            cp_async16(smem_u32(p + r * PITCH), s);
         } else {
-            for (uint32_t e = 0; e < 8; e++) p[e] = c * 8 + e < n ? s[e] : __float2bfloat16_rn(0.f);
+            for (uint32_t e = 0; e < 8; e++) p[r * PITCH + e] = c + e < n ? s[e] : __float2bfloat16_rn(0.f);
         }
-        r += dr;
-        c += dc;
-        if (c >= cpr) { c -= cpr; r++; }
+        s += (size_t)STEP * ld;
     }
 }
+// 2^x (the argument is not positive)
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+constexpr float kLog2e = 1.44269504088896341f;
 __device__ __forceinline__ bool rows_aligned(const void* p, uint32_t ld, uint32_t n) {
     return (reinterpret_cast<uintptr_t>(p) & 15u) == 0 && (ld & 7u) == 0 && (n & 7u) == 0;
 }
-// One warp: la[t] = sum of the log decays of tokens 0 .. t of the chunk (nothing for the tokens past the end), w[t] = step size.
+// One warp: la[t] = sum of the binary logarithms of the decays of tokens 0 .. t of the chunk (nothing for the tokens past the end),
+// w[t] = step size.
 __device__ __forceinline__ void chunk_decays(const LinearRows& d, uint32_t h, uint32_t t0, uint32_t T, float* la, float* w) {
     constexpr int P = kChunk / 32;
     const uint32_t lane = threadIdx.x & 31;
-    const float ld = d.log_decay[h];
+    const float ld = d.log_decay[h] * kLog2e;
     float x[P];
 #pragma unroll
     for (int i = 0; i < P; i++) {
@@ -317,67 +359,75 @@ __device__ __forceinline__ size_t state_fragments(uint32_t chunk, uint32_t heads
 
 // The state is carried as its transpose, 16 value columns x 8 key rows per accumulator tile, which is the layout of those
 // fragments.  grid (heads, dvp / 32), 8 warps: warp = 16 of the CTA's 32 value columns x every fourth block of 16 key rows.  Keys
-// arrive in steps of 64 tokens, three steps deep; the values are weighted on their way into shared memory.  The decays of all
-// chunks are summed up before the walk.
-constexpr uint32_t kStep = 64;
-static size_t chunk_state_smem(uint32_t dkp, uint32_t nc) {
-    return (size_t)3 * kStep * (dkp + 8) * 2 + (size_t)2 * kStep * 40 * 2 + (size_t)nc * kChunk * 8;
-}
-__global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, uint4* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T,
-                                                           uint32_t fresh) {
+// arrive in steps of 64 or 128 tokens, three steps deep; the values are weighted on their way into shared memory.  The decays of all
+// chunks are summed up before the walk.  DK >= dk: the rest is zero.
+template <int DK>
+struct StateCfg {
+    static constexpr uint32_t step = DK <= 128 ? 128 : 64, lv = 40;
+    static size_t smem(uint32_t nc) { return (size_t)3 * step * (DK + 8) * 2 + (size_t)2 * step * lv * 2 + (size_t)nc * kChunk * 8; }
+};
+template <int DK>
+__global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, uint4* __restrict__ states, uint32_t dvp, uint32_t T, uint32_t fresh) {
     extern __shared__ __align__(16) uint8_t smem[];
-    constexpr uint32_t LV = 40;
-    const uint32_t lk = dkp + 8, nb = dkp / 16, nc = (T + kChunk - 1) / kChunk, ns = (T + kStep - 1) / kStep;
-    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [3][kStep][lk]
-    __nv_bfloat16* vS = kS + 3 * kStep * lk;                          // [2][kStep][LV]
-    float* la = reinterpret_cast<float*>(vS + 2 * kStep * LV);        // [nc][kChunk]
+    constexpr uint32_t STEP = StateCfg<DK>::step, LV = StateCfg<DK>::lv, LK = DK + 8, NB = DK / 16, NBW = NB / 4, VP = STEP / 64, PER = kChunk / STEP;
+    const uint32_t nc = (T + kChunk - 1) / kChunk, ns = (T + STEP - 1) / STEP;
+    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [3][STEP][LK]
+    __nv_bfloat16* vS = kS + 3 * STEP * LK;                           // [2][STEP][LV]
+    float* la = reinterpret_cast<float*>(vS + 2 * STEP * LV);         // [nc][kChunk]
     float* wt = la + nc * kChunk;                                     // [nc][kChunk]
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mt = warp & 1, quarter = warp >> 1;
     const uint32_t h = blockIdx.x, j0 = blockIdx.y * 32, grp = h / (d.heads / d.groups);
     const __nv_bfloat16 *k = (const __nv_bfloat16*)d.k + grp * d.dk, *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
     float* S = d.state + (size_t)h * d.dk * d.dv;
     const bool wide = rows_aligned(k, d.ldk, d.dk);
-    // value rows: thread -> token tid / 4 of a step, columns 8 * (tid % 4) ..
+    // value rows: thread -> tokens tid / 4 (+ 64) of a step, columns 8 * (tid % 4) ..
     const uint32_t vt = tid >> 2, vc = (tid & 3) * 8;
     const bool vwide = rows_aligned(v, d.ldv, 8) && j0 + vc + 8 <= d.dv;
-    uint4 vr;
+    uint4 vr[VP];
     auto load_v = [&](uint32_t s) {
-        const uint32_t t = s * kStep + vt;
-        const __nv_bfloat16* p = v + (size_t)t * d.ldv + vc;
-        if (t < T && vwide) {
-            vr = *reinterpret_cast<const uint4*>(p);
-        } else {
-            uint32_t w[4];
 #pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const float x = (t < T && j0 + vc + 2 * i < d.dv) ? __bfloat162float(p[2 * i]) : 0.f;
-                const float y = (t < T && j0 + vc + 2 * i + 1 < d.dv) ? __bfloat162float(p[2 * i + 1]) : 0.f;
-                w[i] = pack_bf2(x, y);
+        for (uint32_t i = 0; i < VP; i++) {
+            const uint32_t t = s * STEP + vt + 64 * i;
+            const __nv_bfloat16* p = v + (size_t)t * d.ldv + vc;
+            if (t < T && vwide) {
+                vr[i] = *reinterpret_cast<const uint4*>(p);
+            } else {
+                uint32_t w[4];
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const float x = (t < T && j0 + vc + 2 * e < d.dv) ? __bfloat162float(p[2 * e]) : 0.f;
+                    const float y = (t < T && j0 + vc + 2 * e + 1 < d.dv) ? __bfloat162float(p[2 * e + 1]) : 0.f;
+                    w[e] = pack_bf2(x, y);
+                }
+                vr[i] = make_uint4(w[0], w[1], w[2], w[3]);
             }
-            vr = make_uint4(w[0], w[1], w[2], w[3]);
         }
     };
     auto put_v = [&](uint32_t s) {         // weighted by what is left of it at the end of its chunk
-        const uint32_t c = s / (kChunk / kStep), t = s * kStep + vt;
-        const float f = wt[t] * expf(la[c * kChunk + kChunk - 1] - la[t]);
-        const uint32_t w[4] = {vr.x, vr.y, vr.z, vr.w};
-        uint32_t p[4];
+        const float end = la[s / PER * kChunk + kChunk - 1];
 #pragma unroll
-        for (int i = 0; i < 4; i++) p[i] = pack_bf2(bf_lo(w[i]) * f, bf_hi(w[i]) * f);
-        *reinterpret_cast<uint4*>(vS + (size_t)(s & 1) * kStep * LV + vt * LV + vc) = make_uint4(p[0], p[1], p[2], p[3]);
+        for (uint32_t i = 0; i < VP; i++) {
+            const uint32_t t = s * STEP + vt + 64 * i;
+            const float f = wt[t] * ex2(end - la[t]);
+            const uint32_t w[4] = {vr[i].x, vr[i].y, vr[i].z, vr[i].w};
+            uint32_t p[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) p[e] = pack_bf2(bf_lo(w[e]) * f, bf_hi(w[e]) * f);
+            *reinterpret_cast<uint4*>(vS + (size_t)(s & 1) * STEP * LV + (vt + 64 * i) * LV + vc) = make_uint4(p[0], p[1], p[2], p[3]);
+        }
     };
-    auto stage_k = [&](uint32_t s) {
-        if (s < ns) stage_rows<kStep>(kS + (size_t)(s % 3) * kStep * lk, lk, k, d.ldk, d.dk, dkp, s * kStep, T, wide);
+    auto stage_k = [&](uint32_t s, uint32_t buf) {
+        if (s < ns) stage_rows<STEP, DK>(kS + buf * STEP * LK, k, d.ldk, d.dk, s * STEP, T, wide);
         cp_async_commit();
     };
-    stage_k(0);
-    stage_k(1);
+    stage_k(0, 0);
+    stage_k(1, 1);
     load_v(0);
     for (uint32_t c = warp; c < nc; c += 8) chunk_decays(d, h, c * kChunk, T, la + c * kChunk, wt + c * kChunk);
-    float acc[4][2][4];                                               // blocks quarter, quarter + 4, ...: two tiles of 8 key rows
+    float acc[NBW][2][4];                                             // blocks quarter, quarter + 4, ...: two tiles of 8 key rows
     auto each = [&](auto f) {
 #pragma unroll
-        for (int b = 0; b < 4; b++)
+        for (uint32_t b = 0; b < NBW; b++)
 #pragma unroll
             for (int n = 0; n < 2; n++)
 #pragma unroll
@@ -390,147 +440,149 @@ __global__ void __launch_bounds__(256) chunk_state_kernel(const LinearRows d, ui
     __syncthreads();
     put_v(0);
     if (ns > 1) load_v(1);
+    const uint32_t k_u = smem_u32(kS + (lane & 15) * LK + (lane >> 4) * 8) + quarter * 32;
+    // V^T: tiles (tokens 0-7 | 8-15) x (columns 0-7 | 8-15), transposed
+    const uint32_t v_u = smem_u32(vS + ((lane >> 4) * 8 + (lane & 7)) * LV + mt * 16 + ((lane >> 3) & 1) * 8);
+    uint4* fr = states + state_fragments(0, d.heads, h, DK, dvp) + (size_t)(j0 / 16 + mt) * NB * 64 + quarter * 64 + lane;
+    const size_t fr_step = state_fragments(1, d.heads, 0, DK, dvp);
+    uint32_t buf = 0;
     for (uint32_t s = 0; s < ns; s++) {
-        if (s % (kChunk / kStep) == 0) {
+        if (s % PER == 0) {
             // the state at the start of the chunk
-            const uint32_t c = s / (kChunk / kStep);
-            uint4* fr = states + state_fragments(c, d.heads, h, dkp, dvp) + (size_t)(j0 / 16 + mt) * nb * 64 + lane;
-            const float e = expf(la[c * kChunk + kChunk - 1]);
+            const float e = ex2(la[s / PER * kChunk + kChunk - 1]);
 #pragma unroll
-            for (int blk = 0; blk < 4; blk++) {
-                const uint32_t kb = quarter + 4 * blk;
-                if (kb >= nb) break;
+            for (uint32_t b = 0; b < NBW; b++) {
                 uint32_t hi[4], lo[4];
 #pragma unroll
                 for (int i = 0; i < 4; i++) {          // i: value column half (i >> 1), tile (i & 1)
-                    float &x = acc[blk][i & 1][(i >> 1) * 2], &y = acc[blk][i & 1][(i >> 1) * 2 + 1];
+                    float &x = acc[b][i & 1][(i >> 1) * 2], &y = acc[b][i & 1][(i >> 1) * 2 + 1];
                     hi[i] = pack_bf2(x, y);
                     lo[i] = pack_bf2(x - bf_lo(hi[i]), y - bf_hi(hi[i]));
                     x *= e;
                     y *= e;
                 }
-                fr[kb * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                fr[kb * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                fr[b * 4 * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                fr[b * 4 * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
             }
+            fr += fr_step;
         }
         cp_async_wait<1>();
         __syncthreads();          // step s has arrived for everyone, step s - 1 has been read by everyone
-        stage_k(s + 2);
-        const uint32_t k_u = smem_u32(kS + (size_t)(s % 3) * kStep * lk + (lane & 15) * lk + (lane >> 4) * 8);
-        // V^T: tiles (tokens 0-7 | 8-15) x (columns 0-7 | 8-15), transposed
-        const uint32_t v_u = smem_u32(vS + (size_t)(s & 1) * kStep * LV + ((lane >> 4) * 8 + (lane & 7)) * LV + mt * 16 + ((lane >> 3) & 1) * 8);
-        uint32_t a[kStep / 16][4];
+        stage_k(s + 2, buf == 0 ? 2 : buf - 1);
+        const uint32_t kb_u = k_u + buf * STEP * LK * 2, vb_u = v_u + (s & 1) * STEP * LV * 2;
 #pragma unroll
-        for (uint32_t kk = 0; kk < kStep / 16; kk++) ldsm_x4_trans(a[kk], v_u + kk * 16 * LV * 2);
+        for (uint32_t kk = 0; kk < STEP / 16; kk++) {
+            uint32_t a[4];
+            ldsm_x4_trans(a, vb_u + kk * 16 * LV * 2);
 #pragma unroll
-        for (int blk = 0; blk < 4; blk++) {
-            const uint32_t kb = quarter + 4 * blk;
-            if (kb >= nb) break;
-#pragma unroll
-            for (uint32_t kk = 0; kk < kStep / 16; kk++) {
+            for (uint32_t b = 0; b < NBW; b++) {
                 uint32_t bk[4];
-                ldsm_x4_trans(bk, k_u + (kk * 16 * lk + kb * 16) * 2);
-                mma_bf16(acc[blk][0], a[kk], bk[0], bk[1]);
-                mma_bf16(acc[blk][1], a[kk], bk[2], bk[3]);
+                ldsm_x4_trans(bk, kb_u + (kk * 16 * LK + b * 64) * 2);
+                mma_bf16(acc[b][0], a, bk[0], bk[1]);
+                mma_bf16(acc[b][1], a, bk[2], bk[3]);
             }
         }
         if (s + 1 < ns) put_v(s + 1);
         if (s + 2 < ns) load_v(s + 2);
+        buf = buf == 2 ? 0 : buf + 1;
     }
     each([&](float& x, bool in, size_t at) { if (in) S[at] = x; });
 }
 
-// grid (chunks, heads, dvp / 64), 8 warps of 16 tokens; KS blocks of 16 key rows (the rest of the last ones is zero).
-template <int KS>
-__global__ void __launch_bounds__(256) chunk_out_kernel(const LinearRows d, const uint4* __restrict__ states, uint32_t dkp, uint32_t dvp, uint32_t T) {
+// grid (chunks, heads, dvp / 64), 8 warps of 16 tokens.  DK >= dk: the rest is zero.
+template <int DK>
+__global__ void __launch_bounds__(256, DK <= 128 ? 2 : 1) chunk_out_kernel(const LinearRows d, const uint4* __restrict__ states, uint32_t dvp, uint32_t T) {
     extern __shared__ __align__(16) uint8_t smem[];
-    constexpr uint32_t LV = 72;
-    const uint32_t lk = dkp + 8, nb = dkp / 16;
-    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [kChunk][lk]: first the queries, then the keys
-    __nv_bfloat16* vS = kS + kChunk * lk;                             // [kChunk][LV]
-    uint4* fS = reinterpret_cast<uint4*>(vS + kChunk * LV);           // [4 column blocks][nb][2][32]: the starting state
-    __shared__ float la[kChunk], wt[kChunk];
+    constexpr uint32_t LV = 72, LK = DK + 8, NB = DK / 16;
+    __nv_bfloat16* kS = reinterpret_cast<__nv_bfloat16*>(smem);       // [kChunk][LK]: first the queries, then the keys
+    __nv_bfloat16* vS = kS + kChunk * LK;                             // [kChunk][LV]
+    uint4* fS = reinterpret_cast<uint4*>(vS + kChunk * LV);           // [4 column blocks][NB][2][32]: the starting state
+    __shared__ __align__(8) float la[kChunk], wt[kChunk];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const uint32_t c = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * 64, grp = h / (d.heads / d.groups), t0 = c * kChunk;
     const __nv_bfloat16 *q = (const __nv_bfloat16*)d.q + grp * d.dk, *k = (const __nv_bfloat16*)d.k + grp * d.dk,
                         *v = (const __nv_bfloat16*)d.v + h * d.dv + j0;
     const uint32_t nv = min(64u, d.dv - j0);
-    stage_rows<kChunk>(kS, lk, q, d.ldq, d.dk, dkp, t0, T, rows_aligned(q, d.ldq, d.dk));
+    stage_rows<kChunk, DK>(kS, q, d.ldq, d.dk, t0, T, rows_aligned(q, d.ldq, d.dk));
     cp_async_commit();
     {
-        const uint4* fr = states + state_fragments(c, d.heads, h, dkp, dvp) + (size_t)(j0 / 16) * nb * 64;
-        for (uint32_t i = tid; i < 4 * nb * 64; i += 256) cp_async16(smem_u32(fS + i), fr + i);
+        const uint4* fr = states + state_fragments(c, d.heads, h, DK, dvp) + (size_t)(j0 / 16) * NB * 64;
+#pragma unroll
+        for (uint32_t i = 0; i < NB; i++) cp_async16(smem_u32(fS + tid + i * 256), fr + tid + i * 256);
     }
     cp_async_commit();
-    stage_rows<kChunk>(vS, LV, v, d.ldv, nv, 64, t0, T, rows_aligned(v, d.ldv, nv));
+    stage_rows<kChunk, 64>(vS, v, d.ldv, nv, t0, T, rows_aligned(v, d.ldv, nv));
     if (warp == 0) chunk_decays(d, h, t0, T, la, wt);
     cp_async_wait<1>();
     __syncthreads();
     // a scheduler's two warps: one with many earlier tokens in the chunk, one with few
     const uint32_t rblk = warp < 4 ? warp : 11 - warp;
-    uint32_t qa[KS][4];
+    uint32_t qa[NB][4];
     {
-        const uint32_t q_u = smem_u32(kS + (rblk * 16 + (lane & 15)) * lk + (lane >> 4) * 8);
+        const uint32_t q_u = smem_u32(kS + (rblk * 16 + (lane & 15)) * LK + (lane >> 4) * 8);
 #pragma unroll
-        for (int ks = 0; ks < KS; ks++) {
-            if ((uint32_t)ks < nb) ldsm_x4(qa[ks], q_u + ks * 32);
-            else qa[ks][0] = qa[ks][1] = qa[ks][2] = qa[ks][3] = 0;
-        }
+        for (uint32_t ks = 0; ks < NB; ks++) ldsm_x4(qa[ks], q_u + ks * 32);
     }
     float o[8][4];
 #pragma unroll
     for (int n = 0; n < 8; n++) { o[n][0] = 0.f; o[n][1] = 0.f; o[n][2] = 0.f; o[n][3] = 0.f; }
     __syncthreads();              // everyone has its queries
-    stage_rows<kChunk>(kS, lk, k, d.ldk, d.dk, dkp, t0, T, rows_aligned(k, d.ldk, d.dk));
+    stage_rows<kChunk, DK>(kS, k, d.ldk, d.dk, t0, T, rows_aligned(k, d.ldk, d.dk));
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
     const uint4* fr = fS + lane;
 #pragma unroll
-    for (int ks = 0; ks < KS; ks++) {
-        if ((uint32_t)ks >= nb) break;
+    for (uint32_t ks = 0; ks < NB; ks++) {
         uint4 hi[4], lo[4];
 #pragma unroll
         for (int n = 0; n < 4; n++) {
-            hi[n] = fr[((size_t)n * nb + ks) * 64];
-            lo[n] = fr[((size_t)n * nb + ks) * 64 + 32];
+            hi[n] = fr[(n * NB + ks) * 64];
+            lo[n] = fr[(n * NB + ks) * 64 + 32];
         }
 #pragma unroll
         for (int n = 0; n < 4; n++) {
             mma_bf16(o[2 * n], qa[ks], hi[n].x, hi[n].y);
             mma_bf16(o[2 * n + 1], qa[ks], hi[n].z, hi[n].w);
+        }
+#pragma unroll
+        for (int n = 0; n < 4; n++) {
             mma_bf16(o[2 * n], qa[ks], lo[n].x, lo[n].y);
             mma_bf16(o[2 * n + 1], qa[ks], lo[n].z, lo[n].w);
         }
     }
+    // The decay from an earlier token j to token i of this warp's block is cut at the block's first token r: r <- j is a factor
+    // of column j, i <- r one of the whole row, which also the starting state's part (decayed up to r) takes.
     const uint32_t ra = rblk * 16 + g, rb = ra + 8;
-    const float la_a = la[ra], la_b = la[rb];
+    const float la_a = la[ra], la_b = la[rb], la_r = la[rblk * 16];
     {
-        const float e_a = expf(la_a), e_b = expf(la_b);
+        const float e = ex2(la_r);
 #pragma unroll
-        for (int n = 0; n < 8; n++) { o[n][0] *= e_a; o[n][1] *= e_a; o[n][2] *= e_b; o[n][3] *= e_b; }
+        for (int n = 0; n < 8; n++) { o[n][0] *= e; o[n][1] *= e; o[n][2] *= e; o[n][3] *= e; }
     }
     cp_async_wait<0>();
     __syncthreads();
     // products within the chunk: 16 tokens at a time up to this warp's own
-    const uint32_t k_u = smem_u32(kS + ((lane >> 4) * 8 + (lane & 7)) * lk + ((lane >> 3) & 1) * 8);
+    const uint32_t k_u = smem_u32(kS + ((lane >> 4) * 8 + (lane & 7)) * LK + ((lane >> 3) & 1) * 8);
     const uint32_t v_u = smem_u32(vS + (lane & 15) * LV + (lane >> 4) * 8);
-    for (uint32_t kk = 0; kk <= rblk; kk++) {
-        float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    auto scores = [&](uint32_t kk, float (&s0)[4], float (&s1)[4]) {
 #pragma unroll
-        for (int ks = 0; ks < KS; ks++) {
-            if ((uint32_t)ks >= nb) break;
-            uint32_t b[4];
-            ldsm_x4(b, k_u + (kk * 16 * lk + ks * 16) * 2);
+        for (int i = 0; i < 4; i++) s0[i] = s1[i] = 0.f;
+        float u0[4] = {0.f, 0.f, 0.f, 0.f}, u1[4] = {0.f, 0.f, 0.f, 0.f};       // two chains of half the length
+#pragma unroll
+        for (uint32_t ks = 0; ks < NB; ks += 2) {
+            uint32_t b[4], b2[4];
+            ldsm_x4(b, k_u + (kk * 16 * LK + ks * 16) * 2);
+            ldsm_x4(b2, k_u + (kk * 16 * LK + ks * 16 + 16) * 2);
             mma_bf16(s0, qa[ks], b[0], b[1]);
             mma_bf16(s1, qa[ks], b[2], b[3]);
+            mma_bf16(u0, qa[ks + 1], b2[0], b2[1]);
+            mma_bf16(u1, qa[ks + 1], b2[2], b2[3]);
         }
-        auto weigh = [&](float s, uint32_t i, float la_i, uint32_t j) { return j <= i ? s * wt[j] * expf(la_i - la[j]) : 0.f; };
-        const uint32_t ja = kk * 16 + 2 * t4;
-        const uint32_t p[4] = {pack_bf2(weigh(s0[0], ra, la_a, ja), weigh(s0[1], ra, la_a, ja + 1)),
-                               pack_bf2(weigh(s0[2], rb, la_b, ja), weigh(s0[3], rb, la_b, ja + 1)),
-                               pack_bf2(weigh(s1[0], ra, la_a, ja + 8), weigh(s1[1], ra, la_a, ja + 9)),
-                               pack_bf2(weigh(s1[2], rb, la_b, ja + 8), weigh(s1[3], rb, la_b, ja + 9))};
+#pragma unroll
+        for (int i = 0; i < 4; i++) { s0[i] += u0[i]; s1[i] += u1[i]; }
+    };
+    auto values = [&](uint32_t kk, const uint32_t (&p)[4]) {
 #pragma unroll
         for (int n = 0; n < 8; n += 2) {
             uint32_t b[4];
@@ -538,6 +590,31 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const LinearRows d, cons
             mma_bf16(o[n], p, b[0], b[1]);
             mma_bf16(o[n + 1], p, b[2], b[3]);
         }
+    };
+    for (uint32_t kk = 0; kk < rblk; kk++) {
+        float s0[4], s1[4];
+        const uint32_t ja = kk * 16 + 2 * t4;
+        const float2 l0 = *reinterpret_cast<const float2*>(la + ja), l1 = *reinterpret_cast<const float2*>(la + ja + 8);
+        const float2 w0 = *reinterpret_cast<const float2*>(wt + ja), w1 = *reinterpret_cast<const float2*>(wt + ja + 8);
+        const float f0 = w0.x * ex2(la_r - l0.x), f1 = w0.y * ex2(la_r - l0.y), f2 = w1.x * ex2(la_r - l1.x), f3 = w1.y * ex2(la_r - l1.y);
+        scores(kk, s0, s1);
+        const uint32_t p[4] = {pack_bf2(s0[0] * f0, s0[1] * f1), pack_bf2(s0[2] * f0, s0[3] * f1), pack_bf2(s1[0] * f2, s1[1] * f3),
+                               pack_bf2(s1[2] * f2, s1[3] * f3)};
+        values(kk, p);
+    }
+    {
+        const float e_a = ex2(la_a - la_r), e_b = ex2(la_b - la_r);
+#pragma unroll
+        for (int n = 0; n < 8; n++) { o[n][0] *= e_a; o[n][1] *= e_a; o[n][2] *= e_b; o[n][3] *= e_b; }
+        float s0[4], s1[4];
+        scores(rblk, s0, s1);
+        auto weigh = [&](float s, uint32_t i, float la_i, uint32_t j) { return j <= i ? s * wt[j] * ex2(la_i - la[j]) : 0.f; };
+        const uint32_t ja = rblk * 16 + 2 * t4;
+        const uint32_t p[4] = {pack_bf2(weigh(s0[0], ra, la_a, ja), weigh(s0[1], ra, la_a, ja + 1)),
+                               pack_bf2(weigh(s0[2], rb, la_b, ja), weigh(s0[3], rb, la_b, ja + 1)),
+                               pack_bf2(weigh(s1[0], ra, la_a, ja + 8), weigh(s1[1], ra, la_a, ja + 9)),
+                               pack_bf2(weigh(s1[2], rb, la_b, ja + 8), weigh(s1[3], rb, la_b, ja + 9))};
+        values(rblk, p);
     }
     const float skip = d.skip ? d.skip[h] : 0.f;
     const bool pairs = (d.dv & 1u) == 0 && (d.ldo & 1u) == 0;
@@ -688,7 +765,7 @@ int32_t ssm_conv_rows(runit_ctx* ctx, const Ssm& m, bool exact, const void* proj
     const uint32_t vec = wide ? 4 : 1, per = kConvThreads * vec;
     const dim3 grid((m.channels() + per - 1) / per + 1, (T + kConvTok - 1) / kConvTok);
     auto go = [&](auto kern, auto* p, auto* o) -> int32_t {
-        kern<<<grid, kConvThreads, 0, ctx->stream>>>(m, p, ld, o, ld_out, dt, T, start);
+        kern<<<grid, kConvThreads, !exact && wide && m.taps == 4 ? kConvTok * kConvThreads * 8 : 0, ctx->stream>>>(m, p, ld, o, ld_out, dt, T, start);
         return runit_after_launch(ctx, "ssm_conv");
     };
 #define RUNIT_CONV(TA, TAPS) (wide ? go(ssm_conv_kernel<TA, TAPS, 4>, (const TA*)proj, (TA*)xbc) : go(ssm_conv_kernel<TA, TAPS, 1>, (const TA*)proj, (TA*)xbc))
@@ -697,27 +774,31 @@ int32_t ssm_conv_rows(runit_ctx* ctx, const Ssm& m, bool exact, const void* proj
 #undef RUNIT_CONV
 }
 
-static bool chunk_sizes(uint32_t dk) { return ((dk + 15) & ~15u) <= 256; }
+// key dimensions of the chunk kernels' variants
+static uint32_t chunk_dk(uint32_t dk) { return dk <= 64 ? 64u : (dk <= 128 ? 128u : (dk <= 256 ? 256u : 0u)); }
 size_t linear_chunk_bytes(uint32_t heads, uint32_t dk, uint32_t dv, uint32_t T) {
-    if (!chunk_sizes(dk)) return 0;
-    return (size_t)((T + kChunk - 1) / kChunk) * heads * pad16(dk) * pad64(dv) * 4;
+    return (size_t)((T + kChunk - 1) / kChunk) * heads * chunk_dk(dk) * pad64(dv) * 4;
 }
 
 int32_t linear_rows(runit_ctx* ctx, const LinearRows& d, bool exact, void* chunk_states, uint32_t T, uint32_t start) {
     RUNIT_REQUIRE(ctx, d.heads > 0 && d.groups > 0 && d.heads % d.groups == 0 && d.dk > 0 && d.dk <= kMaxKeyDim && d.dv > 0, "linear_rows: bad sizes");
     int32_t st;
-    if (!exact && T >= 16 && chunk_states && chunk_sizes(d.dk)) {
-        const uint32_t dkp = pad16(d.dk), dvp = pad64(d.dv), nc = (T + kChunk - 1) / kChunk;
-        const size_t sa = chunk_state_smem(dkp, nc), sb = (size_t)kChunk * (dkp + 8 + 72) * 2 + (size_t)dkp * 64 * 4;
-        if ((st = allow_smem(ctx, "chunk_state", chunk_state_kernel, sa)) != RUNIT_OK) return st;
-        chunk_state_kernel<<<dim3(d.heads, dvp / 32), 256, sa, ctx->stream>>>(d, (uint4*)chunk_states, dkp, dvp, T, start == 0);
-        if ((st = runit_after_launch(ctx, "chunk_state")) != RUNIT_OK) return st;
-        auto go = [&](auto kern) -> int32_t {
-            if ((st = allow_smem(ctx, "chunk_out", kern, sb)) != RUNIT_OK) return st;
-            kern<<<dim3(nc, d.heads, dvp / 64), 256, sb, ctx->stream>>>(d, (const uint4*)chunk_states, dkp, dvp, T);
+    if (!exact && T >= 16 && chunk_states && chunk_dk(d.dk)) {
+        const uint32_t dvp = pad64(d.dv), nc = (T + kChunk - 1) / kChunk;
+        auto go = [&](auto state, auto out, size_t sa, uint32_t dkp) -> int32_t {
+            const size_t sb = (size_t)kChunk * (dkp + 8 + 72) * 2 + (size_t)dkp * 64 * 4;
+            if ((st = allow_smem(ctx, "chunk_state", state, sa)) != RUNIT_OK) return st;
+            state<<<dim3(d.heads, dvp / 32), 256, sa, ctx->stream>>>(d, (uint4*)chunk_states, dvp, T, start == 0);
+            if ((st = runit_after_launch(ctx, "chunk_state")) != RUNIT_OK) return st;
+            if ((st = allow_smem(ctx, "chunk_out", out, sb)) != RUNIT_OK) return st;
+            out<<<dim3(nc, d.heads, dvp / 64), 256, sb, ctx->stream>>>(d, (const uint4*)chunk_states, dvp, T);
             return runit_after_launch(ctx, "chunk_out");
         };
-        return dkp <= 64 ? go(chunk_out_kernel<4>) : (dkp <= 128 ? go(chunk_out_kernel<8>) : go(chunk_out_kernel<16>));
+        switch (chunk_dk(d.dk)) {
+            case 64: return go(chunk_state_kernel<64>, chunk_out_kernel<64>, StateCfg<64>::smem(nc), 64);
+            case 128: return go(chunk_state_kernel<128>, chunk_out_kernel<128>, StateCfg<128>::smem(nc), 128);
+            default: return go(chunk_state_kernel<256>, chunk_out_kernel<256>, StateCfg<256>::smem(nc), 256);
+        }
     }
     const dim3 grid(d.heads, (d.dv + 31) / 32);
 #define RUNIT_SCAN(NR)                                                                                            \
