@@ -671,3 +671,110 @@ def test_trace_through_the_runner(tmp_path):
         assert [x for x in r.stdout.split("\n") if x.startswith("done")] == ["done %d" % i for i in range(4)]
         got = np.concatenate([np.fromfile(out / ("%d.f32" % i), "<f4").reshape(-1, cfg["vocab"]) for i in range(4)])
         assert M.row_errors(got, np.concatenate([rt[[6, 2, 7, 11]], ru[[4]]])).max() <= (1e-4 if dt == "float32" else 0.1)
+
+
+# ── the same parts in other designs ──
+class _Tensors:
+    """A source of tensors from a dict, the values as bf16 holds them."""
+
+    def __init__(self, w):
+        self.w = {k: from_bf16(to_bf16(np.asarray(v))).reshape(np.shape(v)) for k, v in w.items()}
+
+    def shape(self, n):
+        return self.w[n].shape
+
+    def f32(self, n):
+        return self.w[n].astype(np.float32)
+
+    def bf16(self, n):
+        return to_bf16(self.w[n]).reshape(self.w[n].shape)
+
+
+def _serve(ctx, R, up, layers, w, V, W, exact, post):
+    head = {"embed": up.matrix([("embed", V)], W), "final_norm": up.values(w["final"]), "head": up.matrix([("head", V)], W)}
+    cfg = R.LayeredCfg(n_layers=len(layers), width=W, vocab=V, max_seq=200, exact=exact, post_norm=post, eps=1e-5, embed_scale=2.0, logit_cap=9.0)
+    return R.LayeredModel(ctx, cfg, layers, head, keep=up)
+
+
+def _check_served(m, t, ref, exact):
+    for cuts in ([len(t)], [1], [20, 3], [70, 30]):
+        out, pos, i = [], 0, 0
+        while pos < len(t):
+            c = min(cuts[i % len(cuts)], len(t) - pos)
+            out.append(m.forward(t[pos:pos + c], pos, range(c)))
+            pos, i = pos + c, i + 1
+        check_rows(np.concatenate(out), ref, "float32" if exact else "bfloat16")
+    nxt = m.generate(t, 2)
+    assert exact == 0 or int(nxt[0]) == int(np.argmax(ref[-1]))
+
+
+@pytest.mark.parametrize("exact", [1, 0])
+def test_mixers_behind_norms_with_one_gain(ctx, exact):
+    """Attention alone (no window, no bias, queries and keys as they are), retention alone and a state-space layer, each behind
+    a norm with one gain."""
+    import runit_mac_b200 as R
+    from runit_mac_b200 import models
+    W, V, g = 56, 70, np.random.default_rng(2)
+    lin = lambda r, c: g.normal(0, 1.2 / np.sqrt(c), (r, c))
+    at, rt = M.left(4, 2, 16, 24, 10 ** 6), M.right(3, 16, 16, 8)
+    ss = M.mamba(4, 16, 24, groups=2, norm_groups=2)["mixer"]
+    inner, ch = 64, 64 + 96
+    w = {"embed": lin(V, W) * 4, "head": lin(V, W) * 3, "final": np.array([1.2])}
+    w.update({"a.q": lin(64, W), "a.k": lin(32, W), "a.v": lin(48, W), "a.o": lin(W, 96), "r.q": lin(48, W), "r.k": lin(48, W), "r.v": lin(48, W), "r.g": lin(48, W),
+              "r.o": lin(W, 48), "s.in": lin(inner + ch + 4, W), "s.conv": g.normal(0, 0.5, (ch, 4)), "s.conv.b": g.normal(0, 0.2, ch), "s.dt_bias": g.uniform(-3, 0, 4),
+              "s.A_log": g.uniform(-1, 1, 4), "s.D": g.normal(size=4), "s.norm": g.uniform(0.5, 1.5, inner), "s.o": lin(W, inner), "up": lin(40, W), "down": lin(W, 40)})
+    up = models._Uploader(ctx, _Tensors(w))
+    w = {k: np.asarray(v, np.float64) for k, v in up.source.w.items()}
+    gains = [1.25, 0.75, 1.5, 0.875]
+    a = R.LayerDesc(mixer=R.MIX_HEADS, norm1=up.values([gains[0]]), at_heads=4, at_kv_heads=2, at_dim=16, at_vdim=24, at_scale=0.3, at_out_scale=1.0,
+                    w_q=up.matrix([("a.q", 64), ("a.k", 32), ("a.v", 48)], W), w_o=up.matrix([("a.o", W)], 96))
+    r = R.LayerDesc(mixer=R.MIX_HEADS, norm1=up.values([gains[1]]), w_q=up.matrix([("r." + n, 48) for n in "qkvg"], W), w_o=up.matrix([("r.o", W)], 48))
+    models._retention_heads(r, up, rt, "r")
+    r.rt_out_scale = 1.0
+    s = R.LayerDesc(norm1=up.values([gains[2]]), norm2=up.values([gains[3]]))
+    models._mamba2_mixer(up, s, "s.", ss, W)
+    s.ff_kind, s.ff_act, s.ff, s.ff_up, s.ff_down = R.FF_DENSE, R.ACT_RELU2, 40, up.matrix([("up", 40)], W), up.matrix([("down", W)], 40)
+    m = _serve(ctx, R, up, [a, r, s], w, V, W, exact, 0)
+    t = [int(x) for x in g.integers(0, V, 100)]
+    norm = lambda x, k: P.rms(x, 1e-5) * k
+    x = w["embed"][t] * 2.0
+    h = norm(x, gains[0])
+    q, k, v = (h @ w["a.q"].T).reshape(-1, 4, 16), (h @ w["a.k"].T).reshape(-1, 2, 16), (h @ w["a.v"].T).reshape(-1, 2, 24)
+    own = np.arange(4) // 2
+    p = P.softmax_visible(P.biased_scores(q, k[:, own], 0.3, np.zeros(4)), P.window_mask(100, 100))
+    x = x + np.einsum("hij,jhd->ihd", p, v[:, own]).reshape(100, 96) @ w["a.o"].T
+    x = x + P.retention(norm(x, gains[1]), {n: w["r." + n] for n in "qkvgo"}, rt, 1e-5)
+    x = x + P.mamba2(norm(x, gains[2]), {n[2:]: w[n] for n in w if n.startswith("s.")}, ss, 1e-5)
+    x = x + P.relu2_ff(norm(x, gains[3]), w["up"], w["down"])
+    _check_served(m, t, P.softcap(norm(x, float(w["final"][0])) @ w["head"].T, 9.0), exact)
+    m.close()
+
+
+@pytest.mark.parametrize("exact", [1, 0])
+def test_latent_attention_with_norms_on_the_outputs(ctx, exact):
+    import runit_mac_b200 as R
+    from oracle import nuvilorn as N
+    from runit_mac_b200 import models
+    W, V, g = 64, 70, np.random.default_rng(3)
+    lin = lambda r, c: g.normal(0, 1.2 / np.sqrt(c), (r, c))
+    mix = {"heads": 3, "dim": 24, "rot_dim": 8, "vdim": 16, "kv_rank": 40, "rot": {"base": 1000.0, "dims": 8}, "scale": 0.25}
+    w = {"embed": lin(V, W) * 4, "head": lin(V, W) * 3, "final": g.uniform(0.5, 1.5, W), "n1": g.normal(0, 0.3, W), "n2": g.normal(0, 0.3, W)}
+    w.update({"m.q": lin(96, W), "m.dkv": lin(48, W), "m.dkv.norm": g.uniform(0.5, 1.5, 40), "m.uk": lin(72, 40), "m.uv": lin(48, 40), "m.o": lin(W, 48),
+              "f.gate": lin(56, W), "f.up": lin(56, W), "f.down": lin(W, 56)})
+    up = models._Uploader(ctx, _Tensors(w))
+    w = {k: np.asarray(v, np.float64) for k, v in up.source.w.items()}
+    layers = []
+    for _ in range(2):
+        d = R.LayerDesc(norm1=up.gain_offset("n1", W), norm2=up.gain_offset("n2", W))
+        models._latent_mixer(up, d, "m.", mix, W)
+        models._dense_ff(up, d, "f.", {"ff": 56}, W)
+        layers.append(d)
+    m = _serve(ctx, R, up, layers, w, V, W, exact, 1)
+    t = [int(x) for x in g.integers(0, V, 100)]
+    x, pos = w["embed"][t] * 2.0, np.arange(100)
+    mw = {n: w["m." + n] for n in ("q", "uk", "uv", "o")}
+    for _ in range(2):
+        x = x + P.norm_offset(N.latent_attention(x, pos, mw, mix, N.latent_of(x, pos, w["m.dkv"], w["m.dkv.norm"], mix, 1e-5)), w["n1"], 1e-5)
+        x = x + P.norm_offset(N.gated_ff(x, w["f.gate"], w["f.up"], w["f.down"]), w["n2"], 1e-5)
+    _check_served(m, t, P.softcap(P.norm_offset(x, w["final"] - 1, 1e-5) @ w["head"].T, 9.0), exact)
+    m.close()
