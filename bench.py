@@ -951,7 +951,7 @@ def time_pagazen_kernels(R, ctx, torch, stream, size, reps=20, T=2048):
     del caches
     slopes = torch.rand(p["H"], device="cuda")
     decay = torch.rand(2, p["rH"], device="cuda") * 0.1 + 0.85
-    freq = torch.rand(p["rd"] // 2, device="cuda")
+    freq = torch.cat([torch.rand(p["rd"] // 2, device="cuda"), torch.zeros(p["rd"] // 2, device="cuda")])
     proj, tickets, pos = torch.randn(max(in_h, in_s), device="cuda"), torch.zeros(4096, dtype=torch.int32, device="cuda"), torch.tensor([S - 1], dtype=torch.int32, device="cuda")
     part, ao = torch.empty(p["H"] * 64 * (p["dv"] + 2), device="cuda"), torch.empty(max(k_h, inner), device="cuda")
     sets = []

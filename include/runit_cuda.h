@@ -528,8 +528,8 @@ typedef struct {
     void*    v_cache;
 } runit_heads_cfg;
 /* Retention, S <- decay_h S + k v^T, o = S^T q.  A projected row holds [q, k: heads x dim | v, gate: heads x vdim]; the first
- * rot_dims coordinates of q and k rotate (pairs (i, i + rot_dims/2), angle position * freq[i]), k is multiplied by dim^(-1/2).
- * decay f32 [2][heads]: the decays, then their logarithms; state f32 [heads][dim][vdim]. */
+ * rot_dims coordinates of q and k rotate (pairs (i, i + rot_dims/2), angle position * (freq[0][i] + freq[1][i]), freq f32
+ * [2][rot_dims/2]: the frequencies and what their rounding to f32 has left), k is multiplied by dim^(-1/2).  decay f32 [2][heads]: the decays, then their logarithms; state f32 [heads][dim][vdim]. */
 typedef struct {
     uint32_t heads, dim, vdim, rot_dims;
     float    out_scale;

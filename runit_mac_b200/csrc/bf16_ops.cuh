@@ -176,7 +176,7 @@ struct HeadAttn {
 struct Retention {
     uint32_t heads = 0, dim = 0, vdim = 0, rot_dims = 0;
     float out_scale = 1.f, eps = 0.f, k_scale = 1.f;
-    const float* freq = nullptr;       // [rot_dims / 2]
+    const float* freq = nullptr;       // [2][rot_dims / 2]: the frequencies, then what their rounding to f32 has left
     const float* decay = nullptr;      // [2][heads]: the decays, then their logarithms
     float* state = nullptr;            // [heads][dim][vdim]
     __host__ __device__ uint32_t in_rows() const { return 2 * heads * (dim + vdim); }

@@ -320,7 +320,8 @@ __device__ __forceinline__ void retention_cta(const Retention& r, const float* r
             const bool second = i >= half;
             const uint32_t p = second ? i - half : i + half;
             float s, c;
-            sincosf((float)pos * r.freq[second ? p : i], &s, &c);
+            const uint32_t f = second ? p : i;
+            ls::sincos_at(pos, r.freq[f], r.freq[half + f], &s, &c);
             const float qo = q[p], ko = k[p];
             qv = second ? fmaf(qv, c, qo * s) : fmaf(qv, c, -(qo * s));
             kv = second ? fmaf(kv, c, ko * s) : fmaf(kv, c, -(ko * s));
@@ -373,7 +374,7 @@ __global__ void __launch_bounds__(256) heads_rows_kernel(const HeadAttn a, const
     float2* cs = reinterpret_cast<float2*>(sm);
     const uint32_t t = blockIdx.x, pos = start + t, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = r.rot_dims / 2;
     TC* row = proj + (size_t)t * ld;
-    for (uint32_t i = threadIdx.x; i < (r.heads ? half : 0); i += 256) sincosf((float)pos * r.freq[i], &cs[i].y, &cs[i].x);
+    for (uint32_t i = threadIdx.x; i < (r.heads ? half : 0); i += 256) ls::sincos_at(pos, r.freq[i], r.freq[half + i], &cs[i].y, &cs[i].x);
     __syncthreads();
     const bool wide = (ld & 3u) == 0 && (a.dim & 3u) == 0 && (a.vdim & 3u) == 0 && (reinterpret_cast<uintptr_t>(proj) & 7u) == 0;
     const bool pairs = sizeof(TC) == 2 && (ld & 1u) == 0 && (r.dim & 1u) == 0 && (half & 1u) == 0 && (a.in_rows() & 1u) == 0 &&

@@ -592,9 +592,15 @@ int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cf
     };
     size_t q = 0, qe = 0, po = 0, hv = 0, rows = 0, act = 0, routers = 0;
     uint32_t splits = 1;
-    auto angles = [&](int32_t dims, float base) -> const float* {
-        std::vector<float> f(dims / 2);
-        for (int32_t j = 0; j < dims / 2; j++) f[j] = (float)std::pow((double)base, -2.0 * j / dims);
+    // frequencies of a rotation; then (pairs) what their rounding to f32 has left
+    auto angles = [&](int32_t dims, float base, bool pairs) -> const float* {
+        const int32_t half = dims / 2;
+        std::vector<float> f(pairs ? 2 * half : half);
+        for (int32_t j = 0; j < half; j++) {
+            const double x = std::pow((double)base, -2.0 * j / dims);
+            f[j] = (float)x;
+            if (pairs) f[half + j] = (float)(x - (double)f[j]);
+        }
         float* p = nullptr;
         A((void**)&p, f.size() * 4);
         if (st == RUNIT_OK) {
@@ -625,7 +631,7 @@ int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cf
                 Retention& r = l.rt;
                 r.heads = d.rt_heads; r.dim = d.rt_dim; r.vdim = d.rt_vdim; r.rot_dims = d.rt_rot_dims; r.out_scale = d.rt_out_scale; r.eps = c.eps;
                 r.k_scale = (float)(1.0 / std::sqrt((double)r.dim));
-                if (r.rot_dims) r.freq = angles(d.rt_rot_dims, d.rt_rot_base);
+                if (r.rot_dims) r.freq = angles(d.rt_rot_dims, d.rt_rot_base, true);
                 r.decay = (const float*)d.rt_decay;
                 A((void**)&r.state, (size_t)r.heads * r.dim * r.vdim * 4);
                 m->recurrent = true;
@@ -650,7 +656,7 @@ int32_t runit_model_create_layered(runit_ctx_t* ctx, const runit_layered_cfg* cf
             l.w_uv = (const uint8_t*)d.w_ukv + (size_t)d.heads * d.dim * pad8(d.kv_rank) * 2;
             if (own) A(&l.cache, (size_t)c.max_seq * l.lat.pitch() * m->es());
             else l.cache = m->layers[d.kv_from].cache;
-            l.freq = angles(d.rot_dim, d.rot_base);
+            l.freq = angles(d.rot_dim, d.rot_base, false);
             splits = std::max(splits, latent_splits(ctx, l.lat, m->exact, 1));
             qe = std::max<size_t>(qe, (size_t)d.heads * l.lat.pitch());
             po = std::max<size_t>(po, (size_t)d.heads * l.lat.cp());

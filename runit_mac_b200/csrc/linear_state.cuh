@@ -54,6 +54,16 @@ __device__ __forceinline__ float silu_for(float x) {
     else return silu(x);
 }
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+// Sine and cosine of pos * (hi + lo), hi + lo a frequency as the sum of two floats: the product's rounding error (which for far
+// positions is that of the angle) and the low part turn the result by their small angle e.
+__device__ __forceinline__ void sincos_at(uint32_t pos, float hi, float lo, float* s, float* c) {
+    const float p = (float)pos, a = p * hi, e = fmaf(p, lo, fmaf(p, hi, -a));
+    float s0, c0;
+    sincosf(a, &s0, &c0);
+    const float h = -0.5f * e * e;
+    *s = s0 + fmaf(c0, e, s0 * h);
+    *c = c0 + fmaf(-s0, e, c0 * h);
+}
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void put(float* p, float v) { *p = v; }

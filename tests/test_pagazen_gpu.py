@@ -310,7 +310,8 @@ def test_retention_step(ctx, H, d, dv, rot):
     v8 = raw.astype(np.float64)
     q, k = P.rotate_halves(v8[:, :H * d].reshape(n, H, d), np.arange(n), rot, 50.0), P.rotate_halves(v8[:, H * d:2 * H * d].reshape(n, H, d), np.arange(n), rot, 50.0)
     ref = P.linear_scan(q, k * d ** -0.5, v8[:, 2 * H * d:2 * H * d + H * dv].reshape(n, H, dv), np.broadcast_to(decay.astype(np.float64), (n, H)))
-    freq, db = ctx.buffer_from((50.0 ** (-2.0 * np.arange(max(rot // 2, 1)) / max(rot, 1))).astype(np.float32)), ctx.buffer_from(np.stack([decay, np.log(decay)]))
+    f = 50.0 ** (-2.0 * np.arange(max(rot // 2, 1)) / max(rot, 1))
+    freq, db = ctx.buffer_from(np.stack([np.float32(f), np.float32(f - np.float32(f))])), ctx.buffer_from(np.stack([decay, np.log(decay)]))
     state = ctx.buffer_from(np.full(H * d * dv, 3.0, np.float32))
     cfg = R.RetentionCfg(H, d, dv, rot, 0.6, freq.ptr, db.ptr, state.ptr)
     ao, fac, sq = ctx.new_buffer(H * dv * 4), ctx.new_buffer(H * dv * 4), ctx.new_buffer(H * ((dv + 31) // 32) * 4)
@@ -320,6 +321,22 @@ def test_retention_step(ctx, H, d, dv, rot):
         close(ao.download(np.float32, H * dv), ref[t].reshape(-1), 5e-5)
         close(sq.download(np.float32, H * ((dv + 31) // 32)).reshape(H, -1).sum(1), (ref[t] ** 2).sum(1), 2e-4)
         close(fac.download(np.float32, H * dv), 0.6 * P.silu(v8[t, 2 * H * d + H * dv:]), 1e-5)
+
+
+@pytest.mark.parametrize("rot,base", [(64, 10000.0), (20, 50.0)])
+def test_rotation_at_far_positions(ctx, rot, base):
+    """Angles of thousands of radians keep the precision of their sine and cosine."""
+    import runit_mac_b200 as R
+    g, n, start = np.random.default_rng(rot), 16, 30000
+    raw = g.normal(size=(n, 4 * rot)).astype(np.float32)
+    f = base ** (-2.0 * np.arange(rot // 2) / rot)
+    freq, db, state = ctx.buffer_from(np.stack([np.float32(f), np.float32(f - np.float32(f))])), ctx.buffer_from(np.zeros(2, np.float32)), ctx.new_buffer(rot * rot * 4)
+    cfg = R.RetentionCfg(1, rot, rot, rot, 1.0, freq.ptr, db.ptr, state.ptr)
+    pr = Rows(ctx, raw, 1)
+    R.heads_rows(ctx, None, C.byref(cfg), 1, pr.buf, pr.ld, n, start)
+    ctx.flush()
+    ref = P.rotate_halves(raw[:, None, :rot].astype(np.float64), start + np.arange(n), rot, base)[:, 0]
+    assert np.abs(pr.read()[:, :rot] - ref).max() <= 2e-6
 
 
 # ── the model ──
